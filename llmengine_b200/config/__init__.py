@@ -12,6 +12,7 @@ from .funevik import FunevikConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .spec import LayerRun, LayerSpec, ModelSpec, PartSpec
 from .torisun import TorisunConfig
+from .vaderax import VaderaxConfig
 from .vifelix import VifelixConfig
 
 
@@ -73,6 +74,7 @@ register_architecture(BepuzenConfig.ARCHITECTURE, BepuzenConfig)
 register_architecture(TorisunConfig.ARCHITECTURE, TorisunConfig)
 register_architecture(VifelixConfig.ARCHITECTURE, VifelixConfig)
 register_architecture(FunevikConfig.ARCHITECTURE, FunevikConfig)
+register_architecture(VaderaxConfig.ARCHITECTURE, VaderaxConfig)
 
 
 @dataclass
@@ -121,5 +123,5 @@ class EngineConfig:
 
 __all__ = [
     "ARCHITECTURES", "Architecture", "BepuzenConfig", "ConfigError", "EngineConfig", "FunevikConfig", "LayerRun", "LayerSpec", "ModelSpec",
-    "PartSpec", "Qwen3Config", "TorisunConfig", "VifelixConfig", "config_from_dict", "find_architecture", "load_config", "register_architecture",
+    "PartSpec", "Qwen3Config", "TorisunConfig", "VaderaxConfig", "VifelixConfig", "config_from_dict", "find_architecture", "load_config", "register_architecture",
 ]

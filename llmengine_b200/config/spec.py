@@ -67,11 +67,14 @@ class LayerRun:
     `layer` indexes `ModelSpec.layers`; a layer may appear in several runs (its
     weights are shared, each run keeps a cache of its own).  `cache_from`, when
     set, is the index *in the order* of an earlier run whose cache this run
-    reads instead of keeping its own (it then writes nothing).
+    reads instead of keeping its own (it then writes nothing).  `add_embedding`:
+    the embedding output is added to the residual stream right before this run
+    (a design that loops over layers feeds its input in again at every pass).
     """
 
     layer: int
     cache_from: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

@@ -151,6 +151,75 @@ __global__ void window_post_heads_kernel(LlmeWindowPostArgs a) {
     for (int d = lane; d < dv; d += 32) vo[d] = a.v_bias ? from_f32<T>(to_f32(v[d]) + a.v_bias[g * dv + d]) : v[d];
 }
 
+// The same step for designs that divide every query and key head by its root mean square BEHIND the rotation (no weight): a
+// block takes a token (or a share of its heads), forms the token's cosines and sines once, and a warp finishes a head at a time
+// with its values in registers.
+template <typename T, int KR>
+__global__ void __launch_bounds__(256) window_post_unit_kernel(LlmeWindowPostArgs a) {
+    extern __shared__ float cs[];                                    // [rot_dims / 2] cosines, then sines
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, warps = blockDim.x >> 5, lane = threadIdx.x & 31;
+    const int dk = a.dk, dv = a.dv, ps = a.page_size, half = a.inv_freq ? a.rot_dims >> 1 : 0;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf((float)a.positions[t] * a.inv_freq[i], &s, &c);
+        cs[i] = c * a.amplitude;
+        cs[half + i] = s * a.amplitude;
+    }
+    __syncthreads();
+    const int slot = a.k_in ? a.slot_mapping[t] : -1;
+    const int page = slot >= 0 ? slot / ps : 0, off = slot - page * ps;
+    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
+    const int heads = a.nh + (slot >= 0 ? 2 * a.nkv : 0);
+    for (int hh = blockIdx.y * warps + (threadIdx.x >> 5); hh < heads; hh += gridDim.y * warps) {
+        if (hh >= a.nh + a.nkv) {
+            const int g = hh - a.nh - a.nkv;
+            const T* v = (const T*)a.v_in + (size_t)t * a.v_stride + g * dv;
+            T* vo = kpage + (size_t)a.nkv * ps * dk + ((size_t)g * ps + off) * dv;
+            for (int d = lane; d < dv; d += 32) vo[d] = v[d];
+            continue;
+        }
+        const bool query = hh < a.nh;
+        const int g = hh - a.nh;
+        const T* in = query ? (const T*)a.q_in + (size_t)t * a.q_stride + hh * dk : (const T*)a.k_in + (size_t)t * a.k_stride + g * dk;
+        T* out = query ? (T*)a.q_out + ((size_t)t * a.nh + hh) * dk : kpage + ((size_t)g * ps + off) * dk;
+        float x[KR], ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < KR; ++i) {
+            const int d = lane + 32 * i;
+            x[i] = d < dk ? to_f32(in[d]) : 0.0f;
+            if (d < 2 * half) {
+                const int e = a.interleaved ? d >> 1 : (d < half ? d : d - half);
+                const bool first = a.interleaved ? !(d & 1) : d < half;
+                const float other = to_f32(in[a.interleaved ? d ^ 1 : (first ? d + half : d - half)]);
+                x[i] = first ? x[i] * cs[e] - other * cs[half + e] : x[i] * cs[e] + other * cs[half + e];
+            }
+            ss = fmaf(x[i], x[i], ss);
+        }
+        const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)dk + a.eps);
+#pragma unroll
+        for (int i = 0; i < KR; ++i) {
+            const int d = lane + 32 * i;
+            if (d < dk) out[d] = from_f32<T>(x[i] * rinv);
+        }
+    }
+}
+
+template <typename T>
+static int launch_post_unit(const LlmeWindowPostArgs& a, cudaStream_t s) {
+    const int heads = a.nh + (a.k_in ? 2 * a.nkv : 0), most = (heads + 7) / 8, fill = (592 + a.tokens - 1) / a.tokens;
+    const dim3 grid(a.tokens, most < fill ? most : fill), block(256);
+    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float);
+    if (a.dk <= 32) llme_launch(window_post_unit_kernel<T, 1>, grid, block, smem, s, a);
+    else if (a.dk <= 64) llme_launch(window_post_unit_kernel<T, 2>, grid, block, smem, s, a);
+    else if (a.dk <= 128) llme_launch(window_post_unit_kernel<T, 4>, grid, block, smem, s, a);
+    else if (a.dk <= 256) llme_launch(window_post_unit_kernel<T, 8>, grid, block, smem, s, a);
+    else if (a.dk <= 512) llme_launch(window_post_unit_kernel<T, 16>, grid, block, smem, s, a);
+    else LLME_REFUSE("window_post: a query/key size of %d is larger than 512", a.dk);
+    LLME_LAUNCH_STATUS();
+}
+
 LLME_API int llme_window_post(const LlmeWindowPostArgs* args, int dtype, cudaStream_t stream) {
     const LlmeWindowPostArgs& a = *args;
     if (a.tokens <= 0) return 0;
@@ -162,6 +231,13 @@ LLME_API int llme_window_post(const LlmeWindowPostArgs* args, int dtype, cudaStr
         LLME_REFUSE("window_post: %d rotated coordinates of %d need an even count", a.rot_dims, a.dk);
     if ((a.q_gain || a.k_gain) && !(a.eps > 0.0f)) LLME_REFUSE("window_post: eps must be positive");
     const bool wide_in = a.in_f32 && dtype != LLME_F32;     // 32-bit projections, everything else in the type of the products
+    if (a.unit_norm) {
+        if (wide_in || a.q_gain || a.k_gain || a.q_bias || a.k_bias || a.v_bias) LLME_REFUSE("window_post: the norm behind the rotation stands alone");
+        if (!(a.eps > 0.0f)) LLME_REFUSE("window_post: eps must be positive");
+        if (dtype == LLME_F32) return launch_post_unit<float>(a, stream);
+        if (dtype == LLME_BF16) return launch_post_unit<__nv_bfloat16>(a, stream);
+        LLME_REFUSE("window_post: unsupported dtype %d", dtype);
+    }
     if (a.head_norm || a.q_bias || a.k_bias || a.v_bias) {
         if (wide_in) LLME_REFUSE("window_post: 32-bit projections come without biases and without the norm per head");
         if (!a.head_norm && (a.q_gain || a.k_gain)) LLME_REFUSE("window_post: biases come with the norm per head or with no norm");

@@ -123,6 +123,12 @@ __device__ __forceinline__ float xielu_bf16(float z, float a_pos, float a_neg) {
     return z > 0.0f ? fmaf(a_pos * z, z, 0.5f * z) : fmaf(a_neg, (__expf(z) - 1.0f) - z, 0.5f * z);
 }
 
+// max(z, 0)^2
+__device__ __forceinline__ float relu2(float z) {
+    z = fmaxf(z, 0.0f);
+    return z * z;
+}
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 

@@ -80,6 +80,36 @@ LLME_API int llme_embedding(const int* ids, const void* table, int table_dtype, 
     return llme_embedding_scaled(ids, table, table_dtype, out, tokens, hidden, vocab, 1.0f, stream);
 }
 
+// out[t, :] = (out[t, :] + delta[t, :]) + float(table[ids[t], :]) * scale: the embedding output added to the residual stream once
+// more (delta: a contribution that is still to be added, or NULL).  A thread owns columns, so the pass is in place.
+template <typename W>
+__global__ void embedding_add_kernel(const int* __restrict__ ids, const W* __restrict__ table, float* __restrict__ out,
+                                     const float* __restrict__ delta, int hidden, int vocab, float scale) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t];
+    const bool ok = id >= 0 && id < vocab;
+    const W* row = table + (size_t)(ok ? id : 0) * hidden;
+    float* o = out + (size_t)t * hidden;
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < hidden; j += gridDim.y * blockDim.x) {
+        float v = o[j];
+        if (delta) v += delta[(size_t)t * hidden + j];
+        o[j] = v + (ok ? to_f32(row[j]) * scale : 0.0f);
+    }
+}
+
+LLME_API int llme_embedding_add(const int* ids, const void* table, int table_dtype, float* out, const float* delta,
+                                int tokens, int hidden, int vocab, float scale, cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (!ids || !table || !out || hidden <= 0 || vocab <= 0) LLME_REFUSE("embedding_add: null pointer or non-positive size");
+    const int threads = 256, most = (hidden + threads - 1) / threads, fill = (592 + tokens - 1) / tokens;
+    const dim3 grid(tokens, most < fill ? most : fill);
+    if (table_dtype == LLME_F32) llme_launch(embedding_add_kernel<float>, grid, dim3(threads), 0, stream, ids, (const float*)table, out, delta, hidden, vocab, scale);
+    else if (table_dtype == LLME_BF16) llme_launch(embedding_add_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, ids, (const __nv_bfloat16*)table, out, delta, hidden, vocab, scale);
+    else LLME_REFUSE("embedding_add: unsupported table dtype %d", table_dtype);
+    LLME_LAUNCH_STATUS();
+}
+
 // ----------------------------------------------------------------------------- RMS norm (+ residual add)
 // For output row i (source row r = rows ? rows[i] : i):
 //   v = x[r] (+ delta[r], stored back into x[r]);  y[i] = (v * 1/sqrt(mean(v^2) + eps)) * gain.
@@ -248,6 +278,127 @@ LLME_API int llme_rmsnorm_pair(float* x, const void* delta, int delta_dtype, con
     if (delta_dtype == LLME_F32) return dispatch_rmsnorm<float, true>(x, delta, gain, gain_dtype, out, out_dtype, rows, n_out, hidden, eps, stream, gain2, out2);
     if (delta_dtype == LLME_BF16) return dispatch_rmsnorm<__nv_bfloat16, true>(x, delta, gain, gain_dtype, out, out_dtype, rows, n_out, hidden, eps, stream, gain2, out2);
     LLME_REFUSE("rmsnorm: unsupported delta dtype %d", delta_dtype);
+}
+
+// ----------------------------------------------------------------------------- layer norm (+ residual add)
+// For output row i (source row r = rows ? rows[i] : i):
+//   v = x[r] (+ delta[r], stored back into x[r]);  m = mean(v);  y[i] = (v - m) / sqrt(mean((v - m)^2) + eps) * gain + bias.
+// One block per row, both sums in a fixed order; the squares are taken of the deviations themselves.
+template <typename G, typename O>
+__global__ void layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const G* __restrict__ gain, const G* __restrict__ bias,
+                                 O* __restrict__ out, const int* __restrict__ rows, int hidden, float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[32];
+    const int i = blockIdx.x, r = rows ? rows[i] : i;
+    float* xr = x + (size_t)r * hidden;
+    float s = 0.0f;
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+        float v = xr[j];
+        if (delta) {
+            v += delta[(size_t)r * hidden + j];
+            xr[j] = v;
+        }
+        s += v;
+    }
+    const float mean = block_sum(s, scratch) / (float)hidden;
+    float ss = 0.0f;
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+        const float d = xr[j] - mean;                            // same thread wrote xr[j] above
+        ss += d * d;
+    }
+    const float rinv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+    for (int j = threadIdx.x; j < hidden; j += blockDim.x)
+        out[(size_t)i * hidden + j] = from_f32<O>(((xr[j] - mean) * rinv) * to_f32(gain[j]) + to_f32(bias[j]));
+}
+
+// Rows that are a multiple of 4 wide: a thread keeps up to V groups of 4 values of the row in registers.
+template <typename G, typename O, int V>
+__global__ void layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const G* __restrict__ gain, const G* __restrict__ bias,
+                                     O* __restrict__ out, const int* __restrict__ rows, int hidden, float eps) {
+    __shared__ float scratch[32];
+    const int i = blockIdx.x, groups = hidden >> 2;
+    float4 v[V], g[V], b[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) {                                // weights: nothing before this kernel writes them
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j < groups) {
+            g[k] = Vec4<G>::load(gain + 4 * j);
+            b[k] = Vec4<G>::load(bias + 4 * j);
+        }
+    }
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = rows ? rows[i] : i;
+    float* xr = x + (size_t)r * hidden;
+    float s = 0.0f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j < groups) {
+            v[k] = Vec4<float>::load(xr + 4 * j);
+            if (delta) {
+                const float4 d = Vec4<float>::load(delta + (size_t)r * hidden + 4 * j);
+                v[k].x += d.x; v[k].y += d.y; v[k].z += d.z; v[k].w += d.w;
+            }
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j < groups) {
+            if (delta) Vec4<float>::store(xr + 4 * j, v[k]);
+            s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+        }
+    }
+    const float mean = block_sum(s, scratch) / (float)hidden;
+    float ss = 0.0f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j < groups) {
+            v[k].x -= mean; v[k].y -= mean; v[k].z -= mean; v[k].w -= mean;
+            ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+        }
+    }
+    const float rinv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        const int j = threadIdx.x + k * blockDim.x;
+        if (j < groups)
+            Vec4<O>::store(out + (size_t)i * hidden + 4 * j, make_float4((v[k].x * rinv) * g[k].x + b[k].x, (v[k].y * rinv) * g[k].y + b[k].y,
+                                                                         (v[k].z * rinv) * g[k].z + b[k].z, (v[k].w * rinv) * g[k].w + b[k].w));
+    }
+}
+
+template <typename G, typename O>
+static void launch_layernorm(float* x, const float* delta, const void* gain, const void* bias, void* out, const int* rows, int n_out, int hidden,
+                             float eps, cudaStream_t s) {
+    const bool whole = hidden % 4 == 0 && hidden <= 16384 && (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)gain | (uintptr_t)bias | (uintptr_t)out) % 16) == 0;
+    const int groups = hidden / 4;
+    auto threads = [&](int per) { return dim3(((groups + per - 1) / per + 31) / 32 * 32); };
+    if (whole && groups <= 256)
+        llme_launch(layernorm_vec_kernel<G, O, 1>, dim3(n_out), threads(1), 0, s, x, delta, (const G*)gain, (const G*)bias, (O*)out, rows, hidden, eps);
+    else if (whole && groups <= 1024)
+        llme_launch(layernorm_vec_kernel<G, O, 2>, dim3(n_out), threads(2), 0, s, x, delta, (const G*)gain, (const G*)bias, (O*)out, rows, hidden, eps);
+    else if (whole)
+        llme_launch(layernorm_vec_kernel<G, O, 4>, dim3(n_out), threads(4), 0, s, x, delta, (const G*)gain, (const G*)bias, (O*)out, rows, hidden, eps);
+    else
+        llme_launch(layernorm_kernel<G, O>, dim3(n_out), dim3(hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128)), 0, s, x, delta, (const G*)gain, (const G*)bias, (O*)out, rows, hidden, eps);
+}
+
+// x [*, hidden] 32-bit (updated in place when delta, also 32-bit, is given); gain and bias of one type; rows nullable.
+LLME_API int llme_layernorm(float* x, const float* delta, const void* gain, const void* bias, int param_dtype, void* out, int out_dtype,
+                            const int* rows, int n_out, int hidden, float eps, cudaStream_t stream) {
+    if (n_out <= 0) return 0;
+    if (!x || !gain || !bias || !out || hidden <= 0) LLME_REFUSE("layernorm: null pointer or non-positive size");
+    if (!(eps > 0.0f)) LLME_REFUSE("layernorm: eps must be positive");
+    if (param_dtype == LLME_F32 && out_dtype == LLME_F32) launch_layernorm<float, float>(x, delta, gain, bias, out, rows, n_out, hidden, eps, stream);
+    else if (param_dtype == LLME_F32 && out_dtype == LLME_BF16) launch_layernorm<float, __nv_bfloat16>(x, delta, gain, bias, out, rows, n_out, hidden, eps, stream);
+    else if (param_dtype == LLME_BF16 && out_dtype == LLME_F32) launch_layernorm<__nv_bfloat16, float>(x, delta, gain, bias, out, rows, n_out, hidden, eps, stream);
+    else if (param_dtype == LLME_BF16 && out_dtype == LLME_BF16) launch_layernorm<__nv_bfloat16, __nv_bfloat16>(x, delta, gain, bias, out, rows, n_out, hidden, eps, stream);
+    else LLME_REFUSE("layernorm: unsupported parameter/out dtype %d/%d", param_dtype, out_dtype);
+    LLME_LAUNCH_STATUS();
 }
 
 // ----------------------------------------------------------------------------- QK norm + rotary + cache write

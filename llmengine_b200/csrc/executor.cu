@@ -58,7 +58,8 @@ typedef int (*WindowAttnPlainFn)(const LlmeWindowAttnArgs*, int, cudaStream_t);
 typedef int (*WindowAttnTcFn)(const LlmeWindowFastArgs*, int, int, cudaStream_t);
 typedef int (*MoeRouteFn)(const LlmeMoeRouteArgs*, cudaStream_t);
 typedef int (*GroupedFn)(const LlmeGroupedArgs*, int, int, int, cudaStream_t);
-typedef int (*MoeCombineFn)(const float*, long long, const float*, const float*, float*, int, int, int, cudaStream_t);
+typedef int (*MoeCombineFn)(const float*, long long, const float*, const float*, float*, int, int, int, const float*, long long, const int*,
+                            const void*, long long, int, int, cudaStream_t);
 typedef int (*EmbeddingScaledFn)(const int*, const void*, int, float*, int, int, int, float, cudaStream_t);
 typedef int (*SigmoidMulScaledFn)(const void*, long long, const void*, long long, void*, long long, int, int, int, float, cudaStream_t);
 typedef int (*GatedActBiasFn)(const void*, long long, void*, long long, int, int, int, int, float, float, const float*, cudaStream_t);
@@ -70,7 +71,10 @@ typedef int (*GatedNormFn)(const LlmeGatedNormArgs*, cudaStream_t);
 typedef int (*RmsNormPairFn)(float*, const void*, int, const void*, int, void*, int, const int*, int, int, float, const void*, void*, cudaStream_t);
 typedef int (*SigmoidMulGroupedFn)(const void*, long long, const void*, long long, void*, long long, int, int, int, float, int, cudaStream_t);
 typedef int (*ResidualAddScaledFn)(float*, const void*, const void*, int, void*, int, int, int, const float*, const float*, cudaStream_t);
-typedef int (*MoeCombineGatedFn)(const float*, long long, const float*, const float*, float*, int, int, int, const float*, long long, cudaStream_t);
+typedef int (*LayerNormFn)(float*, const float*, const void*, const void*, int, void*, int, const int*, int, int, float, cudaStream_t);
+typedef int (*EmbeddingAddFn)(const int*, const void*, int, float*, const float*, int, int, int, float, cudaStream_t);
+typedef int (*Relu2Fn)(const void*, long long, void*, long long, int, int, int, cudaStream_t);
+typedef int (*DeltaFn)(const LlmeDeltaArgs*, cudaStream_t);
 typedef int (*RowNormFn)(const void*, long long, int, const void*, int, void*, long long, int, int, int, float, cudaStream_t);
 typedef int (*ExpGatesFn)(const LlmeExpGatesArgs*, int, cudaStream_t);
 typedef int (*GemmF32BatchedFn)(const float*, const void*, int, float*, int, int, int, long long, long long, long long, int, long long,
@@ -190,6 +194,8 @@ size_t record_size(int kind) {
         case LLME_OP_GATED_NORM: return sizeof(LlmeGatedNormOp);
         case LLME_OP_ROW_NORM: return sizeof(LlmeRowNormOp);
         case LLME_OP_EXP_GATES: return sizeof(LlmeExpGatesOp);
+        case LLME_OP_LAYERNORM: return sizeof(LlmeLayerNormOp);
+        case LLME_OP_DELTA_RULE: return sizeof(LlmeDeltaRuleOp);
     }
     return 0;
 }
@@ -197,8 +203,8 @@ const char* kind_name(int kind) {
     static const char* names[] = {"?", "embedding", "rmsnorm", "linear", "linear_swiglu", "qkv_post", "attend", "attention", "call",
                                   "linear_act", "pointwise", "batched_linear", "residual_add", "latent_attention", "token_side",
                                   "postnorm", "window_attention", "moe_route", "grouped_linear", "moe_combine", "short_conv", "rotate",
-                                  "recurrence", "gated_norm", "row_norm", "exp_gates"};
-    return kind >= 1 && kind <= 25 ? names[kind] : names[0];
+                                  "recurrence", "gated_norm", "row_norm", "exp_gates", "layernorm", "delta_rule"};
+    return kind >= 1 && kind <= 27 ? names[kind] : names[0];
 }
 
 constexpr int SKINNY_ROWS = 16;      // most rows the weight-streaming product takes (gemm_skinny.cu)
@@ -303,6 +309,11 @@ int product(LlmeExecutor& ex, const LlmeStep& step, const void* x, long long ldx
 }
 
 int op_embedding(LlmeExecutor& ex, const LlmeEmbeddingOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (o.accumulate) {
+        auto* g = (EmbeddingAddFn)ex.find("embedding_add");
+        if (!g) return ex.fail("no kernel that adds an embedding to the stream is registered");
+        return ex.launched(g(s.token_ids, o.table, o.table_dtype, o.out, o.delta, s.num_tokens, o.hidden, o.vocab, o.scale, st), "embedding_add");
+    }
     if (o.scale != 1.0f) {
         auto* g = (EmbeddingScaledFn)ex.find("embedding_scaled");
         if (!g) return ex.fail("no kernel for a scaled embedding is registered");
@@ -325,6 +336,13 @@ int op_rmsnorm(LlmeExecutor& ex, const LlmeRmsNormOp& o, const LlmeStep& s, cuda
     }
     return ex.launched(f(o.x, o.delta, o.delta_dtype, o.gain, o.gain_dtype, o.out, o.out_dtype, some ? s.logit_rows : nullptr,
                          rows_of(s, o.rows), o.size, o.eps, st), "rmsnorm");
+}
+
+int op_layernorm(LlmeExecutor& ex, const LlmeLayerNormOp& o, const LlmeStep& s, cudaStream_t st) {
+    auto* f = (LayerNormFn)ex.find("layernorm");
+    if (!f) return ex.fail("no layernorm kernel is registered");
+    return ex.launched(f(o.x, o.delta, o.gain, o.bias, o.param_dtype, o.out, o.out_dtype, o.rows == LLME_ROWS_LOGITS ? s.logit_rows : nullptr,
+                         rows_of(s, o.rows), o.size, o.eps, st), "layernorm");
 }
 
 int op_linear(LlmeExecutor& ex, const LlmeLinearOp& o, const LlmeStep& s, cudaStream_t st) {
@@ -521,7 +539,7 @@ int op_linear_act(LlmeExecutor& ex, const LlmeLinearActOp& o, const LlmeStep& s,
     const int M = s.num_tokens;
     if (M <= 0) return 0;
     const LlmeLinearOp& p = o.product;
-    if (o.act != LLME_ACT_XIELU) return ex.fail("linear_act: unknown activation %d", o.act);
+    if (o.act != LLME_ACT_XIELU && o.act != LLME_ACT_RELU2) return ex.fail("linear_act: unknown activation %d", o.act);
     // a handful of tokens: the weight-streaming product carries the activation in its epilogue (same rule as the plain product)
     const std::string& dec = ex.choice("linear.decode");
     if (p.x_dtype == LLME_DT_BF16 && p.w_dtype == LLME_DT_BF16 && ex.choice("linear") != "plain" && ex.choice("linear_swiglu") == "fused" &&
@@ -540,6 +558,11 @@ int op_linear_act(LlmeExecutor& ex, const LlmeLinearActOp& o, const LlmeStep& s,
     }
     if (!p.out) return ex.fail("linear_act: the product needs its workspace");
     if (int rc = product(ex, s, p.x, p.ldx, p.x_dtype, p.w, p.ldw, p.w_dtype, p.out, p.ldo, p.out_dtype, M, p.n, p.k, st)) return rc;
+    if (o.act == LLME_ACT_RELU2) {
+        auto* g = (Relu2Fn)ex.find("relu2");
+        if (!g) return ex.fail("no relu2 kernel is registered");
+        return ex.launched(g(p.out, p.ldo, o.out, o.ldo, p.out_dtype, M, p.n, st), "relu2");
+    }
     auto* f = (XieluFn)ex.find("xielu");
     if (!f) return ex.fail("no xielu kernel is registered");
     return ex.launched(f(p.out, p.ldo, o.out, o.ldo, p.out_dtype, M, p.n, o.p0, o.p1, st), "xielu");
@@ -690,8 +713,15 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
     p.positions = s.positions; p.q_out = o.q; p.cache = o.cache; p.slot_mapping = g.slot_mapping;
     p.tokens = s.num_tokens; p.nh = o.nh; p.nkv = o.nkv; p.dk = o.dk; p.dv = o.dv; p.page_size = g.page_size;
     p.q_bias = o.q_bias; p.k_bias = o.k_bias; p.v_bias = o.v_bias; p.head_norm = o.head_norm;
-    p.interleaved = o.interleaved; p.in_f32 = o.in_f32;
+    p.interleaved = o.interleaved; p.in_f32 = o.in_f32; p.unit_norm = o.unit_norm;
     if (int rc = ex.launched(post(&p, o.dtype, st), "window_post")) return rc;
+    // ordinary causal attention with keys and values of one width: a page holds its keys and then its values in both layouts, so the
+    // kernels of plain grouped-query attention (tcgen05 portions, split-context decode) read the cache as it is
+    if (o.decode_scratch && o.dk == o.dv && !o.keep_first && !o.sink && !(o.softcap > 0.0f) && fast_attention(ex, o.dtype, o.dk)) {
+        LlmeAttendOp at = {o.q, o.out, o.dtype, o.cache, o.cache_pages * 2 * o.nkv * g.page_size, o.group, o.nh, o.nkv, o.dk, o.window, o.scale,
+                           o.decode_scratch, o.decode_scratch_floats};
+        return op_attend(ex, at, s, st);
+    }
     // bfloat16 with sizes the tensor-core kernel is built for: prompt portions in one launch, single tokens in another
     auto* tc = (WindowAttnTcFn)ex.find("window_attention_tc/" + std::to_string(o.dk) + "x" + std::to_string(o.dv));
     if (tc && o.dtype == LLME_DT_BF16 && ex.choice("attention") == "fast") {
@@ -732,6 +762,7 @@ int op_short_conv(LlmeExecutor& ex, const LlmeShortConvOp& o, const LlmeStep& s,
     if (!f) return ex.fail("no short_conv kernel is registered");
     LlmeShortConvArgs a = {o.x, o.ldx, o.x_dtype, o.w, o.bias, o.state, o.state_stride, o.out, o.ldo, s.cu_q_lens, s.state_slots,
                            s.num_tokens, s.num_requests, o.channels, o.taps, o.act};
+    if (o.taps > 1 && s.max_portion_len <= 1) return ex.launched(f(&a, 2, st), "short_conv");     // single tokens: outputs and states in one launch
     if (int rc = ex.launched(f(&a, 0, st), "short_conv")) return rc;
     if (o.taps <= 1) return 0;
     return ex.launched(f(&a, 1, st), "short_conv");     // after the outputs, which read the state: it takes the step's last inputs
@@ -765,8 +796,32 @@ int op_gated_norm(LlmeExecutor& ex, const LlmeGatedNormOp& o, const LlmeStep& s,
     auto* f = (GatedNormFn)ex.find("gated_norm");
     if (!f) return ex.fail("no gated_norm kernel is registered");
     LlmeGatedNormArgs a = {o.y, o.ldy, o.gate, o.ldg, o.weight, o.out, o.ldo, o.dtype, s.num_tokens, o.cols, o.group, o.gate_first, o.eps, o.scale,
-                           o.gate_act, o.floor, o.ld_floor, o.den_eps};
+                           o.gate_act, o.floor, o.ld_floor, o.den_eps, o.gate_f32};
     return ex.launched(f(&a, st), "gated_norm");
+}
+
+int op_delta_rule(LlmeExecutor& ex, const LlmeDeltaRuleOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (s.num_tokens <= 0 || s.num_requests <= 0) return 0;
+    auto* step = (DeltaFn)ex.find("delta_step");
+    auto* portions = (DeltaFn)ex.find("delta_portions");
+    if (!step || !portions) return ex.fail("no delta_rule kernels are registered");
+    LlmeDeltaArgs a = {o.q, o.k, o.v, o.ldq, o.ldk, o.ldv, o.write, o.forget, o.ld_gates, o.dt_bias, o.a_log, o.q_scale, o.unit_eps, o.state,
+                       o.state_stride, o.out, o.ldo, s.cu_q_lens, s.state_slots, nullptr, s.num_requests, s.num_requests, s.num_tokens, o.heads,
+                       o.n, o.p, o.qk_groups, o.unit, o.coef};
+    if (ex.choice("delta_rule") == "tokens") return ex.launched(step(&a, st), "delta_step");      // every request, token after token
+    if (s.num_portion > 0) {
+        const long long n4 = (o.n + 3) / 4 * 4, blocks = s.num_tokens / 4 + s.num_requests + 1;
+        if (s.num_tokens * 2 * o.qk_groups * n4 > o.unit_floats || blocks * o.heads * 40 > o.coef_floats)
+            return ex.fail("delta_rule: the workspace is too small for %d tokens of %d requests", s.num_tokens, s.num_requests);
+        a.rows = s.portion_rows; a.n_rows = s.num_portion;
+        if (int rc = ex.launched(portions(&a, st), "delta_portions")) return rc;
+        ++ex.launches;                                          // the blocks' numbers and the walk are two kernels
+    }
+    if (s.num_decode > 0) {
+        a.rows = s.decode_rows; a.n_rows = s.num_decode;
+        if (int rc = ex.launched(step(&a, st), "delta_step")) return rc;
+    }
+    return 0;
 }
 
 int op_row_norm(LlmeExecutor& ex, const LlmeRowNormOp& o, const LlmeStep& s, cudaStream_t st) {
@@ -789,9 +844,10 @@ int op_moe_route(LlmeExecutor& ex, const LlmeMoeRouteOp& o, const LlmeStep& s, c
     if (s.num_tokens <= 0) return 0;
     auto* f = (MoeRouteFn)ex.find("moe_route");
     if (!f) return ex.fail("no moe_route kernel is registered");
-    LlmeMoeRouteArgs a = {o.logits, o.ld, s.num_tokens, o.num_experts, o.top_k, o.scale, o.experts, o.weights, o.offsets, o.order, o.counts, o.mode};
+    LlmeMoeRouteArgs a = {o.logits, o.ld, s.num_tokens, o.num_experts, o.top_k, o.scale, o.experts, o.weights, o.offsets, o.order, o.counts, o.mode,
+                          o.correction, o.groups, o.keep};
     const int rc = ex.launched(f(&a, st), "moe_route");
-    ++ex.launches;                                          // routing and ordering are two kernels
+    if (s.num_tokens > 64) ++ex.launches;                   // routing and ordering are two kernels, one for a few tokens
     return rc;
 }
 
@@ -810,14 +866,10 @@ int op_grouped_linear(LlmeExecutor& ex, const LlmeGroupedLinearOp& o, const Llme
 }
 
 int op_moe_combine(LlmeExecutor& ex, const LlmeMoeCombineOp& o, const LlmeStep& s, cudaStream_t st) {
-    if (o.base_gate) {
-        auto* g = (MoeCombineGatedFn)ex.find("moe_combine_gated");
-        if (!g) return ex.fail("no moe_combine kernel with a gate on the shared part is registered");
-        return ex.launched(g(o.y, o.ldy, o.weights, o.base, o.out, s.num_tokens, o.top_k, o.size, o.base_gate, o.ld_gate, st), "moe_combine");
-    }
     auto* f = (MoeCombineFn)ex.find("moe_combine");
     if (!f) return ex.fail("no moe_combine kernel is registered");
-    return ex.launched(f(o.y, o.ldy, o.weights, o.base, o.out, s.num_tokens, o.top_k, o.size, st), "moe_combine");
+    return ex.launched(f(o.y, o.ldy, o.weights, o.base, o.out, s.num_tokens, o.top_k, o.size, o.base_gate, o.ld_gate, o.experts, o.same, o.ld_same,
+                         o.same_dtype, o.first_identity, st), "moe_combine");
 }
 
 const std::map<std::string, std::vector<std::string>>& variants() {
@@ -828,6 +880,7 @@ const std::map<std::string, std::vector<std::string>>& variants() {
         {"attention", {"fast", "plain"}},
         {"attention.portion", {"tcgen05", "mma"}},
         {"attention.decode", {"fused", "split"}},
+        {"delta_rule", {"blocks", "tokens"}},
     };
     return v;
 }
@@ -872,6 +925,7 @@ LLME_EXPORT int llme_executor_choose(LlmeExecutor* ex, const char* op, const cha
             ex->chosen["linear"] = "plain";
             ex->chosen["linear_swiglu"] = "unfused";
             ex->chosen["attention"] = "plain";
+            ex->chosen["delta_rule"] = "tokens";
         }
         return 0;
     }
@@ -974,6 +1028,8 @@ LLME_EXPORT int llme_plan_run(LlmePlan* p, const LlmeStep* step, int first, int 
             case LLME_OP_RECURRENCE: rc = op_recurrence(ex, *(const LlmeRecurrenceOp*)b, s, stream); break;
             case LLME_OP_GATED_NORM: rc = op_gated_norm(ex, *(const LlmeGatedNormOp*)b, s, stream); break;
             case LLME_OP_ROW_NORM: rc = op_row_norm(ex, *(const LlmeRowNormOp*)b, s, stream); break;
+            case LLME_OP_LAYERNORM: rc = op_layernorm(ex, *(const LlmeLayerNormOp*)b, s, stream); break;
+            case LLME_OP_DELTA_RULE: rc = op_delta_rule(ex, *(const LlmeDeltaRuleOp*)b, s, stream); break;
             case LLME_OP_EXP_GATES: rc = op_exp_gates(ex, *(const LlmeExpGatesOp*)b, s, stream); break;
             case LLME_OP_CALL: {
                 const LlmeCallOp& c = *(const LlmeCallOp*)b;

@@ -164,6 +164,7 @@ __global__ void __launch_bounds__(THREADS, BLOCKS) gemm_skinny_kernel(SkinnyArgs
                 float v = total(i);
                 // the activation sees the product as it is stored when the activation is a kernel of its own
                 if (a.pointwise == 1) v = xielu(__bfloat162float(__float2bfloat16_rn(v)), a.p0, a.p1);
+                else if (a.pointwise == 2) v = relu2(v);
                 reinterpret_cast<O*>(a.out)[(size_t)tok * a.ldo + row] = from_f32<O>(v);
             }
         }
@@ -270,12 +271,12 @@ LLME_API int llme_gemm_skinny_gated_bf16(const void* x, long long ldx, const voi
     LLME_REFUSE("gemm_skinny: unsupported output dtype %d", out_dtype);
 }
 
-// out[M, N] = act(x W^T), elementwise, in the product's epilogue.  act 1: xIELU with coefficients p0 (z > 0) and p1 (z <= 0).
+// out[M, N] = act(x W^T), elementwise, in the product's epilogue.  act 1: xIELU with coefficients p0 (z > 0) and p1 (z <= 0); act 2: max(z, 0)^2.
 LLME_API int llme_gemm_skinny_act_bf16(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
                                        long long ldo, int M, int N, int K, int act, float p0, float p1, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!x || !w || !out) LLME_REFUSE("gemm_skinny: null pointer");
-    if (act != 1) LLME_REFUSE("gemm_skinny: unknown activation %d", act);
+    if (act != 1 && act != 2) LLME_REFUSE("gemm_skinny: unknown activation %d", act);
     if (!llme_gemm_skinny_supports(M, N, K, ldx, ldw)) LLME_REFUSE("gemm_skinny: M=%d N=%d K=%d ldx=%lld ldw=%lld is not supported (M <= 16, K and strides multiples of 8)", M, N, K, ldx, ldw);
     if (((uintptr_t)x | (uintptr_t)w) % 16) LLME_REFUSE("gemm_skinny: operands must be 16-byte aligned");
     if (ldo < N) LLME_REFUSE("gemm_skinny: output row stride shorter than the row");

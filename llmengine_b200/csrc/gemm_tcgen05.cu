@@ -39,7 +39,7 @@ struct TcArgs {
     int M, N, K;
     int m_tiles, n_tiles;
     int inter;      // ACT kernels: W = [gate | up] with `inter` rows each, out[M, inter] = silu(gate) * up
-    int pointwise;  // other kernels: 0 = the product as it is; 1 = xIELU of it (through bfloat16 first), coefficients p0, p1;
+    int pointwise;  // other kernels: 0 = the product as it is; 1 = xIELU of it (through bfloat16 first), coefficients p0, p1; 2 = max(z, 0)^2;
                     // ACT kernels: 0 = silu(gate) * up; 1 = the clamped gate with limit p0 and slope p1
     float p0, p1;
 };
@@ -239,6 +239,9 @@ __device__ __forceinline__ void gemm_tc_body(const CUtensorMap& map_x, const CUt
 #pragma unroll
                             for (int j = 0; j < 32; ++j)
                                 v[j] = __float_as_uint(xielu_bf16(__bfloat162float(__float2bfloat16_rn(__uint_as_float(v[j]))), a.p0, a.p1));
+                        } else if (a.pointwise == 2) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(relu2(__uint_as_float(v[j])));
                         }
                     }
                     if (c + COLS >= OUT_COLS && half == COLS / 32 - 1) {
@@ -423,12 +426,12 @@ static int run_plain(const void* x, long long ldx, const void* w, long long ldw,
     LLME_REFUSE("gemm_tc: unsupported output dtype %d", out_dtype);
 }
 
-// out[M, N] = act(x W^T) elementwise, in the epilogue.  act 1: xIELU with coefficients p0 (z > 0) and p1 (z <= 0).
+// out[M, N] = act(x W^T) elementwise, in the epilogue.  act 1: xIELU with coefficients p0 (z > 0) and p1 (z <= 0); act 2: max(z, 0)^2.
 LLME_API int llme_gemm_tc_act_bf16(const void* x, long long ldx, const void* w, long long ldw, void* out, int out_dtype,
                                    long long ldo, int M, int N, int K, int act, float p0, float p1, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!x || !w || !out) LLME_REFUSE("gemm_tc: null pointer");
-    if (act != 1) LLME_REFUSE("gemm_tc: unknown activation %d", act);
+    if (act != 1 && act != 2) LLME_REFUSE("gemm_tc: unknown activation %d", act);
     if (!llme_gemm_tc_supports(M, N, K, ldx, ldw, ldo)) LLME_REFUSE("gemm_tc: M=%d N=%d K=%d ldx=%lld ldw=%lld ldo=%lld is not supported (K and operand strides must be multiples of 8)", M, N, K, ldx, ldw, ldo);
     if (((uintptr_t)x | (uintptr_t)w) % 16) LLME_REFUSE("gemm_tc: operands must be 16-byte aligned");
     TcArgs a{out, ldo, M, N, K, 0, 0, 0, act, p0, p1};

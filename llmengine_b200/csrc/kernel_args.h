@@ -87,6 +87,7 @@ typedef struct LlmeWindowPostArgs {
     int head_norm;
     int interleaved;                                         /* 1: the rotation pairs coordinate 2i with 2i + 1, not i with i + rot_dims / 2 */
     int in_f32;                                              /* 1: q_in, k_in and v_in are 32-bit whatever the type of q_out and the cache */
+    int unit_norm;                                           /* 1: behind the rotation every query and key head is divided by its own root mean square (eps inside the root) */
 } LlmeWindowPostArgs;
 
 /* Attention over such a cache: query i sees key j if j <= i and (i - j < window or j < keep_first). */
@@ -117,7 +118,10 @@ typedef struct LlmeMoeRouteArgs {
     int tokens, num_experts, top_k; float scale;
     int* experts; float* weights;                            /* [T, top_k] */
     int* offsets; int* order; int* counts;                   /* [E + 1], [T * top_k], [E] (zero between launches) */
-    int mode;                                                /* 0: sigmoid scores normalised over the chosen; 1: softmax over the chosen logits */
+    int mode;                                                /* 0: sigmoid scores normalised over the chosen; 1: softmax over the chosen logits; 2: softmax over all */
+    /* mode 2: the choice goes by softmax + correction (32-bit [E], or NULL); the E choices form `groups` equal groups of neighbours,
+     * of which the `keep` with the largest best member offer theirs; the weights are scale * softmax */
+    const float* correction; int groups, keep;
 } LlmeMoeRouteArgs;
 
 /* One product per expert over the rows routed to it. */
@@ -128,7 +132,7 @@ typedef struct LlmeGroupedArgs {
     const int* offsets; const int* order;
     int pairs, num_experts, top_k, n, k;                     /* pairs = tokens * top_k */
     int gather, scatter;                                     /* x row = order[r] / top_k; out row = order[r] */
-    int act;                                                 /* 1: w[e] = [gate | up], the row written is silu(gate) * up, n / 2 wide */
+    int act;                                                 /* 1: w[e] = [gate | up], the row written is silu(gate) * up, n / 2 wide; 2: max(product, 0)^2 */
 } LlmeGroupedArgs;
 
 /* Causal convolution per channel over the tokens of each request (csrc/recurrent.cu): y_t = bias + sum_j w[:, K-1-j] x_(t-j),
@@ -190,7 +194,25 @@ typedef struct LlmeGatedNormArgs {
     /* with `floor` [T, cols / group] every group of y is one value wider than `group`: the extra value d stands behind the
      * group's own, and the group is divided by max(|d|, floor) + den_eps before anything else */
     const float* floor; long long ld_floor; float den_eps;
+    int gate_f32;                                            /* 1: the gate is 32-bit whatever `dtype` is */
 } LlmeGatedNormArgs;
+
+/* The gated delta rule with a matrix state per head and request (csrc/delta_rule.cu): with unit queries and keys,
+ *   S <- a_t S (S is n x p),  u = b_t (v_t - S^T k_t),  S <- S + k_t u^T,  o_t = S^T q_t,
+ * b_t = sigmoid(write[t, h]), a_t = exp(-exp(a_log[h]) softplus(forget[t, h] + dt_bias[h])).  q and k come in `qk_groups` groups of n,
+ * head h reads group h / (heads / qk_groups).  The state lives in 32-bit in the request's slot, one column of S after the other
+ * ([heads, p, n]), and goes from step to step.  `rows`: the batch rows that a launch serves. */
+typedef struct LlmeDeltaArgs {
+    const float* q; const float* k; const float* v; long long ldq, ldk, ldv;     /* [T, qk_groups * n] twice, [T, heads * p] */
+    const float* write; const float* forget; long long ld_gates;                 /* [T, heads] each */
+    const float* dt_bias; const float* a_log;
+    float q_scale, unit_eps;
+    float* state; long long state_stride;                    /* slot s: [heads, p, n] at state + s * state_stride */
+    float* out; long long ldo;                               /* [T, heads * p] */
+    const int* cu_q_lens; const int* state_slots; const int* rows;
+    int n_rows, requests, tokens, heads, n, p, qk_groups;
+    float* unit; float* coef;                                /* workspace of portions: [T, 2 qk_groups n'], n' = n rounded up to fours; 40 values per block and head */
+} LlmeDeltaArgs;
 
 /* The gates of a matrix memory with exponential gating (csrc/recurrent.cu), per request and head over the request's tokens:
  * a_t = cap tanh(i_pre / cap), b_t = logsigmoid(cap tanh(f_pre / cap)) (cap 0: uncapped), M_t = max(b_t + M_(t-1), a_t) with M

@@ -1,6 +1,6 @@
 // The grouped product of a mixture of experts on the tensor cores (bfloat16 operands, 32-bit sums): one product per
 // expert over the (token, choice) pairs that were routed to it, rows gathered by token on the way in and scattered by
-// pair on the way out where asked, silu(gate) * up in the epilogue of the gate|up product.
+// pair on the way out where asked, silu(gate) * up (or max(., 0)^2 of a product without a gate) in the epilogue.
 //
 // A block owns a tile of BM pairs of ONE expert x BN output columns and walks K in steps of 32 through a cp.async
 // pipeline of two or three stages; its four warps share the tile by columns (mma.sync m16n8k16, fragments by ldmatrix).
@@ -66,10 +66,11 @@ template <> __device__ __forceinline__ void store2<bf16>(bf16* p, float a, float
     if (two) p[1] = __float2bfloat16_rn(b);
 }
 
-// BM x BN tile on WM x WNW warps, STAGES stages; ACT: the weight rows of a column are its gate row and, n_out further on, its up row.
-template <int BM, int BN, int WM, int WNW, int STAGES, bool ACT, typename O>
+// BM x BN tile on WM x WNW warps, STAGES stages; ACT 1: the weight rows of a column are its gate row and, n_out further on, its up row;
+// ACT 2: max(product, 0)^2 in the epilogue.
+template <int BM, int BN, int WM, int WNW, int STAGES, int ACT, typename O>
 __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedArgs a) {
-    constexpr int THREADS = 32 * WM * WNW, MT = BM / WM / 16, WN = BN / WNW, NT = WN / 8, HALVES = ACT ? 2 : 1;
+    constexpr int THREADS = 32 * WM * WNW, MT = BM / WM / 16, WN = BN / WNW, NT = WN / 8, HALVES = ACT == 1 ? 2 : 1;
     constexpr int A_STAGE = BM * LDS, B_STAGE = HALVES * BN * LDS;
     static_assert(MT >= 1 && NT >= 2 && NT % 2 == 0, "warp tiles are whole 16 x 16 pieces");
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -93,7 +94,7 @@ __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedAr
         s_dst[r] = r < rows ? (a.scatter ? pair : first + r) : -1;
     }
     __syncthreads();
-    const int n_out = ACT ? a.n / 2 : a.n;
+    const int n_out = ACT == 1 ? a.n / 2 : a.n;
     const int col0 = blockIdx.x * BN;
     const bf16* x = (const bf16*)a.x;
     const bf16* w = (const bf16*)a.w + (size_t)e * a.w_expert;
@@ -171,7 +172,11 @@ __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedAr
                 const int col = col0 + wn * WN + n * 8 + (lane & 3) * 2;
                 if (col >= n_out) continue;
                 float v0 = acc[0][m][n][half_rows * 2], v1 = acc[0][m][n][half_rows * 2 + 1];
-                if (ACT) {
+                if (ACT == 2) {
+                    v0 = relu2(v0);
+                    v1 = relu2(v1);
+                }
+                if (ACT == 1) {
                     // gate and up pass through bfloat16 first, as they do when the activation is a kernel of its own
                     const float g0 = __bfloat162float(__float2bfloat16_rn(v0)), g1 = __bfloat162float(__float2bfloat16_rn(v1));
                     const float u0 = __bfloat162float(__float2bfloat16_rn(acc[HALVES - 1][m][n][half_rows * 2]));
@@ -184,10 +189,10 @@ __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedAr
         }
 }
 
-template <int BM, int BN, int WM, int WNW, int STAGES, bool ACT, typename O>
+template <int BM, int BN, int WM, int WNW, int STAGES, int ACT, typename O>
 int launch(const LlmeGroupedArgs& a, cudaStream_t s) {
-    constexpr int SMEM = STAGES * (BM + (ACT ? 2 : 1) * BN) * LDS * (int)sizeof(bf16);
-    const int n_out = ACT ? a.n / 2 : a.n;
+    constexpr int SMEM = STAGES * (BM + (ACT == 1 ? 2 : 1) * BN) * LDS * (int)sizeof(bf16);
+    const int n_out = ACT == 1 ? a.n / 2 : a.n;
     const int most = a.num_experts < a.pairs ? a.num_experts : a.pairs;
     int tiles = (a.pairs + BM - 1) / BM + most;           // every expert may add one tile that is not full
     if (tiles > a.pairs) tiles = a.pairs;
@@ -208,7 +213,7 @@ int launch(const LlmeGroupedArgs& a, cudaStream_t s) {
     LLME_LAUNCH_STATUS();
 }
 
-template <bool ACT, typename O>
+template <int ACT, typename O>
 int dispatch(const LlmeGroupedArgs& a, cudaStream_t s) {
     // few rows per expert: tiles of 16 rows, so that little of a tile is padding and every weight is read once
     if ((long long)a.pairs < 32LL * a.num_experts) return launch<16, 128, 1, 4, 4, ACT, O>(a, s);     // three steps of weights in flight per block
@@ -222,12 +227,10 @@ LLME_API int llme_grouped_linear_tc(const LlmeGroupedArgs* args, int x_dtype, in
     if (a.pairs <= 0 || a.n <= 0) return 0;
     if (!a.x || !a.w || !a.out || !a.offsets || !a.order) LLME_REFUSE("grouped_linear_tc: null pointer");
     if (x_dtype != LLME_BF16 || w_dtype != LLME_BF16) LLME_REFUSE("grouped_linear_tc: bfloat16 operands only");
-    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || (a.act && a.n % 2)) LLME_REFUSE("grouped_linear_tc: bad size");
+    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || a.act < 0 || a.act > 2 || (a.act == 1 && a.n % 2)) LLME_REFUSE("grouped_linear_tc: bad size");
     if (a.k % 8 || a.ldx % 8 || a.ldw % 8 || a.w_expert % 8 || (((uintptr_t)a.x | (uintptr_t)a.w) & 15))
         LLME_REFUSE("grouped_linear_tc: rows must be whole 16-byte pieces");
-    if (a.act && out_dtype == LLME_BF16) return dispatch<true, bf16>(a, stream);
-    if (a.act && out_dtype == LLME_F32) return dispatch<true, float>(a, stream);
-    if (!a.act && out_dtype == LLME_BF16) return dispatch<false, bf16>(a, stream);
-    if (!a.act && out_dtype == LLME_F32) return dispatch<false, float>(a, stream);
+    if (out_dtype == LLME_BF16) return a.act == 1 ? dispatch<1, bf16>(a, stream) : a.act == 2 ? dispatch<2, bf16>(a, stream) : dispatch<0, bf16>(a, stream);
+    if (out_dtype == LLME_F32) return a.act == 1 ? dispatch<1, float>(a, stream) : a.act == 2 ? dispatch<2, float>(a, stream) : dispatch<0, float>(a, stream);
     LLME_REFUSE("grouped_linear_tc: unsupported output dtype %d", out_dtype);
 }

@@ -71,6 +71,50 @@ LLME_API int llme_xielu(const void* in, long long ld_in, void* out, long long ld
     LLME_LAUNCH_STATUS();
 }
 
+// ----------------------------------------------------------------------------- out = max(in, 0)^2
+template <typename T>
+__global__ void relu2_kernel(const T* __restrict__ in, long long ld_in, T* __restrict__ out, long long ld_out, int cols) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const T* i = in + (size_t)blockIdx.x * ld_in;
+    T* o = out + (size_t)blockIdx.x * ld_out;
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < cols; j += gridDim.y * blockDim.x) o[j] = from_f32<T>(relu2(to_f32(i[j])));
+}
+
+// bfloat16 rows of whole 16-byte pieces: eight values per thread and load
+__global__ void relu2_bf16x8_kernel(const __nv_bfloat16* __restrict__ in, long long ld_in, __nv_bfloat16* __restrict__ out, long long ld_out,
+                                    int cols) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const uint4* i = reinterpret_cast<const uint4*>(in + (size_t)blockIdx.x * ld_in);
+    uint4* o = reinterpret_cast<uint4*>(out + (size_t)blockIdx.x * ld_out);
+    for (int j = blockIdx.y * blockDim.x + threadIdx.x; j < cols / 8; j += gridDim.y * blockDim.x) {
+        uint4 v = i[j];
+        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const float2 f = __bfloat1622float2(h[e]);
+            h[e] = __floats2bfloat162_rn(relu2(f.x), relu2(f.y));
+        }
+        o[j] = v;
+    }
+}
+
+LLME_API int llme_relu2(const void* in, long long ld_in, void* out, long long ld_out, int dtype, int rows, int cols, cudaStream_t stream) {
+    if (rows <= 0 || cols <= 0) return 0;
+    if (!in || !out) LLME_REFUSE("relu2: null pointer");
+    const int threads = 128;
+    if (dtype == LLME_BF16 && cols % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+        llme_launch(relu2_bf16x8_kernel, grid_for(rows, cols / 8, threads), dim3(threads), 0, stream, (const __nv_bfloat16*)in, ld_in,
+                    (__nv_bfloat16*)out, ld_out, cols);
+        LLME_LAUNCH_STATUS();
+    }
+    if (dtype == LLME_F32) llme_launch(relu2_kernel<float>, grid_for(rows, cols, threads), dim3(threads), 0, stream, (const float*)in, ld_in, (float*)out, ld_out, cols);
+    else if (dtype == LLME_BF16) llme_launch(relu2_kernel<__nv_bfloat16>, grid_for(rows, cols, threads), dim3(threads), 0, stream, (const __nv_bfloat16*)in, ld_in, (__nv_bfloat16*)out, ld_out, cols);
+    else LLME_REFUSE("relu2: unsupported dtype %d", dtype);
+    LLME_LAUNCH_STATUS();
+}
+
 // ----------------------------------------------------------------------------- out = a * sigmoid(b) * scale
 // `group` > 1: b has one value for every `group` neighbouring columns of a (one gate per head).
 template <typename T>

@@ -194,6 +194,36 @@ __global__ void short_conv_state_kernel(LlmeShortConvArgs a) {
     }
 }
 
+// A step of single tokens: the thread that owns a channel of a request reads its K - 1 stored inputs and the present one, writes
+// the output (the sums in the order of the kernels above) and moves the stored inputs on, all in one launch.
+__global__ void short_conv_step_kernel(LlmeShortConvArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x, t = a.cu_q_lens[r], K = a.taps;
+    if (a.cu_q_lens[r + 1] == t) return;
+    float* st = a.state + (size_t)a.state_slots[r] * a.state_stride;
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < a.channels; c += gridDim.y * blockDim.x) {
+        float old[MAX_TAPS], w[MAX_TAPS];
+#pragma unroll
+        for (int m = 0; m < MAX_TAPS; ++m) {
+            old[m] = m < K - 1 ? st[(size_t)m * a.channels + c] : 0.0f;
+            w[m] = m < K ? a.w[(size_t)c * K + m] : 0.0f;
+        }
+        const float x = load_as_f32(a.x, a.x_dtype, (size_t)t * a.ldx + c);
+        float y = a.bias ? a.bias[c] : 0.0f;
+#pragma unroll
+        for (int m = 0; m < MAX_TAPS; ++m) {                     // the oldest input first, the present one last
+            if (m < K) y = fmaf(w[m], m == K - 1 ? x : old[m], y);
+        }
+        a.out[(size_t)t * a.ldo + c] = a.act == 1 ? silu32(y) : y;
+#pragma unroll
+        for (int m = 0; m + 1 < MAX_TAPS; ++m)
+            if (m < K - 1) st[(size_t)m * a.channels + c] = m == K - 2 ? x : old[m + 1];
+    }
+}
+
+// `update` 0: the outputs; 1: the states take the step's last inputs (after the outputs); 2: both at once, for a step in which no
+// request has more than one token.
 LLME_API int llme_short_conv(const LlmeShortConvArgs* args, int update, cudaStream_t stream) {
     const LlmeShortConvArgs& a = *args;
     if (a.tokens <= 0 || a.requests <= 0 || a.channels <= 0) return 0;
@@ -202,7 +232,9 @@ LLME_API int llme_short_conv(const LlmeShortConvArgs* args, int update, cudaStre
     if (a.x_dtype != LLME_F32 && a.x_dtype != LLME_BF16) LLME_REFUSE("short_conv: unsupported dtype %d", a.x_dtype);
     const int threads = 128;
     int pieces = (a.channels + threads - 1) / threads;
-    if (update) {
+    if (update == 2) {
+        llme_launch(short_conv_step_kernel, dim3(a.requests, pieces), dim3(threads), 0, stream, a);
+    } else if (update) {
         if (a.taps > 1) llme_launch(short_conv_state_kernel, dim3(a.requests, pieces), dim3(threads), 0, stream, a);
     } else {
         // a thread takes up to four channels of its token, more where the step has too few tokens to fill the GPU otherwise
@@ -763,7 +795,8 @@ LLME_API int llme_exp_gates(const LlmeExpGatesArgs* args, int max_len, cudaStrea
 // ----------------------------------------------------------------------------- grouped RMS norm with a silu gate
 __device__ __forceinline__ float gate32(float z, int act) { return act == 1 ? 1.0f / (1.0f + expf(-z)) : silu32(z); }
 
-template <typename T>
+// T: the type of the result, GT: of the gate (that of the result, or 32-bit).
+template <typename T, typename GT>
 __global__ void gated_norm_kernel(LlmeGatedNormArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -773,7 +806,7 @@ __global__ void gated_norm_kernel(LlmeGatedNormArgs a) {
     if (item >= (long long)a.tokens * groups) return;
     const int t = (int)(item / groups), gi = (int)(item - (long long)t * groups), c0 = gi * a.group;
     const float* y = a.y + (size_t)t * a.ldy + (a.floor ? c0 + gi : c0);       // with a floor every group of y is one value wider
-    const T* g = (const T*)a.gate + (size_t)t * a.ldg + c0;
+    const GT* g = (const GT*)a.gate + (size_t)t * a.ldg + c0;
     T* o = (T*)a.out + (size_t)t * a.ldo + c0;
     const float den = a.floor ? fmaxf(fabsf(y[a.group]), a.floor[(size_t)t * a.ld_floor + gi]) + a.den_eps : 1.0f;
     float ss = 0.0f;
@@ -796,7 +829,7 @@ __global__ void gated_norm_kernel(LlmeGatedNormArgs a) {
 // Groups of more than 128 and up to 1,024 columns: a block per (token, group), a thread for every eight columns (whole warps),
 // keeps its values in registers between the sum of squares and the output, so y and the gate are read once and all loads are on
 // their way together.
-template <typename T>
+template <typename T, typename GT>
 __global__ void __launch_bounds__(128) gated_norm_block_kernel(LlmeGatedNormArgs a) {
     __shared__ float red[32];
     pdl_launch_dependents();
@@ -804,7 +837,7 @@ __global__ void __launch_bounds__(128) gated_norm_block_kernel(LlmeGatedNormArgs
     const int groups = a.cols / a.group;
     const int t = blockIdx.x / groups, gi = blockIdx.x - t * groups, c0 = gi * a.group;
     const float* y = a.y + (size_t)t * a.ldy + (a.floor ? c0 + gi : c0);
-    const T* g = (const T*)a.gate + (size_t)t * a.ldg + c0;
+    const GT* g = (const GT*)a.gate + (size_t)t * a.ldg + c0;
     T* o = (T*)a.out + (size_t)t * a.ldo + c0;
     float u[8], gate[8], ss = 0.0f;
 #pragma unroll
@@ -843,14 +876,16 @@ LLME_API int llme_gated_norm(const LlmeGatedNormArgs* args, cudaStream_t stream)
     const long long items = (long long)a.tokens * (a.cols / a.group);
     if (a.group > 128 && a.group <= 1024 && items < (1LL << 31) && (a.dtype == LLME_F32 || a.dtype == LLME_BF16)) {
         const dim3 block(((a.group + 7) / 8 + 31) / 32 * 32);
-        if (a.dtype == LLME_F32) llme_launch(gated_norm_block_kernel<float>, dim3((unsigned)items), block, 0, stream, a);
-        else llme_launch(gated_norm_block_kernel<__nv_bfloat16>, dim3((unsigned)items), block, 0, stream, a);
+        if (a.dtype == LLME_F32) llme_launch(gated_norm_block_kernel<float, float>, dim3((unsigned)items), block, 0, stream, a);
+        else if (a.gate_f32) llme_launch(gated_norm_block_kernel<__nv_bfloat16, float>, dim3((unsigned)items), block, 0, stream, a);
+        else llme_launch(gated_norm_block_kernel<__nv_bfloat16, __nv_bfloat16>, dim3((unsigned)items), block, 0, stream, a);
         LLME_LAUNCH_STATUS();
     }
     const int warps = 4;
     const dim3 grid((unsigned)((items + warps - 1) / warps)), block(32 * warps);
-    if (a.dtype == LLME_F32) llme_launch(gated_norm_kernel<float>, grid, block, 0, stream, a);
-    else if (a.dtype == LLME_BF16) llme_launch(gated_norm_kernel<__nv_bfloat16>, grid, block, 0, stream, a);
+    if (a.dtype == LLME_F32) llme_launch(gated_norm_kernel<float, float>, grid, block, 0, stream, a);
+    else if (a.dtype == LLME_BF16 && a.gate_f32) llme_launch(gated_norm_kernel<__nv_bfloat16, float>, grid, block, 0, stream, a);
+    else if (a.dtype == LLME_BF16) llme_launch(gated_norm_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, stream, a);
     else LLME_REFUSE("gated_norm: unsupported dtype %d", a.dtype);
     LLME_LAUNCH_STATUS();
 }

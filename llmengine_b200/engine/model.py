@@ -8,7 +8,8 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from ..config.spec import ModelSpec
-from ..parts.base import (Part, Runtime, WeightSpec, build_part, emit_block, emit_embedding, emit_head, emit_norm)
+from ..parts.base import (Part, Runtime, WeightSpec, build_part, emit_block, emit_embedding, emit_embedding_again, emit_head,
+                          emit_norm)
 from .plan import ROWS_LOGITS, Plan
 
 
@@ -71,11 +72,18 @@ class Model:
         plan = Plan()
         x = emit_embedding(plan, self.embedding, self.spec.hidden_size)
         delta = None
-        for i, run in enumerate(self.order):
-            x, delta = emit_block(plan, self.blocks[run.layer], x, delta, caches[i])
+        for i in range(len(self.order)):
+            x, delta = self.emit_run(plan, i, x, delta, caches)
         h = emit_norm(plan, self.final_norm, x, delta=delta, rows=ROWS_LOGITS)
         emit_head(plan, self.head, h)
         return plan
+
+    def emit_run(self, plan: Plan, i: int, x: torch.Tensor, delta: Optional[torch.Tensor], caches):
+        """Run i of the order: what is added to the stream before it, and its block."""
+        run = self.order[i]
+        if run.add_embedding:
+            x, delta = emit_embedding_again(plan, self.embedding, x, delta)
+        return emit_block(plan, self.blocks[run.layer], x, delta, caches[i])
 
     def forward(self, batch, caches) -> Optional[torch.Tensor]:
         """Runs the batch's tokens through every run of the order and returns 32-bit logits

@@ -49,9 +49,22 @@ class Plan:
     def _add(self, kind: str, **a: Any) -> None:
         self.ops.append(Op(kind, a))
 
-    def embedding(self, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-        """out[t] = table[token_ids[t]] * scale as 32-bit, for the step's tokens."""
-        self._add("embedding", table=table, out=out, scale=float(scale))
+    def embedding(self, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0, accumulate: bool = False,
+                  delta: Optional[torch.Tensor] = None) -> None:
+        """out[t] = table[token_ids[t]] * scale as 32-bit, for the step's tokens; with `accumulate`, out[t] = (out[t] + delta[t])
+        + that row (`delta`, a pending contribution, may be None)."""
+        if delta is not None and not accumulate:
+            raise ValueError("embedding: a contribution is only added to a stream that exists")
+        self._add("embedding", table=table, out=out, scale=float(scale), accumulate=bool(accumulate), delta=delta)
+        if accumulate:
+            self.note_copy(out, None)
+
+    def layernorm(self, x: torch.Tensor, gain: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+                  delta: Optional[torch.Tensor] = None, rows: str = ROWS_TOKENS) -> None:
+        """x += delta (if given), out = (x - mean) / sqrt(mean of (x - mean)^2 + eps) * gain + bias; `rows` as for `rmsnorm`."""
+        self._add("layernorm", x=x, gain=gain, bias=bias, eps=float(eps), out=out, delta=delta, rows=rows)
+        if delta is not None:
+            self.note_copy(x, None)
 
     def rmsnorm(self, x: torch.Tensor, gain: torch.Tensor, eps: float, out: torch.Tensor,
                 delta: Optional[torch.Tensor] = None, rows: str = ROWS_TOKENS, gain2: Optional[torch.Tensor] = None,
@@ -105,7 +118,8 @@ class Plan:
     def linear_act(self, x: torch.Tensor, w: torch.Tensor, mid: torch.Tensor, out: torch.Tensor, act: str,
                    params: tuple = ()) -> None:
         """out = act(x w^T), elementwise; `mid` is the workspace of the form that runs product and activation as two
-        kernels.  Activations: "xielu" with params (a_pos, a_neg): z > 0: a_pos z^2 + z/2, else a_neg (exp(z) - 1 - z) + z/2."""
+        kernels.  Activations: "xielu" with params (a_pos, a_neg): z > 0: a_pos z^2 + z/2, else a_neg (exp(z) - 1 - z) + z/2;
+        "relu2": max(z, 0)^2."""
         self._add("linear_act", x=x, w=w, mid=mid, out=out, act=act, params=tuple(float(p) for p in params))
 
     def pointwise(self, kind: str, a: torch.Tensor, b: Optional[torch.Tensor], out: torch.Tensor, scale: float = 1.0,
@@ -160,7 +174,8 @@ class Plan:
     def window_attention(self, *, q_in, k_in, v_in, q_gain, k_gain, eps: float, inv_freq, rot_dims: int, amplitude: float,
                          q, out, cache, group: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int,
                          window: int, keep_first: int, scale: float, sink=None, scratch=None, q_bias=None, k_bias=None,
-                         v_bias=None, head_norm: bool = False, softcap: float = 0.0, interleaved: bool = False) -> None:
+                         v_bias=None, head_norm: bool = False, softcap: float = 0.0, interleaved: bool = False,
+                         unit_norm: bool = False, decode_scratch=None) -> None:
         """Grouped-query attention over a cache whose keys are `qk_dim` and whose values are `v_dim` wide, from the raw
         projections: q_in [T, H qk_dim] and, for a layer that stores, k_in [T, G qk_dim] and v_in [T, G v_dim] (column
         ranges of one product).  With gains, queries and keys are RMS-normed over the WHOLE projection (all heads at
@@ -174,40 +189,50 @@ class Plan:
         coordinates and the gains are [qk_dim], shared by the heads; `v_in` may be `k_in` itself (the values are then the
         keys as projected, before norm and rotation); `softcap` c > 0: s_ij <- c tanh(s_ij / c) behind the scale;
         `interleaved`: the rotation pairs coordinate 2i with 2i + 1 instead of i with i + rot_dims / 2.  The projections may
-        be 32-bit where everything else has the type of the products (they then come from a convolution, not a product)."""
+        be 32-bit where everything else has the type of the products (they then come from a convolution, not a product).
+        `unit_norm`: behind the rotation every query and key head is divided by its own sqrt(mean(x^2) + eps) (no gains).
+        `decode_scratch`: scratch memory of the kernels of ordinary grouped-query attention, which serve the record where its
+        mask and softmax are theirs (one width for keys and values, no kept first positions, no sink, no cap)."""
         self._add("window_attention", q_bias=q_bias, k_bias=k_bias, v_bias=v_bias, head_norm=bool(head_norm), q_in=q_in, k_in=k_in, v_in=v_in, q_gain=q_gain, k_gain=k_gain, eps=float(eps),
                   inv_freq=inv_freq, rot_dims=int(rot_dims), amplitude=float(amplitude), q=q, out=out, cache=cache, group=group,
                   num_heads=num_heads, num_kv_heads=num_kv_heads, qk_dim=qk_dim, v_dim=v_dim, window=int(window),
                   keep_first=int(keep_first), scale=float(scale), sink=sink, scratch=scratch, softcap=float(softcap),
-                  interleaved=bool(interleaved))
+                  interleaved=bool(interleaved), unit_norm=bool(unit_norm), decode_scratch=decode_scratch)
 
     def moe_route(self, *, logits, top_k: int, scale: float, experts, weights, offsets, order, counts,
-                  mode: str = "sigmoid") -> None:
+                  mode: str = "sigmoid", correction=None, groups: tuple = (1, 1)) -> None:
         """Routing of every token of the step from its router `logits` [T, E] (32-bit, any row stride): s = sigmoid(logits);
         C = the `top_k` experts of largest s (`experts` [T, top_k] int32, best first); `weights` [T, top_k]: w_e = scale *
         s_e / (sum over C of s + 1e-20).  `mode` "softmax_chosen": C = the experts of largest logits and w_e = scale *
-        exp(z_e) / sum over C of exp(z).  The (token, choice) pairs are then listed expert by expert:
+        exp(z_e) / sum over C of exp(z).  `mode` "softmax": s = softmax(z) over all E; the choice goes by s (+ `correction` [E],
+        32-bit), C = the `top_k` largest among the members of the groups[1] groups with the largest best member (the E choices
+        form groups[0] equal groups of neighbours); w_e = scale * s_e.  The (token, choice) pairs are then listed expert by expert:
         `offsets` [E + 1] int32 with the pairs of expert e at order[offsets[e] : offsets[e + 1]], a pair being
         token * top_k + choice.  `counts` [E] int32 is scratch that is zero between launches."""
-        if mode not in ("sigmoid", "softmax_chosen"):
+        if mode not in ("sigmoid", "softmax_chosen", "softmax"):
             raise ValueError(f"moe_route: unknown mode {mode!r}")
+        if mode != "softmax" and (correction is not None or tuple(groups) != (1, 1)):
+            raise ValueError("moe_route: corrections and groups belong to the mode 'softmax'")
         self._add("moe_route", logits=logits, top_k=int(top_k), scale=float(scale), experts=experts, weights=weights,
-                  offsets=offsets, order=order, counts=counts, mode=mode)
+                  offsets=offsets, order=order, counts=counts, mode=mode, correction=correction, groups=(int(groups[0]), int(groups[1])))
 
     def grouped_linear(self, *, x, w, out, offsets, order, top_k: int, gather: bool, scatter: bool, mid=None,
                        act: Optional[str] = None) -> None:
         """One product per expert over the rows that were routed to it: for place r of expert e's range of `order`,
         out_row = w[e] x_row, with x_row = x[order[r] // top_k] if `gather` (the token's row) else x[r], and written
-        to out[order[r]] if `scatter` (the pair's row) else out[r].  w is [E, n, k].  With `act` ("silu"), w[e] is
-        [gate | up] by rows and the row written is silu(gate) * up, half as wide (`mid` [pairs, n]: workspace of the
-        form that runs product and activation apart)."""
+        to out[order[r]] if `scatter` (the pair's row) else out[r].  w is [E, n, k].  With `act` "silu", w[e] is
+        [gate | up] by rows and the row written is silu(gate) * up, half as wide; with `act` "relu2" the row written is
+        max(product, 0)^2 (`mid` [pairs, n]: workspace of the form that runs product and activation apart)."""
         self._add("grouped_linear", x=x, w=w, out=out, offsets=offsets, order=order, top_k=int(top_k), gather=bool(gather),
                   scatter=bool(scatter), mid=mid, act=act)
 
-    def moe_combine(self, *, y, weights, base, out, base_gate=None) -> None:
+    def moe_combine(self, *, y, weights, base, out, base_gate=None, experts=None, identity=None, first_identity: int = 0) -> None:
         """out[t] = base[t] (if given) + sum_k weights[t, k] * y[t * top_k + k], the choices added in their order,
-        in 32-bit.  With `base_gate` [T, 1] (32-bit, any row stride) base[t] is first multiplied by sigmoid(base_gate[t])."""
-        self._add("moe_combine", y=y, weights=weights, base=base, out=out, base_gate=base_gate)
+        in 32-bit.  With `base_gate` [T, 1] (32-bit, any row stride) base[t] is first multiplied by sigmoid(base_gate[t]).
+        With `identity` [T, D] and `experts` [T, top_k]: a choice whose expert is `first_identity` or a later one stands for
+        identity[t] instead of a row of y."""
+        self._add("moe_combine", y=y, weights=weights, base=base, out=out, base_gate=base_gate, experts=experts, identity=identity,
+                  first_identity=int(first_identity))
 
     def short_conv(self, *, x, w, bias, state, out, act: Optional[str] = "silu") -> None:
         """Causal convolution per channel over each request's tokens: y_t = bias + sum_j w[:, K-1-j] x_(t-j) with zeros
@@ -234,6 +259,18 @@ class Plan:
         self._add("recurrence", q=q, k=k, v=v, state=state, out=out, heads=int(heads), n=int(n), p=int(p), qk_groups=int(qk_groups),
                   decay=decay, dt=dt, dt_bias=dt_bias, a_log=a_log, skip=skip, scratch=scratch, keep=keep, take=take,
                   unit_column=bool(unit_column))
+
+    def delta_rule(self, *, q, k, v, write, forget, dt_bias, a_log, q_scale: float, unit_eps: float, state, out, heads: int, n: int,
+                   p: int, qk_groups: int, unit, coef) -> None:
+        """The gated delta rule, per request and head over the request's tokens in order, all 32-bit.  q, k [T, qk_groups * n] are
+        first made unit vectors per group, x / sqrt(sum(x^2) + unit_eps), q then times q_scale; head h reads group h // (H / qk_groups).
+        b_t = sigmoid(write[t, h]); a_t = exp(-exp(a_log_h) softplus(forget[t, h] + dt_bias_h)); S <- a_t S (S is n x p);
+        u = b_t (v_t - S^T k_t); S <- S + k_t u^T; out[t, h] = S^T q_t.  v and out are [T, H p]; `write` and `forget` [T, H] share
+        their row stride.  `state` [slots, H, p, n] goes from step to step.  `unit` and `coef`: workspace of the form that takes a
+        portion's tokens four at a time (Runtime.delta_workspace)."""
+        self._add("delta_rule", q=q, k=k, v=v, write=write, forget=forget, dt_bias=dt_bias, a_log=a_log, q_scale=float(q_scale),
+                  unit_eps=float(unit_eps), state=state, out=out, heads=int(heads), n=int(n), p=int(p), qk_groups=int(qk_groups),
+                  unit=unit, coef=coef)
 
     def gated_norm(self, *, y, gate, weight, out, group: int, gate_first: bool, eps: float, scale: float = 1.0,
                    gate_act: str = "silu", floor=None, den_eps: float = 0.0) -> None:

@@ -70,10 +70,10 @@ enum LlmeOpKind {
     LLME_OP_ATTENTION, LLME_OP_CALL, LLME_OP_LINEAR_ACT, LLME_OP_POINTWISE, LLME_OP_BATCHED_LINEAR, LLME_OP_RESIDUAL_ADD,
     LLME_OP_LATENT_ATTENTION, LLME_OP_TOKEN_SIDE, LLME_OP_POSTNORM, LLME_OP_WINDOW_ATTENTION, LLME_OP_MOE_ROUTE,
     LLME_OP_GROUPED_LINEAR, LLME_OP_MOE_COMBINE, LLME_OP_SHORT_CONV, LLME_OP_ROTATE, LLME_OP_RECURRENCE, LLME_OP_GATED_NORM,
-    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES
+    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES, LLME_OP_LAYERNORM, LLME_OP_DELTA_RULE
 };
 
-enum { LLME_ACT_XIELU = 1 };
+enum { LLME_ACT_XIELU = 1, LLME_ACT_RELU2 = 2 };   /* 2: max(z, 0)^2 */
 /* activations of a (gate, up) pair: g sigmoid(g) u; with p0 = limit, p1 = slope: g' = min(g, limit),
  * u' = clamp(u, -limit, limit), g' sigmoid(slope g') (u' + 1) */
 enum { LLME_GATE_SILU = 0, LLME_GATE_CLAMPED_SWISH = 1, LLME_GATE_GELU_TANH = 2 };   /* 2: gelu(g) u, the tanh form of gelu */
@@ -85,6 +85,8 @@ typedef struct LlmeEmbeddingOp {
     const void* table; int table_dtype, vocab, hidden;
     float* out;                /* [T, hidden] */
     float scale;               /* every row times this constant, in 32-bit (1: none) */
+    int accumulate;            /* 1: out = (out + delta) + row: the embedding output added to a stream that exists */
+    const float* delta;        /* with accumulate: a contribution still to be added, or NULL */
 } LlmeEmbeddingOp;
 
 typedef struct LlmeRmsNormOp {
@@ -96,6 +98,16 @@ typedef struct LlmeRmsNormOp {
     int rows;                  /* LLME_ROWS_TOKENS: every row; LLME_ROWS_LOGITS: the step's logit rows only */
     const void* gain2; void* out2;   /* a second gain and place for the same normed rows (the types of the first), or NULL */
 } LlmeRmsNormOp;
+
+/* x += delta (if given); out = (x - mean) / sqrt(mean of (x - mean)^2 + eps) * gain + bias. */
+typedef struct LlmeLayerNormOp {
+    float* x;                  /* [T, size] the residual stream, updated in place when delta is given */
+    const float* delta;
+    const void* gain; const void* bias; int param_dtype;
+    void* out; int out_dtype;
+    int size; float eps;
+    int rows;                  /* LLME_ROWS_TOKENS or LLME_ROWS_LOGITS */
+} LlmeLayerNormOp;
 
 typedef struct LlmeLinearOp {
     const void* x; long long ldx; int x_dtype;
@@ -231,6 +243,10 @@ typedef struct LlmeWindowAttentionOp {
     float softcap;                                           /* c > 0: a score s becomes c tanh(s / c) behind the scale */
     int interleaved;                                         /* 1: the rotation pairs coordinate 2i with 2i + 1 */
     int in_f32;                                              /* 1: q_in, k_in, v_in are 32-bit whatever `dtype` is (they come from a convolution) */
+    int unit_norm;                                           /* 1: behind the rotation every query and key head is divided by its own root mean square */
+    /* scratch of the kernels of ordinary grouped-query attention, which serve the record where its mask and softmax are theirs
+     * (dk = dv, keep_first 0, no sink, no cap); NULL: they do not */
+    float* decode_scratch; long long decode_scratch_floats; long long cache_pages;
 } LlmeWindowAttentionOp;
 
 /* Routing of a mixture of experts: s = sigmoid(logits), the top_k largest, w_e = scale * s_e / (sum of the chosen s + 1e-20);
@@ -238,7 +254,9 @@ typedef struct LlmeWindowAttentionOp {
 typedef struct LlmeMoeRouteOp {
     const float* logits; long long ld; int num_experts, top_k; float scale;
     int* experts; float* weights; int* offsets; int* order; int* counts;
-    int mode;                  /* 0: as above; 1: the largest logits chosen, w_e = scale * softmax over the chosen logits alone */
+    int mode;                  /* 0: as above; 1: the largest logits chosen, w_e = scale * softmax over the chosen logits alone; 2: s = softmax over all */
+    const float* correction;   /* mode 2: added to s for the choice alone ([E], or NULL); the choices form `groups` equal groups of */
+    int groups, keep;          /* neighbours, and the members of the `keep` groups with the largest best member can be chosen; w_e = scale s_e */
 } LlmeMoeRouteOp;
 
 /* One product per expert over the pairs routed to it. */
@@ -248,13 +266,15 @@ typedef struct LlmeGroupedLinearOp {
     void* out; long long ldo; int out_dtype;
     void* mid; long long ld_mid;                              /* [pairs, n]: workspace of the unfused activation, or NULL */
     const int* offsets; const int* order;
-    int num_experts, top_k, n, k, gather, scatter, act;       /* act 1: w[e] = [gate | up], out = silu(gate) * up */
+    int num_experts, top_k, n, k, gather, scatter, act;       /* act 1: w[e] = [gate | up], out = silu(gate) * up; 2: out = max(product, 0)^2 */
 } LlmeGroupedLinearOp;
 
 /* out[t] = base[t] (times sigmoid(base_gate[t * ld_gate]) where base_gate is given) + sum_k weights[t, k] y[t top_k + k]. */
 typedef struct LlmeMoeCombineOp {
     const float* y; long long ldy; const float* weights; const float* base; float* out; int top_k, size;
     const float* base_gate; long long ld_gate;
+    /* with `same` [T, size]: a choice whose expert is first_identity or a later one stands for same[t] instead of a row of y */
+    const int* experts; const void* same; long long ld_same; int same_dtype, first_identity;
 } LlmeMoeCombineOp;
 
 /* Causal convolution per channel over each request's tokens, y_t = bias + sum_j w[:, K-1-j] x_(t-j), then silu (act 1);
@@ -307,7 +327,22 @@ typedef struct LlmeGatedNormOp {
     /* with `floor` [T, cols / group] every group of y is one value wider: the extra value d stands behind the group's own, and
      * the group is divided by max(|d|, floor) + den_eps before anything else */
     const float* floor; long long ld_floor; float den_eps;
+    int gate_f32;                                            /* 1: the gate is 32-bit whatever `dtype` is */
 } LlmeGatedNormOp;
+
+/* The gated delta rule per request and head (csrc/delta_rule.cu): unit queries (times q_scale) and keys per group,
+ * S <- a_t S, u = b_t (v_t - S^T k_t), S <- S + k_t u^T, out_t = S^T q_t, with b_t = sigmoid(write[t, h]) and a_t =
+ * exp(-exp(a_log[h]) softplus(forget[t, h] + dt_bias[h])).  State [heads, p, n] 32-bit per slot, zero when the request starts. */
+typedef struct LlmeDeltaRuleOp {
+    const float* q; const float* k; const float* v; long long ldq, ldk, ldv; int qk_groups;
+    const float* write; const float* forget; long long ld_gates;
+    const float* dt_bias; const float* a_log;
+    float q_scale, unit_eps;
+    float* state; long long state_stride;
+    float* out; long long ldo;
+    int heads, n, p;
+    float* unit; float* coef; long long unit_floats, coef_floats;   /* workspace of portions */
+} LlmeDeltaRuleOp;
 
 /* out = x / sqrt(mean(x^2) + eps) * gain over the rows of x: a norm on (a column range of) a product. */
 typedef struct LlmeRowNormOp {
@@ -342,7 +377,7 @@ void llme_executor_destroy(LlmeExecutor*);
  * "postnorm", "gated_act", "gemm_skinny_gated", "gemm_tc_gated", "window_post", "window_attention_plain", per pair of
  * key and value sizes "window_attention_tc/<dk>x<dv>", "moe_route", "grouped_linear", "grouped_linear_tc", "moe_combine";
  * "short_conv", "rotate", "recurrence", "gated_norm", "row_norm", "exp_gates", "sigmoid_mul_grouped", "residual_add_scaled",
- * "moe_combine_gated". */
+ * "layernorm", "embedding_add", "relu2", "delta_step", "delta_portions". */
 int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
 /* Which implementation an operation takes.  Operations and their variants:
  *   "linear":            "auto" | "tcgen05" | "cublas" | "plain"   (bfloat16 products of 128 tokens or more / all)
@@ -350,6 +385,7 @@ int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
  *   "linear_swiglu":     "fused" | "unfused"
  *   "attention.portion": "tcgen05" | "mma" | "plain"
  *   "attention.decode":  "fused" | "split" | "plain"
+ *   "delta_rule":        "blocks" | "tokens"                        (portions: four tokens at a time / one after the other)
  *   "*":                 "fast" | "plain"                           (all of the above at once)
  * Returns 0, or -1 for an unknown operation or variant. */
 int llme_executor_choose(LlmeExecutor*, const char* op, const char* variant);
@@ -433,6 +469,8 @@ public:
     int add(const LlmeGatedNormOp& r) { return add(LLME_OP_GATED_NORM, &r, sizeof r); }
     int add(const LlmeRowNormOp& r) { return add(LLME_OP_ROW_NORM, &r, sizeof r); }
     int add(const LlmeExpGatesOp& r) { return add(LLME_OP_EXP_GATES, &r, sizeof r); }
+    int add(const LlmeLayerNormOp& r) { return add(LLME_OP_LAYERNORM, &r, sizeof r); }
+    int add(const LlmeDeltaRuleOp& r) { return add(LLME_OP_DELTA_RULE, &r, sizeof r); }
     /* One step through the whole plan; throws with the failing record's message. */
     void run(const LlmeStep& step, cudaStream_t stream) {
         if (llme_plan_run(h_, &step, 0, -1, stream)) throw std::runtime_error(ex_.error());

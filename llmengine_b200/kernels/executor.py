@@ -14,10 +14,11 @@ ROWS = {"tokens": 0, "logits": 1}
 (OP_EMBEDDING, OP_RMSNORM, OP_LINEAR, OP_LINEAR_SWIGLU, OP_QKV_POST, OP_ATTEND, OP_ATTENTION, OP_CALL, OP_LINEAR_ACT,
  OP_POINTWISE, OP_BATCHED_LINEAR, OP_RESIDUAL_ADD, OP_LATENT_ATTENTION, OP_TOKEN_SIDE, OP_POSTNORM, OP_WINDOW_ATTENTION,
  OP_MOE_ROUTE, OP_GROUPED_LINEAR, OP_MOE_COMBINE, OP_SHORT_CONV, OP_ROTATE, OP_RECURRENCE, OP_GATED_NORM, OP_ROW_NORM,
- OP_EXP_GATES) = range(1, 26)
+ OP_EXP_GATES, OP_LAYERNORM, OP_DELTA_RULE) = range(1, 28)
 GATES = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}
-ROUTING = {"sigmoid": 0, "softmax_chosen": 1}
-ACTIVATIONS = {"xielu": 1}
+ROUTING = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
+ACTIVATIONS = {"xielu": 1, "relu2": 2}
+EXPERT_ACTIVATIONS = {None: 0, "silu": 1, "relu2": 2}
 POINTWISE = {"sigmoid_mul": 1}
 
 
@@ -54,7 +55,12 @@ CallFn = CFUNCTYPE(c_int, c_void_p, POINTER(Step), c_void_p)
 
 class EmbeddingOp(Structure):
     _fields_ = [("table", c_void_p), ("table_dtype", c_int), ("vocab", c_int), ("hidden", c_int), ("out", c_void_p),
-                ("scale", c_float)]
+                ("scale", c_float), ("accumulate", c_int), ("delta", c_void_p)]
+
+
+class LayerNormOp(Structure):
+    _fields_ = [("x", c_void_p), ("delta", c_void_p), ("gain", c_void_p), ("bias", c_void_p), ("param_dtype", c_int), ("out", c_void_p),
+                ("out_dtype", c_int), ("size", c_int), ("eps", c_float), ("rows", c_int)]
 
 
 class RmsNormOp(Structure):
@@ -145,13 +151,14 @@ class WindowAttentionOp(Structure):
                 ("cache", c_void_p), ("group", c_int), ("nh", c_int), ("nkv", c_int), ("dk", c_int), ("dv", c_int),
                 ("window", c_int), ("keep_first", c_int), ("scale", c_float), ("sink", c_void_p), ("scratch", c_void_p),
                 ("scratch_floats", c_longlong), ("q_bias", c_void_p), ("k_bias", c_void_p), ("v_bias", c_void_p),
-                ("head_norm", c_int), ("softcap", c_float), ("interleaved", c_int), ("in_f32", c_int)]
+                ("head_norm", c_int), ("softcap", c_float), ("interleaved", c_int), ("in_f32", c_int), ("unit_norm", c_int),
+                ("decode_scratch", c_void_p), ("decode_scratch_floats", c_longlong), ("cache_pages", c_longlong)]
 
 
 class MoeRouteOp(Structure):
     _fields_ = [("logits", c_void_p), ("ld", c_longlong), ("num_experts", c_int), ("top_k", c_int), ("scale", c_float),
                 ("experts", c_void_p), ("weights", c_void_p), ("offsets", c_void_p), ("order", c_void_p), ("counts", c_void_p),
-                ("mode", c_int)]
+                ("mode", c_int), ("correction", c_void_p), ("groups", c_int), ("keep", c_int)]
 
 
 class GroupedLinearOp(Structure):
@@ -163,7 +170,8 @@ class GroupedLinearOp(Structure):
 
 class MoeCombineOp(Structure):
     _fields_ = [("y", c_void_p), ("ldy", c_longlong), ("weights", c_void_p), ("base", c_void_p), ("out", c_void_p),
-                ("top_k", c_int), ("size", c_int), ("base_gate", c_void_p), ("ld_gate", c_longlong)]
+                ("top_k", c_int), ("size", c_int), ("base_gate", c_void_p), ("ld_gate", c_longlong), ("experts", c_void_p),
+                ("same", c_void_p), ("ld_same", c_longlong), ("same_dtype", c_int), ("first_identity", c_int)]
 
 
 class ShortConvOp(Structure):
@@ -190,7 +198,15 @@ class GatedNormOp(Structure):
     _fields_ = [("y", c_void_p), ("ldy", c_longlong), ("gate", c_void_p), ("ldg", c_longlong), ("weight", c_void_p),
                 ("out", c_void_p), ("ldo", c_longlong), ("dtype", c_int), ("cols", c_int), ("group", c_int),
                 ("gate_first", c_int), ("eps", c_float), ("scale", c_float), ("gate_act", c_int), ("floor", c_void_p),
-                ("ld_floor", c_longlong), ("den_eps", c_float)]
+                ("ld_floor", c_longlong), ("den_eps", c_float), ("gate_f32", c_int)]
+
+
+class DeltaRuleOp(Structure):
+    _fields_ = [("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("ldq", c_longlong), ("ldk", c_longlong), ("ldv", c_longlong),
+                ("qk_groups", c_int), ("write", c_void_p), ("forget", c_void_p), ("ld_gates", c_longlong), ("dt_bias", c_void_p),
+                ("a_log", c_void_p), ("q_scale", c_float), ("unit_eps", c_float), ("state", c_void_p), ("state_stride", c_longlong),
+                ("out", c_void_p), ("ldo", c_longlong), ("heads", c_int), ("n", c_int), ("p", c_int), ("unit", c_void_p), ("coef", c_void_p),
+                ("unit_floats", c_longlong), ("coef_floats", c_longlong)]
 
 
 class RowNormOp(Structure):
@@ -278,7 +294,17 @@ def records(op, keep: List[Any]):
     if k == "embedding":
         t, out = a["table"], a["out"]
         assert out.dtype == torch.float32 and t.is_contiguous() and out.is_contiguous()
-        return OP_EMBEDDING, EmbeddingOp(t.data_ptr(), code(t.dtype), t.shape[0], t.shape[1], out.data_ptr(), float(a.get("scale", 1.0)))
+        d = a.get("delta")
+        assert d is None or (d.dtype == torch.float32 and d.is_contiguous() and d.shape == out.shape)
+        return OP_EMBEDDING, EmbeddingOp(t.data_ptr(), code(t.dtype), t.shape[0], t.shape[1], out.data_ptr(), float(a.get("scale", 1.0)),
+                                         1 if a.get("accumulate") else 0, ptr(d))
+    if k == "layernorm":
+        x, d, g, b, out = a["x"], a["delta"], a["gain"], a["bias"], a["out"]
+        assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[1] == x.shape[1]
+        assert d is None or (d.dtype == torch.float32 and d.is_contiguous() and d.shape == x.shape)
+        assert g.dtype == b.dtype and g.is_contiguous() and b.is_contiguous() and g.numel() == b.numel() == x.shape[1]
+        return OP_LAYERNORM, LayerNormOp(x.data_ptr(), ptr(d), g.data_ptr(), b.data_ptr(), code(g.dtype), out.data_ptr(), code(out.dtype),
+                                         x.shape[1], a["eps"], ROWS[a["rows"]])
     if k == "rmsnorm":
         x, d, g, out = a["x"], a["delta"], a["gain"], a["out"]
         assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and (d is None or d.is_contiguous())
@@ -400,7 +426,8 @@ def records(op, keep: List[Any]):
             q.data_ptr(), out.data_ptr(), cache.data_ptr(), a["group"], H, G, dk, dv, a["window"], a["keep_first"], a["scale"],
             ptr(a["sink"]), ptr(a.get("scratch")), a["scratch"].numel() if a.get("scratch") is not None else 0,
             ptr(a.get("q_bias")), ptr(a.get("k_bias")), ptr(a.get("v_bias")), 1 if a.get("head_norm") else 0,
-            float(a.get("softcap", 0.0)), 1 if a.get("interleaved") else 0, 1 if wide else 0)
+            float(a.get("softcap", 0.0)), 1 if a.get("interleaved") else 0, 1 if wide else 0, 1 if a.get("unit_norm") else 0,
+            ptr(a.get("decode_scratch")), a["decode_scratch"].numel() if a.get("decode_scratch") is not None else 0, cache.shape[0])
     if k == "moe_route":
         z, ex_, wt, off, order, counts = a["logits"], a["experts"], a["weights"], a["offsets"], a["order"], a["counts"]
         assert z.dtype == wt.dtype == torch.float32 and z.stride(1) == 1 and ex_.is_contiguous() and wt.is_contiguous()
@@ -408,12 +435,13 @@ def records(op, keep: List[Any]):
         E, top = z.shape[1], a["top_k"]
         assert ex_.shape[1] == wt.shape[1] == top and off.numel() == E + 1 and counts.numel() == E and order.numel() >= ex_.shape[0] * top
         return OP_MOE_ROUTE, MoeRouteOp(z.data_ptr(), z.stride(0), E, top, a["scale"], ex_.data_ptr(), wt.data_ptr(), off.data_ptr(),
-                                        order.data_ptr(), counts.data_ptr(), ROUTING[a.get("mode", "sigmoid")])
+                                        order.data_ptr(), counts.data_ptr(), ROUTING[a.get("mode", "sigmoid")], ptr(a.get("correction")),
+                                        a.get("groups", (1, 1))[0], a.get("groups", (1, 1))[1])
     if k == "grouped_linear":
         x, w, out, mid = a["x"], a["w"], a["out"], a["mid"]
-        act = 1 if a["act"] else 0
-        assert a["act"] in (None, "silu") and w.dim() == 3 and w.is_contiguous() and x.stride(1) == 1 and out.stride(1) == 1
-        assert w.shape[2] == x.shape[1] and out.shape[1] == (w.shape[1] // 2 if act else w.shape[1]) and x.dtype == w.dtype
+        act = EXPERT_ACTIVATIONS[a["act"]]
+        assert w.dim() == 3 and w.is_contiguous() and x.stride(1) == 1 and out.stride(1) == 1
+        assert w.shape[2] == x.shape[1] and out.shape[1] == (w.shape[1] // 2 if act == 1 else w.shape[1]) and x.dtype == w.dtype
         return OP_GROUPED_LINEAR, GroupedLinearOp(
             x.data_ptr(), x.stride(0), code(x.dtype), w.data_ptr(), w.stride(1), w.stride(0), code(w.dtype), out.data_ptr(), out.stride(0),
             code(out.dtype), ptr(mid), mid.stride(0) if mid is not None else 0, a["offsets"].data_ptr(), a["order"].data_ptr(), w.shape[0],
@@ -422,10 +450,15 @@ def records(op, keep: List[Any]):
         y, wt, base, out = a["y"], a["weights"], a["base"], a["out"]
         assert y.dtype == wt.dtype == out.dtype == torch.float32 and y.stride(1) == 1 and wt.is_contiguous() and out.is_contiguous()
         assert base is None or (base.dtype == torch.float32 and base.is_contiguous() and base.shape[1] == out.shape[1])
-        bg = a.get("base_gate")
+        bg, experts, same = a.get("base_gate"), a.get("experts"), a.get("identity")
+        assert (experts is None) == (same is None)
+        assert same is None or (same.stride(1) == 1 and same.shape[1] == out.shape[1] and experts.dtype == torch.int32 and experts.is_contiguous()
+                                and experts.shape == wt.shape)
         assert bg is None or (base is not None and bg.dtype == torch.float32 and bg.dim() == 2 and bg.shape[1] == 1)
         return OP_MOE_COMBINE, MoeCombineOp(y.data_ptr(), y.stride(0), wt.data_ptr(), ptr(base), out.data_ptr(), wt.shape[1], out.shape[1],
-                                            ptr(bg), bg.stride(0) if bg is not None else 0)
+                                            ptr(bg), bg.stride(0) if bg is not None else 0, ptr(experts), ptr(same),
+                                            same.stride(0) if same is not None else 0, code(same.dtype) if same is not None else 0,
+                                            int(a.get("first_identity", 0)))
     if k == "short_conv":
         x, w, b, st, out = a["x"], a["w"], a["bias"], a["state"], a["out"]
         C, K = w.shape
@@ -470,7 +503,7 @@ def records(op, keep: List[Any]):
     if k == "gated_norm":
         y, g, w, out = a["y"], a["gate"], a["weight"], a["out"]
         cols, floor = out.shape[1], a.get("floor")
-        assert y.dtype == torch.float32 and y.stride(1) == g.stride(1) == out.stride(1) == 1 and g.dtype == out.dtype
+        assert y.dtype == torch.float32 and y.stride(1) == g.stride(1) == out.stride(1) == 1 and g.dtype in (out.dtype, torch.float32)
         assert g.shape[1] == cols and cols % a["group"] == 0 and _f32(w, cols)
         groups = cols // a["group"]
         assert y.shape[1] == (cols + groups if floor is not None else cols)
@@ -478,7 +511,20 @@ def records(op, keep: List[Any]):
         return OP_GATED_NORM, GatedNormOp(y.data_ptr(), y.stride(0), g.data_ptr(), g.stride(0), ptr(w), out.data_ptr(), out.stride(0),
                                           code(out.dtype), cols, a["group"], 1 if a["gate_first"] else 0, a["eps"], a["scale"],
                                           1 if a.get("gate_act", "silu") == "sigmoid" else 0, ptr(floor),
-                                          floor.stride(0) if floor is not None else 0, float(a.get("den_eps", 0.0)))
+                                          floor.stride(0) if floor is not None else 0, float(a.get("den_eps", 0.0)),
+                                          1 if g.dtype == torch.float32 else 0)
+    if k == "delta_rule":
+        q, kk, v, wr, fg, st, out, unit, coef = (a[n] for n in ("q", "k", "v", "write", "forget", "state", "out", "unit", "coef"))
+        H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]
+        for t in (q, kk, v, wr, fg, out, unit):
+            assert t.dtype == torch.float32 and t.stride(1) == 1
+        assert q.shape[1] == kk.shape[1] == G * n and v.shape[1] == out.shape[1] == H * p and wr.shape[1] == fg.shape[1] == H and H % G == 0
+        assert wr.stride(0) == fg.stride(0) and _f32(a["dt_bias"], H) and _f32(a["a_log"], H) and _state(st) and tuple(st.shape[1:]) == (H, p, n)
+        assert unit.is_contiguous() and _f32(coef)
+        return OP_DELTA_RULE, DeltaRuleOp(q.data_ptr(), kk.data_ptr(), v.data_ptr(), q.stride(0), kk.stride(0), v.stride(0), G, wr.data_ptr(),
+                                          fg.data_ptr(), wr.stride(0), a["dt_bias"].data_ptr(), a["a_log"].data_ptr(), a["q_scale"],
+                                          a["unit_eps"], st.data_ptr(), st.stride(0), out.data_ptr(), out.stride(0), H, n, p, unit.data_ptr(),
+                                          coef.data_ptr(), unit.numel(), coef.numel())
     if k == "row_norm":
         x, g, out = a["x"], a["gain"], a["out"]
         assert x.stride(1) == 1 and out.stride(1) == 1 and x.shape[1] == out.shape[1] == g.numel() and g.is_contiguous()

@@ -192,20 +192,21 @@ class CudaOps:
 
     _ENTRY_POINTS = {
         "elementwise": {"embedding": "llme_embedding", "rmsnorm": "llme_rmsnorm", "qkv_post": "llme_qkv_post",
-                        "swiglu": "llme_swiglu", "embedding_scaled": "llme_embedding_scaled", "rmsnorm_pair": "llme_rmsnorm_pair"},
+                        "swiglu": "llme_swiglu", "embedding_scaled": "llme_embedding_scaled", "rmsnorm_pair": "llme_rmsnorm_pair",
+                        "embedding_add": "llme_embedding_add", "layernorm": "llme_layernorm"},
         "gemm_f32": {"gemm_f32": "llme_gemm_nt_f32", "gemm_f32_batched": "llme_gemm_nt_f32_batched"},
         "pointwise": {"xielu": "llme_xielu", "sigmoid_mul": "llme_sigmoid_mul", "residual_add": "llme_residual_add",
                       "gelu_gather_mul": "llme_gelu_gather_mul", "rmsnorm_add": "llme_rmsnorm_add",
                       "latent_post": "llme_latent_post", "postnorm": "llme_postnorm", "gated_act": "llme_gated_act",
                       "sigmoid_mul_scaled": "llme_sigmoid_mul_scaled", "gated_act_bias": "llme_gated_act_bias",
                       "bias_add": "llme_bias_add", "sigmoid_mul_grouped": "llme_sigmoid_mul_grouped",
-                      "residual_add_scaled": "llme_residual_add_scaled", "row_norm": "llme_row_norm"},
+                      "residual_add_scaled": "llme_residual_add_scaled", "row_norm": "llme_row_norm", "relu2": "llme_relu2"},
         "recurrent": {"short_conv": "llme_short_conv", "rotate": "llme_rotate", "recurrence": "llme_recurrence",
                       "gated_norm": "llme_gated_norm", "exp_gates": "llme_exp_gates"},
+        "delta_rule": {"delta_step": "llme_delta_step", "delta_portions": "llme_delta_portions"},
         "attention_window": {"window_post": "llme_window_post", "window_attention_plain": "llme_window_attention_plain"},
         "attention_window_tc": {"window_attention_tc/{hd}": "llme_window_attention_tc"},
-        "moe": {"moe_route": "llme_moe_route", "grouped_linear": "llme_grouped_linear", "moe_combine": "llme_moe_combine",
-                "moe_combine_gated": "llme_moe_combine_gated"},
+        "moe": {"moe_route": "llme_moe_route", "grouped_linear": "llme_grouped_linear", "moe_combine": "llme_moe_combine"},
         "moe_tc": {"grouped_linear_tc": "llme_grouped_linear_tc"},
         "attention_latent": {"latent_attention_plain": "llme_latent_attention_plain"},
         "attention_latent_tc": {"latent_attention_tc/{hd}": "llme_latent_attention_tc",
@@ -243,7 +244,7 @@ class CudaOps:
         fast_attention = self.chosen("attention") == "fast"
         for op in plan.ops:
             a = op.a
-            if op.kind in ("embedding", "rmsnorm", "qkv_post", "attention"):
+            if op.kind in ("embedding", "rmsnorm", "layernorm", "qkv_post", "attention"):
                 want("elementwise")
             if op.kind in ("linear_act", "pointwise", "residual_add", "latent_attention", "token_side", "postnorm", "row_norm"):
                 want("pointwise")
@@ -253,9 +254,15 @@ class CudaOps:
                 want("pointwise")
             if op.kind in ("short_conv", "rotate", "recurrence", "gated_norm", "exp_gates"):
                 want("recurrent")
+            if op.kind == "delta_rule":
+                want("delta_rule")
             if op.kind == "window_attention":
                 want("attention_window")
-                if fast_attention and build.has_source("attention_window_tc") and self.window_tc_supports(a["qk_dim"], a["v_dim"], a["q"].dtype):
+                if fast_attention and a.get("decode_scratch") is not None and self.fast_attention_supports(a["qk_dim"], a["q"].dtype):
+                    want(f"attention_fast@HEAD_DIM={a['qk_dim']}")       # ordinary attention: the grouped-query kernels
+                    if a["qk_dim"] in (64, 128) and self.chosen("attention.portion") == "tcgen05":
+                        want(f"attention_tc@HEAD_DIM={a['qk_dim']}")
+                elif fast_attention and build.has_source("attention_window_tc") and self.window_tc_supports(a["qk_dim"], a["v_dim"], a["q"].dtype):
                     want(f"attention_window_tc@DK={a['qk_dim']},DV={a['v_dim']}")
             if op.kind in ("moe_route", "grouped_linear", "moe_combine"):
                 want("moe")

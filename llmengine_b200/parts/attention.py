@@ -172,7 +172,9 @@ class WindowSinkAttention(Part):
       before the request's start); the request's last K - 1 projected values are a state beside the pages;
     * `softcap` c > 0: a score s becomes c tanh(s / c) behind the scale;
     * `unit_sink`: the softmax's denominator holds one more term of one (a sink whose logit is zero);
-    * a position part with `interleaved` pairs coordinate 2i with 2i + 1.
+    * a position part with `interleaved` pairs coordinate 2i with 2i + 1;
+    * `unit_norm_eps`: BEHIND the rotation every query and key head is divided by its own root mean square,
+      sqrt(mean(x^2) + eps), without a weight (it excludes the norm before the rotation).
 
     Tensors: q, k, v, o; q.norm, k.norm; sink; g; q.b, k.b, v.b; q.conv, k.conv, v.conv.
 
@@ -185,8 +187,11 @@ class WindowSinkAttention(Part):
                  window: int = 0, keep_first: int = 0, sink: bool = False, own_kv: bool = True,
                  retain_window: Optional[int] = None, retain_first: Optional[int] = None, head_norm: bool = False,
                  biases: bool = False, values_are_keys: bool = False, gate: Optional[str] = None, conv_taps: int = 0,
-                 softcap: float = 0.0, unit_sink: bool = False):
+                 softcap: float = 0.0, unit_sink: bool = False, unit_norm_eps: Optional[float] = None):
         super().__init__(rt, prefix)
+        self.unit_eps = None if unit_norm_eps is None else float(unit_norm_eps)
+        if self.unit_eps is not None and (norm_eps is not None or biases or conv_taps):
+            raise ValueError(f"{prefix}: the norm behind the rotation stands alone, behind plain projections")
         self.taps, self.softcap, self.unit_sink = int(conv_taps), float(softcap), bool(unit_sink)
         if self.unit_sink and sink:
             raise ValueError(f"{prefix}: a learned sink and a sink of one exclude each other")
@@ -268,6 +273,12 @@ class WindowSinkAttention(Part):
             self.v_bias = t[self.name("v.b")].float().contiguous() if self.has_v else (self.k_bias if self.values_are_keys else None)
 
     @property
+    def ordinary(self) -> bool:
+        """Whether mask and softmax are those of `GQAttention`: keys and values of one width, no kept first positions beside a
+        window, no sink, no cap."""
+        return self.dk == self.dv and not (self.keep_first or self.has_sink or self.unit_sink or self.softcap)
+
+    @property
     def in_size(self) -> int:
         """Rows of `w_in`: the width of the product that holds every projection of the mixer's input."""
         return self.q_size + (self.k_size if self.own_kv else 0) + (self.v_size if self.has_v else 0) + self.gate_size
@@ -305,13 +316,16 @@ class WindowSinkAttention(Part):
         pos = self.position
         plan.window_attention(
             q_in=src[:, :qs], k_in=k_in, v_in=v_in,
-            q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps or 0.0,
+            q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps or self.unit_eps or 0.0, unit_norm=self.unit_eps is not None,
             inv_freq=pos.frequencies() if pos is not None else None, rot_dims=pos.dims if pos is not None else 0,
             amplitude=pos.amplitude if pos is not None else 1.0, q=q, out=heads, cache=cache.kv, group=cache.group,
             num_heads=self.nh, num_kv_heads=self.nkv, qk_dim=self.dk, v_dim=self.dv, window=self.window,
             keep_first=self.keep_first, scale=self.scale, sink=self.sink,
             q_bias=self.q_bias, k_bias=self.k_bias, v_bias=self.v_bias, head_norm=self.head_norm, softcap=self.softcap,
             interleaved=bool(pos is not None and getattr(pos, "interleaved", False)),
+            # an ordinary causal softmax over keys and values of one width: the kernels of plain grouped-query attention serve it
+            decode_scratch=(rt.attention_scratch(self.nh, self.nkv, self.dk)
+                            if rt.dtype == torch.bfloat16 and self.ordinary else None),
             # up to 8 key ranges per decoded token: a maximum, a sum and an output row per range and head
             scratch=(rt.buffer("window_attention_scratch", 1, rt.max_requests * self.nh * 8 * (self.dv + 2), torch.float32,
                                exact=True).view(-1) if rt.dtype == torch.bfloat16 else None))

@@ -26,7 +26,8 @@ feed_forward    `emit(plan, h) -> delta` / `forward(h, batch) -> delta [T, hidde
 block           arranges mixer, feed-forward and norms: `emit(plan, x, delta, cache) -> (x, delta)` /
                 `forward(x, delta, batch, cache) -> (x, delta)`, where `delta` is a contribution
                 not yet added to the residual stream `x` (the next norm adds it).
-embedding       `emit(plan) -> x` / `forward(token_ids) -> x`.
+embedding       `emit(plan) -> x` / `forward(token_ids) -> x`; for designs that add the embedding output to the stream again
+                later: `emit_again(plan, x, delta)`.
 head            `emit(plan, h)` (writes the step's logits) / `forward(h) -> logits` (32-bit).
 
 Cache specs
@@ -276,6 +277,17 @@ class Runtime:
         self._recurrence_scratch_floats = max(getattr(self, "_recurrence_scratch_floats", 0), pieces * heads * (p * n + 1))
         return self.buffer("recurrence_scratch", 1, self._recurrence_scratch_floats, torch.float32, exact=True).view(-1)
 
+    def delta_workspace(self, heads: int, qk_heads: int, n: int) -> Tuple[torch.Tensor, torch.Tensor]:
+        """What the delta rule over portions works from: the unit queries and keys of every token ([tokens, 2 * qk_heads * n'],
+        n' = n rounded up to whole groups of four), and per block of four tokens of a request and head the 40 numbers that the
+        block's triangular solve needs (one buffer each for all layers; blocks are numbered floor(first token / 4) + place of
+        the request in the step + block of the request)."""
+        n4 = (n + 3) // 4 * 4
+        blocks = self.max_tokens // 4 + self.max_requests + 1
+        self._delta_coef_floats = max(getattr(self, "_delta_coef_floats", 0), blocks * heads * 40)
+        return (self.workspace("delta_unit", 2 * qk_heads * n4, torch.float32),
+                self.buffer("delta_coef", 1, self._delta_coef_floats, torch.float32, exact=True).view(-1))
+
     def latent_scratch(self, num_heads: int, kv_rank: int) -> Optional[torch.Tensor]:
         """Scratch memory of the latent attention whose requests are cut into several key ranges (one buffer for all
         layers, as large as the widest of them needs)."""
@@ -349,6 +361,24 @@ def emit_embedding(plan, part: Part, hidden: int) -> torch.Tensor:
     x = rt.workspace("residual", hidden, torch.float32)
     plan.call(lambda batch: _copy_rows(x, part.forward(batch.token_ids)), f"embedding {part.prefix}")
     return x
+
+
+def emit_embedding_again(plan, part: Part, x: torch.Tensor, delta: Optional[torch.Tensor]):
+    """x += delta (if a contribution is pending) + the embedding output; nothing is pending afterwards."""
+    if hasattr(part, "emit_again"):
+        part.emit_again(plan, x, delta)
+        return x, None
+    rt = part.rt
+
+    def call(batch):
+        rows = rt.rows(x)
+        if delta is not None:
+            rows += rt.rows(delta).float()
+        rows += part.forward(batch.token_ids).to(rows.dtype)
+    if hasattr(part, "emit"):
+        raise ValueError(f"{part.prefix}: this embedding cannot be added to the stream a second time (no emit_again)")
+    plan.call(call, f"embedding {part.prefix}, added again")
+    return x, None
 
 
 def emit_norm(plan, part: Part, x: torch.Tensor, delta: Optional[torch.Tensor] = None, rows: str = "tokens") -> torch.Tensor:

@@ -18,23 +18,27 @@ class PreNormResidualBlock(Part):
 
     The residual stream `x` stays 32-bit.  A contribution is not added where it is produced:
     it travels as `delta` to the next norm, whose kernel adds it to `x` and normalises in one
-    pass.  The block reads the parts "mixer", "mixer_norm", "feed_forward" and "feed_forward_norm" of its
-    layer; the names under which their tensors are stored come with the spec.
+    pass.  The block reads the parts "mixer", "mixer_norm" and, where the layer has a feed-forward, "feed_forward" and
+    "feed_forward_norm" of its layer; the names under which their tensors are stored come with the spec.
     """
 
     def __init__(self, rt: Runtime, prefix: str, layer: LayerSpec, mixer_name: str = "mixer",
                  feed_forward_name: str = "feed_forward", mixer_norm_name: str = "mixer_norm",
                  feed_forward_norm_name: str = "feed_forward_norm"):
         super().__init__(rt, prefix)
-        need = ("mixer", "mixer_norm", "feed_forward", "feed_forward_norm")
-        missing = [n for n in need if n not in layer.parts]
+        missing = [n for n in ("mixer", "mixer_norm") if n not in layer.parts]
+        has_ffn = "feed_forward" in layer.parts
+        if has_ffn and "feed_forward_norm" not in layer.parts:
+            missing.append("feed_forward_norm")
         if missing:
             raise ValueError(f"layer {prefix!r}: a prenorm_residual block needs the parts {', '.join(missing)}")
         self.mixer_norm = build_part("norm", layer.parts["mixer_norm"], rt, self.name(mixer_norm_name))
         self.mixer = build_part("mixer", layer.parts["mixer"], rt, self.name(mixer_name))
-        self.ffn_norm = build_part("norm", layer.parts["feed_forward_norm"], rt, self.name(feed_forward_norm_name))
-        self.ffn = build_part("feed_forward", layer.parts["feed_forward"], rt, self.name(feed_forward_name))
-        self.parts = (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn)
+        self.ffn_norm = self.ffn = None
+        if has_ffn:
+            self.ffn_norm = build_part("norm", layer.parts["feed_forward_norm"], rt, self.name(feed_forward_norm_name))
+            self.ffn = build_part("feed_forward", layer.parts["feed_forward"], rt, self.name(feed_forward_name))
+        self.parts = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
         self.capture_safe = all(p.capture_safe and hasattr(p, "emit") for p in self.parts)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -54,6 +58,8 @@ class PreNormResidualBlock(Part):
         hidden = x.shape[1]
         h = emit_norm(plan, self.mixer_norm, x, delta=delta)
         a = emit_mixer(plan, self.mixer, h, cache, hidden)
+        if self.ffn is None:
+            return x, a
         h = emit_norm(plan, self.ffn_norm, x, delta=a)
         return x, emit_feed_forward(plan, self.ffn, h, hidden)
 

@@ -62,6 +62,12 @@ class TokenEmbedding(Part):
             plan.postnorm(x, x, self.norm_gain, self.norm_eps, accumulate=False, copy=copy)
         return x
 
+    def emit_again(self, plan: Plan, x: torch.Tensor, delta: Optional[torch.Tensor]) -> None:
+        """x += delta (where a contribution is pending) + the embedding output, the rows gathered anew."""
+        if self.norm_leaf is not None:
+            raise ValueError(f"{self.prefix}: an embedding with a norm of its own is not added to the stream a second time")
+        plan.embedding(self.table, x, scale=self.scale, accumulate=True, delta=delta)
+
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         from ..engine.batch import StepBatch
         plan = Plan()

@@ -1,7 +1,7 @@
 """Feed-forward parts."""
 from __future__ import annotations
 
-from typing import Dict, Optional
+from typing import Dict, Optional, Tuple
 
 import torch
 
@@ -97,7 +97,43 @@ class DenseXIELU(Part):
         return delta[: h.shape[0]]
 
 
+@register_part("feed_forward", "dense")
+class Dense(Part):
+    """down( act(up(h)) ), tensors up / down, no biases, an activation without learned numbers: "relu2": max(z, 0)^2.  The
+    activation rides in the epilogue of the up product where a kernel has it."""
+
+    def __init__(self, rt: Runtime, prefix: str, hidden_size: int, intermediate_size: int, activation: str):
+        super().__init__(rt, prefix)
+        if activation not in PLAIN_ACTIVATIONS:
+            raise ValueError(f"{prefix}: unknown activation {activation!r}; known: {', '.join(PLAIN_ACTIVATIONS)}")
+        self.hidden, self.inter, self.act = int(hidden_size), int(intermediate_size), activation
+        self.w_up = self.w_down = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.name("up"): WeightSpec((self.inter, self.hidden)), self.name("down"): WeightSpec((self.hidden, self.inter))}
+
+    def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        self.w_up, self.w_down = t[self.name("up")].contiguous(), t[self.name("down")].contiguous()
+
+    def emit(self, plan: Plan, h: torch.Tensor) -> torch.Tensor:
+        rt = self.rt
+        up = rt.workspace("ffn_up", self.inter, rt.dtype)
+        act = rt.workspace("act", self.inter, rt.dtype)
+        plan.linear_act(h, self.w_up, up, act, self.act)
+        delta = rt.workspace("ffn_out", self.hidden, torch.float32)
+        plan.linear(act, self.w_down, delta)
+        return delta
+
+    def forward(self, h: torch.Tensor, batch=None) -> torch.Tensor:
+        from ..engine.batch import StepBatch
+        plan = Plan()
+        delta = self.emit(plan, h)
+        run_alone(self.rt, plan, batch if batch is not None else StepBatch.bare(h.shape[0], h.device))
+        return delta[: h.shape[0]]
+
+
 GATED_ACTIVATIONS = ("silu", "clamped_swish", "gelu_tanh")
+PLAIN_ACTIVATIONS = ("relu2",)
 
 
 @register_part("feed_forward", "gated_dense")
@@ -160,10 +196,16 @@ class RoutedExperts(Part):
     """A mixture of `num_experts` small feed-forwards down(silu(gate h) * (up h)) of which every token uses `top_k`:
     z = W_router h (+ a bias with `router_bias`) in 32-bit.  `routing` "sigmoid": s = sigmoid(z), C = the `top_k` experts of
     largest s, w_e = route_scale * s_e / (sum over C of s + 1e-20); "softmax_chosen": C = the experts of largest z and w_e =
-    route_scale * softmax over the chosen logits alone.  Output = sum over C of w_e expert_e(h), plus, with `shared_size` > 0,
+    route_scale * softmax over the chosen logits alone; "softmax": s = softmax(z) over all, C = the experts of largest s (with
+    `correction`, a tensor of that name: of largest s + correction), w_e = route_scale * s_e, not renormalised.  Output = sum over C of w_e expert_e(h), plus, with `shared_size` > 0,
     one more expert of that size that takes every token, with weight one or, with `shared_gate`, with weight
-    sigmoid(W_sg h), one number a token.  Tensors: router (router.b); e<i>.gate / up / down; shared.gate / up / down
+    sigmoid(W_sg h), one number a token.  Tensors: router (router.b, correction); e<i>.gate / up / down; shared.gate / up / down
     (shared.sg [1, hidden]).
+
+    Options of the "softmax" routing: `groups` (count, keep): the choices form `count` equal groups of neighbours, and only the
+    members of the `keep` groups whose largest choice score is largest can be chosen; `identity` I: the router has I outputs
+    more than there are experts, and these stand for the input itself (output h, times the weight; no tensors).
+    `activation` "relu2": an expert is down(max(up h, 0)^2), without a gate.
 
     The experts' matrices are stacked ([E, 2 ff, D] and [E, D, ff]) and run as two grouped products over the
     (token, choice) pairs listed expert by expert; the pairs' outputs are combined per token in the order of the
@@ -172,13 +214,23 @@ class RoutedExperts(Part):
 
     def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_experts: int, top_k: int, expert_size: int,
                  route_scale: float = 1.0, shared_size: int = 0, routing: str = "sigmoid", router_bias: bool = False,
-                 shared_gate: bool = False):
+                 shared_gate: bool = False, activation: str = "silu", correction: bool = False, identity: int = 0,
+                 groups: Tuple[int, int] = (1, 1)):
         super().__init__(rt, prefix)
         self.hidden, self.E, self.top, self.ff = int(hidden_size), int(num_experts), int(top_k), int(expert_size)
-        if not 0 < self.top <= self.E:
-            raise ValueError(f"{prefix}: {self.top} of {self.E} experts cannot be chosen")
-        if routing not in ("sigmoid", "softmax_chosen"):
-            raise ValueError(f"{prefix}: unknown routing {routing!r}; known: sigmoid, softmax_chosen")
+        self.identity, self.choices = int(identity), int(num_experts) + int(identity)
+        self.groups, self.has_correction, self.correction = (int(groups[0]), int(groups[1])), bool(correction), None
+        if activation not in ("silu",) + PLAIN_ACTIVATIONS:
+            raise ValueError(f"{prefix}: unknown activation {activation!r} of an expert")
+        self.act = activation
+        if not 0 < self.top <= self.choices:
+            raise ValueError(f"{prefix}: {self.top} of {self.choices} experts cannot be chosen")
+        if routing not in ("sigmoid", "softmax_chosen", "softmax"):
+            raise ValueError(f"{prefix}: unknown routing {routing!r}; known: sigmoid, softmax_chosen, softmax")
+        if routing != "softmax" and (correction or identity or self.groups[1] < self.groups[0]):
+            raise ValueError(f"{prefix}: corrections, identity experts and groups belong to the routing by a softmax over all")
+        if self.choices % self.groups[0] or not 0 < self.groups[1] <= self.groups[0] or self.top > self.choices // self.groups[0] * self.groups[1]:
+            raise ValueError(f"{prefix}: {self.groups[1]} of {self.groups[0]} groups of {self.choices} experts do not offer {self.top}")
         self.route_scale, self.routing, self.router_bias = float(route_scale), routing, bool(router_bias)
         self.shared = (GatedDense(rt, self.name("shared"), hidden_size, int(shared_size)) if shared_size else None)
         self.shared_gate = bool(shared_gate)
@@ -187,11 +239,14 @@ class RoutedExperts(Part):
         self.w_router = self.w_gate_up = self.w_down = self.b_router = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
-        s = {self.name("router"): WeightSpec((self.E, self.hidden))}
+        s = {self.name("router"): WeightSpec((self.choices, self.hidden))}
         if self.router_bias:
-            s[self.name("router.b")] = WeightSpec((self.E,), role="vector")
+            s[self.name("router.b")] = WeightSpec((self.choices,), role="vector")
+        if self.has_correction:
+            s[self.name("correction")] = WeightSpec((self.choices,), role="vector")
         for e in range(self.E):
-            s[self.name(f"e{e}.gate")] = WeightSpec((self.ff, self.hidden))
+            if self.act == "silu":
+                s[self.name(f"e{e}.gate")] = WeightSpec((self.ff, self.hidden))
             s[self.name(f"e{e}.up")] = WeightSpec((self.ff, self.hidden))
             s[self.name(f"e{e}.down")] = WeightSpec((self.hidden, self.ff))
         if self.shared is not None:
@@ -209,16 +264,18 @@ class RoutedExperts(Part):
         self.w_router = torch.cat(rows, 0).contiguous()
         if self.router_bias:
             b = t[self.name("router.b")].float()
-            self.b_router = torch.cat([b, b.new_zeros(self.w_router.shape[0] - self.E)]).contiguous()
-        self.w_gate_up = torch.stack([torch.cat([t[self.name(f"e{e}.gate")], t[self.name(f"e{e}.up")]], 0)
-                                      for e in range(self.E)]).contiguous()
+            self.b_router = torch.cat([b, b.new_zeros(self.w_router.shape[0] - self.choices)]).contiguous()
+        if self.has_correction:
+            self.correction = t[self.name("correction")].float().contiguous()
+        leaves = ("gate", "up") if self.act == "silu" else ("up",)
+        self.w_gate_up = torch.stack([torch.cat([t[self.name(f"e{e}.{n}")] for n in leaves], 0) for e in range(self.E)]).contiguous()
         self.w_down = torch.stack([t[self.name(f"e{e}.down")] for e in range(self.E)]).contiguous()
         if self.shared is not None:
             self.shared.load_weights({n: t[n] for n in self.shared.weight_specs()})
 
     def emit(self, plan: Plan, h: torch.Tensor) -> torch.Tensor:
         rt = self.rt
-        T, E, top = rt.max_tokens, self.E, self.top
+        T, E, top = rt.max_tokens, self.choices, self.top      # E: what a token chooses from; the last `identity` of them have no product
         wide = rt.workspace("router_logits", self.w_router.shape[0], torch.float32)    # [logits | gate of the shared expert]
         plan.linear(h, self.w_router, wide, bias=self.b_router)
         logits = wide[:, :E]
@@ -228,16 +285,17 @@ class RoutedExperts(Part):
         counts = rt.buffer("route_counts", 1, E, torch.int32, exact=True, zero=True).view(-1)
         order = rt.buffer("route_order", T * top, 1, torch.int32).view(-1)
         plan.moe_route(logits=logits, top_k=top, scale=self.route_scale, experts=experts, weights=weights,
-                       offsets=offsets, order=order, counts=counts, mode=self.routing)
+                       offsets=offsets, order=order, counts=counts, mode=self.routing, correction=self.correction, groups=self.groups)
         act = rt.buffer("expert_act", T * top, self.ff, rt.dtype)
-        mid = rt.buffer("expert_gate_up", T * top, 2 * self.ff, rt.dtype)
+        mid = rt.buffer("expert_gate_up", T * top, self.w_gate_up.shape[1], rt.dtype)
         plan.grouped_linear(x=h, w=self.w_gate_up, out=act, offsets=offsets, order=order, top_k=top, gather=True,
-                            scatter=False, mid=mid, act="silu")
+                            scatter=False, mid=mid, act=self.act)
         y = rt.buffer("expert_out", T * top, self.hidden, torch.float32)
         plan.grouped_linear(x=act, w=self.w_down, out=y, offsets=offsets, order=order, top_k=top, gather=False, scatter=True)
         base = self.shared.emit(plan, h, out_name="shared_out") if self.shared is not None else None
         delta = rt.workspace("ffn_out", self.hidden, torch.float32)
-        plan.moe_combine(y=y, weights=weights, base=base, out=delta, base_gate=wide[:, E:E + 1] if self.shared_gate else None)
+        plan.moe_combine(y=y, weights=weights, base=base, out=delta, base_gate=wide[:, E:E + 1] if self.shared_gate else None,
+                         experts=experts if self.identity else None, identity=h if self.identity else None, first_identity=self.E)
         return delta
 
     def forward(self, h: torch.Tensor, batch=None) -> torch.Tensor:

@@ -1,4 +1,4 @@
-"""RMS norm over the residual stream, fused with the pending residual add."""
+"""Norms over the residual stream, fused with the pending residual add."""
 from __future__ import annotations
 
 from typing import Dict, Optional
@@ -81,3 +81,40 @@ class OnePlusRMSNorm(RMSNorm):
 
     def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.gain = (1.0 + tensors[self.name(self.leaf)].float()).contiguous()
+
+
+@register_part("norm", "layernorm")
+class LayerNorm(Part):
+    """y = (x - mean) / sqrt(mean of (x - mean)^2 + eps) * w + b, the tensors `leaf` and `bias_leaf` (below the prefix; an
+    empty leaf is the prefix itself).  The pending contribution is added in the same pass, as in `RMSNorm`."""
+
+    def __init__(self, rt: Runtime, prefix: str, size: int, eps: float, leaf: str = "weight", bias_leaf: str = "bias"):
+        super().__init__(rt, prefix)
+        self.size, self.eps = int(size), float(eps)
+        self.leaf, self.bias_leaf = leaf, bias_leaf
+        self.gain: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.name(self.leaf): WeightSpec((self.size,), role="vector", init="gain"),
+                self.name(self.bias_leaf): WeightSpec((self.size,), role="vector")}
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        w, b = tensors[self.name(self.leaf)], tensors[self.name(self.bias_leaf)]
+        if w.dtype != b.dtype:                # one kernel launch takes one type for both
+            w, b = w.float(), b.float()
+        self.gain, self.bias = w.contiguous(), b.contiguous()
+
+    def emit(self, plan: Plan, x: torch.Tensor, delta: Optional[torch.Tensor] = None, rows: str = ROWS_TOKENS,
+             out_name: Optional[str] = None) -> torch.Tensor:
+        out = self.rt.workspace(out_name or ("normed" if rows == ROWS_TOKENS else "normed_rows"), self.size, self.rt.dtype)
+        plan.layernorm(x, self.gain, self.bias, self.eps, out, delta=delta, rows=rows)
+        return out
+
+    def forward(self, x: torch.Tensor, delta: Optional[torch.Tensor] = None,
+                out_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        from ..engine.batch import StepBatch
+        plan = Plan()
+        out = self.emit(plan, x, delta=delta, rows=ROWS_TOKENS if out_rows is None else ROWS_LOGITS)
+        run_alone(self.rt, plan, StepBatch.bare(x.shape[0], x.device, logit_rows=out_rows))
+        return out[: x.shape[0] if out_rows is None else out_rows.numel()]

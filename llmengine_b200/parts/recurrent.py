@@ -16,6 +16,11 @@
   o_t = S_t^T q_t / (max(|n_t . q_t|, exp(-M_t)) + 1e-6); every head's o is divided by its root mean square, the heads are
   multiplied by a weight vector and by sigmoid(W_g h), and projected.  State per request: S and n (n is one more column of
   S, whose v is one) and M, all 32-bit.
+* `GatedDelta` (kind `gated_delta`): the delta rule with a decay and a write strength per head and token.  q, k and v pass a
+  short causal convolution per channel and silu; q and k become unit vectors, q then times qk_dim^(-1/2); b_t = sigmoid(W_b h),
+  a_t = exp(-exp(A_log) softplus(W_a h + dt_bias)); S <- a_t S, u = b_t (v_t - S^T k_t), S <- S + k_t u^T, o_t = S^T q_t; every
+  head's o is divided by its root mean square, times a weight shared by the heads, times silu(W_g h), and projected.  State per
+  request: the matrices S (32-bit) and the convolution's last taps - 1 inputs.
 * `ParallelMixer` (kind `parallel`): branches that read the same input; the result is sum_b scale_b branch_b(h).  The
   branches' input projections are ONE product, and so are their output projections: every branch writes its gated heads,
   times its scale, into its columns of one row, and the output matrices stand side by side.
@@ -223,6 +228,78 @@ class MatrixMemory(Part):
         heads = rt.workspace("memory_heads", hs, rt.dtype)
         plan.gated_norm(y=o, gate=proj[:, 2 * qs + hs:], weight=self.norm_w, out=heads, group=self.dv, gate_first=False,
                         eps=self.eps, gate_act="sigmoid", floor=gates[:, 2 * H:], den_eps=self.DEN_EPS)
+        delta = rt.workspace("mixer_out", self.hidden, torch.float32)
+        plan.linear(heads, self.w_o, delta)
+        return delta
+
+    def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:
+        plan = Plan()
+        buf = self.rt.workspace("normed", self.hidden, self.rt.dtype)
+        buf[: h.shape[0]].copy_(h)
+        delta = self.emit(plan, buf, cache)
+        run_alone(self.rt, plan, batch)
+        return delta[: h.shape[0]]
+
+
+@register_part("mixer", "gated_delta")
+class GatedDelta(Part):
+    """Tensors: q, k [qk_heads qk_dim, hidden]; v, g [heads v_dim, hidden]; q.conv, k.conv, v.conv [channels, taps]; b, a
+    [heads, hidden]; A_log, dt_bias [heads]; norm [v_dim]; o [hidden, heads v_dim]; no biases.  Head i uses the q and k of head
+    i // (heads / qk_heads).  All six projections of the input are ONE product with 32-bit results: the write strengths and the
+    decays enter the recurrence unrounded, and no second, small product is needed for them."""
+
+    UNIT_EPS = 1e-6                      # inside the root of the norm that makes q and k unit vectors
+
+    def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, num_qk_heads: int, qk_dim: int, v_dim: int,
+                 taps: int, norm_eps: float):
+        super().__init__(rt, prefix)
+        self.hidden, self.nh, self.nqk = int(hidden_size), int(num_heads), int(num_qk_heads)
+        self.dk, self.dv, self.taps, self.eps = int(qk_dim), int(v_dim), int(taps), float(norm_eps)
+        if self.nh % self.nqk:
+            raise ValueError(f"{prefix}: {self.nh} heads are not a multiple of {self.nqk} query/key heads")
+        if self.taps < 1:
+            raise ValueError(f"{prefix}: a convolution needs at least one tap")
+        self.qk_size, self.heads_size = self.nqk * self.dk, self.nh * self.dv
+        self.conv_channels = 2 * self.qk_size + self.heads_size
+        used = self.conv_channels + self.heads_size + 2 * self.nh
+        self.in_size = used + -used % 8          # rows of zeros up to a multiple of 8: the product's rows start on 32 bytes
+        self.w_in = self.w_o = self.conv_w = self.dt_bias = self.a_log = self.norm_w = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        m = lambda n: WeightSpec((n, self.hidden))
+        v = lambda n, init: WeightSpec((n,), role="vector", init=init)
+        conv = lambda n: WeightSpec((n, self.taps), role="vector", init="unit")
+        return {self.name("q"): m(self.qk_size), self.name("q.conv"): conv(self.qk_size), self.name("k"): m(self.qk_size),
+                self.name("k.conv"): conv(self.qk_size), self.name("v"): m(self.heads_size), self.name("v.conv"): conv(self.heads_size),
+                self.name("g"): m(self.heads_size), self.name("b"): m(self.nh), self.name("a"): m(self.nh),
+                self.name("A_log"): v(self.nh, "unit"), self.name("dt_bias"): v(self.nh, "unit"), self.name("norm"): v(self.dv, "gain"),
+                self.name("o"): WeightSpec((self.hidden, self.heads_size))}
+
+    def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        rows = [t[self.name(n)] for n in ("q", "k", "v", "g", "b", "a")]
+        rows.append(rows[0].new_zeros(self.in_size - sum(r.shape[0] for r in rows), self.hidden))
+        self.w_in, self.w_o = torch.cat(rows, 0).contiguous(), t[self.name("o")].contiguous()
+        self.conv_w = torch.cat([t[self.name(n + ".conv")].float() for n in ("q", "k", "v")], 0).contiguous()
+        self.dt_bias, self.a_log = t[self.name("dt_bias")].float().contiguous(), t[self.name("A_log")].float().contiguous()
+        self.norm_w = t[self.name("norm")].float().repeat(self.nh).contiguous()
+
+    def cache_spec(self) -> StatesSpec:
+        return StatesSpec((("conv", (max(self.taps - 1, 1), self.conv_channels)), ("state", (self.nh, self.dv, self.dk))))
+
+    def emit(self, plan: Plan, h: torch.Tensor, cache: StatesView) -> torch.Tensor:
+        rt, H, qs, hs, C = self.rt, self.nh, self.qk_size, self.heads_size, self.conv_channels
+        proj = rt.workspace("delta_in", self.in_size, torch.float32)
+        plan.linear(h, self.w_in, proj)
+        qkv = rt.workspace("delta_conv", C, torch.float32)
+        plan.short_conv(x=proj[:, :C], w=self.conv_w, bias=None, state=cache.states["conv"], out=qkv, act="silu")
+        o = rt.workspace("delta_o", hs, torch.float32)
+        unit, coef = rt.delta_workspace(H, self.nqk, self.dk)
+        gates = C + hs
+        plan.delta_rule(q=qkv[:, :qs], k=qkv[:, qs:2 * qs], v=qkv[:, 2 * qs:], write=proj[:, gates:gates + H], forget=proj[:, gates + H:gates + 2 * H],
+                        dt_bias=self.dt_bias, a_log=self.a_log, q_scale=float(self.dk) ** -0.5, unit_eps=self.UNIT_EPS,
+                        state=cache.states["state"], out=o, heads=H, n=self.dk, p=self.dv, qk_groups=self.nqk, unit=unit, coef=coef)
+        heads = rt.workspace("delta_heads", hs, rt.dtype)
+        plan.gated_norm(y=o, gate=proj[:, C:C + hs], weight=self.norm_w, out=heads, group=self.dv, gate_first=False, eps=self.eps)
         delta = rt.workspace("mixer_out", self.hidden, torch.float32)
         plan.linear(heads, self.w_o, delta)
         return delta

@@ -23,9 +23,22 @@ class HostOps:
     def compile(self, plan):
         return HostPlan(self, plan)
 
-    def embedding(self, ids, table, out, scale=1.0):
-        out.copy_(table[ids.long()].float() * scale)
+    def embedding(self, ids, table, out, scale=1.0, accumulate=False, delta=None):
+        rows = table[ids.long()].float() * scale
+        if delta is not None:
+            out += delta.float()
+        out.copy_(out + rows if accumulate else rows)
         return out
+
+    def layernorm(self, x, gain, bias, eps, out, delta=None, rows=None):
+        if delta is not None:
+            if rows is None:
+                x += delta.float()
+            else:
+                x[rows.long()] += delta.float()[rows.long()]
+        src = x if rows is None else x[rows.long()]
+        c = src - src.mean(-1, keepdim=True)
+        out.copy_((c / torch.sqrt((c * c).mean(-1, keepdim=True) + eps) * gain.float() + bias.float()).to(out.dtype))
 
     def rmsnorm(self, x, gain, eps, out, delta=None, rows=None, gain2=None, out2=None):
         if delta is not None:
@@ -113,8 +126,11 @@ class HostOps:
         return out
 
     def activation(self, act, params, x, out):
-        assert act == "xielu"
         z = x.float()
+        if act == "relu2":
+            out.copy_((torch.clamp(z, min=0) ** 2).to(out.dtype))
+            return
+        assert act == "xielu"
         ap, an = params
         out.copy_(torch.where(z > 0, ap * z * z + 0.5 * z, an * (torch.expm1(torch.clamp(z, max=0)) - z) + 0.5 * z).to(out.dtype))
 
@@ -184,6 +200,22 @@ class HostOps:
                 if a["skip"] is not None:
                     y = y + a["skip"][:, None] * v
                 a["out"][t] = y.reshape(-1)
+
+    def delta_rule(self, a, batch):
+        H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]
+        rep = H // G
+        unit = lambda x: x / torch.sqrt((x * x).sum(-1, keepdim=True) + a["unit_eps"])
+        for lo, hi, slot in self._requests(batch):
+            S = a["state"][slot]                                           # [H, p, n]
+            for t in range(lo, hi):
+                q = (unit(a["q"][t].view(G, n)) * a["q_scale"]).repeat_interleave(rep, 0)
+                k = unit(a["k"][t].view(G, n)).repeat_interleave(rep, 0)
+                v, z = a["v"][t].view(H, p), a["forget"][t] + a["dt_bias"]
+                keep = torch.exp(-torch.exp(a["a_log"]) * (torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))))
+                S.mul_(keep[:, None, None])
+                u = torch.sigmoid(a["write"][t])[:, None] * (v - torch.einsum("hpn,hn->hp", S, k))
+                S.add_(u[:, :, None] * k[:, None, :])
+                a["out"][t] = torch.einsum("hpn,hn->hp", S, q).reshape(-1)
 
     def gated_norm(self, a, T):
         y, g = a["y"][:T], a["gate"][:T].float()
@@ -307,6 +339,8 @@ class HostOps:
             x = x.view(T, heads, dk)
             if a["inv_freq"] is not None:
                 x = self._rotate(x, positions, a["inv_freq"], a["rot_dims"], bool(a.get("interleaved")), a["amplitude"])
+            if a.get("unit_norm"):
+                x = x / torch.sqrt((x * x).mean(-1, keepdim=True) + a["eps"])
             return x
         q = finish(a["q_in"], H, a["q_gain"], a.get("q_bias")).to(cache.dtype)
         a["q"][:T] = q.reshape(T, -1)
@@ -343,6 +377,14 @@ class HostOps:
         if a.get("mode", "sigmoid") == "softmax_chosen":
             val, idx = torch.topk(a["logits"][:T].float(), top, dim=-1)
             wt = torch.softmax(val, -1) * a["scale"]
+        elif a["mode"] == "softmax":
+            s = torch.softmax(a["logits"][:T].float(), -1)
+            c = s if a["correction"] is None else s + a["correction"]
+            count, keep = a["groups"]
+            kept = torch.topk(c.view(T, count, -1).amax(-1), keep, dim=-1).indices
+            allowed = torch.zeros(T, count, dtype=torch.bool).scatter_(1, kept, True).repeat_interleave(E // count, 1)
+            idx = torch.topk(c.masked_fill(~allowed, float("-inf")), top, dim=-1).indices
+            wt = s.gather(1, idx) * a["scale"]
         else:
             s = torch.sigmoid(a["logits"][:T].float())
             val, idx = torch.topk(s, top, dim=-1)
@@ -364,7 +406,9 @@ class HostOps:
                 pair = int(order[r])
                 row = a["x"][pair // top if a["gather"] else r].float()
                 y = w[e].float() @ row
-                if a["act"]:
+                if a["act"] == "relu2":
+                    y = torch.clamp(y, min=0) ** 2
+                elif a["act"]:
                     n = y.numel() // 2
                     g, u = y[:n].to(a["x"].dtype).float(), y[n:].to(a["x"].dtype).float()
                     y = g * torch.sigmoid(g) * u
@@ -413,7 +457,10 @@ class HostPlan:
         for op in self.plan.ops[first:last]:
             a, k = op.a, op.kind
             if k == "embedding":
-                o.embedding(batch.token_ids, a["table"], a["out"][:T], a.get("scale", 1.0))
+                o.embedding(batch.token_ids, a["table"], a["out"][:T], a.get("scale", 1.0), bool(a.get("accumulate")), cut(a.get("delta")))
+            elif k == "layernorm":
+                o.layernorm(a["x"][:T], a["gain"], a["bias"], a["eps"], a["out"][:n_rows(a["rows"])], delta=cut(a["delta"]),
+                            rows=batch.logit_rows if a["rows"] == "logits" else None)
             elif k == "rmsnorm":
                 some = a["rows"] == "logits"
                 o.rmsnorm(a["x"][:T], a["gain"], a["eps"], a["out"][:n_rows(a["rows"])], delta=cut(a["delta"]),
@@ -429,6 +476,8 @@ class HostPlan:
                 o.rotate(a, T, batch.positions)
             elif k == "recurrence":
                 o.recurrence(a, batch)
+            elif k == "delta_rule":
+                o.delta_rule(a, batch)
             elif k == "gated_norm":
                 o.gated_norm(a, T)
             elif k == "row_norm":
@@ -454,6 +503,9 @@ class HostPlan:
             elif k == "moe_combine":
                 top = a["weights"].shape[1]
                 y = a["y"][:T * top].view(T, top, -1)
+                if a.get("identity") is not None:
+                    same = a["experts"][:T] >= a["first_identity"]
+                    y = torch.where(same[:, :, None], a["identity"][:T, None, :].float(), y)
                 v = (a["weights"][:T, :, None] * y).sum(1)
                 base = a["base"][:T] if a["base"] is not None else None
                 if base is not None and a.get("base_gate") is not None:
