@@ -1,4 +1,4 @@
-"""A design beside its closest existing model at equal size (`python bench.py --design bepuzen | torisun | vifelix | funevik`).
+"""A design beside its closest existing model at equal size (`python bench.py --design bepuzen | torisun | vifelix | funevik | vaderax`).
 
 For each size: prefill of one 2,048-token prompt and decode at batch 1 / 8 / 64 over 2,048 cached tokens, tokens/s,
 for the design and for the grouped-query model of the same width, depth and (active) weight count per layer;
@@ -16,6 +16,8 @@ L1, L2 = "latent_attention", "latent_attention_2"
 # a 32-bit operation outside the tensor cores counts as this many operations of the bf16 product peak that the tables divide
 # by (set by `run` from the measured peak), so that `ideal` is its time at the 32-bit ceiling
 FP32_SHARE = 1.0
+# (experts, choices per token) -> share of the choices that go to experts with a product, where a router has identity experts
+ROUTED_SHARE: Dict[tuple, float] = {}
 
 
 def bepuzen_shape(layers: int, width: int, heads: int, ff: int, kv_rank: int = 512, dim: int = 128, rot: int = 64,
@@ -94,6 +96,22 @@ def funevik_shape(width: int, heads: int, kv_heads: int, ff: int, experts: int, 
             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in kinds]}
 
 
+def vaderax_shape(width: int, heads: int, kv_heads: int, ff: int, experts: int, top: int, expert_ff: int, delta_heads: int,
+                  dim: int = 128, vocab: int = 32768) -> Dict[str, Any]:
+    """Four stored layers that run as six: a delta layer (value heads of 128 on half as many query/key heads of 128, four taps) with
+    a dense feed-forward, a loop of two passes over a delta and an attention layer with routed experts (identity experts beside
+    them, half of the groups kept), and a delta layer with a dense feed-forward again.  A dense or an active routed feed-forward has
+    about the weights of the grouped-query model's gated one (two matrices of one and a half times the columns)."""
+    de = {"heads": delta_heads, "kv_heads": delta_heads // 2, "dim": dim, "vdim": dim, "conv": 4}
+    at = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 10000.0, "dims": dim // 2}}
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "identity": experts // 8,
+                                                                     "groups": {"count": 8, "keep": 4}}}
+    kinds = [("delta", de, dense), ("delta", de, routed), ("attention", at, routed), ("delta", de, dense)]
+    return {"architecture": "Vaderax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in kinds], "loop": {"start": 1, "stop": 3, "times": 2}}
+
+
 # 32-bit multiply-adds outside the tensor cores: 148 SMs x 128 lanes x 2 x 1.965 GHz (nominal), the compute ceiling of a
 # recurrence whose state and inputs are 32-bit
 FP32_TFLOPS = 74.4
@@ -114,6 +132,10 @@ VIFELIX_SIZES = {
 FUNEVIK_SIZES = {
     "2048": (6, funevik_shape(2048, 16, 4, 5504, 32, 4, 1024, 8), gqa_shape(6, 2048, 16, 5504)),
     "4096": (6, funevik_shape(4096, 32, 8, 10944, 64, 4, 2048, 16), gqa_shape(6, 4096, 32, 10944)),
+}
+VADERAX_SIZES = {
+    "2048": (6, vaderax_shape(2048, 16, 4, 8192, 32, 4, 2048, 16), gqa_shape(6, 2048, 16, 5504)),
+    "4096": (6, vaderax_shape(4096, 32, 8, 16384, 64, 4, 4096, 32), gqa_shape(6, 4096, 32, 10944)),
 }
 CACHED, PROMPT = 2048, 2048
 
@@ -180,12 +202,20 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
         w, top = a["w"], a["top_k"]
         E, n, kk = w.shape
         used = E * (1.0 - (1.0 - top / E) ** T)                       # experts that some token of the step uses, in the mean
-        n_out = n // 2 if a["act"] else n
-        return (f"grouped {'gate|up + silu' if a['act'] else 'down'} {E}x{n}x{kk}", 2.0 * T * top * n * kk,
+        n_out = n // 2 if a["act"] == "silu" else n
+        what = {"silu": "gate|up + silu", "relu2": "up + relu^2", None: "down"}[a["act"]]
+        if (E, top) in ROUTED_SHARE:                                  # identity experts take their share of the pairs
+            top = top * ROUTED_SHARE[E, top]
+            used = E * (1.0 - (1.0 - top / E) ** T)
+        return (f"grouped {what} {E}x{n}x{kk}", 2.0 * T * top * n * kk,
                 used * n * kk * el + T * top * (kk * el + n_out * a["out"].element_size()))
     if k == "moe_combine":
         D, top = a["out"].shape[1], a["weights"].shape[1]
         return "weighted sum of the chosen experts", 0.0, T * D * (top * 4 + (4 if a["base"] is not None else 0) + 4)
+    if k == "layernorm":
+        return "layer norm + residual add", 0.0, T * a["x"].shape[1] * ((12 if a["delta"] is not None else 4) + el)
+    if k == "embedding":
+        return "embedding added again", 0.0, T * a["out"].shape[1] * (12 + el)
     if k == "rmsnorm":
         return "rmsnorm + residual add", 0.0, T * a["x"].shape[1] * (4 + 4 + 4 + el)
     if k == "token_side":
@@ -212,9 +242,13 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
         return (f"recurrence {H} heads, state {n}x{p}" + (", decay per token" if a.get("dt") is not None else
                                                           ", given gates" if a.get("keep") is not None else ", fixed decay"),
                 4.0 * T * H * n * p * FP32_SHARE, requests * 2 * H * n * p * 4 + T * (2 * G * n * 4 + H * p * (a["v"].element_size() + 4)))
+    if k == "delta_rule":
+        H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]
+        return (f"delta rule {H} heads, state {n}x{p}", 6.0 * T * H * n * p * FP32_SHARE,
+                requests * 2 * H * n * p * 4 + T * (2 * G * n * 4 + 2 * H * p * 4 + 2 * H * 4))
     if k == "gated_norm":
         cols = a["y"].shape[1]
-        return f"gate + norm in groups of {a['group']}" + (", normalised" if a.get("floor") is not None else ""), 0.0, T * cols * (4 + 2 * el)
+        return f"gate + norm in groups of {a['group']}" + (", normalised" if a.get("floor") is not None else ""), 0.0, T * cols * (4 + a["gate"].element_size() + el)
     return k, 0.0, 0.0
 
 
@@ -239,13 +273,13 @@ def layer_table(cfg, layers: int, batch: int, page: int, pk) -> Dict[str, List[D
     compiled = eng.ops.compile(plan)
     # which records belong to which layer: every block emits once more into a plan of its own, and is counted
     from .engine.plan import Plan
-    from .parts.base import emit_block, emit_embedding
+    from .parts.base import emit_embedding
     scratch = Plan()
     x = emit_embedding(scratch, eng.model.embedding, eng.spec.hidden_size)
     per_layer, delta = [], None
-    for i, run_ in enumerate(eng.model.order):
+    for i in range(len(eng.model.order)):
         at = len(scratch.ops)
-        x, delta = emit_block(scratch, eng.model.blocks[run_.layer], x, delta, eng._caches[i])
+        x, delta = eng.model.emit_run(scratch, i, x, delta, eng._caches)
         per_layer.append(list(range(at, len(scratch.ops))))
     assert len(scratch.ops) + 2 == len(plan.ops), "the plan is not embedding, layers, final norm, head"
     assert all(a.kind == b.kind for a, b in zip(scratch.ops, plan.ops))
@@ -359,13 +393,20 @@ def run(args, pk) -> int:
 
     import torch
     design_name = getattr(args, "design", None) or "bepuzen"
-    table_of_sizes = {"bepuzen": SIZES, "torisun": TORISUN_SIZES, "vifelix": VIFELIX_SIZES, "funevik": FUNEVIK_SIZES}[design_name]
+    table_of_sizes = {"bepuzen": SIZES, "torisun": TORISUN_SIZES, "vifelix": VIFELIX_SIZES, "funevik": FUNEVIK_SIZES,
+                      "vaderax": VADERAX_SIZES}[design_name]
     global FP32_SHARE
     FP32_SHARE = pk["bf16_tflops"] / FP32_TFLOPS
     sizes = [args.size] if getattr(args, "size", None) else list(table_of_sizes)
     rec: Dict[str, Any] = {"metric": f"{design_name.capitalize()} beside the grouped-query model of equal size, bf16: tokens/s and per-record rooflines",
                            "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic token ids, random weights",
                            "peaks": pk["source"], "page_size": args.page_size, "cached_tokens": CACHED, "sizes": {}}
+    ROUTED_SHARE.clear()
+    for _, design, _ in table_of_sizes.values():
+        for L in design.get("layers", []):
+            r = (L.get("mlp") or {}).get("router", {})
+            if r.get("identity"):
+                ROUTED_SHARE[r["experts"], r["top"]] = r["experts"] / (r["experts"] + r["identity"])
     for name in sizes:
         layers, design, closest = table_of_sizes[name]
         entry: Dict[str, Any] = {"layers": layers}
