@@ -106,7 +106,7 @@ def vaderax_shape(width: int, heads: int, kv_heads: int, ff: int, experts: int, 
     at = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": {"base": 10000.0, "dims": dim // 2}}
     dense = {"kind": "dense", "ff": ff}
     routed = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "identity": experts // 8,
-                                                                     "groups": {"count": 8, "keep": 4}}}
+                                                                     "groups": {"count": 4, "keep": 2}}}
     kinds = [("delta", de, dense), ("delta", de, routed), ("attention", at, routed), ("delta", de, dense)]
     return {"architecture": "Vaderax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5},
             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in kinds], "loop": {"start": 1, "stop": 3, "times": 2}}

@@ -77,9 +77,10 @@ def causal_conv(u: torch.Tensor, taps: torch.Tensor) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------- mixers
-def delta_rule(q, k, v, beta, keep, S=None):
+def delta_rule(q, k, v, beta, keep, S=None, sizes=None):
     """q, k [T, H, d], v [T, H, P], beta and keep [T, H].  Per head: the memory decays, S <- keep S; what it answers to k is
-    corrected towards v, u = beta (v - S^T k), S <- S + k u^T; then it is read, o = S^T q.  Returns o [T, H, P], S [H, d, P]."""
+    corrected towards v, u = beta (v - S^T k), S <- S + k u^T; then it is read, o = S^T q.  Returns o [T, H, P], S [H, d, P];
+    `sizes` (a list) receives the norm of every head's S per token."""
     T, H, d = q.shape
     if S is None:
         S = torch.zeros(H, d, v.shape[-1], dtype=q.dtype)
@@ -89,6 +90,8 @@ def delta_rule(q, k, v, beta, keep, S=None):
         u = beta[t][:, None] * (v[t] - torch.einsum("adp,ad->ap", S, k[t]))
         S = S + k[t][:, :, None] * u[:, None, :]
         out.append(torch.einsum("adp,ad->ap", S, q[t]))
+        if sizes is not None:
+            sizes.append(S.flatten(1).norm(dim=-1))
     return torch.stack(out), S
 
 
@@ -109,16 +112,11 @@ def delta_mixer(h, w, pre, m, eps, round_to, calls=None):
     v = mix("v").view(T, H, P)
     beta = torch.sigmoid(h @ w[pre + "b"].t())
     keep = torch.exp(-torch.exp(w[pre + "A_log"]) * softplus(h @ w[pre + "a"].t() + w[pre + "dt_bias"]))
-    if calls is None:
-        o, _ = delta_rule(q, k, v, beta, keep)
-    else:
-        o, away, S = torch.empty(T, H, P, dtype=h.dtype), torch.empty(T), None
-        for t in range(T):
-            step = slice(t, t + 1)
-            o[step], S = delta_rule(q[step], k[step], v[step], beta[step], keep[step], S)
-            hold = S.flatten(1).norm(dim=-1) * q[t].norm(dim=-1)
-            away[t] = 2.5 * math.sqrt(d) * float((o[t].norm(dim=-1) / hold.clamp_min(1e-30)).min())
-        calls.append(away)
+    sizes = None if calls is None else []
+    o, _ = delta_rule(q, k, v, beta, keep, sizes=sizes)
+    if calls is not None:
+        hold = torch.stack(sizes) * q.norm(dim=-1)
+        calls.append((2.5 * math.sqrt(d) * (o.norm(dim=-1) / hold.clamp_min(1e-30)).amin(-1)).to(torch.float32))
     o = (unit_rms(o, eps) * w[pre + "norm"]).reshape(T, H * P)
     return o * silu(_r(h @ w[pre + "g"].t(), round_to))
 

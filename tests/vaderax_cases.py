@@ -2,6 +2,8 @@
 plain implementation."""
 from __future__ import annotations
 
+import hashlib
+import os
 from typing import Dict, List, Optional, Sequence
 
 import torch
@@ -21,11 +23,15 @@ def keep_away_from_close_calls(model: PlainVaderax, reqs: Dict[str, List[int]], 
     vocabulary (positions before it are not affected: the model is causal)."""
     vocab = model.cfg["vocab"]
     for r, ids in reqs.items():
-        for _ in range(40 * len(ids)):
-            model.logits(ids)
+        n = 8                                  # a beginning that grows: the model is causal, so what is settled stays settled
+        for _ in range(60 * len(ids)):
+            model.logits(ids[:n])
             close = (model.gaps < margin).nonzero()
             if not close.numel():
-                break
+                if n >= len(ids):
+                    break
+                n = n * 5 // 4 + 2
+                continue
             p = int(close[0])
             ids[p] = (ids[p] + 1) % vocab
         else:
@@ -38,15 +44,30 @@ def reference_logits(model_dir: str, reqs: Dict[str, List[int]], dtype: str):
     and only a run that rounds where the engine rounds takes the same choices.  The yardstick of the tolerance is the model's
     own sensitivity to rounding (the distance between the rounded and the unrounded plain run): the engine must stay within two
     yardsticks of the rounded run (it also rounds the attention's probabilities and adds in another order)."""
+    with open(os.path.join(model_dir, "config.json"), "rb") as f, open(os.path.join(model_dir, "model.safetensors"), "rb") as g:
+        key = (f.read(), hashlib.sha256(g.read()).hexdigest(), dtype, repr(reqs))
+    if key not in _SETTLED:                    # the same model and requests serve several tests (both kernel sets, two page sizes)
+        _SETTLED[key] = _settle(model_dir, reqs, dtype)
+    settled, ref, tol = _SETTLED[key]
+    for r, ids in settled.items():
+        reqs[r][:] = ids
+    return ref, tol
+
+
+_SETTLED: Dict[tuple, tuple] = {}
+
+
+def _settle(model_dir: str, reqs: Dict[str, List[int]], dtype: str):
+    reqs = {r: list(ids) for r, ids in reqs.items()}
     plain = PlainVaderax(model_dir)
     rounded = PlainVaderax(model_dir, round_to=torch.bfloat16)
-    keep_away_from_close_calls(rounded if dtype == "bfloat16" else plain, reqs, 0.25 if dtype == "bfloat16" else 2e-4)
+    keep_away_from_close_calls(rounded if dtype == "bfloat16" else plain, reqs, 0.12 if dtype == "bfloat16" else 2e-4)
     ref = {r: plain.logits(ids) for r, ids in reqs.items()}
     if dtype != "bfloat16":
-        return ref, TOL_F32 * max(1.0, max(float(v.abs().max()) for v in ref.values()) / 10.0)
+        return reqs, ref, TOL_F32 * max(1.0, max(float(v.abs().max()) for v in ref.values()) / 10.0)
     ref16 = {r: rounded.logits(ids) for r, ids in reqs.items()}
     inherent = max(float((ref16[r] - ref[r]).abs().max()) for r in ref)
-    return ref16, max(5e-3, 2.0 * inherent)
+    return reqs, ref16, max(5e-3, 2.0 * inherent)
 
 
 def replay_all_schedules(model_dir: str, cfg: dict, dtype: str, lens: Sequence[int], page: int, ops, device: str,
