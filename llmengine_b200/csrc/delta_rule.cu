@@ -9,16 +9,17 @@
 // norms and gates are formed in the kernel.  The kernel takes any number of tokens, one after the other: it is also the plain
 // form of portions.
 //
-// Portions (delta_prepare_kernel, delta_tile_kernel): a request's tokens are taken FOUR at a time.  With G(i, j) = the product of
+// Portions (delta_prepare_kernel, delta_tile_kernel): a request's tokens are taken EIGHT at a time.  With G(i, j) = the product of
 // the decays of tokens j + 1 .. i (G(i) from the block's start) and S0 the state before the block,
-//   u_i = b_i (v_i - G(i) S0^T k_i - sum_(j < i) G(i, j) (k_j . k_i) u_j),
-//   o_i = G(i) S0^T q_i + sum_(j <= i) G(i, j) (k_j . q_i) u_j,
-//   S   = G(3) S0 + sum_j G(3, j) k_j u_j^T,
-// which is the rule above written out: the eight products with S0 do not wait for one another, their sums over the lanes are
-// formed together, and what is left in sequence is a triangular solve of four numbers per column.  The numbers that do not
-// depend on a column (40 per block and head) and the unit vectors are made by delta_prepare_kernel for all blocks side by side.
-// No quotient of decays is ever formed, so a decay of zero is harmless.  A block at a portion's end is filled up with tokens that
-// change nothing (k = q = 0, b = 0, a = 1); how a prompt is cut into steps changes the order of the sums and nothing else.
+//   u_i = r_i - sum_(j < i) A_ij u_j,   r_i = b_i (v_i - G(i) S0^T k_i),   A_ij = b_i G(i, j) k_j . k_i,
+//   o_i = G(i) S0^T q_i + sum_(j <= i) B_ij u_j,   B_ij = G(i, j) k_j . q_i,
+//   S   = G(7) S0 + sum_j G(7, j) k_j u_j^T,
+// which is the rule above written out.  The sixteen products with S0 do not wait for one another, and their sums over the lanes are
+// formed together.  What does not depend on a column is made by delta_prepare_kernel for all blocks side by side: the unit vectors,
+// the inverse N of the unit lower triangular I + A, and B N, so that u = N r and o = G S0^T q + (B N) r: lane i of a column forms
+// u_i and o_i from the eight r's, and nothing is left to be solved in sequence.  No quotient of decays is ever formed, so a decay of
+// zero is harmless.  A block at a portion's end is filled up with tokens that change nothing (k = q = 0, b = 0, a = 1); how a
+// prompt is cut into steps changes the order of the sums and nothing else.
 #include "common.cuh"
 #include "kernel_args.h"
 
@@ -26,7 +27,8 @@ LLME_API const char* llme_last_error() { return llme_error_buffer(); }
 
 namespace {
 
-constexpr int BLOCK = 4, QUADS = 10;             // tokens of a block; groups of four numbers that a block and head need
+constexpr int BLOCK = 8, ROW_NUMBERS = 20;       // tokens of a block; numbers that a token of a block and head needs: b, b G, G, G(7, .),
+constexpr int NUMBERS = BLOCK * ROW_NUMBERS;      // a row of N, a row of B N
 
 __device__ __forceinline__ float softplus32(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float write_strength(float z) { return 1.0f / (1.0f + expf(-z)); }
@@ -182,17 +184,29 @@ void launch_step(const LlmeDeltaArgs& a, int vec_state, int vec_qk, cudaStream_t
 }
 
 // ----------------------------------------------------------------------------- portions: what no column has a say in
-// Block number of request r's b-th block: floor(first token / 4) + r + b (distinct for all blocks of a step).
-__device__ __forceinline__ int first_block(const int* __restrict__ cu, int r) { return (cu[r] >> 2) + r; }
+// Block number of request r's b-th block: floor(first token / 8) + r + b (distinct for all blocks of a step).
+__device__ __forceinline__ int first_block(const int* __restrict__ cu, int r) { return cu[r] / BLOCK + r; }
 
-// One warp per (block, query/key group): unit queries and keys, their products within the block, and per head of the group
-//   0: b_i   1: b_i G(i)   2: A10 A20 A21 A30   3: A31 A32 0 G(3)   4: G(3, i)   5: G(i)   6 + i: B_i0 .. B_i3
-// with A_ij = b_i G(i, j) k_j . k_i and B_ij = G(i, j) k_j . q_i (zero for j > i).
-template <int R>
-__global__ void __launch_bounds__(128) delta_prepare_kernel(LlmeDeltaArgs a) {
+// Sums over the warp of 32 values a lane: lane i ends with the sum of everybody's v[i].
+__device__ __forceinline__ float sums_of_32(float (&v)[32], int lane) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < o; ++i) v[i] = (up ? v[i + o] : v[i]) + __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + o], o);
+    }
+    return v[0];
+}
+
+// One warp per (block, query/key group).
+constexpr int PREPARE_WARPS = 4;
+
+__global__ void __launch_bounds__(32 * PREPARE_WARPS) delta_prepare_kernel(LlmeDeltaArgs a) {
+    // sums: [0, 36) k_j . q_i at i (i + 1) / 2 + j; [36, 64) k_j . k_i (j < i) at i (i - 1) / 2 + j; [64, 72) |q_i|^2; [72, 80) |k_i|^2
+    __shared__ float sums_of[PREPARE_WARPS][96];
     pdl_launch_dependents();
     pdl_wait();
-    const int lane = threadIdx.x & 31, id = blockIdx.x, g = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, id = blockIdx.x, g = blockIdx.y * PREPARE_WARPS + warp;
     if (g >= a.qk_groups) return;
     int lo = 0, hi = a.requests;                                // the last request whose first block is not behind `id`
     while (hi - lo > 1) {
@@ -202,56 +216,59 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(LlmeDeltaArgs a) {
     const int len = a.cu_q_lens[lo + 1] - a.cu_q_lens[lo], at = BLOCK * (id - first_block(a.cu_q_lens, lo));
     if (at < 0 || at >= len || len < 2) return;                 // a number no block has, or a single token
     const int t0 = a.cu_q_lens[lo] + at, count = min(BLOCK, len - at), n = a.n, n4 = (n + 3) & ~3;
-    float q[BLOCK][R], k[BLOCK][R];
+    float* sums = sums_of[warp];
+    const float* qp = a.q + (size_t)t0 * a.ldq + (size_t)g * n;
+    const float* kp = a.k + (size_t)t0 * a.ldk + (size_t)g * n;
+    {
+        float s0[32], s1[32], s2[32];
 #pragma unroll
-    for (int j = 0; j < BLOCK; ++j)
+        for (int i = 0; i < 32; ++i) s0[i] = s1[i] = s2[i] = 0.0f;
+        auto slot = [&](int i) -> float& { return i < 32 ? s0[i] : i < 64 ? s1[i - 32] : s2[i - 64]; };
+        for (int e = lane; e < n; e += 32) {
+            float q[BLOCK], k[BLOCK];
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int e = lane + 32 * i;
-            const bool ok = j < count && e < n;
-            q[j][i] = ok ? a.q[(size_t)(t0 + j) * a.ldq + (size_t)g * n + e] : 0.0f;
-            k[j][i] = ok ? a.k[(size_t)(t0 + j) * a.ldk + (size_t)g * n + e] : 0.0f;
+            for (int j = 0; j < BLOCK; ++j) {
+                q[j] = j < count ? qp[(size_t)j * a.ldq + e] : 0.0f;
+                k[j] = j < count ? kp[(size_t)j * a.ldk + e] : 0.0f;
+            }
+#pragma unroll
+            for (int i = 0; i < BLOCK; ++i) {
+                slot(64 + i) = fmaf(q[i], q[i], slot(64 + i));
+                slot(72 + i) = fmaf(k[i], k[i], slot(72 + i));
+#pragma unroll
+                for (int j = 0; j <= i; ++j) {
+                    slot(i * (i + 1) / 2 + j) = fmaf(k[j], q[i], slot(i * (i + 1) / 2 + j));
+                    if (j < i) slot(36 + i * (i - 1) / 2 + j) = fmaf(k[j], k[i], slot(36 + i * (i - 1) / 2 + j));
+                }
+            }
         }
+        sums[lane] = sums_of_32(s0, lane);
+        sums[32 + lane] = sums_of_32(s1, lane);
+        sums[64 + lane] = sums_of_32(s2, lane);
+    }
+    __syncwarp();
+    // 1 / |.| of the queries (times their constant) and of the keys, in the places of their squares
+    if (lane < 2 * BLOCK) sums[64 + lane] = (lane < BLOCK ? a.q_scale : 1.0f) / sqrtf(sums[64 + lane] + a.unit_eps);
+    __syncwarp();
+    float iq[BLOCK], ik[BLOCK];
 #pragma unroll
     for (int j = 0; j < BLOCK; ++j) {
-        float sq = 0.0f, sk = 0.0f;
+        iq[j] = sums[64 + j];
+        ik[j] = sums[72 + j];
+    }
+    for (int e = lane; e < n4; e += 32) {
+        float* uq = a.unit + ((size_t)t0 * 2 * a.qk_groups + g) * n4 + e;
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-            sq = fmaf(q[j][i], q[j][i], sq);
-            sk = fmaf(k[j][i], k[j][i], sk);
-        }
-        const float iq = a.q_scale / sqrtf(warp_sum(sq) + a.unit_eps), ik = 1.0f / sqrtf(warp_sum(sk) + a.unit_eps);
-        float* uq = a.unit + ((size_t)(t0 + j) * 2 * a.qk_groups + g) * n4;
-        float* uk = uq + (size_t)a.qk_groups * n4;
-#pragma unroll
-        for (int i = 0; i < R; ++i) {
-            const int e = lane + 32 * i;
-            q[j][i] *= iq;
-            k[j][i] *= ik;
-            if (j < count && e < n4) {
-                uq[e] = q[j][i];
-                uk[e] = k[j][i];
-            }
+        for (int j = 0; j < BLOCK; ++j) {
+            if (j >= count) break;
+            uq[(size_t)j * 2 * a.qk_groups * n4] = e < n ? qp[(size_t)j * a.ldq + e] * iq[j] : 0.0f;
+            uq[((size_t)j * 2 + 1) * a.qk_groups * n4] = e < n ? kp[(size_t)j * a.ldk + e] * ik[j] : 0.0f;
         }
     }
-    float kk[BLOCK][BLOCK], qk[BLOCK][BLOCK];                   // [i][j], j < i and j <= i
-#pragma unroll
-    for (int i = 0; i < BLOCK; ++i)
-#pragma unroll
-        for (int j = 0; j <= i; ++j) {
-            float x = 0.0f, y = 0.0f;
-#pragma unroll
-            for (int e = 0; e < R; ++e) {
-                if (j < i) x = fmaf(k[j][e], k[i][e], x);
-                y = fmaf(k[j][e], q[i][e], y);
-            }
-            if (j < i) kk[i][j] = warp_sum(x);
-            qk[i][j] = warp_sum(y);
-        }
-    // four lanes per head: each forms its token's two gates, all four then hold the block's
-    const int rep = a.heads / a.qk_groups, j = lane & 3;
-    for (int x0 = 0; x0 < rep; x0 += 8) {
-        const int x = x0 + (lane >> 2), h = g * rep + x;
+    // eight lanes per head: each forms its token's two gates, all eight then hold the block's, and lane j forms column j of N and B N
+    const int rep = a.heads / a.qk_groups, j = lane & 7;
+    for (int x0 = 0; x0 < rep; x0 += 4) {
+        const int x = x0 + (lane >> 3), h = g * rep + x;
         float beta = 0.0f, keep = 1.0f;
         if (x < rep && j < count) {
             beta = write_strength(a.write[(size_t)(t0 + j) * a.ld_gates + h]);
@@ -260,31 +277,34 @@ __global__ void __launch_bounds__(128) delta_prepare_kernel(LlmeDeltaArgs a) {
         float b[BLOCK], w[BLOCK];
 #pragma unroll
         for (int i = 0; i < BLOCK; ++i) {
-            b[i] = __shfl_sync(0xffffffffu, beta, (lane & ~3) + i);
-            w[i] = __shfl_sync(0xffffffffu, keep, (lane & ~3) + i);
+            b[i] = __shfl_sync(0xffffffffu, beta, (lane & ~7) + i);
+            w[i] = __shfl_sync(0xffffffffu, keep, (lane & ~7) + i);
         }
         if (x >= rep) continue;
-        const float g1 = w[0] * w[1], g2 = g1 * w[2], g3 = g2 * w[3], w12 = w[1] * w[2], w23 = w[2] * w[3], w123 = w12 * w[3];
-        float4* o = (float4*)(a.coef + ((size_t)id * a.heads + h) * (4 * QUADS));
-        if (j == 0) {
-            o[0] = make_float4(b[0], b[1], b[2], b[3]);
-            o[4] = make_float4(w123, w23, w[3], 1.0f);
-            o[8] = make_float4(w12 * qk[2][0], w[2] * qk[2][1], qk[2][2], 0.0f);
-        } else if (j == 1) {
-            o[1] = make_float4(b[0] * w[0], b[1] * g1, b[2] * g2, b[3] * g3);
-            o[5] = make_float4(w[0], g1, g2, g3);
-            o[9] = make_float4(w123 * qk[3][0], w23 * qk[3][1], w[3] * qk[3][2], qk[3][3]);
-        } else if (j == 2) {
-            o[2] = make_float4(b[1] * w[1] * kk[1][0], b[2] * w12 * kk[2][0], b[2] * w[2] * kk[2][1], b[3] * w123 * kk[3][0]);
-            o[6] = make_float4(qk[0][0], 0.0f, 0.0f, 0.0f);
-        } else {
-            o[3] = make_float4(b[3] * w23 * kk[3][1], b[3] * w[3] * kk[3][2], 0.0f, g3);
-            o[7] = make_float4(w[1] * qk[1][0], qk[1][1], 0.0f, 0.0f);
+        float* o = a.coef + ((size_t)id * a.heads + h) * NUMBERS;
+        float G[BLOCK], N[BLOCK], from_start = 1.0f, to_end = 1.0f;
+#pragma unroll
+        for (int i = 0; i < BLOCK; ++i) {
+#pragma unroll
+            for (int m = 0; m < i; ++m) G[m] *= w[i];            // G(i, m)
+            G[i] = 1.0f;
+            float below = 0.0f, read = 0.0f;
+#pragma unroll
+            for (int m = 0; m < i; ++m) below = fmaf(G[m] * (sums[36 + i * (i - 1) / 2 + m] * ik[m]), N[m], below);
+            N[i] = i == j ? 1.0f : -(b[i] * ik[i]) * below;      // zero above the diagonal: `below` is zero there
+#pragma unroll
+            for (int m = 0; m <= i; ++m) read = fmaf(G[m] * (sums[i * (i + 1) / 2 + m] * ik[m]), N[m], read);
+            o[i * ROW_NUMBERS + 4 + j] = N[i];
+            o[i * ROW_NUMBERS + 12 + j] = read * iq[i];
+            if (i <= j) from_start *= w[i];
+            else to_end *= w[i];
         }
+        const float mine = beta;
+        *(float4*)(o + j * ROW_NUMBERS) = make_float4(mine, mine * from_start, from_start, to_end);
     }
 }
 
-// ----------------------------------------------------------------------------- portions: four tokens at a time
+// ----------------------------------------------------------------------------- portions: eight tokens at a time
 // A block of W warps takes W * 32 / L * C neighbouring columns of one (request, head).  Unit queries and keys, values and the
 // blocks' numbers come into shared memory TT tokens at a time by asynchronous copies, NS tiles deep.
 constexpr int TT = 16;
@@ -292,7 +312,7 @@ constexpr int TT = 16;
 template <int L, int M, int C, int W, int NS>
 struct DeltaTile {
     static constexpr int ROW = 4 * L * M, COLS = W * (32 / L) * C;
-    float q[NS][TT][ROW], k[NS][TT][ROW], v[NS][TT][COLS], coef[NS][TT / BLOCK][4 * QUADS];
+    float q[NS][TT][ROW], k[NS][TT][ROW], v[NS][TT][COLS], coef[NS][TT / BLOCK][NUMBERS];
 };
 
 template <int L, int M, int C, int W, int NS>
@@ -301,9 +321,7 @@ __global__ void __launch_bounds__(32 * W) delta_tile_kernel(LlmeDeltaArgs a, int
     constexpr int ROW = Tile::ROW, COLS = Tile::COLS, P2 = 2 * M;         // packed pairs of rows a lane holds per column
     extern __shared__ __align__(16) unsigned char smem_raw[];
     Tile& sm = *reinterpret_cast<Tile*>(smem_raw);
-    pdl_launch_dependents();
-    pdl_wait();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane % L;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane % L, row = sub & 7, base = lane & ~(L - 1);
     const int jb = blockIdx.x * COLS, mine = (warp * (32 / L) + lane / L) * C, col0 = jb + mine;
     const int h = blockIdx.y, r = a.rows ? a.rows[blockIdx.z] : (int)blockIdx.z, n = a.n, p = a.p, n4 = (n + 3) & ~3;
     const int first = a.cu_q_lens[r], last = a.cu_q_lens[r + 1], g = h / (a.heads / a.qk_groups);
@@ -326,10 +344,10 @@ __global__ void __launch_bounds__(32 * W) delta_tile_kernel(LlmeDeltaArgs a, int
                 const bool ok = t0 + u < last && jb + c < p;
                 copy_async_4(&sm.v[s][u][c], ok ? a.v + (size_t)(t0 + u) * a.ldv + (size_t)h * p + jb + c : a.v, ok);
             }
-            for (int i = tid; i < TT / BLOCK * QUADS; i += 32 * W) {
-                const int b = i / QUADS, e = (i % QUADS) * 4;
+            for (int i = tid; i < TT / BLOCK * (NUMBERS / 4); i += 32 * W) {
+                const int b = i / (NUMBERS / 4), e = (i % (NUMBERS / 4)) * 4;
                 const bool ok = t0 + BLOCK * b < last;
-                copy_async_16(&sm.coef[s][b][e], ok ? a.coef + ((size_t)(block0 + tile * (TT / BLOCK) + b) * a.heads + h) * (4 * QUADS) + e : a.coef, ok);
+                copy_async_16(&sm.coef[s][b][e], ok ? a.coef + ((size_t)(block0 + tile * (TT / BLOCK) + b) * a.heads + h) * NUMBERS + e : a.coef, ok);
             }
         }
         copy_async_commit();                                    // one group a tile, also an empty one: the waits below count them
@@ -352,78 +370,96 @@ __global__ void __launch_bounds__(32 * W) delta_tile_kernel(LlmeDeltaArgs a, int
         __syncthreads();                                        // ... for every thread, and the tile before has been read by all
         fetch(tile + NS - 1);
         const int s = tile % NS, t0 = first + tile * TT;
-#pragma unroll
+#pragma unroll 1
         for (int b = 0; b < TT / BLOCK; ++b) {
             if (t0 + BLOCK * b >= last) break;                  // (uniform over the block)
             f32x2 k[BLOCK][P2];
             float part[C][2 * BLOCK];                           // this lane's share of S0^T k_i, then of S0^T q_i
 #pragma unroll
-            for (int i = 0; i < BLOCK; ++i) {
-                f32x2 acc[C];
-#pragma unroll
-                for (int c = 0; c < C; ++c) acc[c] = pack2(0.0f, 0.0f);
+            for (int i = 0; i < BLOCK; ++i)
 #pragma unroll
                 for (int m = 0; m < M; ++m) {
                     const ulonglong2 f = *(const ulonglong2*)&sm.k[s][BLOCK * b + i][4 * (sub + L * m)];
                     k[i][2 * m] = f.x;
                     k[i][2 * m + 1] = f.y;
-#pragma unroll
-                    for (int c = 0; c < C; ++c) acc[c] = fma2(S[c][2 * m + 1], f.y, fma2(S[c][2 * m], f.x, acc[c]));
                 }
-#pragma unroll
-                for (int c = 0; c < C; ++c) part[c][i] = sum2(acc[c]);
-            }
-#pragma unroll
-            for (int i = 0; i < BLOCK; ++i) {
-                f32x2 acc[C];
-#pragma unroll
-                for (int c = 0; c < C; ++c) acc[c] = pack2(0.0f, 0.0f);
-#pragma unroll
-                for (int m = 0; m < M; ++m) {
-                    const ulonglong2 f = *(const ulonglong2*)&sm.q[s][BLOCK * b + i][4 * (sub + L * m)];
-#pragma unroll
-                    for (int c = 0; c < C; ++c) acc[c] = fma2(S[c][2 * m + 1], f.y, fma2(S[c][2 * m], f.x, acc[c]));
-                }
-#pragma unroll
-                for (int c = 0; c < C; ++c) part[c][BLOCK + i] = sum2(acc[c]);
-            }
-            const float4* cf = (const float4*)sm.coef[s][b];
-            const float4 cb = cf[0], cbg = cf[1], ca = cf[2], ca2 = cf[3], cu = cf[4];
-            const int mi = sub & 3;
-            const float gi = sm.coef[s][b][20 + mi];
-            const float4 cB = cf[6 + mi];
+            const float* cf = sm.coef[s][b] + row * ROW_NUMBERS;
+            const float4 own = *(const float4*)cf;              // b, b G, G and G(7, .) of the token this lane stands for
+            const float total = sm.coef[s][b][(BLOCK - 1) * ROW_NUMBERS + 2];
 #pragma unroll
             for (int c = 0; c < C; ++c) {
-                // lanes exchange halves of what they hold until lane `sub` has the whole sum number sub % 8: 0..3 with the
-                // keys, 4..7 with the queries
+                f32x2 acc[BLOCK];
+#pragma unroll
+                for (int i = 0; i < BLOCK; ++i) acc[i] = mul2(S[c][0], k[i][0]);
+#pragma unroll
+                for (int e = 1; e < P2; ++e)
+#pragma unroll
+                    for (int i = 0; i < BLOCK; ++i) acc[i] = fma2(S[c][e], k[i][e], acc[i]);
+#pragma unroll
+                for (int i = 0; i < BLOCK; ++i) part[c][i] = sum2(acc[i]);
+            }
+            {
+                f32x2 acc[C][BLOCK];
+#pragma unroll
+                for (int m = 0; m < M; ++m)
+#pragma unroll
+                    for (int i = 0; i < BLOCK; ++i) {
+                        const ulonglong2 f = *(const ulonglong2*)&sm.q[s][BLOCK * b + i][4 * (sub + L * m)];
+#pragma unroll
+                        for (int c = 0; c < C; ++c)
+                            acc[c][i] = fma2(S[c][2 * m + 1], f.y, m == 0 ? mul2(S[c][0], f.x) : fma2(S[c][2 * m], f.x, acc[c][i]));
+                    }
+#pragma unroll
+                for (int c = 0; c < C; ++c)
+#pragma unroll
+                    for (int i = 0; i < BLOCK; ++i) part[c][BLOCK + i] = sum2(acc[c][i]);
+            }
+            const float4 n0 = *(const float4*)(cf + 4), n1 = *(const float4*)(cf + 8), r0 = *(const float4*)(cf + 12), r1 = *(const float4*)(cf + 16);
+#pragma unroll
+            for (int c = 0; c < C; ++c) {
+                // lanes exchange halves of what they hold until every lane has two whole sums: those of token sub % 8 with its key
+                // and with its query
                 const bool up4 = sub & 4, up2 = sub & 2, up1 = sub & 1;
-                float x[4], y[2], z;
+                float x[2][4], y[2][2], z[2];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) x[i] = (up4 ? part[c][i + 4] : part[c][i]) + __shfl_xor_sync(0xffffffffu, up4 ? part[c][i] : part[c][i + 4], 4);
+                for (int f = 0; f < 2; ++f)
 #pragma unroll
-                for (int i = 0; i < 2; ++i) y[i] = (up2 ? x[i + 2] : x[i]) + __shfl_xor_sync(0xffffffffu, up2 ? x[i] : x[i + 2], 2);
-                z = (up1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, up1 ? y[0] : y[1], 1);
+                    for (int i = 0; i < 4; ++i) {
+                        const float low = part[c][BLOCK * f + i], high = part[c][BLOCK * f + i + 4];
+                        x[f][i] = (up4 ? high : low) + __shfl_xor_sync(0xffffffffu, up4 ? low : high, 4);
+                    }
 #pragma unroll
-                for (int o = 8; o < L; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-                const int base = lane & ~(L - 1);
-                const float d0 = __shfl_sync(0xffffffffu, z, base), d1 = __shfl_sync(0xffffffffu, z, base + 1);
-                const float d2 = __shfl_sync(0xffffffffu, z, base + 2), d3 = __shfl_sync(0xffffffffu, z, base + 3);
-                const float v0 = sm.v[s][BLOCK * b][mine + c], v1 = sm.v[s][BLOCK * b + 1][mine + c];
-                const float v2 = sm.v[s][BLOCK * b + 2][mine + c], v3 = sm.v[s][BLOCK * b + 3][mine + c];
-                const float u0 = fmaf(-cbg.x, d0, cb.x * v0);
-                const float u1 = fmaf(-ca.x, u0, fmaf(-cbg.y, d1, cb.y * v1));
-                const float u2 = fmaf(-ca.z, u1, fmaf(-ca.y, u0, fmaf(-cbg.z, d2, cb.z * v2)));
-                const float u3 = fmaf(-ca2.y, u2, fmaf(-ca2.x, u1, fmaf(-ca.w, u0, fmaf(-cbg.w, d3, cb.w * v3))));
-                if (sub >= 4 && sub < 8) {
-                    const int t = t0 + BLOCK * b + mi;
-                    const float o = fmaf(cB.w, u3, fmaf(cB.z, u2, fmaf(cB.y, u1, fmaf(cB.x, u0, gi * z))));
-                    if (t < last && col0 + c < p) a.out[(size_t)t * a.ldo + (size_t)h * p + col0 + c] = o;
+                for (int f = 0; f < 2; ++f)
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) y[f][i] = (up2 ? x[f][i + 2] : x[f][i]) + __shfl_xor_sync(0xffffffffu, up2 ? x[f][i] : x[f][i + 2], 2);
+#pragma unroll
+                for (int f = 0; f < 2; ++f) {
+                    z[f] = (up1 ? y[f][1] : y[f][0]) + __shfl_xor_sync(0xffffffffu, up1 ? y[f][0] : y[f][1], 1);
+#pragma unroll
+                    for (int o = 8; o < L; o <<= 1) z[f] += __shfl_xor_sync(0xffffffffu, z[f], o);
                 }
-                const float w0 = cu.x * u0, w1 = cu.y * u1, w2 = cu.z * u2, w3 = cu.w * u3;
-                const f32x2 p0 = pack2(w0, w0), p1 = pack2(w1, w1), p2 = pack2(w2, w2), p3 = pack2(w3, w3), gt = pack2(ca2.w, ca2.w);
+                const f32x2 kept = pack2(total, total);
 #pragma unroll
-                for (int i = 0; i < P2; ++i)
-                    S[c][i] = fma2(k[3][i], p3, fma2(k[2][i], p2, fma2(k[1][i], p1, fma2(k[0][i], p0, mul2(gt, S[c][i])))));
+                for (int e = 0; e < P2; ++e) S[c][e] = mul2(kept, S[c][e]);
+                // r of this lane's token, everybody's r, then u and o of this lane's token
+                const float mine_r = fmaf(-own.y, z[0], own.x * sm.v[s][BLOCK * b + row][mine + c]);
+                float rr[BLOCK];
+#pragma unroll
+                for (int i = 0; i < BLOCK; ++i) rr[i] = __shfl_sync(0xffffffffu, mine_r, base + i);
+                const float u = fmaf(n1.w, rr[7], n1.z * rr[6]) + fmaf(n1.y, rr[5], n1.x * rr[4]) + (fmaf(n0.w, rr[3], n0.z * rr[2]) + fmaf(n0.y, rr[1], n0.x * rr[0]));
+                const float write = own.w * u;
+                float o = own.z * z[1];
+                o = fmaf(r0.x, rr[0], o); o = fmaf(r0.y, rr[1], o); o = fmaf(r0.z, rr[2], o); o = fmaf(r0.w, rr[3], o);
+                o = fmaf(r1.x, rr[4], o); o = fmaf(r1.y, rr[5], o); o = fmaf(r1.z, rr[6], o); o = fmaf(r1.w, rr[7], o);
+                const int t = t0 + BLOCK * b + row;
+                if (sub < BLOCK && t < last && col0 + c < p) a.out[(size_t)t * a.ldo + (size_t)h * p + col0 + c] = o;
+#pragma unroll
+                for (int i = 0; i < BLOCK; ++i) {
+                    const float wi = __shfl_sync(0xffffffffu, write, base + i);
+                    const f32x2 w2 = pack2(wi, wi);
+#pragma unroll
+                    for (int e = 0; e < P2; ++e) S[c][e] = fma2(k[i][e], w2, S[c][e]);
+                }
             }
         }
     }
@@ -447,7 +483,9 @@ int launch_tile(const LlmeDeltaArgs& a, int vec_state, cudaStream_t s) {
             LLME_REFUSE("delta_rule: %zu bytes of shared memory are not available", sizeof(Tile));
         configured = true;
     }
-    llme_launch(kernel, dim3((a.p + Tile::COLS - 1) / Tile::COLS, a.heads, a.n_rows), dim3(32 * W), sizeof(Tile), s, a, vec_state);
+    // An ordinary launch, which waits for the kernel before it: let in early, the blocks would crowd on the first SMs that have
+    // room (there are about as many blocks as SMs), and the walk would take twice its time.
+    kernel<<<dim3((a.p + Tile::COLS - 1) / Tile::COLS, a.heads, a.n_rows), 32 * W, sizeof(Tile), s>>>(a, vec_state);
     LLME_LAUNCH_STATUS();
 }
 
@@ -479,22 +517,22 @@ LLME_API int llme_delta_step(const LlmeDeltaArgs* args, cudaStream_t stream) {
     LLME_LAUNCH_STATUS();
 }
 
-// The requests `rows`, each with two tokens or more, four tokens at a time.
+// The requests `rows`, each with two tokens or more, eight tokens at a time.
 LLME_API int llme_delta_portions(const LlmeDeltaArgs* args, cudaStream_t stream) {
     const LlmeDeltaArgs& a = *args;
     if (a.n_rows <= 0) return 0;
     if (int rc = check(a)) return rc;
     if (!a.unit || !a.coef || ((uintptr_t)a.unit | (uintptr_t)a.coef) % 16) LLME_REFUSE("delta_rule: portions need their workspace");
-    const dim3 blocks(a.tokens / BLOCK + a.requests + 1, (a.qk_groups + 3) / 4);
-    if (a.n <= 32) llme_launch(delta_prepare_kernel<1>, blocks, dim3(128), 0, stream, a);
-    else if (a.n <= 64) llme_launch(delta_prepare_kernel<2>, blocks, dim3(128), 0, stream, a);
-    else if (a.n <= 128) llme_launch(delta_prepare_kernel<4>, blocks, dim3(128), 0, stream, a);
-    else if (a.n <= 256) llme_launch(delta_prepare_kernel<8>, blocks, dim3(128), 0, stream, a);
-    else llme_launch(delta_prepare_kernel<16>, blocks, dim3(128), 0, stream, a);
+    const dim3 blocks(a.tokens / BLOCK + a.requests + 1, (a.qk_groups + PREPARE_WARPS - 1) / PREPARE_WARPS);
+    llme_launch(delta_prepare_kernel, blocks, dim3(32 * PREPARE_WARPS), 0, stream, a);
     const int vs = rows_of_16(a.state, a.state_stride, a.n);
-    if (a.n <= 32) return launch_tile<8, 1, 1, 4, 3>(a, vs, stream);
-    if (a.n <= 64) return launch_tile<8, 2, 1, 4, 3>(a, vs, stream);
-    if (a.n <= 128) return launch_tile<8, 4, 1, 4, 3>(a, vs, stream);
+    // 16 columns a block either way: one a lane on four warps where there are few blocks (the walk's latency counts: 297 against
+    // 350 us for 2,048 tokens of 16 heads of 128 x 128), two a lane on two warps where there are many (what is read from shared
+    // memory counts: 410 against 465 us for 32 heads, 168 against 237 us for four requests of 512 tokens)
+    const bool many = (long long)((a.p + 15) / 16) * a.heads * a.n_rows >= 200;
+    if (a.n <= 32) return many ? launch_tile<8, 1, 2, 2, 3>(a, vs, stream) : launch_tile<8, 1, 1, 4, 3>(a, vs, stream);
+    if (a.n <= 64) return many ? launch_tile<8, 2, 2, 2, 3>(a, vs, stream) : launch_tile<8, 2, 1, 4, 3>(a, vs, stream);
+    if (a.n <= 128) return many ? launch_tile<8, 4, 2, 2, 3>(a, vs, stream) : launch_tile<8, 4, 1, 4, 3>(a, vs, stream);
     if (a.n <= 256) return launch_tile<16, 4, 1, 4, 3>(a, vs, stream);
     return launch_tile<32, 4, 1, 4, 2>(a, vs, stream);
 }

@@ -810,8 +810,8 @@ int op_delta_rule(LlmeExecutor& ex, const LlmeDeltaRuleOp& o, const LlmeStep& s,
                        o.n, o.p, o.qk_groups, o.unit, o.coef};
     if (ex.choice("delta_rule") == "tokens") return ex.launched(step(&a, st), "delta_step");      // every request, token after token
     if (s.num_portion > 0) {
-        const long long n4 = (o.n + 3) / 4 * 4, blocks = s.num_tokens / 4 + s.num_requests + 1;
-        if (s.num_tokens * 2 * o.qk_groups * n4 > o.unit_floats || blocks * o.heads * 40 > o.coef_floats)
+        const long long n4 = (o.n + 3) / 4 * 4, blocks = s.num_tokens / 8 + s.num_requests + 1;
+        if (s.num_tokens * 2 * o.qk_groups * n4 > o.unit_floats || blocks * o.heads * 160 > o.coef_floats)
             return ex.fail("delta_rule: the workspace is too small for %d tokens of %d requests", s.num_tokens, s.num_requests);
         a.rows = s.portion_rows; a.n_rows = s.num_portion;
         if (int rc = ex.launched(portions(&a, st), "delta_portions")) return rc;

@@ -211,7 +211,7 @@ typedef struct LlmeDeltaArgs {
     float* out; long long ldo;                               /* [T, heads * p] */
     const int* cu_q_lens; const int* state_slots; const int* rows;
     int n_rows, requests, tokens, heads, n, p, qk_groups;
-    float* unit; float* coef;                                /* workspace of portions: [T, 2 qk_groups n'], n' = n rounded up to fours; 40 values per block and head */
+    float* unit; float* coef;                                /* workspace of portions: [T, 2 qk_groups n'], n' = n rounded up to fours; 160 values per block of 8 tokens and head */
 } LlmeDeltaArgs;
 
 /* The gates of a matrix memory with exponential gating (csrc/recurrent.cu), per request and head over the request's tokens:

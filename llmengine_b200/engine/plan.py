@@ -267,7 +267,7 @@ class Plan:
         b_t = sigmoid(write[t, h]); a_t = exp(-exp(a_log_h) softplus(forget[t, h] + dt_bias_h)); S <- a_t S (S is n x p);
         u = b_t (v_t - S^T k_t); S <- S + k_t u^T; out[t, h] = S^T q_t.  v and out are [T, H p]; `write` and `forget` [T, H] share
         their row stride.  `state` [slots, H, p, n] goes from step to step.  `unit` and `coef`: workspace of the form that takes a
-        portion's tokens four at a time (Runtime.delta_workspace)."""
+        portion's tokens eight at a time (Runtime.delta_workspace)."""
         self._add("delta_rule", q=q, k=k, v=v, write=write, forget=forget, dt_bias=dt_bias, a_log=a_log, q_scale=float(q_scale),
                   unit_eps=float(unit_eps), state=state, out=out, heads=int(heads), n=int(n), p=int(p), qk_groups=int(qk_groups),
                   unit=unit, coef=coef)

@@ -385,7 +385,7 @@ int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
  *   "linear_swiglu":     "fused" | "unfused"
  *   "attention.portion": "tcgen05" | "mma" | "plain"
  *   "attention.decode":  "fused" | "split" | "plain"
- *   "delta_rule":        "blocks" | "tokens"                        (portions: four tokens at a time / one after the other)
+ *   "delta_rule":        "blocks" | "tokens"                        (portions: eight tokens at a time / one after the other)
  *   "*":                 "fast" | "plain"                           (all of the above at once)
  * Returns 0, or -1 for an unknown operation or variant. */
 int llme_executor_choose(LlmeExecutor*, const char* op, const char* variant);

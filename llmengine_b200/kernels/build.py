@@ -39,7 +39,7 @@ SOURCES: Dict[str, str] = {
     # mixture of experts: routing, the grouped product (plain form), the weighted sum; and the grouped product on tensor cores
     # layers with a state of fixed size per request: short convolution, linear recurrence, gated group norm
     "recurrent": "recurrent.cu",
-    # the gated delta rule: single tokens, and portions four tokens at a time
+    # the gated delta rule: single tokens, and portions eight tokens at a time
     "delta_rule": "delta_rule.cu",
     "moe": "moe.cu",
     "moe_tc": "moe_tc.cu",

@@ -279,12 +279,12 @@ class Runtime:
 
     def delta_workspace(self, heads: int, qk_heads: int, n: int) -> Tuple[torch.Tensor, torch.Tensor]:
         """What the delta rule over portions works from: the unit queries and keys of every token ([tokens, 2 * qk_heads * n'],
-        n' = n rounded up to whole groups of four), and per block of four tokens of a request and head the 40 numbers that the
-        block's triangular solve needs (one buffer each for all layers; blocks are numbered floor(first token / 4) + place of
+        n' = n rounded up to whole groups of four), and per block of eight tokens of a request and head the 160 numbers that
+        its columns share (one buffer each for all layers; blocks are numbered floor(first token / 8) + place of
         the request in the step + block of the request)."""
         n4 = (n + 3) // 4 * 4
-        blocks = self.max_tokens // 4 + self.max_requests + 1
-        self._delta_coef_floats = max(getattr(self, "_delta_coef_floats", 0), blocks * heads * 40)
+        blocks = self.max_tokens // 8 + self.max_requests + 1
+        self._delta_coef_floats = max(getattr(self, "_delta_coef_floats", 0), blocks * heads * 160)
         return (self.workspace("delta_unit", 2 * qk_heads * n4, torch.float32),
                 self.buffer("delta_coef", 1, self._delta_coef_floats, torch.float32, exact=True).view(-1))
 

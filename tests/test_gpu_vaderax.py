@@ -31,7 +31,7 @@ def _step_spans(lens, cuts, step):
 
 @pytest.mark.parametrize("kernels", ["fast", "plain"])
 @pytest.mark.parametrize("H,G,n,p", [(1, 1, 4, 3), (4, 2, 8, 16), (3, 1, 6, 5), (2, 2, 32, 48), (6, 2, 64, 33), (4, 1, 128, 20), (2, 1, 100, 64),
-                                     (2, 2, 200, 9), (1, 1, 500, 6), (40, 4, 12, 8)])
+                                     (2, 2, 200, 9), (1, 1, 500, 6), (40, 4, 12, 24), (24, 12, 60, 70), (48, 8, 128, 17)])
 def test_delta_rule_kernels(H, G, n, p, kernels):
     """Single tokens beside portions (down to two tokens, no multiples of four, hundreds) in slots that are not in order; the second
     step starts every request from the state the first one left.  Keys come again (the write replaces what the memory holds), write
@@ -53,7 +53,7 @@ def test_delta_rule_kernels(H, G, n, p, kernels):
     state = torch.zeros(max(slots) + 2, H, p, n, device=DEV)
     T = sum(lens)
     unit = torch.full((T, 2 * G * ((n + 3) // 4 * 4)), float("nan"), device=DEV)
-    coef = torch.full(((T // 4 + len(lens) + 1) * H * 40,), float("nan"), device=DEV)
+    coef = torch.full(((T // 8 + len(lens) + 1) * H * 160,), float("nan"), device=DEV)
     got = [[] for _ in lens]
     for step in range(2):
         spans = _step_spans(lens, cuts, step)
@@ -275,7 +275,7 @@ def test_constants_that_are_one_off(tmp_path, dtype):
     router = lambda c: c["layers"][0]["mlp"]["router"]
     changes = {
         "more coordinates rotated": lambda c: c["layers"][0]["mixer"]["rot"].__setitem__("dims", 10),
-        "another base": lambda c: c["layers"][0]["mixer"]["rot"].__setitem__("base", 400.0),
+        "another base": lambda c: c["layers"][0]["mixer"]["rot"].__setitem__("base", 4.0),
         "another scale": lambda c: c["layers"][0]["mixer"].__setitem__("scale", 0.6),
         "one expert per token": lambda c: router(c).__setitem__("top", 1),
         "three groups kept": lambda c: router(c)["groups"].__setitem__("keep", 3),
