@@ -74,6 +74,8 @@ typedef int (*ResidualAddScaledFn)(float*, const void*, const void*, int, void*,
 typedef int (*LayerNormFn)(float*, const float*, const void*, const void*, int, void*, int, const int*, int, int, float, cudaStream_t);
 typedef int (*EmbeddingAddFn)(const int*, const void*, int, float*, const float*, int, int, int, float, cudaStream_t);
 typedef int (*Relu2Fn)(const void*, long long, void*, long long, int, int, int, cudaStream_t);
+typedef int (*GroupedTcgen05Fn)(const LlmeGroupedArgs*, void*, int, cudaStream_t);
+typedef int (*GroupedFitsFn)(const LlmeGroupedArgs*, int);
 typedef int (*DeltaFn)(const LlmeDeltaArgs*, cudaStream_t);
 typedef int (*RowNormFn)(const void*, long long, int, const void*, int, void*, long long, int, int, int, float, cudaStream_t);
 typedef int (*ExpGatesFn)(const LlmeExpGatesArgs*, int, cudaStream_t);
@@ -851,11 +853,22 @@ int op_moe_route(LlmeExecutor& ex, const LlmeMoeRouteOp& o, const LlmeStep& s, c
     return rc;
 }
 
+constexpr long long GROUPED_ROWS = 64;      // rows an expert gets in the mean, from which on tiles of 128 rows pay
+
 int op_grouped_linear(LlmeExecutor& ex, const LlmeGroupedLinearOp& o, const LlmeStep& s, cudaStream_t st) {
     if (s.num_tokens <= 0) return 0;
     LlmeGroupedArgs a = {o.x, o.ldx, o.w, o.ldw, o.w_expert, o.out, o.ldo, o.offsets, o.order, s.num_tokens * o.top_k, o.num_experts,
                          o.top_k, o.n, o.k, o.gather, o.scatter, o.act};
     // bfloat16 operands in whole 16-byte pieces: the tensor-core form (the activation in its epilogue)
+    // many rows an expert: the tcgen05 kernel, on tiles of 128 rows
+    const std::string& how = ex.choice("grouped_linear");
+    auto* t5 = (GroupedTcgen05Fn)ex.find("grouped_tcgen05");
+    auto* fits = (GroupedFitsFn)ex.find("grouped_tcgen05_supports");
+    if (t5 && fits && o.x_dtype == LLME_DT_BF16 && o.w_dtype == LLME_DT_BF16 && ex.choice("linear") != "plain" && (!o.gather || o.rows) &&
+        (how == "tcgen05" || (how == "auto" && (long long)a.pairs >= GROUPED_ROWS * o.num_experts)) && fits(&a, o.out_dtype)) {
+        if (o.gather) ++ex.launches;
+        return ex.launched(t5(&a, o.rows, o.out_dtype, st), "grouped_tcgen05");
+    }
     auto* tc = (GroupedFn)ex.find("grouped_linear_tc");
     if (tc && o.x_dtype == LLME_DT_BF16 && o.w_dtype == LLME_DT_BF16 && ex.choice("linear") != "plain" && o.k % 8 == 0 && o.ldx % 8 == 0 &&
         o.ldw % 8 == 0 && o.w_expert % 8 == 0 && aligned16(o.x, o.w))
@@ -881,6 +894,7 @@ const std::map<std::string, std::vector<std::string>>& variants() {
         {"attention.portion", {"tcgen05", "mma"}},
         {"attention.decode", {"fused", "split"}},
         {"delta_rule", {"blocks", "tokens"}},
+        {"grouped_linear", {"auto", "tcgen05", "mma"}},
     };
     return v;
 }

@@ -429,6 +429,7 @@ class Engine:
         """Raise if a bounded wait inside a kernel ever gave up (synchronises the device)."""
         libs = getattr(self.ops, "_libs", {})
         status = self.ops.linear_tc_status() if "gemm_tcgen05" in libs else 0
+        status = status or (self.ops.grouped_tcgen05_status() if "moe_tcgen05" in libs else 0)
         for key in libs:
             if key.startswith("attention_tc@HEAD_DIM="):
                 status = status or self.ops.attention_tc_status(int(key.split("=")[1]))

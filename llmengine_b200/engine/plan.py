@@ -217,14 +217,15 @@ class Plan:
                   offsets=offsets, order=order, counts=counts, mode=mode, correction=correction, groups=(int(groups[0]), int(groups[1])))
 
     def grouped_linear(self, *, x, w, out, offsets, order, top_k: int, gather: bool, scatter: bool, mid=None,
-                       act: Optional[str] = None) -> None:
+                       act: Optional[str] = None, rows=None) -> None:
         """One product per expert over the rows that were routed to it: for place r of expert e's range of `order`,
         out_row = w[e] x_row, with x_row = x[order[r] // top_k] if `gather` (the token's row) else x[r], and written
         to out[order[r]] if `scatter` (the pair's row) else out[r].  w is [E, n, k].  With `act` "silu", w[e] is
         [gate | up] by rows and the row written is silu(gate) * up, half as wide; with `act` "relu2" the row written is
-        max(product, 0)^2 (`mid` [pairs, n]: workspace of the form that runs product and activation apart)."""
+        max(product, 0)^2 (`mid` [pairs, n]: workspace of the form that runs product and activation apart).  `rows` [pairs, k]: where a kernel that wants its rows side by side puts gathered
+        ones."""
         self._add("grouped_linear", x=x, w=w, out=out, offsets=offsets, order=order, top_k=int(top_k), gather=bool(gather),
-                  scatter=bool(scatter), mid=mid, act=act)
+                  scatter=bool(scatter), mid=mid, act=act, rows=rows)
 
     def moe_combine(self, *, y, weights, base, out, base_gate=None, experts=None, identity=None, first_identity: int = 0) -> None:
         """out[t] = base[t] (if given) + sum_k weights[t, k] * y[t * top_k + k], the choices added in their order,

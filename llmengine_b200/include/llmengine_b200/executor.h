@@ -267,6 +267,7 @@ typedef struct LlmeGroupedLinearOp {
     void* mid; long long ld_mid;                              /* [pairs, n]: workspace of the unfused activation, or NULL */
     const int* offsets; const int* order;
     int num_experts, top_k, n, k, gather, scatter, act;       /* act 1: w[e] = [gate | up], out = silu(gate) * up; 2: out = max(product, 0)^2 */
+    void* rows;                                               /* [pairs, k] in the type of x: where gathered rows come to stand side by side, or NULL */
 } LlmeGroupedLinearOp;
 
 /* out[t] = base[t] (times sigmoid(base_gate[t * ld_gate]) where base_gate is given) + sum_k weights[t, k] y[t top_k + k]. */
@@ -377,7 +378,8 @@ void llme_executor_destroy(LlmeExecutor*);
  * "postnorm", "gated_act", "gemm_skinny_gated", "gemm_tc_gated", "window_post", "window_attention_plain", per pair of
  * key and value sizes "window_attention_tc/<dk>x<dv>", "moe_route", "grouped_linear", "grouped_linear_tc", "moe_combine";
  * "short_conv", "rotate", "recurrence", "gated_norm", "row_norm", "exp_gates", "sigmoid_mul_grouped", "residual_add_scaled",
- * "layernorm", "embedding_add", "relu2", "delta_step", "delta_portions". */
+ * "layernorm", "embedding_add", "relu2", "delta_step", "delta_portions", "grouped_tcgen05",
+ * "grouped_tcgen05_supports". */
 int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
 /* Which implementation an operation takes.  Operations and their variants:
  *   "linear":            "auto" | "tcgen05" | "cublas" | "plain"   (bfloat16 products of 128 tokens or more / all)
@@ -385,6 +387,7 @@ int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
  *   "linear_swiglu":     "fused" | "unfused"
  *   "attention.portion": "tcgen05" | "mma" | "plain"
  *   "attention.decode":  "fused" | "split" | "plain"
+ *   "grouped_linear":    "auto" | "tcgen05" | "mma"                 (bfloat16: many rows an expert / all / none)
  *   "delta_rule":        "blocks" | "tokens"                        (portions: eight tokens at a time / one after the other)
  *   "*":                 "fast" | "plain"                           (all of the above at once)
  * Returns 0, or -1 for an unknown operation or variant. */

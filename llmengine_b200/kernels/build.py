@@ -43,6 +43,8 @@ SOURCES: Dict[str, str] = {
     "delta_rule": "delta_rule.cu",
     "moe": "moe.cu",
     "moe_tc": "moe_tc.cu",
+    # the same on tcgen05, for many rows an expert
+    "moe_tcgen05": "moe_tcgen05.cu",
     "gemm_f32": "gemm_f32.cu",
     "sampling": "sampling.cu",
     "gemm_skinny": "gemm_skinny.cu",

@@ -165,7 +165,7 @@ class GroupedLinearOp(Structure):
     _fields_ = [("x", c_void_p), ("ldx", c_longlong), ("x_dtype", c_int), ("w", c_void_p), ("ldw", c_longlong),
                 ("w_expert", c_longlong), ("w_dtype", c_int), ("out", c_void_p), ("ldo", c_longlong), ("out_dtype", c_int),
                 ("mid", c_void_p), ("ld_mid", c_longlong), ("offsets", c_void_p), ("order", c_void_p), ("num_experts", c_int),
-                ("top_k", c_int), ("n", c_int), ("k", c_int), ("gather", c_int), ("scatter", c_int), ("act", c_int)]
+                ("top_k", c_int), ("n", c_int), ("k", c_int), ("gather", c_int), ("scatter", c_int), ("act", c_int), ("rows", c_void_p)]
 
 
 class MoeCombineOp(Structure):
@@ -439,13 +439,14 @@ def records(op, keep: List[Any]):
                                         a.get("groups", (1, 1))[0], a.get("groups", (1, 1))[1])
     if k == "grouped_linear":
         x, w, out, mid = a["x"], a["w"], a["out"], a["mid"]
-        act = EXPERT_ACTIVATIONS[a["act"]]
+        act, rows = EXPERT_ACTIVATIONS[a["act"]], a.get("rows")
+        assert rows is None or (rows.dtype == x.dtype and rows.is_contiguous() and rows.shape[1] == x.shape[1] and rows.shape[0] >= x.shape[0] * a["top_k"])
         assert w.dim() == 3 and w.is_contiguous() and x.stride(1) == 1 and out.stride(1) == 1
         assert w.shape[2] == x.shape[1] and out.shape[1] == (w.shape[1] // 2 if act == 1 else w.shape[1]) and x.dtype == w.dtype
         return OP_GROUPED_LINEAR, GroupedLinearOp(
             x.data_ptr(), x.stride(0), code(x.dtype), w.data_ptr(), w.stride(1), w.stride(0), code(w.dtype), out.data_ptr(), out.stride(0),
             code(out.dtype), ptr(mid), mid.stride(0) if mid is not None else 0, a["offsets"].data_ptr(), a["order"].data_ptr(), w.shape[0],
-            a["top_k"], w.shape[1], w.shape[2], 1 if a["gather"] else 0, 1 if a["scatter"] else 0, act)
+            a["top_k"], w.shape[1], w.shape[2], 1 if a["gather"] else 0, 1 if a["scatter"] else 0, act, ptr(rows))
     if k == "moe_combine":
         y, wt, base, out = a["y"], a["weights"], a["base"], a["out"]
         assert y.dtype == wt.dtype == out.dtype == torch.float32 and y.stride(1) == 1 and wt.is_contiguous() and out.is_contiguous()

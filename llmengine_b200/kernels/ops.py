@@ -207,6 +207,7 @@ class CudaOps:
         "attention_window": {"window_post": "llme_window_post", "window_attention_plain": "llme_window_attention_plain"},
         "attention_window_tc": {"window_attention_tc/{hd}": "llme_window_attention_tc"},
         "moe": {"moe_route": "llme_moe_route", "grouped_linear": "llme_grouped_linear", "moe_combine": "llme_moe_combine"},
+        "moe_tcgen05": {"grouped_tcgen05": "llme_grouped_tcgen05", "grouped_tcgen05_supports": "llme_grouped_tcgen05_supports"},
         "moe_tc": {"grouped_linear_tc": "llme_grouped_linear_tc"},
         "attention_latent": {"latent_attention_plain": "llme_latent_attention_plain"},
         "attention_latent_tc": {"latent_attention_tc/{hd}": "llme_latent_attention_tc",
@@ -268,6 +269,10 @@ class CudaOps:
                 want("moe")
             if op.kind == "grouped_linear" and a["x"].dtype == torch.bfloat16 and self.chosen("linear") != "plain" and build.has_source("moe_tc"):
                 want("moe_tc")
+                # (the same sizes the kernel itself asks for: whole 16-byte pieces)
+                w = a["w"]
+                if self.chosen("grouped_linear") != "mma" and w.shape[2] % 8 == 0 and a["out"].shape[1] % 8 == 0:
+                    want("moe_tcgen05")
             if op.kind == "latent_attention":
                 want("attention_latent")
                 if fast_attention and self.latent_tc_supports(a["kv_rank"], a["rot_dim"], a["q"].dtype):
@@ -580,6 +585,9 @@ class CudaOps:
     def linear_tc_status(self) -> int:
         """0 if no bounded wait of the tcgen05 kernels ever gave up (synchronises the device)."""
         return int(self._lib("gemm_tcgen05").llme_gemm_tc_status())
+
+    def grouped_tcgen05_status(self) -> int:
+        return int(self._lib("moe_tcgen05").llme_grouped_tcgen05_status())
 
     def random_fill(self, out: torch.Tensor, key: int, start: int, scale: float, offset: float,
                     round_bf16_first: bool = False) -> torch.Tensor:

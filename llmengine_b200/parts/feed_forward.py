@@ -289,7 +289,8 @@ class RoutedExperts(Part):
         act = rt.buffer("expert_act", T * top, self.ff, rt.dtype)
         mid = rt.buffer("expert_gate_up", T * top, self.w_gate_up.shape[1], rt.dtype)
         plan.grouped_linear(x=h, w=self.w_gate_up, out=act, offsets=offsets, order=order, top_k=top, gather=True,
-                            scatter=False, mid=mid, act=self.act)
+                            scatter=False, mid=mid, act=self.act,
+                            rows=rt.buffer("expert_rows", T * top, self.hidden, rt.dtype) if rt.dtype == torch.bfloat16 else None)
         y = rt.buffer("expert_out", T * top, self.hidden, torch.float32)
         plan.grouped_linear(x=act, w=self.w_down, out=y, offsets=offsets, order=order, top_k=top, gather=False, scatter=True)
         base = self.shared.emit(plan, h, out_name="shared_out") if self.shared is not None else None
