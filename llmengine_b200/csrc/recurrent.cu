@@ -87,10 +87,10 @@ __global__ void short_conv_taps_kernel(LlmeShortConvArgs a) {
 }
 
 // Prompt portions whose rows allow loads of four channels at once: a thread owns four neighbouring channels and walks over
-// CONV_TOKENS tokens of the step, keeping the K - 1 inputs before the present one in registers, so an input is read once (and
+// U tokens of the step, keeping the K - 1 inputs before the present one in registers, so an input is read once (and
 // once more by the block that takes the next tokens); where a request begins inside the walk the window is read anew (from the
 // request's state).  The sums are those of the kernel above, in its order.
-constexpr int CONV_TOKENS = 16;
+constexpr int CONV_TOKENS = 16, CONV_TOKENS_F32 = 8;      // tokens of a walk (a 32-bit input takes twice the registers)
 
 template <typename T> __device__ __forceinline__ void load_four(const T* p, float (&v)[4]);
 template <> __device__ __forceinline__ void load_four<float>(const float* p, float (&v)[4]) {
@@ -103,13 +103,13 @@ template <> __device__ __forceinline__ void load_four<__nv_bfloat16>(const __nv_
     v[0] = __low2float(lo); v[1] = __high2float(lo); v[2] = __low2float(hi); v[3] = __high2float(hi);
 }
 
-template <int K, typename T>
+template <int K, typename T, int U>
 __global__ void __launch_bounds__(128) short_conv_walk_kernel(LlmeShortConvArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
     if (c >= a.channels) return;
-    const int t0 = blockIdx.x * CONV_TOKENS, t1 = min(a.tokens, t0 + CONV_TOKENS);
+    const int t0 = blockIdx.x * U, t1 = min(a.tokens, t0 + U);
     float w[4][K], bias[4];
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
@@ -118,15 +118,15 @@ __global__ void __launch_bounds__(128) short_conv_walk_kernel(LlmeShortConvArgs 
         for (int j = 0; j < K; ++j) w[m][j] = a.w[(size_t)(c + m) * K + (K - 1 - j)];      // w[m][j] meets the input j tokens back
     }
     const T* x = (const T*)a.x;
-    float present[CONV_TOKENS][4];                                      // all of the walk's inputs are on their way at once
+    float present[U][4];                                      // all of the walk's inputs are on their way at once
 #pragma unroll
-    for (int u = 0; u < CONV_TOKENS; ++u)
+    for (int u = 0; u < U; ++u)
         if (t0 + u < t1) load_four<T>(x + (size_t)(t0 + u) * a.ldx + c, present[u]);
     float back[K][4];                                                   // back[j]: the input j tokens before the present one
     int r = row_of_token(a.cu_q_lens, a.requests, t0), begin = a.cu_q_lens[r], end = a.cu_q_lens[r + 1];
     bool fresh = true;
 #pragma unroll
-    for (int u = 0; u < CONV_TOKENS; ++u) {
+    for (int u = 0; u < U; ++u) {
         const int t = t0 + u;
         if (t >= t1) break;
         while (t >= end) {                                              // the next request that has tokens
@@ -164,9 +164,10 @@ __global__ void __launch_bounds__(128) short_conv_walk_kernel(LlmeShortConvArgs 
 
 template <int K>
 static void short_conv_walk(const LlmeShortConvArgs& a, cudaStream_t stream) {
-    const dim3 grid((a.tokens + CONV_TOKENS - 1) / CONV_TOKENS, (a.channels / 4 + 127) / 128), block(128);
-    if (a.x_dtype == LLME_F32) llme_launch(short_conv_walk_kernel<K, float>, grid, block, 0, stream, a);
-    else llme_launch(short_conv_walk_kernel<K, __nv_bfloat16>, grid, block, 0, stream, a);
+    const int walk = a.x_dtype == LLME_F32 ? CONV_TOKENS_F32 : CONV_TOKENS;
+    const dim3 grid((a.tokens + walk - 1) / walk, (a.channels / 4 + 127) / 128), block(128);
+    if (a.x_dtype == LLME_F32) llme_launch(short_conv_walk_kernel<K, float, CONV_TOKENS_F32>, grid, block, 0, stream, a);
+    else llme_launch(short_conv_walk_kernel<K, __nv_bfloat16, CONV_TOKENS>, grid, block, 0, stream, a);
 }
 
 __global__ void short_conv_state_kernel(LlmeShortConvArgs a) {
@@ -826,6 +827,75 @@ __global__ void gated_norm_kernel(LlmeGatedNormArgs a) {
     }
 }
 
+// Groups of 4 to 512 columns in fours, rows that start on 16 bytes (8 for bfloat16), the gate behind the norm: a warp per (token,
+// group), a lane holds up to V pieces of four values between the sum of squares and the output; y and gate are read once, with all
+// loads on their way together.
+template <typename T> __device__ __forceinline__ void store_four(T* p, const float (&v)[4]);
+template <> __device__ __forceinline__ void store_four<float>(float* p, const float (&v)[4]) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
+template <> __device__ __forceinline__ void store_four<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[4]) {
+    uint2 raw;
+    *(__nv_bfloat162*)&raw.x = __floats2bfloat162_rn(v[0], v[1]);
+    *(__nv_bfloat162*)&raw.y = __floats2bfloat162_rn(v[2], v[3]);
+    *(uint2*)p = raw;
+}
+
+template <typename T, typename GT, int V>
+__global__ void __launch_bounds__(128) gated_norm_fours_kernel(LlmeGatedNormArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, groups = a.cols / a.group;
+    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);          // (token, group)
+    if (item >= (long long)a.tokens * groups) return;
+    const int t = (int)(item / groups), c0 = (int)(item - (long long)t * groups) * a.group;
+    const float* y = a.y + (size_t)t * a.ldy + c0;
+    const GT* g = (const GT*)a.gate + (size_t)t * a.ldg + c0;
+    T* o = (T*)a.out + (size_t)t * a.ldo + c0;
+    float u[V][4], gate[V][4], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c < a.group) {
+            load_four<float>(y + c, u[i]);
+            load_four<GT>(g + c, gate[i]);
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) u[i][e] = gate[i][e] = 0.0f;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) ss = fmaf(u[i][e], u[i][e], ss);
+    const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.group + a.eps);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int c = 4 * (lane + 32 * i);
+        if (c >= a.group) continue;
+        float w[4] = {1.0f, 1.0f, 1.0f, 1.0f};
+        if (a.weight) load_four<float>(a.weight + c0 + c, w);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            // (a result that goes to bfloat16 takes the hardware's exponential and reciprocal)
+            const float z = gate[i][e];
+            const float s = sizeof(T) == 2 ? __frcp_rn(1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+            u[i][e] = u[i][e] * rinv * w[e] * (a.gate_act == 1 ? s : z * s) * a.scale;
+        }
+        store_four<T>(o + c, u[i]);
+    }
+}
+
+template <typename T, typename GT>
+static bool launch_fours(const LlmeGatedNormArgs& a, long long items, cudaStream_t s) {
+    const size_t bytes = 4 * sizeof(T), gate_bytes = 4 * sizeof(GT);
+    if (a.gate_first || a.floor || a.group % 4 || a.group > 512 || items > (1LL << 32)) return false;
+    if (a.ldy % 4 || a.ldg % 4 || a.ldo % 4 || (uintptr_t)a.y % 16 || (uintptr_t)a.weight % 16 || (uintptr_t)a.gate % gate_bytes || (uintptr_t)a.out % bytes) return false;
+    const dim3 grid((unsigned)((items + 3) / 4)), block(128);
+    if (a.group <= 128) llme_launch(gated_norm_fours_kernel<T, GT, 1>, grid, block, 0, s, a);
+    else if (a.group <= 256) llme_launch(gated_norm_fours_kernel<T, GT, 2>, grid, block, 0, s, a);
+    else llme_launch(gated_norm_fours_kernel<T, GT, 4>, grid, block, 0, s, a);
+    return true;
+}
+
 // Groups of more than 128 and up to 1,024 columns: a block per (token, group), a thread for every eight columns (whole warps),
 // keeps its values in registers between the sum of squares and the output, so y and the gate are read once and all loads are on
 // their way together.
@@ -874,6 +944,11 @@ LLME_API int llme_gated_norm(const LlmeGatedNormArgs* args, cudaStream_t stream)
     if (a.group <= 0 || a.cols % a.group) LLME_REFUSE("gated_norm: %d columns are not whole groups of %d", a.cols, a.group);
     if (!(a.eps > 0.0f)) LLME_REFUSE("gated_norm: eps must be positive");
     const long long items = (long long)a.tokens * (a.cols / a.group);
+    const bool fours = a.dtype == LLME_F32 ? launch_fours<float, float>(a, items, stream)
+                     : a.dtype != LLME_BF16 ? false
+                     : a.gate_f32 ? launch_fours<__nv_bfloat16, float>(a, items, stream)
+                                  : launch_fours<__nv_bfloat16, __nv_bfloat16>(a, items, stream);
+    if (fours) LLME_LAUNCH_STATUS();
     if (a.group > 128 && a.group <= 1024 && items < (1LL << 31) && (a.dtype == LLME_F32 || a.dtype == LLME_BF16)) {
         const dim3 block(((a.group + 7) / 8 + 31) / 32 * 32);
         if (a.dtype == LLME_F32) llme_launch(gated_norm_block_kernel<float, float>, dim3((unsigned)items), block, 0, stream, a);

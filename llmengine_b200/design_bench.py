@@ -213,7 +213,7 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
         D, top = a["out"].shape[1], a["weights"].shape[1]
         return "weighted sum of the chosen experts", 0.0, T * D * (top * 4 + (4 if a["base"] is not None else 0) + 4)
     if k == "layernorm":
-        return "layer norm + residual add", 0.0, T * a["x"].shape[1] * ((12 if a["delta"] is not None else 4) + el)
+        return "layer norm" + (" + residual add" if a["delta"] is not None else ""), 0.0, T * a["x"].shape[1] * ((12 if a["delta"] is not None else 4) + el)
     if k == "embedding":
         return "embedding added again", 0.0, T * a["out"].shape[1] * (12 + el)
     if k == "rmsnorm":
