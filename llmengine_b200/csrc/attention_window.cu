@@ -206,11 +206,92 @@ __global__ void __launch_bounds__(256) window_post_unit_kernel(LlmeWindowPostArg
     }
 }
 
+// The same for heads of up to 128 coordinates in fours, rotate-half pairs in fours, rows that start on whole pieces: a lane holds four
+// neighbouring coordinates and gets their partners from the lane that holds them; a warp has two heads on their way at a time.
+template <typename T> struct Four;
+template <> struct Four<float> {
+    static __device__ __forceinline__ float4 load(const float* p) { return *(const float4*)p; }
+    static __device__ __forceinline__ void store(float* p, float4 v) { *(float4*)p = v; }
+};
+template <> struct Four<__nv_bfloat16> {
+    static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
+        const uint2 raw = *(const uint2*)p;
+        const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
+        return make_float4(a.x, a.y, b.x, b.y);
+    }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
+        uint2 raw;
+        *(__nv_bfloat162*)&raw.x = __floats2bfloat162_rn(v.x, v.y);
+        *(__nv_bfloat162*)&raw.y = __floats2bfloat162_rn(v.z, v.w);
+        *(uint2*)p = raw;
+    }
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowPostArgs a) {
+    extern __shared__ __align__(16) float cs4[];                     // [rot_dims / 2] cosines, then sines
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, warps = blockDim.x >> 5, lane = threadIdx.x & 31, d = 4 * lane;
+    const int dk = a.dk, dv = a.dv, ps = a.page_size, half = a.inv_freq ? a.rot_dims >> 1 : 0;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s, c;
+        sincosf((float)a.positions[t] * a.inv_freq[i], &s, &c);
+        cs4[i] = c * a.amplitude;
+        cs4[half + i] = s * a.amplitude;
+    }
+    const int slot = a.k_in ? a.slot_mapping[t] : -1;
+    const int page = slot >= 0 ? slot / ps : 0, off = slot - page * ps;
+    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
+    const int heads = a.nh + (slot >= 0 ? 2 * a.nkv : 0), stride = gridDim.y * warps;
+    const T* qrow = (const T*)a.q_in + (size_t)t * a.q_stride;
+    const T* krow = (const T*)a.k_in + (size_t)t * a.k_stride;
+    const T* vrow = (const T*)a.v_in + (size_t)t * a.v_stride;
+    const bool turned = d < 2 * half, first = d < half, inside = d < dk;
+    const int partner = !turned ? lane : first ? lane + half / 4 : lane - half / 4;
+    auto source = [&](int hh) -> const T* {
+        return hh < a.nh ? qrow + hh * dk : hh < a.nh + a.nkv ? krow + (hh - a.nh) * dk : vrow + (hh - a.nh - a.nkv) * dv;
+    };
+    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    int hh = blockIdx.y * warps + (threadIdx.x >> 5);
+    float4 x = zero, ahead = zero;
+    if (hh < heads && d < (hh < a.nh + a.nkv ? dk : dv)) x = Four<T>::load(source(hh) + d);
+    __syncthreads();
+    float4 c = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s = zero;
+    if (turned) {
+        c = *(const float4*)&cs4[first ? d : d - half];
+        s = *(const float4*)&cs4[half + (first ? d : d - half)];
+        if (first) s = make_float4(-s.x, -s.y, -s.z, -s.w);          // u cos - v sin, v cos + u sin
+    }
+    for (; hh < heads; hh += stride, x = ahead) {
+        const int nx = hh + stride;
+        ahead = nx < heads && d < (nx < a.nh + a.nkv ? dk : dv) ? Four<T>::load(source(nx) + d) : zero;
+        if (hh >= a.nh + a.nkv) {
+            if (d < dv) Four<T>::store(kpage + (size_t)a.nkv * ps * dk + ((size_t)(hh - a.nh - a.nkv) * ps + off) * dv + d, x);
+            continue;
+        }
+        const float4 o = make_float4(__shfl_sync(0xffffffffu, x.x, partner), __shfl_sync(0xffffffffu, x.y, partner),
+                                     __shfl_sync(0xffffffffu, x.z, partner), __shfl_sync(0xffffffffu, x.w, partner));
+        if (turned) x = make_float4(x.x * c.x + o.x * s.x, x.y * c.y + o.y * s.y, x.z * c.z + o.z * s.z, x.w * c.w + o.w * s.w);
+        const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+        const float rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
+        T* out = hh < a.nh ? (T*)a.q_out + ((size_t)t * a.nh + hh) * dk : kpage + ((size_t)(hh - a.nh) * ps + off) * dk;
+        if (inside) Four<T>::store(out + d, make_float4(x.x * rinv, x.y * rinv, x.z * rinv, x.w * rinv));
+    }
+}
+
 template <typename T>
 static int launch_post_unit(const LlmeWindowPostArgs& a, cudaStream_t s) {
     const int heads = a.nh + (a.k_in ? 2 * a.nkv : 0), most = (heads + 7) / 8, fill = (592 + a.tokens - 1) / a.tokens;
     const dim3 grid(a.tokens, most < fill ? most : fill), block(256);
-    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float);
+    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float), piece = 4 * sizeof(T);
+    const bool fours = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && a.dv <= 128 && !a.interleaved && (!a.inv_freq || a.rot_dims % 8 == 0) &&
+                       a.q_stride % 4 == 0 && a.k_stride % 4 == 0 && a.v_stride % 4 == 0 &&
+                       ((uintptr_t)a.q_in | (uintptr_t)a.k_in | (uintptr_t)a.v_in | (uintptr_t)a.q_out | (uintptr_t)a.cache) % piece == 0;
+    if (fours) {
+        llme_launch(window_post_unit_fours_kernel<T>, grid, block, smem, s, a);
+        LLME_LAUNCH_STATUS();
+    }
     if (a.dk <= 32) llme_launch(window_post_unit_kernel<T, 1>, grid, block, smem, s, a);
     else if (a.dk <= 64) llme_launch(window_post_unit_kernel<T, 2>, grid, block, smem, s, a);
     else if (a.dk <= 128) llme_launch(window_post_unit_kernel<T, 4>, grid, block, smem, s, a);

@@ -290,6 +290,7 @@ def layer_table(cfg, layers: int, batch: int, page: int, pk) -> Dict[str, List[D
         def run_all():
             for i in indices:
                 compiled.run(batch_obj, i, 1)
+        compiled.run(batch_obj)                 # a whole step: every workspace holds what the record meets in a model
         run_all()
         torch.cuda.synchronize()
         g = torch.cuda.CUDAGraph()
@@ -307,6 +308,7 @@ def layer_table(cfg, layers: int, batch: int, page: int, pk) -> Dict[str, List[D
 
     def table(batch_obj, tokens, keys_per_row, cache_rows):
         out = []
+        batch_obj.logits = eng.rt.buffer("logits", batch_obj.logit_rows.numel(), V, torch.float32)
         # the same record of different layers is timed together; layers may differ in kind (two mixers in turn)
         members: Dict[tuple, List[int]] = {}
         for idx in per_layer:

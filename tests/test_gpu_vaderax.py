@@ -280,6 +280,13 @@ def test_replay_gpu(tmp_path, name, cfg, page, lens, dtype, kernels):
     print(f"replay {name} {dtype} {kernels}: share of the tolerance: " + ", ".join(f"{k} {v:.2f}" for k, v in worst.items()))
 
 
+def test_replay_with_the_experts_products_on_tcgen05(tmp_path):
+    """Every step's experts through the kernel that otherwise serves long prompts alone: tiles of a few rows, rows that run on into
+    the next expert's."""
+    d = make_vaderax_dir(str(tmp_path / "m"), BIG, seed=11)
+    replay_all_schedules(d, BIG, "bfloat16", [150, 40, 129, 2, 64], 64, None, DEV, kernels={"grouped_linear": "tcgen05"})
+
+
 # ----------------------------------------------------------------------------- constants that are one off
 EDGE = model(50, 64, 1e-5, 6.0, [
     layer("attention", attention(4, 2, 32, 32, 0.2, base=200.0, dims=8), moe(6, 3, 32, identity=2, groups=(4, 2))),
