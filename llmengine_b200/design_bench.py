@@ -325,7 +325,7 @@ def layer_table(cfg, layers: int, batch: int, page: int, pk) -> Dict[str, List[D
                         "of_roofline": round(ideal / us, 3) if us > 0 else None, "layers": len(which)})
         return out
 
-    dec = eng._build_batch([StepEntry(n, [5], [0]) for n in names], [CACHED] * batch)
+    dec = eng._build_batch([StepEntry(n, [(5 + 97 * i) % V], [0]) for i, n in enumerate(names)], [CACHED] * batch)
     eng.cache.flush()
     result = {"decode": table(dec, batch, CACHED + 1, batch * (CACHED + 1))}
     eng.cache.add_request("prefill")
@@ -371,7 +371,7 @@ def throughput(cfg, batches, page: int, steps: int, warmup: int) -> Dict[str, An
             eng.step([StepEntry(n, torch.randint(0, V, (CACHED,), generator=gen).tolist(), [])])
 
         def one():
-            logits = eng.step([StepEntry(n, [7], [0]) for n in names])
+            logits = eng.step([StepEntry(n, [(7 + 97 * i) % V], [0]) for i, n in enumerate(names)])   # (routers see different tokens)
             llm.sampler.sample(logits, [greedy] * batch, [0] * batch)
         for _ in range(warmup):
             one()
