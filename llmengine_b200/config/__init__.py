@@ -9,6 +9,7 @@ from typing import Any, Callable, Dict, Mapping, Optional, Type
 
 from .bepuzen import BepuzenConfig
 from .funevik import FunevikConfig
+from .lopilix import LopilixConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .spec import LayerRun, LayerSpec, ModelSpec, PartSpec
 from .torisun import TorisunConfig
@@ -75,6 +76,7 @@ register_architecture(TorisunConfig.ARCHITECTURE, TorisunConfig)
 register_architecture(VifelixConfig.ARCHITECTURE, VifelixConfig)
 register_architecture(FunevikConfig.ARCHITECTURE, FunevikConfig)
 register_architecture(VaderaxConfig.ARCHITECTURE, VaderaxConfig)
+register_architecture(LopilixConfig.ARCHITECTURE, LopilixConfig)
 
 
 @dataclass
@@ -122,6 +124,6 @@ class EngineConfig:
 
 
 __all__ = [
-    "ARCHITECTURES", "Architecture", "BepuzenConfig", "ConfigError", "EngineConfig", "FunevikConfig", "LayerRun", "LayerSpec", "ModelSpec",
+    "ARCHITECTURES", "Architecture", "BepuzenConfig", "ConfigError", "EngineConfig", "FunevikConfig", "LayerRun", "LayerSpec", "LopilixConfig", "ModelSpec",
     "PartSpec", "Qwen3Config", "TorisunConfig", "VaderaxConfig", "VifelixConfig", "config_from_dict", "find_architecture", "load_config", "register_architecture",
 ]

@@ -10,6 +10,11 @@
 
 LLME_API const char* llme_last_error() { return llme_error_buffer(); }
 
+// Value heads of a layer, and the values of a page: with a `value_share` n of more than one, n neighbouring key heads share one value
+// head (the maps of a differential attention).
+__device__ __forceinline__ int value_heads(int nkv, int share) { return share > 1 ? nkv / share : nkv; }
+__device__ __forceinline__ size_t page_values(int nkv, int nv, int ps, int dk, int dv) { return (size_t)ps * ((size_t)nkv * dk + (size_t)nv * dv); }
+
 // ----------------------------------------------------------------------------- norm, rotation, cache write
 // One value of a projection row after the norm (x * rinv * gain) and the rotation of its head's first `dims`
 // coordinates in rotate-half pairs (i, i + dims/2) by position * inv_freq[i], cosine and sine times `amp`.
@@ -42,7 +47,8 @@ __global__ void window_post_kernel(LlmeWindowPostArgs a) {
     __shared__ float scratch[32];
     const int t = blockIdx.x, dk = a.dk, dv = a.dv, ps = a.page_size;
     const int pos = a.positions[t];
-    const int qn = a.nh * dk, kn = a.nkv * dk, vn = a.nkv * dv;
+    const int nv = value_heads(a.nkv, a.value_share);
+    const int qn = a.nh * dk, kn = a.nkv * dk, vn = nv * dv;
     const I* q = (const I*)a.q_in + (size_t)t * a.q_stride;
     float rq = 1.0f, rk = 1.0f;
     if (a.q_gain) {
@@ -69,7 +75,7 @@ __global__ void window_post_kernel(LlmeWindowPostArgs a) {
         rk = 1.0f / sqrtf(block_sum(ss, scratch) / (float)kn + a.eps);
     }
     const int page = slot / ps, off = slot - page * ps;
-    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
+    T* kpage = (T*)a.cache + (size_t)page * page_values(a.nkv, nv, ps, dk, dv);
     T* vpage = kpage + (size_t)a.nkv * ps * dk;
     for (int j = threadIdx.x; j < kn; j += blockDim.x) {
         const int g = j / dk, d = j - g * dk;
@@ -126,7 +132,7 @@ __global__ void window_post_heads_kernel(LlmeWindowPostArgs a) {
     const int warps = blockDim.x >> 5, lane = threadIdx.x & 31;
     const int item = blockIdx.x * warps + (threadIdx.x >> 5);       // (token, head of q | head of k | head of v)
     const bool stores = a.k_in != nullptr;
-    const int per_token = a.nh + (stores ? 2 * a.nkv : 0);
+    const int nv = value_heads(a.nkv, a.value_share), per_token = a.nh + (stores ? a.nkv + nv : 0);
     if (item >= a.tokens * per_token) return;
     const int t = item / per_token, hh = item - t * per_token;
     const int dk = a.dk, dv = a.dv, ps = a.page_size, pos = a.positions[t];
@@ -138,7 +144,7 @@ __global__ void window_post_heads_kernel(LlmeWindowPostArgs a) {
     const int slot = a.slot_mapping[t];
     if (slot < 0) return;
     const int page = slot / ps, off = slot - page * ps;
-    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
+    T* kpage = (T*)a.cache + (size_t)page * page_values(a.nkv, nv, ps, dk, dv);
     if (hh < a.nh + a.nkv) {
         const int g = hh - a.nh;
         finish_head((const T*)a.k_in + (size_t)t * a.k_stride + g * dk, a.k_bias ? a.k_bias + g * dk : nullptr, a.k_gain, a.eps, dk,
@@ -170,8 +176,9 @@ __global__ void __launch_bounds__(256) window_post_unit_kernel(LlmeWindowPostArg
     __syncthreads();
     const int slot = a.k_in ? a.slot_mapping[t] : -1;
     const int page = slot >= 0 ? slot / ps : 0, off = slot - page * ps;
-    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
-    const int heads = a.nh + (slot >= 0 ? 2 * a.nkv : 0);
+    const int nv = value_heads(a.nkv, a.value_share);
+    T* kpage = (T*)a.cache + (size_t)page * page_values(a.nkv, nv, ps, dk, dv);
+    const int heads = a.nh + (slot >= 0 ? a.nkv + nv : 0);
     for (int hh = blockIdx.y * warps + (threadIdx.x >> 5); hh < heads; hh += gridDim.y * warps) {
         if (hh >= a.nh + a.nkv) {
             const int g = hh - a.nh - a.nkv;
@@ -206,8 +213,10 @@ __global__ void __launch_bounds__(256) window_post_unit_kernel(LlmeWindowPostArg
     }
 }
 
-// The same for heads of up to 128 coordinates in fours, rotate-half pairs in fours, rows that start on whole pieces: a lane holds four
-// neighbouring coordinates and gets their partners from the lane that holds them; a warp has two heads on their way at a time.
+// The same for heads of up to 128 coordinates in fours, rotated coordinates in eights (neighbouring pairs: in fours), rows that start on
+// whole pieces: a lane holds four neighbouring coordinates and has their partners itself (neighbouring pairs) or gets them from the
+// lane that holds them; a warp has two heads on their way at a time.  It also serves designs that norm every head by itself with
+// gains BEFORE the rotation (`head_norm`, no biases).
 template <typename T> struct Four;
 template <> struct Four<float> {
     static __device__ __forceinline__ float4 load(const float* p) { return *(const float4*)p; }
@@ -242,8 +251,9 @@ __global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowP
     }
     const int slot = a.k_in ? a.slot_mapping[t] : -1;
     const int page = slot >= 0 ? slot / ps : 0, off = slot - page * ps;
-    T* kpage = (T*)a.cache + (size_t)page * ((size_t)a.nkv * ps * (dk + dv));
-    const int heads = a.nh + (slot >= 0 ? 2 * a.nkv : 0), stride = gridDim.y * warps;
+    const int nv = value_heads(a.nkv, a.value_share);
+    T* kpage = (T*)a.cache + (size_t)page * page_values(a.nkv, nv, ps, dk, dv);
+    const int heads = a.nh + (slot >= 0 ? a.nkv + nv : 0), stride = gridDim.y * warps;
     const T* qrow = (const T*)a.q_in + (size_t)t * a.q_stride;
     const T* krow = (const T*)a.k_in + (size_t)t * a.k_stride;
     const T* vrow = (const T*)a.v_in + (size_t)t * a.v_stride;
@@ -257,8 +267,16 @@ __global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowP
     float4 x = zero, ahead = zero;
     if (hh < heads && d < (hh < a.nh + a.nkv ? dk : dv)) x = Four<T>::load(source(hh) + d);
     __syncthreads();
-    float4 c = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s = zero;
-    if (turned) {
+    float4 c = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s = zero, gq = c, gk = c;
+    if (a.head_norm && inside && a.q_gain) {
+        gq = *(const float4*)(a.q_gain + d);
+        gk = a.k_gain ? *(const float4*)(a.k_gain + d) : gk;
+    }
+    if (turned && a.interleaved) {                                   // pairs (d, d + 1) and (d + 2, d + 3): frequencies d/2, d/2 + 1
+        const float c0 = cs4[d >> 1], c1 = cs4[(d >> 1) + 1], s0 = cs4[half + (d >> 1)], s1 = cs4[half + (d >> 1) + 1];
+        c = make_float4(c0, c0, c1, c1);
+        s = make_float4(-s0, s0, -s1, s1);
+    } else if (turned) {
         c = *(const float4*)&cs4[first ? d : d - half];
         s = *(const float4*)&cs4[half + (first ? d : d - half)];
         if (first) s = make_float4(-s.x, -s.y, -s.z, -s.w);          // u cos - v sin, v cos + u sin
@@ -270,28 +288,48 @@ __global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowP
             if (d < dv) Four<T>::store(kpage + (size_t)a.nkv * ps * dk + ((size_t)(hh - a.nh - a.nkv) * ps + off) * dv + d, x);
             continue;
         }
-        const float4 o = make_float4(__shfl_sync(0xffffffffu, x.x, partner), __shfl_sync(0xffffffffu, x.y, partner),
-                                     __shfl_sync(0xffffffffu, x.z, partner), __shfl_sync(0xffffffffu, x.w, partner));
+        if (a.head_norm) {
+            const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+            const float rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
+            const float4 g = hh < a.nh ? gq : gk;
+            x = make_float4(x.x * rinv * g.x, x.y * rinv * g.y, x.z * rinv * g.z, x.w * rinv * g.w);
+        }
+        const float4 o = a.interleaved ? make_float4(x.y, x.x, x.w, x.z)
+                                       : make_float4(__shfl_sync(0xffffffffu, x.x, partner), __shfl_sync(0xffffffffu, x.y, partner),
+                                                     __shfl_sync(0xffffffffu, x.z, partner), __shfl_sync(0xffffffffu, x.w, partner));
         if (turned) x = make_float4(x.x * c.x + o.x * s.x, x.y * c.y + o.y * s.y, x.z * c.z + o.z * s.z, x.w * c.w + o.w * s.w);
-        const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
-        const float rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
+        float rinv = 1.0f;
+        if (a.unit_norm) {
+            const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+            rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
+        }
         T* out = hh < a.nh ? (T*)a.q_out + ((size_t)t * a.nh + hh) * dk : kpage + ((size_t)(hh - a.nh) * ps + off) * dk;
         if (inside) Four<T>::store(out + d, make_float4(x.x * rinv, x.y * rinv, x.z * rinv, x.w * rinv));
     }
 }
 
+// A block per token, or several where the step has few.
+static dim3 post_grid(const LlmeWindowPostArgs& a) {
+    const int heads = a.nh + (a.k_in ? a.nkv + (a.value_share > 1 ? a.nkv / a.value_share : a.nkv) : 0), most = (heads + 7) / 8;
+    const int fill = (592 + a.tokens - 1) / a.tokens;
+    return dim3(a.tokens, most < fill ? most : fill);
+}
+
+template <typename T>
+static bool launch_post_fours(const LlmeWindowPostArgs& a, cudaStream_t s) {
+    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float), piece = 4 * sizeof(T);
+    const bool fours = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && a.dv <= 128 && (!a.inv_freq || a.rot_dims % (a.interleaved ? 4 : 8) == 0) &&
+                       a.q_stride % 4 == 0 && a.k_stride % 4 == 0 && a.v_stride % 4 == 0 && ((uintptr_t)a.q_gain | (uintptr_t)a.k_gain) % 16 == 0 &&
+                       ((uintptr_t)a.q_in | (uintptr_t)a.k_in | (uintptr_t)a.v_in | (uintptr_t)a.q_out | (uintptr_t)a.cache) % piece == 0;
+    if (fours) llme_launch(window_post_unit_fours_kernel<T>, post_grid(a), dim3(256), smem, s, a);
+    return fours;
+}
+
 template <typename T>
 static int launch_post_unit(const LlmeWindowPostArgs& a, cudaStream_t s) {
-    const int heads = a.nh + (a.k_in ? 2 * a.nkv : 0), most = (heads + 7) / 8, fill = (592 + a.tokens - 1) / a.tokens;
-    const dim3 grid(a.tokens, most < fill ? most : fill), block(256);
-    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float), piece = 4 * sizeof(T);
-    const bool fours = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && a.dv <= 128 && !a.interleaved && (!a.inv_freq || a.rot_dims % 8 == 0) &&
-                       a.q_stride % 4 == 0 && a.k_stride % 4 == 0 && a.v_stride % 4 == 0 &&
-                       ((uintptr_t)a.q_in | (uintptr_t)a.k_in | (uintptr_t)a.v_in | (uintptr_t)a.q_out | (uintptr_t)a.cache) % piece == 0;
-    if (fours) {
-        llme_launch(window_post_unit_fours_kernel<T>, grid, block, smem, s, a);
-        LLME_LAUNCH_STATUS();
-    }
+    const dim3 grid = post_grid(a), block(256);
+    const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float);
+    if (launch_post_fours<T>(a, s)) LLME_LAUNCH_STATUS();
     if (a.dk <= 32) llme_launch(window_post_unit_kernel<T, 1>, grid, block, smem, s, a);
     else if (a.dk <= 64) llme_launch(window_post_unit_kernel<T, 2>, grid, block, smem, s, a);
     else if (a.dk <= 128) llme_launch(window_post_unit_kernel<T, 4>, grid, block, smem, s, a);
@@ -308,6 +346,7 @@ LLME_API int llme_window_post(const LlmeWindowPostArgs* args, int dtype, cudaStr
     if ((a.k_in == nullptr) != (a.v_in == nullptr)) LLME_REFUSE("window_post: keys and values are stored together");
     if (a.k_in && (!a.cache || !a.slot_mapping || a.page_size <= 0)) LLME_REFUSE("window_post: keys without a cache to store them in");
     if (a.nh <= 0 || a.nkv <= 0 || a.dk <= 0 || a.dv <= 0) LLME_REFUSE("window_post: non-positive size");
+    if (a.value_share > 1 && a.nkv % a.value_share) LLME_REFUSE("window_post: %d key heads do not share values %d at a time", a.nkv, a.value_share);
     if (a.inv_freq && (a.rot_dims <= 0 || a.rot_dims % 2 || a.rot_dims > a.dk))
         LLME_REFUSE("window_post: %d rotated coordinates of %d need an even count", a.rot_dims, a.dk);
     if ((a.q_gain || a.k_gain) && !(a.eps > 0.0f)) LLME_REFUSE("window_post: eps must be positive");
@@ -322,7 +361,11 @@ LLME_API int llme_window_post(const LlmeWindowPostArgs* args, int dtype, cudaStr
     if (a.head_norm || a.q_bias || a.k_bias || a.v_bias) {
         if (wide_in) LLME_REFUSE("window_post: 32-bit projections come without biases and without the norm per head");
         if (!a.head_norm && (a.q_gain || a.k_gain)) LLME_REFUSE("window_post: biases come with the norm per head or with no norm");
-        const long long items = (long long)a.tokens * (a.nh + (a.k_in ? 2 * a.nkv : 0));
+        if (a.head_norm && a.q_gain && (a.k_gain || !a.k_in) && !a.q_bias && !a.k_bias && !a.v_bias && !a.unit_norm) {
+            if (dtype == LLME_F32 ? launch_post_fours<float>(a, stream) : dtype == LLME_BF16 ? launch_post_fours<__nv_bfloat16>(a, stream) : false)
+                LLME_LAUNCH_STATUS();
+        }
+        const long long items = (long long)a.tokens * (a.nh + (a.k_in ? a.nkv + (a.value_share > 1 ? a.nkv / a.value_share : a.nkv) : 0));
         const int wpb = 4;
         if (dtype == LLME_F32) llme_launch(window_post_heads_kernel<float>, dim3((unsigned)((items + wpb - 1) / wpb)), dim3(wpb * 32), 0, stream, a);
         else if (dtype == LLME_BF16) llme_launch(window_post_heads_kernel<__nv_bfloat16>, dim3((unsigned)((items + wpb - 1) / wpb)), dim3(wpb * 32), 0, stream, a);
@@ -354,7 +397,8 @@ __global__ void window_attention_plain_kernel(LlmeWindowAttnArgs a) {
     const int lo = (a.window > 0 && p - a.window + 1 > 0) ? p - a.window + 1 : 0;
     const int first = a.keep_first < lo ? a.keep_first : lo;       // keys 0 .. first-1 are seen beside the window
     const int* bt = a.block_tables + (size_t)a.token_request[t] * a.max_blocks;
-    const size_t page_elems = (size_t)a.nkv * ps * (dk + dv);
+    const int share = a.value_share > 1 ? a.value_share : 1;
+    const size_t page_elems = page_values(a.nkv, a.nkv / share, ps, dk, dv);
 
     float q[KR], acc[VR];
     const T* qp = (const T*)a.q + ((size_t)t * a.nh + h) * dk;
@@ -372,7 +416,7 @@ __global__ void window_attention_plain_kernel(LlmeWindowAttnArgs a) {
         const int page = bt[j / ps];
         const int off = j - (j / ps) * ps;
         const T* kp = (const T*)a.cache + (size_t)page * page_elems + ((size_t)kvh * ps + off) * dk;
-        const T* vp = (const T*)a.cache + (size_t)page * page_elems + (size_t)a.nkv * ps * dk + ((size_t)kvh * ps + off) * dv;
+        const T* vp = (const T*)a.cache + (size_t)page * page_elems + (size_t)a.nkv * ps * dk + ((size_t)(kvh / share) * ps + off) * dv;
         float s = 0.0f;
 #pragma unroll
         for (int i = 0; i < KR; ++i) {
@@ -433,6 +477,7 @@ LLME_API int llme_window_attention_plain(const LlmeWindowAttnArgs* args, int dty
     if (a.nh <= 0 || a.nkv <= 0 || a.nh % a.nkv) LLME_REFUSE("window attention: %d query heads are not a multiple of %d key/value heads", a.nh, a.nkv);
     if (a.dk <= 0 || a.dv <= 0 || a.page_size <= 0 || a.max_blocks <= 0 || a.window < 0 || a.keep_first < 0) LLME_REFUSE("window attention: bad size");
     if (a.nh > 65535) LLME_REFUSE("window attention: more than 65535 query heads");
+    if (a.value_share > 1 && a.nkv % a.value_share) LLME_REFUSE("window attention: %d key heads do not share values %d at a time", a.nkv, a.value_share);
     if (dtype == LLME_F32) return launch_plain<float>(a, stream);
     if (dtype == LLME_BF16) return launch_plain<__nv_bfloat16>(a, stream);
     LLME_REFUSE("window attention: unsupported dtype %d", dtype);

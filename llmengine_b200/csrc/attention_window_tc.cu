@@ -81,7 +81,8 @@ __global__ void __launch_bounds__(THREADS) window_tc_kernel(LlmeWindowFastArgs a
     const int c_first = split ? min(n_chunks, (int)blockIdx.x * per) : 0;
     const int c_stop = split ? min(n_chunks, c_first + per) : n_chunks;
     const int* bt = a.block_tables + (size_t)a.table_rows[req] * a.max_blocks;
-    const size_t page_elems = (size_t)a.nkv * ps * (DK + DV);
+    const int share = a.value_share > 1 ? a.value_share : 1;            // neighbouring key heads that attend to one value head
+    const size_t page_elems = (size_t)ps * ((size_t)a.nkv * DK + (size_t)(a.nkv / share) * DV);
     const bf16* cache = (const bf16*)a.cache;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
@@ -101,7 +102,7 @@ __global__ void __launch_bounds__(THREADS) window_tc_kernel(LlmeWindowFastArgs a
             const bool ok = page >= 0;
             const int off = j - blk * ps;
             const bf16* krow = ok ? cache + (size_t)page * page_elems + ((size_t)kvh * ps + off) * DK : cache;
-            const bf16* vrow = ok ? cache + (size_t)page * page_elems + (size_t)a.nkv * ps * DK + ((size_t)kvh * ps + off) * DV : cache;
+            const bf16* vrow = ok ? cache + (size_t)page * page_elems + (size_t)a.nkv * ps * DK + ((size_t)(kvh / share) * ps + off) * DV : cache;
 #pragma unroll
             for (int c = c0; c < KC; c += TPR) cp_async16(Ks + r * LDK + c * 8, ok ? krow + c * 8 : cache, ok);
 #pragma unroll
@@ -350,6 +351,7 @@ LLME_API int llme_window_attention_tc(const LlmeWindowFastArgs* args, int max_q_
         LLME_REFUSE("window attention: null pointer");
     if (a.nh <= 0 || a.nkv <= 0 || a.nh % a.nkv) LLME_REFUSE("window attention: %d query heads are not a multiple of %d key/value heads", a.nh, a.nkv);
     if (a.page_size <= 0 || a.max_blocks <= 0 || a.window < 0 || a.keep_first < 0) LLME_REFUSE("window attention: bad size");
+    if (a.value_share > 1 && a.nkv % a.value_share) LLME_REFUSE("window attention: %d key heads do not share values %d at a time", a.nkv, a.value_share);
     if (a.nkv > 65535 || a.n_rows > 65535) LLME_REFUSE("window attention: more than 65535 key/value heads or requests");
     if ((((uintptr_t)a.q | (uintptr_t)a.cache | (uintptr_t)a.out) & 15)) LLME_REFUSE("window attention: operands must be 16-byte aligned");
     static bool configured = false;

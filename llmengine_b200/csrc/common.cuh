@@ -129,6 +129,9 @@ __device__ __forceinline__ float relu2(float z) {
     return z * z;
 }
 
+// z times the normal distribution's share below z: gelu in its erf form
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+
 __device__ __forceinline__ float to_f32(float v) { return v; }
 __device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 

@@ -167,6 +167,56 @@ template <> struct Vec4<__nv_bfloat16> {
     }
 };
 
+// out[t, s, :] = float(table[ids[t], :]) * scale + float(pos_table[positions[t], :]) for every stream s: a design that learns its
+// positions and keeps several copies of the residual stream.  A position outside the table adds nothing (the engine refuses such
+// requests on the host).
+template <typename W, int N>
+__global__ void embedding_streams_kernel(const int* __restrict__ ids, const W* __restrict__ table, const int* __restrict__ positions,
+                                         const W* __restrict__ pos_table, int max_positions, float* __restrict__ out, int hidden, int vocab,
+                                         float scale, int streams) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, id = ids[t], p = pos_table ? positions[t] : -1;
+    const bool ok = id >= 0 && id < vocab, placed = p >= 0 && p < max_positions;
+    const W* row = table + (size_t)(ok ? id : 0) * hidden;
+    const W* at = placed ? pos_table + (size_t)p * hidden : row;
+    float* o = out + (size_t)t * streams * hidden;
+    for (int j = N * (blockIdx.y * blockDim.x + threadIdx.x); j < hidden; j += N * gridDim.y * blockDim.x) {
+        __align__(16) float v[N], q[N];
+        if (N == 4) {
+            *(float4*)v = Vec4<W>::load(row + j);
+            *(float4*)q = Vec4<W>::load(at + j);
+        } else {
+            v[0] = to_f32(row[j]);
+            q[0] = to_f32(at[j]);
+        }
+#pragma unroll
+        for (int e = 0; e < N; ++e) v[e] = (ok ? v[e] * scale : 0.0f) + (placed ? q[e] : 0.0f);
+        for (int s = 0; s < streams; ++s) {
+            if (N == 4) Vec4<float>::store(o + (size_t)s * hidden + j, *(const float4*)v);
+            else o[(size_t)s * hidden + j] = v[0];
+        }
+    }
+}
+
+LLME_API int llme_embedding_streams(const int* ids, const void* table, int table_dtype, const int* positions, const void* pos_table,
+                                    int max_positions, float* out, int tokens, int hidden, int vocab, float scale, int streams,
+                                    cudaStream_t stream) {
+    if (tokens <= 0) return 0;
+    if (!ids || !table || !out || hidden <= 0 || vocab <= 0 || streams <= 0) LLME_REFUSE("embedding: null pointer or non-positive size");
+    if (pos_table && (!positions || max_positions <= 0)) LLME_REFUSE("embedding: a position table without positions or rows");
+    if (table_dtype != LLME_F32 && table_dtype != LLME_BF16) LLME_REFUSE("embedding: unsupported table dtype %d", table_dtype);
+    const size_t piece = table_dtype == LLME_F32 ? 16 : 8;
+    const bool fours = hidden % 4 == 0 && ((uintptr_t)table | (uintptr_t)pos_table) % piece == 0 && (uintptr_t)out % 16 == 0;
+    const int threads = 128, each = fours ? 4 * threads : threads, most = (hidden + each - 1) / each, fill = (592 + tokens - 1) / tokens;
+    const dim3 grid(tokens, most < fill ? most : fill);
+#define LLME_ES(W, N) llme_launch(embedding_streams_kernel<W, N>, grid, dim3(threads), 0, stream, ids, (const W*)table, positions, (const W*)pos_table, max_positions, out, hidden, vocab, scale, streams)
+    if (table_dtype == LLME_F32) { if (fours) LLME_ES(float, 4); else LLME_ES(float, 1); }
+    else { if (fours) LLME_ES(__nv_bfloat16, 4); else LLME_ES(__nv_bfloat16, 1); }
+#undef LLME_ES
+    LLME_LAUNCH_STATUS();
+}
+
 template <typename D, typename G, typename O, bool HAS_DELTA, int V>
 __global__ void rmsnorm_vec_kernel(float* __restrict__ x, const D* __restrict__ delta, const G* __restrict__ gain,
                                    O* __restrict__ out, const int* __restrict__ rows, int hidden, float eps,

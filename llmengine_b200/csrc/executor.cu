@@ -77,6 +77,10 @@ typedef int (*Relu2Fn)(const void*, long long, void*, long long, int, int, int, 
 typedef int (*GroupedTcgen05Fn)(const LlmeGroupedArgs*, void*, int, cudaStream_t);
 typedef int (*GroupedFitsFn)(const LlmeGroupedArgs*, int);
 typedef int (*DeltaFn)(const LlmeDeltaArgs*, cudaStream_t);
+typedef int (*EmbeddingStreamsFn)(const int*, const void*, int, const int*, const void*, int, float*, int, int, int, float, int, cudaStream_t);
+typedef int (*StreamNormFn)(const LlmeStreamNormArgs*, cudaStream_t);
+typedef int (*ForgetGatesFn)(const LlmeForgetGatesArgs*, cudaStream_t);
+typedef int (*DifferenceNormFn)(const LlmeDifferenceNormArgs*, cudaStream_t);
 typedef int (*RowNormFn)(const void*, long long, int, const void*, int, void*, long long, int, int, int, float, cudaStream_t);
 typedef int (*ExpGatesFn)(const LlmeExpGatesArgs*, int, cudaStream_t);
 typedef int (*GemmF32BatchedFn)(const float*, const void*, int, float*, int, int, int, long long, long long, long long, int, long long,
@@ -198,6 +202,9 @@ size_t record_size(int kind) {
         case LLME_OP_EXP_GATES: return sizeof(LlmeExpGatesOp);
         case LLME_OP_LAYERNORM: return sizeof(LlmeLayerNormOp);
         case LLME_OP_DELTA_RULE: return sizeof(LlmeDeltaRuleOp);
+        case LLME_OP_STREAM_NORM: return sizeof(LlmeStreamNormOp);
+        case LLME_OP_FORGET_GATES: return sizeof(LlmeForgetGatesOp);
+        case LLME_OP_DIFFERENCE_NORM: return sizeof(LlmeDifferenceNormOp);
     }
     return 0;
 }
@@ -205,8 +212,9 @@ const char* kind_name(int kind) {
     static const char* names[] = {"?", "embedding", "rmsnorm", "linear", "linear_swiglu", "qkv_post", "attend", "attention", "call",
                                   "linear_act", "pointwise", "batched_linear", "residual_add", "latent_attention", "token_side",
                                   "postnorm", "window_attention", "moe_route", "grouped_linear", "moe_combine", "short_conv", "rotate",
-                                  "recurrence", "gated_norm", "row_norm", "exp_gates", "layernorm", "delta_rule"};
-    return kind >= 1 && kind <= 27 ? names[kind] : names[0];
+                                  "recurrence", "gated_norm", "row_norm", "exp_gates", "layernorm", "delta_rule",
+                                  "stream_norm", "forget_gates", "difference_norm"};
+    return kind >= 1 && kind <= 30 ? names[kind] : names[0];
 }
 
 constexpr int SKINNY_ROWS = 16;      // most rows the weight-streaming product takes (gemm_skinny.cu)
@@ -315,6 +323,12 @@ int op_embedding(LlmeExecutor& ex, const LlmeEmbeddingOp& o, const LlmeStep& s, 
         auto* g = (EmbeddingAddFn)ex.find("embedding_add");
         if (!g) return ex.fail("no kernel that adds an embedding to the stream is registered");
         return ex.launched(g(s.token_ids, o.table, o.table_dtype, o.out, o.delta, s.num_tokens, o.hidden, o.vocab, o.scale, st), "embedding_add");
+    }
+    if (o.pos_table || o.streams > 1) {
+        auto* g = (EmbeddingStreamsFn)ex.find("embedding_streams");
+        if (!g) return ex.fail("no embedding kernel with positions and streams is registered");
+        return ex.launched(g(s.token_ids, o.table, o.table_dtype, s.positions, o.pos_table, o.max_positions, o.out, s.num_tokens, o.hidden, o.vocab, o.scale,
+                             o.streams > 1 ? o.streams : 1, st), "embedding_streams");
     }
     if (o.scale != 1.0f) {
         auto* g = (EmbeddingScaledFn)ex.find("embedding_scaled");
@@ -647,6 +661,7 @@ int op_latent_attention(LlmeExecutor& ex, const LlmeLatentAttentionOp& o, const 
     p.c_gain = o.c_gain; p.gain_dtype = o.gain_dtype; p.eps = o.eps; p.inv_freq = o.inv_freq; p.rot_dims = o.rot_dims;
     p.positions = s.positions; p.q = o.q; p.cache = o.cache; p.slot_mapping = g.slot_mapping;
     p.tokens = s.num_tokens; p.nh = o.nh; p.rank = o.rank; p.rot = o.rot; p.interleaved = o.interleaved;
+    p.amplitude = o.amplitude;
     if (int rc = ex.launched(post(&p, o.dtype, st), "latent_post")) return rc;
     // bfloat16 with a latent size the tensor-core kernel is built for: prompt portions in one launch, single tokens in
     // another whose requests may be cut into several key ranges
@@ -716,10 +731,11 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
     p.tokens = s.num_tokens; p.nh = o.nh; p.nkv = o.nkv; p.dk = o.dk; p.dv = o.dv; p.page_size = g.page_size;
     p.q_bias = o.q_bias; p.k_bias = o.k_bias; p.v_bias = o.v_bias; p.head_norm = o.head_norm;
     p.interleaved = o.interleaved; p.in_f32 = o.in_f32; p.unit_norm = o.unit_norm;
+    p.value_share = o.value_share;
     if (int rc = ex.launched(post(&p, o.dtype, st), "window_post")) return rc;
     // ordinary causal attention with keys and values of one width: a page holds its keys and then its values in both layouts, so the
     // kernels of plain grouped-query attention (tcgen05 portions, split-context decode) read the cache as it is
-    if (o.decode_scratch && o.dk == o.dv && !o.keep_first && !o.sink && !(o.softcap > 0.0f) && fast_attention(ex, o.dtype, o.dk)) {
+    if (o.decode_scratch && o.dk == o.dv && o.value_share <= 1 && !o.keep_first && !o.sink && !(o.softcap > 0.0f) && fast_attention(ex, o.dtype, o.dk)) {
         LlmeAttendOp at = {o.q, o.out, o.dtype, o.cache, o.cache_pages * 2 * o.nkv * g.page_size, o.group, o.nh, o.nkv, o.dk, o.window, o.scale,
                            o.decode_scratch, o.decode_scratch_floats};
         return op_attend(ex, at, s, st);
@@ -731,6 +747,7 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
         f.q = o.q; f.cache = o.cache; f.out = o.out; f.sink = o.sink; f.cu_q_lens = s.cu_q_lens; f.ctx_lens = s.ctx_lens;
         f.table_rows = s.state_slots; f.block_tables = g.block_tables; f.max_blocks = g.max_blocks; f.nh = o.nh; f.nkv = o.nkv;
         f.page_size = g.page_size; f.window = o.window; f.keep_first = o.keep_first; f.scale = o.scale; f.softcap = o.softcap;
+        f.value_share = o.value_share;
         if (s.num_portion > 0) {
             f.rows = s.portion_rows; f.n_rows = s.num_portion;
             if (int rc = ex.launched(tc(&f, s.max_portion_len, 0, st), "window_attention_tc")) return rc;
@@ -754,7 +771,7 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
     auto* plain = (WindowAttnPlainFn)ex.find("window_attention_plain");
     if (!plain) return ex.fail("no window attention kernel is registered");
     LlmeWindowAttnArgs a = {o.q, o.cache, o.out, o.sink, s.positions, s.token_request, g.block_tables, g.max_blocks, s.num_tokens,
-                            o.nh, o.nkv, o.dk, o.dv, g.page_size, o.window, o.keep_first, o.scale, o.softcap};
+                            o.nh, o.nkv, o.dk, o.dv, g.page_size, o.window, o.keep_first, o.scale, o.softcap, o.value_share};
     return ex.launched(plain(&a, o.dtype, st), "window_attention_plain");
 }
 
@@ -831,6 +848,31 @@ int op_row_norm(LlmeExecutor& ex, const LlmeRowNormOp& o, const LlmeStep& s, cud
     auto* f = (RowNormFn)ex.find("row_norm");
     if (!f) return ex.fail("no row_norm kernel is registered");
     return ex.launched(f(o.x, o.ldx, o.x_dtype, o.gain, o.gain_dtype, o.out, o.ldo, o.out_dtype, s.num_tokens, o.cols, o.eps, st), "row_norm");
+}
+
+int op_stream_norm(LlmeExecutor& ex, const LlmeStreamNormOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (rows_of(s, o.rows) <= 0) return 0;
+    auto* f = (StreamNormFn)ex.find("stream_norm");
+    if (!f) return ex.fail("no stream_norm kernel is registered");
+    LlmeStreamNormArgs a = {o.x, o.streams, o.size, o.y, o.gate, o.ldg, o.gate_dtype, o.gate_bias, o.mix, o.put, o.read, o.gain, o.eps, o.out, o.out_dtype,
+                            o.rows == LLME_ROWS_LOGITS ? s.logit_rows : nullptr, rows_of(s, o.rows)};
+    return ex.launched(f(&a, st), "stream_norm");
+}
+
+int op_forget_gates(LlmeExecutor& ex, const LlmeForgetGatesOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (s.num_tokens <= 0) return 0;
+    auto* f = (ForgetGatesFn)ex.find("forget_gates");
+    if (!f) return ex.fail("no forget_gates kernel is registered");
+    LlmeForgetGatesArgs a = {o.q_in, o.f_in, o.ld_in, o.f_bias, o.lower, o.q, o.f, o.ldq, o.ldf, s.num_tokens, o.cols};
+    return ex.launched(f(&a, st), "forget_gates");
+}
+
+int op_difference_norm(LlmeExecutor& ex, const LlmeDifferenceNormOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (s.num_tokens <= 0) return 0;
+    auto* f = (DifferenceNormFn)ex.find("difference_norm");
+    if (!f) return ex.fail("no difference_norm kernel is registered");
+    LlmeDifferenceNormArgs a = {o.a, o.lda, o.out, o.ldo, o.dtype, s.num_tokens, o.heads, o.rep, o.dim, o.weight, o.scale, o.eps};
+    return ex.launched(f(&a, st), "difference_norm");
 }
 
 int op_exp_gates(LlmeExecutor& ex, const LlmeExpGatesOp& o, const LlmeStep& s, cudaStream_t st) {
@@ -1044,6 +1086,9 @@ LLME_EXPORT int llme_plan_run(LlmePlan* p, const LlmeStep* step, int first, int 
             case LLME_OP_ROW_NORM: rc = op_row_norm(ex, *(const LlmeRowNormOp*)b, s, stream); break;
             case LLME_OP_LAYERNORM: rc = op_layernorm(ex, *(const LlmeLayerNormOp*)b, s, stream); break;
             case LLME_OP_DELTA_RULE: rc = op_delta_rule(ex, *(const LlmeDeltaRuleOp*)b, s, stream); break;
+            case LLME_OP_STREAM_NORM: rc = op_stream_norm(ex, *(const LlmeStreamNormOp*)b, s, stream); break;
+            case LLME_OP_FORGET_GATES: rc = op_forget_gates(ex, *(const LlmeForgetGatesOp*)b, s, stream); break;
+            case LLME_OP_DIFFERENCE_NORM: rc = op_difference_norm(ex, *(const LlmeDifferenceNormOp*)b, s, stream); break;
             case LLME_OP_EXP_GATES: rc = op_exp_gates(ex, *(const LlmeExpGatesOp*)b, s, stream); break;
             case LLME_OP_CALL: {
                 const LlmeCallOp& c = *(const LlmeCallOp*)b;

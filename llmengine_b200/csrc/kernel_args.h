@@ -58,6 +58,7 @@ typedef struct LlmeLatentPostArgs {
     void* cache; const int* slot_mapping;         /* rows of rank + rot; slot < 0: not stored */
     int tokens, nh, rank, rot;
     int interleaved;                              /* 1: the rotation pairs coordinate 2i with 2i + 1, not i with i + rot_dims / 2 */
+    float amplitude;                              /* cosine and sine times this constant */
 } LlmeLatentPostArgs;
 
 /* Attention over cached latent rows [c | rotated key part], one row per token for all heads. */
@@ -88,6 +89,7 @@ typedef struct LlmeWindowPostArgs {
     int interleaved;                                         /* 1: the rotation pairs coordinate 2i with 2i + 1, not i with i + rot_dims / 2 */
     int in_f32;                                              /* 1: q_in, k_in and v_in are 32-bit whatever the type of q_out and the cache */
     int unit_norm;                                           /* 1: behind the rotation every query and key head is divided by its own root mean square (eps inside the root) */
+    int value_share;                                         /* n > 1: n neighbouring key heads share a value head: v_in and a page hold nkv / n of them */
 } LlmeWindowPostArgs;
 
 /* Attention over such a cache: query i sees key j if j <= i and (i - j < window or j < keep_first). */
@@ -98,6 +100,7 @@ typedef struct LlmeWindowAttnArgs {
     int max_blocks, tokens, nh, nkv, dk, dv, page_size, window, keep_first;
     float scale;
     float softcap;                                           /* c > 0: a score s becomes c tanh(s / c) behind the scale */
+    int value_share;                                         /* n > 1: key head g reads value head g / n of nkv / n */
 } LlmeWindowAttnArgs;
 
 /* The same for the tensor-core kernel: the requests `rows` of the batch, each with its tokens
@@ -110,6 +113,7 @@ typedef struct LlmeWindowFastArgs {
     float scale;
     float* scratch; int splits;      /* single tokens: each request's keys cut into `splits` ranges whose parts meet in `scratch` */
     float softcap;                   /* c > 0: a score s becomes c tanh(s / c) behind the scale */
+    int value_share;                 /* n > 1: key head g reads value head g / n of nkv / n */
 } LlmeWindowFastArgs;
 
 /* Routing of a mixture of experts (csrc/moe.cu). */
@@ -121,7 +125,7 @@ typedef struct LlmeMoeRouteArgs {
     int mode;                                                /* 0: sigmoid scores normalised over the chosen; 1: softmax over the chosen logits; 2: softmax over all */
     /* mode 2: the choice goes by softmax + correction (32-bit [E], or NULL); the E choices form `groups` equal groups of neighbours,
      * of which the `keep` with the largest best member offer theirs; the weights are scale * softmax */
-    const float* correction; int groups, keep;
+    const float* correction; int groups, keep;               /* mode 0, keep < groups: the groups with the largest sum of their two largest scores offer theirs */
 } LlmeMoeRouteArgs;
 
 /* One product per expert over the rows routed to it. */
@@ -132,7 +136,7 @@ typedef struct LlmeGroupedArgs {
     const int* offsets; const int* order;
     int pairs, num_experts, top_k, n, k;                     /* pairs = tokens * top_k */
     int gather, scatter;                                     /* x row = order[r] / top_k; out row = order[r] */
-    int act;                                                 /* 1: w[e] = [gate | up], the row written is silu(gate) * up, n / 2 wide; 2: max(product, 0)^2 */
+    int act;                                                 /* 1: w[e] = [gate | up], the row written is silu(gate) * up, n / 2 wide; 2: max(product, 0)^2; 3: gelu (erf) */
 } LlmeGroupedArgs;
 
 /* Causal convolution per channel over the tokens of each request (csrc/recurrent.cu): y_t = bias + sum_j w[:, K-1-j] x_(t-j),
@@ -178,6 +182,7 @@ typedef struct LlmeRecurrenceArgs {
     /* gate 2: a_t = keep[t, h], s_t = take[t, h], 32-bit, made by an earlier kernel (row stride ld_gates) */
     const float* keep; const float* take; long long ld_gates;
     int unit_column;                                         /* 1: column p - 1 has no v behind it, its v_t is one; v is [T, heads * (p - 1)] */
+    /* gate 3: k holds a forget gate f per row of S: S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T */
 } LlmeRecurrenceArgs;
 
 /* RMS norm in groups of `group` columns with a gate (silu of a second tensor) before or after it:
@@ -190,7 +195,7 @@ typedef struct LlmeGatedNormArgs {
     void* out; long long ldo;
     int dtype, tokens, cols, group, gate_first;
     float eps, scale;
-    int gate_act;                                            /* 0: silu(g); 1: sigmoid(g) */
+    int gate_act;                                            /* 0: silu(g); 1: sigmoid(g); 2: no gate (gate NULL) */
     /* with `floor` [T, cols / group] every group of y is one value wider than `group`: the extra value d stands behind the
      * group's own, and the group is divided by max(|d|, floor) + den_eps before anything else */
     const float* floor; long long ld_floor; float den_eps;
@@ -225,3 +230,32 @@ typedef struct LlmeExpGatesArgs {
     const int* cu_q_lens; const int* state_slots;
     int requests, heads;
 } LlmeExpGatesArgs;
+
+/* Residual streams x [tokens, streams * size], 32-bit (csrc/streams.cu): with y, x_t <- sum_s mix[s, t] x_s + put[t] y sigmoid(gate +
+ * gate_bias) (gate NULL: no gate); with out, u = sum_s read[s] x_s and out = u / sqrt(mean(u^2) + eps) * gain.  With `rows` [tokens]
+ * (row indices) output row i is made from row rows[i], and x stays as it is. */
+typedef struct LlmeStreamNormArgs {
+    float* x; int streams, size;
+    const float* y;
+    const void* gate; long long ldg; int gate_dtype; const float* gate_bias;
+    const float* mix; const float* put;                      /* [streams, streams] (from, to), [streams] */
+    const float* read; const float* gain; float eps;
+    void* out; int out_dtype;
+    const int* rows; int tokens;
+} LlmeStreamNormArgs;
+
+/* q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in + f_bias), elementwise over [tokens, cols], 32-bit. */
+typedef struct LlmeForgetGatesArgs {
+    const float* q_in; const float* f_in; long long ld_in;
+    const float* f_bias; const float* lower;
+    float* q; float* f; long long ldq, ldf;
+    int tokens, cols;
+} LlmeForgetGatesArgs;
+
+/* The maps of a differential attention become its heads (u = a1 - weight a2, divided by its root mean square, times scale). */
+typedef struct LlmeDifferenceNormArgs {
+    const void* a; long long lda;                            /* [tokens, 2 heads dim]: per group of rep heads map 1's, then map 2's */
+    void* out; long long ldo;                                /* [tokens, heads dim] */
+    int dtype, tokens, heads, rep, dim;
+    float weight, scale, eps;
+} LlmeDifferenceNormArgs;

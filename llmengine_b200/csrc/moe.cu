@@ -1,4 +1,5 @@
-// A mixture of experts: routing (sigmoid scores, the largest few chosen, weights normalised over the chosen; or the
+// A mixture of experts: routing (sigmoid scores, the largest few chosen, perhaps only inside the groups with the largest sums of
+// their two best scores, weights normalised over the chosen; or the
 // softmax over the chosen logits alone; or the softmax over all with a correction of the choice and a limit to the best
 // groups), the list
 // of (token, choice) pairs expert by expert, one product per expert over its pairs (plain form: any sizes, both types,
@@ -19,6 +20,11 @@ __device__ __forceinline__ void warp_argmax(float& best, int& bi) {
         const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
         if (oi >= 0 && (bi < 0 || ob > best || (ob == best && oi < bi))) { best = ob; bi = oi; }
     }
+}
+
+// 32-bit values of shared memory that a warp's routing needs
+__host__ __device__ __forceinline__ int route_place(const LlmeMoeRouteArgs& a) {
+    return a.mode == 2 ? a.num_experts : (a.mode == 0 && a.keep > 0 && a.keep < a.groups) ? a.num_experts + a.groups : 0;
 }
 
 __device__ __forceinline__ void route_token(const LlmeMoeRouteArgs& a, int t, int lane, float* __restrict__ choice) {
@@ -50,6 +56,37 @@ __device__ __forceinline__ void route_token(const LlmeMoeRouteArgs& a, int t, in
             }
             taken = ~offered;
         }
+    }
+    if (a.mode == 0 && a.keep > 0 && a.keep < a.groups) {
+        // a group is as good as the sum of its two largest scores: lane g adds them up for the groups g, g + 32, ...
+        const int size = E / a.groups;
+        float* total_of = choice + E;
+        for (int i = lane; i < E; i += 32) choice[i] = 1.0f / (1.0f + expf(-z[i]));
+        __syncwarp();
+        for (int g = lane; g < a.groups; g += 32) {
+            float one = -1.0f, two = -1.0f;
+            for (int i = g * size; i < (g + 1) * size; ++i) {
+                const float s = choice[i];
+                two = fmaxf(two, fminf(one, s));
+                one = fmaxf(one, s);
+            }
+            total_of[g] = size > 1 ? one + two : one;
+        }
+        __syncwarp();
+        unsigned offered = 0;
+        for (int k = 0; k < a.keep; ++k) {
+            float best = -INFINITY;
+            int bi = -1;
+            for (int g = lane; g < a.groups; g += 32)
+                if (total_of[g] >= 0.0f && (bi < 0 || total_of[g] > best)) { best = total_of[g]; bi = g; }
+            warp_argmax(best, bi);
+            for (int i = lane, n = 0; i < E; i += 32, ++n)
+                if (i / size == bi) offered |= 1u << n;
+            __syncwarp();
+            if (lane == 0) total_of[bi] = -1.0f;               // kept: out of the next rounds
+            __syncwarp();
+        }
+        taken = ~offered;
     }
     float score[8];
     int chosen[8];
@@ -90,13 +127,13 @@ __device__ __forceinline__ void route_token(const LlmeMoeRouteArgs& a, int t, in
 }
 
 __global__ void moe_route_kernel(LlmeMoeRouteArgs a) {
-    extern __shared__ float choices[];                    // mode 2: [warps][E]
+    extern __shared__ float choices[];                    // mode 2: [warps][E]; mode 0 with groups: [warps][E + groups]
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= a.tokens) return;
-    route_token(a, t, lane, choices + (size_t)warp * a.num_experts);
+    route_token(a, t, lane, choices + (size_t)warp * route_place(a));
     for (int k = lane; k < a.top_k; k += 32) atomicAdd(a.counts + a.experts[(size_t)t * a.top_k + k], 1);
 }
 
@@ -148,14 +185,14 @@ __global__ void moe_order_kernel(LlmeMoeRouteArgs a) {
 constexpr int ROUTE_FEW = 64, ROUTE_WARPS = 16;
 
 __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_few_kernel(LlmeMoeRouteArgs a) {
-    extern __shared__ float choices[];                    // [warps][E], then the cursors [E + 1] and the counts [E]
+    extern __shared__ float choices[];                    // [warps][route_place], then the cursors [E + 1] and the counts [E]
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, E = a.num_experts, P = a.tokens * a.top_k;
-    int* cursor = (int*)(choices + (size_t)ROUTE_WARPS * (a.mode == 2 ? E : 0));
+    int* cursor = (int*)(choices + (size_t)ROUTE_WARPS * route_place(a));
     int* counts = cursor + E + 1;
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
-    for (int t = warp; t < a.tokens; t += ROUTE_WARPS) route_token(a, t, lane, choices + (size_t)warp * E);
+    for (int t = warp; t < a.tokens; t += ROUTE_WARPS) route_token(a, t, lane, choices + (size_t)warp * route_place(a));
     __syncthreads();
     for (int i = threadIdx.x; i < P; i += blockDim.x) atomicAdd(counts + a.experts[i], 1);
     __syncthreads();
@@ -171,9 +208,10 @@ LLME_API int llme_moe_route(const LlmeMoeRouteArgs* args, cudaStream_t stream) {
     if (a.mode < 0 || a.mode > 2) LLME_REFUSE("moe_route: unknown mode %d", a.mode);
     if (a.num_experts <= 0 || a.num_experts > 1024 || a.top_k <= 0 || a.top_k > a.num_experts)
         LLME_REFUSE("moe_route: %d of %d experts (at most 1024)", a.top_k, a.num_experts);
-    if (a.mode == 2 && (a.groups <= 0 || a.num_experts % a.groups || a.keep <= 0 || a.keep > a.groups || a.top_k > a.num_experts / a.groups * a.keep))
+    const bool grouped = a.mode == 2 || (a.mode == 0 && a.keep > 0 && a.keep < a.groups);
+    if (grouped && (a.groups <= 0 || a.num_experts % a.groups || a.keep <= 0 || a.keep > a.groups || a.top_k > a.num_experts / a.groups * a.keep))
         LLME_REFUSE("moe_route: %d of %d groups of %d experts do not offer %d", a.keep, a.groups, a.num_experts, a.top_k);
-    const size_t lists = (size_t)(2 * a.num_experts + 1) * sizeof(int), place = a.mode == 2 ? (size_t)a.num_experts * sizeof(float) : 0;
+    const size_t lists = (size_t)(2 * a.num_experts + 1) * sizeof(int), place = (size_t)route_place(a) * sizeof(float);
     if (a.tokens <= ROUTE_FEW && ROUTE_WARPS * place + lists <= 48 * 1024) {
         llme_launch(moe_route_few_kernel, dim3(1), dim3(32 * ROUTE_WARPS), ROUTE_WARPS * place + lists, stream, a);
         LLME_LAUNCH_STATUS();
@@ -270,6 +308,7 @@ __global__ void __launch_bounds__(256) grouped_linear_kernel(LlmeGroupedArgs a) 
         if (col >= n_out) continue;
         float v = acc[0][c];
         if (a.act == 2) v = relu2(v);
+        if (a.act == 3) v = gelu_erf(v);
         if (gated) {
             // gate and up pass through the type of the activations first, as they do when the activation is a kernel of its own
             const float g = to_f32(from_f32<T>(acc[0][c])), u = to_f32(from_f32<T>(acc[1][c]));
@@ -283,7 +322,7 @@ LLME_API int llme_grouped_linear(const LlmeGroupedArgs* args, int x_dtype, int w
     const LlmeGroupedArgs& a = *args;
     if (a.pairs <= 0 || a.n <= 0) return 0;
     if (!a.x || !a.w || !a.out || !a.offsets || !a.order) LLME_REFUSE("grouped_linear: null pointer");
-    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || a.act < 0 || a.act > 2 || (a.act == 1 && a.n % 2)) LLME_REFUSE("grouped_linear: bad size");
+    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || a.act < 0 || a.act > 3 || (a.act == 1 && a.n % 2)) LLME_REFUSE("grouped_linear: bad size");
     const int n_out = a.act == 1 ? a.n / 2 : a.n;
     const int most = a.num_experts < a.pairs ? a.num_experts : a.pairs;
     int tiles = (a.pairs + GM - 1) / GM + most;

@@ -67,7 +67,7 @@ template <> __device__ __forceinline__ void store2<bf16>(bf16* p, float a, float
 }
 
 // BM x BN tile on WM x WNW warps, STAGES stages; ACT 1: the weight rows of a column are its gate row and, n_out further on, its up row;
-// ACT 2: max(product, 0)^2 in the epilogue.
+// ACT 2: max(product, 0)^2 in the epilogue; ACT 3: gelu in its erf form.
 template <int BM, int BN, int WM, int WNW, int STAGES, int ACT, typename O>
 __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedArgs a) {
     constexpr int THREADS = 32 * WM * WNW, MT = BM / WM / 16, WN = BN / WNW, NT = WN / 8, HALVES = ACT == 1 ? 2 : 1;
@@ -176,6 +176,10 @@ __global__ void __launch_bounds__(32 * WM * WNW) grouped_tc_kernel(LlmeGroupedAr
                     v0 = relu2(v0);
                     v1 = relu2(v1);
                 }
+                if (ACT == 3) {
+                    v0 = gelu_erf(v0);
+                    v1 = gelu_erf(v1);
+                }
                 if (ACT == 1) {
                     // gate and up pass through bfloat16 first, as they do when the activation is a kernel of its own
                     const float g0 = __bfloat162float(__float2bfloat16_rn(v0)), g1 = __bfloat162float(__float2bfloat16_rn(v1));
@@ -227,10 +231,10 @@ LLME_API int llme_grouped_linear_tc(const LlmeGroupedArgs* args, int x_dtype, in
     if (a.pairs <= 0 || a.n <= 0) return 0;
     if (!a.x || !a.w || !a.out || !a.offsets || !a.order) LLME_REFUSE("grouped_linear_tc: null pointer");
     if (x_dtype != LLME_BF16 || w_dtype != LLME_BF16) LLME_REFUSE("grouped_linear_tc: bfloat16 operands only");
-    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || a.act < 0 || a.act > 2 || (a.act == 1 && a.n % 2)) LLME_REFUSE("grouped_linear_tc: bad size");
+    if (a.num_experts <= 0 || a.top_k <= 0 || a.k <= 0 || a.act < 0 || a.act > 3 || (a.act == 1 && a.n % 2)) LLME_REFUSE("grouped_linear_tc: bad size");
     if (a.k % 8 || a.ldx % 8 || a.ldw % 8 || a.w_expert % 8 || (((uintptr_t)a.x | (uintptr_t)a.w) & 15))
         LLME_REFUSE("grouped_linear_tc: rows must be whole 16-byte pieces");
-    if (out_dtype == LLME_BF16) return a.act == 1 ? dispatch<1, bf16>(a, stream) : a.act == 2 ? dispatch<2, bf16>(a, stream) : dispatch<0, bf16>(a, stream);
-    if (out_dtype == LLME_F32) return a.act == 1 ? dispatch<1, float>(a, stream) : a.act == 2 ? dispatch<2, float>(a, stream) : dispatch<0, float>(a, stream);
+    if (out_dtype == LLME_BF16) return a.act == 1 ? dispatch<1, bf16>(a, stream) : a.act == 2 ? dispatch<2, bf16>(a, stream) : a.act == 3 ? dispatch<3, bf16>(a, stream) : dispatch<0, bf16>(a, stream);
+    if (out_dtype == LLME_F32) return a.act == 1 ? dispatch<1, float>(a, stream) : a.act == 2 ? dispatch<2, float>(a, stream) : a.act == 3 ? dispatch<3, float>(a, stream) : dispatch<0, float>(a, stream);
     LLME_REFUSE("grouped_linear_tc: unsupported output dtype %d", out_dtype);
 }

@@ -194,6 +194,10 @@ grouped_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_c
 #pragma unroll
                             for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(relu2(__uint_as_float(v[j])));
                         }
+                        if (ACT == 3) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) v[j] = __float_as_uint(gelu_erf(__uint_as_float(v[j])));
+                        }
                     }
                     if (c + COLS >= OUT_COLS && half == COLS / 32 - 1) {     // the tile has left tensor memory
                         asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -281,7 +285,7 @@ LLME_API int llme_grouped_tcgen05(const LlmeGroupedArgs* args, void* rows, int o
     const LlmeGroupedArgs& a = *args;
     if (a.pairs <= 0 || a.n <= 0) return 0;
     if (!a.x || !a.w || !a.out || !a.offsets || !a.order || a.top_k <= 0) LLME_REFUSE("grouped_tcgen05: null pointer or no choices");
-    if (a.act < 0 || a.act > 2 || (out_dtype != LLME_F32 && out_dtype != LLME_BF16) || !llme_grouped_tcgen05_supports(args, out_dtype))
+    if (a.act < 0 || a.act > 3 || (out_dtype != LLME_F32 && out_dtype != LLME_BF16) || !llme_grouped_tcgen05_supports(args, out_dtype))
         LLME_REFUSE("grouped_tcgen05: sizes or strides that are not whole 16-byte pieces");
     const void* x = a.x;
     long long ldx = a.ldx;
@@ -294,8 +298,8 @@ LLME_API int llme_grouped_tcgen05(const LlmeGroupedArgs* args, void* rows, int o
         ldx = a.k;
     }
     if (out_dtype == LLME_F32)
-        return a.act == 1 ? launch<1, float>(a, x, ldx, stream) : a.act == 2 ? launch<2, float>(a, x, ldx, stream) : launch<0, float>(a, x, ldx, stream);
-    return a.act == 1 ? launch<1, bf16>(a, x, ldx, stream) : a.act == 2 ? launch<2, bf16>(a, x, ldx, stream) : launch<0, bf16>(a, x, ldx, stream);
+        return a.act == 1 ? launch<1, float>(a, x, ldx, stream) : a.act == 2 ? launch<2, float>(a, x, ldx, stream) : a.act == 3 ? launch<3, float>(a, x, ldx, stream) : launch<0, float>(a, x, ldx, stream);
+    return a.act == 1 ? launch<1, bf16>(a, x, ldx, stream) : a.act == 2 ? launch<2, bf16>(a, x, ldx, stream) : a.act == 3 ? launch<3, bf16>(a, x, ldx, stream) : launch<0, bf16>(a, x, ldx, stream);
 }
 
 // Reads and clears the error flag of the kernel (synchronises the device).  0 = no wait ever gave up.

@@ -279,15 +279,17 @@ LLME_API int llme_rmsnorm_add(float* x, const float* y, const void* gain, int ga
 // ----------------------------------------------------------------------------- latent: norm, rotation, cache write
 // One value of a vector whose first `dims` coordinates are rotated in rotate-half pairs (i, i + dims/2) by the angle
 // position * inv_freq[i], formed in 32-bit; coordinates from `dims` on pass unchanged.
-// `interleaved`: the pairs are (2i, 2i + 1) instead.
+// `interleaved`: the pairs are (2i, 2i + 1) instead.  Cosine and sine times `amplitude`.
 template <typename T>
 __device__ __forceinline__ float rotated_value(const T* __restrict__ v, int idx, int dims, const float* __restrict__ inv_freq, int position,
-                                               int interleaved = 0) {
+                                               int interleaved, float amplitude) {
     if (idx >= dims) return to_f32(v[idx]);
     const int half = dims >> 1, i = interleaved ? idx >> 1 : (idx < half ? idx : idx - half);
     const float angle = (float)position * inv_freq[i];
     float s, c;
     sincosf(angle, &s, &c);
+    s *= amplitude;
+    c *= amplitude;
     const float u = to_f32(v[interleaved ? 2 * i : i]), w = to_f32(v[interleaved ? 2 * i + 1 : i + half]);
     const bool first = interleaved ? !(idx & 1) : idx < half;
     return first ? u * c - w * s : w * c + u * s;
@@ -313,7 +315,7 @@ __global__ void latent_post_kernel(LlmeLatentPostArgs a) {
         const float rinv = 1.0f / sqrtf(ss / (float)rank + a.eps);
         const G* gain = (const G*)a.c_gain;
         for (int j = threadIdx.x; j < rank; j += blockDim.x) row[j] = from_f32<T>((to_f32(kv[j]) * rinv) * to_f32(gain[j]));
-        for (int j = threadIdx.x; j < rot; j += blockDim.x) row[rank + j] = from_f32<T>(rotated_value(kv + rank, j, a.rot_dims, a.inv_freq, pos, a.interleaved));
+        for (int j = threadIdx.x; j < rot; j += blockDim.x) row[rank + j] = from_f32<T>(rotated_value(kv + rank, j, a.rot_dims, a.inv_freq, pos, a.interleaved, a.amplitude));
     }
     if (rot > 0 && a.q_rot && a.q && (gridDim.y == 1 || blockIdx.y > 0)) {
         const T* qr = (const T*)a.q_rot + (size_t)t * a.q_rot_stride;
@@ -321,7 +323,7 @@ __global__ void latent_post_kernel(LlmeLatentPostArgs a) {
         const int first = gridDim.y == 1 ? 0 : blockIdx.y - 1, stride = gridDim.y == 1 ? 1 : gridDim.y - 1;
         for (int e = first * blockDim.x + threadIdx.x; e < a.nh * rot; e += stride * blockDim.x) {
             const int h = e / rot, j = e - h * rot;
-            q[(size_t)h * width + rank + j] = from_f32<T>(rotated_value(qr + (size_t)h * a.q_rot_head_stride, j, a.rot_dims, a.inv_freq, pos, a.interleaved));
+            q[(size_t)h * width + rank + j] = from_f32<T>(rotated_value(qr + (size_t)h * a.q_rot_head_stride, j, a.rot_dims, a.inv_freq, pos, a.interleaved, a.amplitude));
         }
     }
 }
@@ -390,6 +392,98 @@ LLME_API int llme_row_norm(const void* x, long long ldx, int x_dtype, const void
     else LLME_REFUSE("row_norm: unsupported dtypes %d / %d / %d", x_dtype, gain_dtype, out_dtype);
 #undef LLME_RN
     LLME_LAUNCH_STATUS();
+}
+
+// ----------------------------------------------------------------------------- differential attention: the maps become heads
+// Per token and head u = a1 - weight a2 (the two maps' outputs), out = u / sqrt(mean(u^2) + eps) * scale.  The maps' heads lie group
+// by group (`rep` heads of map 1, then the same of map 2).  One warp per (token, head); in the N = 4 form a lane holds V pieces of
+// four values between the sum of squares and the output.
+template <typename T> __device__ __forceinline__ float4 piece_of(const T* p);
+template <> __device__ __forceinline__ float4 piece_of<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 piece_of<__nv_bfloat16>(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128) difference_norm_kernel(LlmeDifferenceNormArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, dim = a.dim;
+    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (item >= (long long)a.tokens * a.heads) return;
+    const int t = (int)(item / a.heads), h = (int)(item - (long long)t * a.heads), g = h / a.rep, first = g * 2 * a.rep + (h - g * a.rep);
+    const T* a1 = (const T*)a.a + (size_t)t * a.lda + (size_t)first * dim;
+    const T* a2 = a1 + (size_t)a.rep * dim;
+    T* o = (T*)a.out + (size_t)t * a.ldo + (size_t)h * dim;
+    float ss = 0.0f;
+    for (int d = lane; d < dim; d += 32) {
+        const float u = to_f32(a1[d]) - a.weight * to_f32(a2[d]);
+        ss = fmaf(u, u, ss);
+    }
+    const float r = a.scale / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+    for (int d = lane; d < dim; d += 32) o[d] = from_f32<T>((to_f32(a1[d]) - a.weight * to_f32(a2[d])) * r);
+}
+
+__device__ __forceinline__ void store4(float* p, float a, float b, float c, float d);
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float c, float d);
+
+template <typename T, int V>
+__global__ void __launch_bounds__(128) difference_norm_fours_kernel(LlmeDifferenceNormArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, dim = a.dim;
+    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (item >= (long long)a.tokens * a.heads) return;
+    const int t = (int)(item / a.heads), h = (int)(item - (long long)t * a.heads), g = h / a.rep, first = g * 2 * a.rep + (h - g * a.rep);
+    const T* a1 = (const T*)a.a + (size_t)t * a.lda + (size_t)first * dim;
+    const T* a2 = a1 + (size_t)a.rep * dim;
+    float4 u[V], v[V];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int d = 4 * (lane + 32 * i);
+        u[i] = v[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (d < dim) {
+            u[i] = piece_of<T>(a1 + d);
+            v[i] = piece_of<T>(a2 + d);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        u[i] = make_float4(u[i].x - a.weight * v[i].x, u[i].y - a.weight * v[i].y, u[i].z - a.weight * v[i].z, u[i].w - a.weight * v[i].w);
+        ss = fmaf(u[i].x, u[i].x, fmaf(u[i].y, u[i].y, fmaf(u[i].z, u[i].z, fmaf(u[i].w, u[i].w, ss))));
+    }
+    const float r = a.scale / sqrtf(warp_sum(ss) / (float)dim + a.eps);
+    T* o = (T*)a.out + (size_t)t * a.ldo + (size_t)h * dim;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+        const int d = 4 * (lane + 32 * i);
+        if (d < dim) store4(o + d, u[i].x * r, u[i].y * r, u[i].z * r, u[i].w * r);
+    }
+}
+
+template <typename T>
+static int launch_difference(const LlmeDifferenceNormArgs& a, cudaStream_t s) {
+    const long long items = (long long)a.tokens * a.heads;
+    const dim3 grid((unsigned)((items + 3) / 4)), block(128);
+    const bool fours = a.dim % 4 == 0 && a.dim <= 512 && a.lda % 4 == 0 && a.ldo % 4 == 0 && ((uintptr_t)a.a | (uintptr_t)a.out) % (4 * sizeof(T)) == 0;
+    if (!fours) llme_launch(difference_norm_kernel<T>, grid, block, 0, s, a);
+    else if (a.dim <= 128) llme_launch(difference_norm_fours_kernel<T, 1>, grid, block, 0, s, a);
+    else if (a.dim <= 256) llme_launch(difference_norm_fours_kernel<T, 2>, grid, block, 0, s, a);
+    else llme_launch(difference_norm_fours_kernel<T, 4>, grid, block, 0, s, a);
+    LLME_LAUNCH_STATUS();
+}
+
+LLME_API int llme_difference_norm(const LlmeDifferenceNormArgs* args, cudaStream_t stream) {
+    const LlmeDifferenceNormArgs& a = *args;
+    if (a.tokens <= 0) return 0;
+    if (!a.a || !a.out || a.heads <= 0 || a.dim <= 0 || a.rep <= 0 || a.heads % a.rep) LLME_REFUSE("difference_norm: null pointer or bad size");
+    if (!(a.eps > 0.0f)) LLME_REFUSE("difference_norm: eps must be positive");
+    if (a.dtype == LLME_F32) return launch_difference<float>(a, stream);
+    if (a.dtype == LLME_BF16) return launch_difference<__nv_bfloat16>(a, stream);
+    LLME_REFUSE("difference_norm: unsupported dtype %d", a.dtype);
 }
 
 // ----------------------------------------------------------------------------- the norm on a sublayer's output

@@ -308,7 +308,8 @@ LLME_API int llme_rotate(const LlmeRotateArgs* args, cudaStream_t stream) {
 // one coordinate of v): lane l holds S[l + 32 i], i < R, in registers; a token costs R multiply-adds for the update, R for the
 // output and one sum over the lanes.  Columns are independent, so no warp waits for another.  A block takes WARPS columns of
 // one (request, head); the state is stored column by column, so a warp's loads and stores of it are contiguous.
-template <int R>
+// CHANNEL: every row has a decay of its own, f, and takes 1 - f of v (gate 3: k holds f).
+template <int R, bool CHANNEL>
 __global__ void __launch_bounds__(256) recurrence_column_kernel(LlmeRecurrenceArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -345,7 +346,8 @@ __global__ void __launch_bounds__(256) recurrence_column_kernel(LlmeRecurrenceAr
         for (int i = 0; i < R; ++i) {
             const int e = lane + 32 * i;
             if (e < n) {
-                S[i] = fmaf(decay, S[i], (step * k[e]) * v);
+                if (CHANNEL) S[i] = fmaf(k[e], S[i], (1.0f - k[e]) * v);
+                else S[i] = fmaf(decay, S[i], (step * k[e]) * v);
                 y = fmaf(S[i], q[e], y);
             }
         }
@@ -363,6 +365,9 @@ __global__ void __launch_bounds__(256) recurrence_column_kernel(LlmeRecurrenceAr
 // block needs the same q and k, and no token's operands come from global memory when they are due.  A token costs a warp 4 R
 // multiply-adds for the update, 4 R for the output, and six exchanges that sum the four columns over the lanes (each lane
 // ending with the sum of one column).
+//
+// With a forget gate per row (CHANNEL, gate 3) the k tile holds f: a row's decay is f, what it takes of v is 1 - f, and a piece leaves a
+// product of decays per row instead of one per head.
 //
 // A request with many tokens in the step is cut into pieces of `chunk` tokens that run side by side, in three launches:
 // every piece but a request's last starts from zero and leaves E_c, what its tokens alone add to the state, and D_c, the
@@ -421,7 +426,7 @@ template <int R> struct RecTile {
     float sums[8][TOKENS][16];                                         // per warp and token: four partial sums of each of four columns
 };
 
-template <int R, bool LOCAL>
+template <int R, bool LOCAL, bool CHANNEL>
 __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(LlmeRecurrenceArgs a, int pass, int chunk, int slots, int vec) {
     using Tile = RecTile<R>;
     constexpr int TT = Tile::TOKENS, ROW = Tile::ROW, V_EACH = Tile::V_EACH;
@@ -464,6 +469,7 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
 
     const int vp = a.unit_column ? p - 1 : p;                           // columns that have a v behind them
     float v_next[V_EACH], dt_next = 0.0f, keep_next = 1.0f;
+    constexpr float NO_K = CHANNEL ? 1.0f : 0.0f;                       // what stands for k behind the last token and in the rows' padding: it changes nothing
     // Sends for the tokens t0 .. t0 + TT - 1: q and k straight into buffer b, v and dt into registers for now.
     auto fetch = [&](int t0, int b) {
         if (vec) {
@@ -475,7 +481,7 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
                     copy_async_16(&sm.k[b][u][e], kg + (size_t)t * a.ldk + e);
                 } else {
                     *(float4*)&sm.q[b][u][e] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                    *(float4*)&sm.k[b][u][e] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+                    *(float4*)&sm.k[b][u][e] = make_float4(NO_K, NO_K, NO_K, NO_K);
                 }
             }
         } else {
@@ -485,7 +491,10 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
                 if (t < last) {
                     copy_async_4(&sm.q[b][u][e], qg + (size_t)t * a.ldq + e);
                     copy_async_4(&sm.k[b][u][e], kg + (size_t)t * a.ldk + e);
-                } else sm.q[b][u][e] = sm.k[b][u][e] = 0.0f;
+                } else {
+                    sm.q[b][u][e] = 0.0f;
+                    sm.k[b][u][e] = NO_K;
+                }
             }
         }
 #pragma unroll
@@ -523,7 +532,10 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
     const int tiles = (last - first + TT - 1) / TT;
     if (n < ROW)                                                       // the rows' padding stays zero
         for (int idx = tid; idx < 2 * TT * ROW; idx += 256)
-            if (idx % ROW >= n) (&sm.q[0][0][0])[idx] = (&sm.k[0][0][0])[idx] = 0.0f;
+            if (idx % ROW >= n) {
+                (&sm.q[0][0][0])[idx] = 0.0f;
+                (&sm.k[0][0][0])[idx] = NO_K;
+            }
     if (tiles > 0) {
         const int t0 = first + (LOCAL ? tiles - 1 : 0) * TT;
         fetch(t0, 0);
@@ -531,7 +543,10 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
     }
     // A piece's own addition to the state is taken from its last token backwards: E = sum_u (s_u prod_(u' > u) a_u') k_u v_u^T,
     // one multiply-add an element and token, with `total` the product of the decays of the tokens behind.
-    float total = 1.0f;
+    float total = 1.0f, row_total[CHANNEL && LOCAL ? R : 1];
+    if (CHANNEL && LOCAL)
+#pragma unroll
+        for (int r = 0; r < R; ++r) row_total[r] = 1.0f;
     for (int i = 0; i < tiles; ++i) {
         const int b = i & 1, tile = LOCAL ? tiles - 1 - i : i, t0 = first + tile * TT;
         const int next = first + (LOCAL ? tile - 1 : tile + 1) * TT;
@@ -544,7 +559,8 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
                 const f32x2 v01 = pack2(v4.x, v4.y), v23 = pack2(v4.z, v4.w);
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
-                    const float kw = w * sm.k[b][u][lane * R + r];
+                    const float kr = sm.k[b][u][lane * R + r], kw = CHANNEL ? (1.0f - kr) * row_total[CHANNEL && LOCAL ? r : 0] : w * kr;
+                    if (CHANNEL) row_total[CHANNEL && LOCAL ? r : 0] *= kr;
                     const f32x2 kw2 = pack2(kw, kw);
                     S[0][r] = fma2(kw2, v01, S[0][r]);
                     S[1][r] = fma2(kw2, v23, S[1][r]);
@@ -560,10 +576,10 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
                 f32x2 y01 = pack2(0.0f, 0.0f), y23 = y01;
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
-                    const float qi = sm.q[b][u][lane * R + r], ks = step * sm.k[b][u][lane * R + r];
-                    const f32x2 qi2 = pack2(qi, qi), ks2 = pack2(ks, ks);
-                    S[0][r] = fma2(decay2, S[0][r], mul2(ks2, v01));      // S = a S + (s k) v, as the single-token kernel rounds it
-                    S[1][r] = fma2(decay2, S[1][r], mul2(ks2, v23));
+                    const float kr = sm.k[b][u][lane * R + r], qi = sm.q[b][u][lane * R + r], ks = CHANNEL ? 1.0f - kr : step * kr;
+                    const f32x2 qi2 = pack2(qi, qi), ks2 = pack2(ks, ks), keep2 = CHANNEL ? pack2(kr, kr) : decay2;
+                    S[0][r] = fma2(keep2, S[0][r], mul2(ks2, v01));       // S = a S + (s k) v, as the single-token kernel rounds it
+                    S[1][r] = fma2(keep2, S[1][r], mul2(ks2, v23));
                     y01 = fma2(S[0][r], qi2, y01);
                     y23 = fma2(S[1][r], qi2, y23);
                 }
@@ -602,7 +618,12 @@ __global__ void __launch_bounds__(256, R <= 4 ? 3 : 1) recurrence_tile_kernel(Ll
                 if (j0 + 2 * c + 1 < p && lane * R + i < n) to[(size_t)(2 * c + 1) * n + lane * R + i] = hi;
             }
     }
-    if (LOCAL && j0 == 0 && lane == 0) a.scratch[(size_t)slots * hpn + (size_t)pc.slot * a.heads + h] = total;
+    if (LOCAL && CHANNEL && j0 == 0) {
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+            if (lane * R + r < n) a.scratch[(size_t)slots * hpn + ((size_t)pc.slot * a.heads + h) * n + lane * R + r] = row_total[CHANNEL && LOCAL ? r : 0];
+    }
+    if (LOCAL && !CHANNEL && j0 == 0 && lane == 0) a.scratch[(size_t)slots * hpn + (size_t)pc.slot * a.heads + h] = total;
 }
 
 // The second of the three launches: one thread per element of a request's state walks over the request's pieces.
@@ -619,9 +640,10 @@ __global__ void recurrence_join_kernel(LlmeRecurrenceArgs a, int chunk, int slot
     }
     const size_t hpn = (size_t)a.heads * a.p * a.n, pn = (size_t)a.p * a.n;
     const float* kept = a.state + (size_t)a.state_slots[r] * a.state_stride;
-    const float* products = a.scratch + (size_t)slots * hpn + (size_t)base * a.heads;
+    const size_t decays = a.gate == 3 ? (size_t)a.heads * a.n : a.heads;     // products of decays that a piece has left
+    const float* products = a.scratch + (size_t)slots * hpn + (size_t)base * decays;
     for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < hpn; e += (size_t)gridDim.x * blockDim.x) {
-        const int h = (int)(e / pn);
+        const size_t h = a.gate == 3 ? e / pn * a.n + e % a.n : e / pn;      // the element's among them
         float* at = a.scratch + (size_t)base * hpn + e;
         float S = kept[e];
         int c = 0;
@@ -630,7 +652,7 @@ __global__ void recurrence_join_kernel(LlmeRecurrenceArgs a, int chunk, int slot
 #pragma unroll
             for (int m = 0; m < 4; ++m) {
                 added[m] = at[(size_t)m * hpn];
-                product[m] = products[(size_t)(c + m) * a.heads + h];
+                product[m] = products[(size_t)(c + m) * decays + h];
             }
 #pragma unroll
             for (int m = 0; m < 4; ++m) {
@@ -641,20 +663,35 @@ __global__ void recurrence_join_kernel(LlmeRecurrenceArgs a, int chunk, int slot
         for (; c + 1 < pieces; ++c, at += hpn) {
             const float added = *at;
             *at = S;
-            S = fmaf(products[(size_t)c * a.heads + h], S, added);
+            S = fmaf(products[(size_t)c * decays + h], S, added);
         }
         *at = S;
     }
 }
 
+template <bool LOCAL, bool CHANNEL>
+static void recurrence_tiles_of(const LlmeRecurrenceArgs& a, dim3 grid, int pass, int chunk, int slots, int vec, cudaStream_t stream) {
+    const dim3 block(256);
+    if (a.n <= 32) llme_launch(recurrence_tile_kernel<1, LOCAL, CHANNEL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+    else if (a.n <= 64) llme_launch(recurrence_tile_kernel<2, LOCAL, CHANNEL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+    else if (a.n <= 128) llme_launch(recurrence_tile_kernel<4, LOCAL, CHANNEL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+    else if (a.n <= 256) llme_launch(recurrence_tile_kernel<8, LOCAL, CHANNEL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+    else llme_launch(recurrence_tile_kernel<16, LOCAL, CHANNEL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+}
+
 template <bool LOCAL>
 static void recurrence_tiles(const LlmeRecurrenceArgs& a, dim3 grid, int pass, int chunk, int slots, int vec, cudaStream_t stream) {
-    const dim3 block(256);
-    if (a.n <= 32) llme_launch(recurrence_tile_kernel<1, LOCAL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
-    else if (a.n <= 64) llme_launch(recurrence_tile_kernel<2, LOCAL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
-    else if (a.n <= 128) llme_launch(recurrence_tile_kernel<4, LOCAL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
-    else if (a.n <= 256) llme_launch(recurrence_tile_kernel<8, LOCAL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
-    else llme_launch(recurrence_tile_kernel<16, LOCAL>, grid, block, 0, stream, a, pass, chunk, slots, vec);
+    if (a.gate == 3) recurrence_tiles_of<LOCAL, true>(a, grid, pass, chunk, slots, vec, stream);
+    else recurrence_tiles_of<LOCAL, false>(a, grid, pass, chunk, slots, vec, stream);
+}
+
+template <bool CHANNEL>
+static void recurrence_columns(const LlmeRecurrenceArgs& a, dim3 grid, dim3 block, cudaStream_t stream) {
+    if (a.n <= 32) llme_launch(recurrence_column_kernel<1, CHANNEL>, grid, block, 0, stream, a);
+    else if (a.n <= 64) llme_launch(recurrence_column_kernel<2, CHANNEL>, grid, block, 0, stream, a);
+    else if (a.n <= 128) llme_launch(recurrence_column_kernel<4, CHANNEL>, grid, block, 0, stream, a);
+    else if (a.n <= 256) llme_launch(recurrence_column_kernel<8, CHANNEL>, grid, block, 0, stream, a);
+    else llme_launch(recurrence_column_kernel<16, CHANNEL>, grid, block, 0, stream, a);
 }
 
 // The chunk a step of `tokens` tokens whose longest request brings `max_len` is cut by, with room for `slots` piece states
@@ -676,7 +713,7 @@ LLME_API int llme_recurrence(const LlmeRecurrenceArgs* args, cudaStream_t stream
     if (a.requests <= 0) return 0;
     if (!a.q || !a.k || !a.v || !a.state || !a.out || !a.cu_q_lens || !a.state_slots) LLME_REFUSE("recurrence: null pointer");
     if (a.heads <= 0 || a.n <= 0 || a.p <= 0 || a.qk_groups <= 0 || a.heads % a.qk_groups) LLME_REFUSE("recurrence: %d heads in %d groups", a.heads, a.qk_groups);
-    if (a.gate == 0 ? !a.decay : a.gate == 1 ? (!a.dt || !a.a_log) : (a.gate != 2 || !a.keep || !a.take))
+    if (a.gate == 0 ? !a.decay : a.gate == 1 ? (!a.dt || !a.a_log) : a.gate == 3 ? (a.skip || a.unit_column) : (a.gate != 2 || !a.keep || !a.take))
         LLME_REFUSE("recurrence: gate %d lacks its constants", a.gate);
     if (a.unit_column && (a.p < 2 || a.skip)) LLME_REFUSE("recurrence: a column without v stands beside others and has no skip");
     if (a.n > 512) LLME_REFUSE("recurrence: a state of %d rows per column, this build takes up to 512", a.n);
@@ -684,15 +721,12 @@ LLME_API int llme_recurrence(const LlmeRecurrenceArgs* args, cudaStream_t stream
     if (a.max_len <= 1 || a.p < 4) {                                    // single tokens, or too few columns for four a warp
         const int warps = a.p >= 8 ? 8 : a.p;
         const dim3 grid((a.p + warps - 1) / warps, a.heads, a.requests), block(32 * warps);
-        if (a.n <= 32) llme_launch(recurrence_column_kernel<1>, grid, block, 0, stream, a);
-        else if (a.n <= 64) llme_launch(recurrence_column_kernel<2>, grid, block, 0, stream, a);
-        else if (a.n <= 128) llme_launch(recurrence_column_kernel<4>, grid, block, 0, stream, a);
-        else if (a.n <= 256) llme_launch(recurrence_column_kernel<8>, grid, block, 0, stream, a);
-        else llme_launch(recurrence_column_kernel<16>, grid, block, 0, stream, a);
+        if (a.gate == 3) recurrence_columns<true>(a, grid, block, stream);
+        else recurrence_columns<false>(a, grid, block, stream);
         LLME_LAUNCH_STATUS();
     }
     const long long hpn = (long long)a.heads * a.p * a.n;
-    const long long slots = a.scratch ? a.scratch_floats / (hpn + a.heads) : 0;
+    const long long slots = a.scratch ? a.scratch_floats / (hpn + (a.gate == 3 ? (long long)a.heads * a.n : a.heads)) : 0;
     const int chunk = recurrence_chunk(a.tokens, a.max_len, slots, (long long)((a.p + REC_COLUMNS - 1) / REC_COLUMNS) * a.heads);
     // 16-byte copies where every row of q and k starts on such a boundary
     const int vec = ((uintptr_t)a.q % 16 == 0 && (uintptr_t)a.k % 16 == 0 && a.ldq % 4 == 0 && a.ldk % 4 == 0 && a.n % 4 == 0) ? 1 : 0;
@@ -708,6 +742,55 @@ LLME_API int llme_recurrence(const LlmeRecurrenceArgs* args, cudaStream_t stream
     const long long blocks = (hpn + 255) / 256;
     llme_launch(recurrence_join_kernel, dim3((unsigned)(blocks < 1024 ? blocks : 1024), a.requests), dim3(256), 0, stream, a, chunk, (int)slots);
     recurrence_tiles<false>(a, grid, REC_FROM_START, chunk, (int)slots, vec, stream);
+    LLME_LAUNCH_STATUS();
+}
+
+// ----------------------------------------------------------------------------- forget gates per channel
+// q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in + f_bias): what enters a memory with a forget gate per row, formed once per token
+// (every column of the memory reads it).  N columns a thread.
+template <int N>
+__global__ void __launch_bounds__(128) forget_gates_kernel(LlmeForgetGatesArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    for (int c = N * (blockIdx.y * blockDim.x + threadIdx.x); c < a.cols; c += N * gridDim.y * blockDim.x) {
+        __align__(16) float q[N], f[N], b[N], l[N];
+        if (N == 4) {
+            *(float4*)q = *(const float4*)(a.q_in + (size_t)t * a.ld_in + c);
+            *(float4*)f = *(const float4*)(a.f_in + (size_t)t * a.ld_in + c);
+            *(float4*)b = *(const float4*)(a.f_bias + c);
+            *(float4*)l = *(const float4*)(a.lower + c);
+        } else {
+            q[0] = a.q_in[(size_t)t * a.ld_in + c];
+            f[0] = a.f_in[(size_t)t * a.ld_in + c];
+            b[0] = a.f_bias[c];
+            l[0] = a.lower[c];
+        }
+#pragma unroll
+        for (int e = 0; e < N; ++e) {
+            q[e] = silu32(q[e]);
+            f[e] = fmaf(1.0f - l[e], 1.0f / (1.0f + expf(-(f[e] + b[e]))), l[e]);
+        }
+        if (N == 4) {
+            *(float4*)(a.q + (size_t)t * a.ldq + c) = *(const float4*)q;
+            *(float4*)(a.f + (size_t)t * a.ldf + c) = *(const float4*)f;
+        } else {
+            a.q[(size_t)t * a.ldq + c] = q[0];
+            a.f[(size_t)t * a.ldf + c] = f[0];
+        }
+    }
+}
+
+LLME_API int llme_forget_gates(const LlmeForgetGatesArgs* args, cudaStream_t stream) {
+    const LlmeForgetGatesArgs& a = *args;
+    if (a.tokens <= 0 || a.cols <= 0) return 0;
+    if (!a.q_in || !a.f_in || !a.f_bias || !a.lower || !a.q || !a.f) LLME_REFUSE("forget_gates: null pointer");
+    const bool fours = a.cols % 4 == 0 && a.ld_in % 4 == 0 && a.ldq % 4 == 0 && a.ldf % 4 == 0 &&
+                       (((uintptr_t)a.q_in | (uintptr_t)a.f_in | (uintptr_t)a.f_bias | (uintptr_t)a.lower | (uintptr_t)a.q | (uintptr_t)a.f) & 15) == 0;
+    const int each = fours ? 512 : 128, most = (a.cols + each - 1) / each, fill = (592 + a.tokens - 1) / a.tokens;
+    const dim3 grid(a.tokens, most < fill ? most : fill);
+    if (fours) llme_launch(forget_gates_kernel<4>, grid, dim3(128), 0, stream, a);
+    else llme_launch(forget_gates_kernel<1>, grid, dim3(128), 0, stream, a);
     LLME_LAUNCH_STATUS();
 }
 
@@ -794,7 +877,7 @@ LLME_API int llme_exp_gates(const LlmeExpGatesArgs* args, int max_len, cudaStrea
 }
 
 // ----------------------------------------------------------------------------- grouped RMS norm with a silu gate
-__device__ __forceinline__ float gate32(float z, int act) { return act == 1 ? 1.0f / (1.0f + expf(-z)) : silu32(z); }
+__device__ __forceinline__ float gate32(float z, int act) { return act == 2 ? 1.0f : act == 1 ? 1.0f / (1.0f + expf(-z)) : silu32(z); }
 
 // T: the type of the result, GT: of the gate (that of the result, or 32-bit).
 template <typename T, typename GT>
@@ -818,7 +901,7 @@ __global__ void gated_norm_kernel(LlmeGatedNormArgs a) {
     }
     const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.group + a.eps);
     for (int c = lane; c < a.group; c += 32) {
-        const float gate = gate32(to_f32(g[c]), a.gate_act);
+        const float gate = a.gate ? gate32(to_f32(g[c]), a.gate_act) : 1.0f;
         const float yc = a.floor ? y[c] / den : y[c];
         float u = (a.gate_first ? yc * gate : yc) * rinv;
         if (a.weight) u *= a.weight[c0 + c];
@@ -856,7 +939,7 @@ __global__ void __launch_bounds__(128) gated_norm_fours_kernel(LlmeGatedNormArgs
         const int c = 4 * (lane + 32 * i);
         if (c < a.group) {
             load_four<float>(y + c, u[i]);
-            load_four<GT>(g + c, gate[i]);
+            if (a.gate) load_four<GT>(g + c, gate[i]);
         } else {
 #pragma unroll
             for (int e = 0; e < 4; ++e) u[i][e] = gate[i][e] = 0.0f;
@@ -876,9 +959,9 @@ __global__ void __launch_bounds__(128) gated_norm_fours_kernel(LlmeGatedNormArgs
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             // (a result that goes to bfloat16 takes the hardware's exponential and reciprocal)
-            const float z = gate[i][e];
+            const float z = a.gate ? gate[i][e] : 0.0f;
             const float s = sizeof(T) == 2 ? __frcp_rn(1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
-            u[i][e] = u[i][e] * rinv * w[e] * (a.gate_act == 1 ? s : z * s) * a.scale;
+            u[i][e] = u[i][e] * rinv * w[e] * (!a.gate ? 1.0f : a.gate_act == 1 ? s : z * s) * a.scale;
         }
         store_four<T>(o + c, u[i]);
     }
@@ -914,7 +997,7 @@ __global__ void __launch_bounds__(128) gated_norm_block_kernel(LlmeGatedNormArgs
     for (int i = 0; i < 8; ++i) {
         const int c = threadIdx.x + blockDim.x * i;
         u[i] = c < a.group ? y[c] : 0.0f;
-        gate[i] = c < a.group ? to_f32(g[c]) : 0.0f;
+        gate[i] = a.gate && c < a.group ? to_f32(g[c]) : 0.0f;
     }
     // (the normaliser and its floor are asked for with the row's values, not before them)
     const float den = a.floor ? fmaxf(fabsf(y[a.group]), a.floor[(size_t)t * a.ld_floor + gi]) + a.den_eps : 1.0f;
@@ -940,7 +1023,7 @@ __global__ void __launch_bounds__(128) gated_norm_block_kernel(LlmeGatedNormArgs
 LLME_API int llme_gated_norm(const LlmeGatedNormArgs* args, cudaStream_t stream) {
     const LlmeGatedNormArgs& a = *args;
     if (a.tokens <= 0 || a.cols <= 0) return 0;
-    if (!a.y || !a.gate || !a.out) LLME_REFUSE("gated_norm: null pointer");
+    if (!a.y || !a.out || (!a.gate && (a.gate_first || a.gate_act != 2))) LLME_REFUSE("gated_norm: null pointer");
     if (a.group <= 0 || a.cols % a.group) LLME_REFUSE("gated_norm: %d columns are not whole groups of %d", a.cols, a.group);
     if (!(a.eps > 0.0f)) LLME_REFUSE("gated_norm: eps must be positive");
     const long long items = (long long)a.tokens * (a.cols / a.group);

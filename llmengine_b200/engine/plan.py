@@ -29,6 +29,19 @@ class Op:
     a: Dict[str, Any] = field(default_factory=dict)
 
 
+@dataclass(frozen=True)
+class StreamUpdate:
+    """A sublayer's result on its way into S residual streams: x_t <- sum_s mix[s, t] x_s + put[t] * y * sigmoid(gate + bias),
+    all streams from the old ones.  y [T, D] 32-bit; gate [T, D] (any type) and bias [D], or neither: no gate; mix [S, S] and
+    put [S] 32-bit."""
+
+    y: torch.Tensor
+    gate: Optional[torch.Tensor]
+    bias: Optional[torch.Tensor]
+    mix: torch.Tensor
+    put: torch.Tensor
+
+
 class Plan:
     def __init__(self) -> None:
         self.ops: List[Op] = []
@@ -50,12 +63,16 @@ class Plan:
         self.ops.append(Op(kind, a))
 
     def embedding(self, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0, accumulate: bool = False,
-                  delta: Optional[torch.Tensor] = None) -> None:
+                  delta: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None, streams: int = 1) -> None:
         """out[t] = table[token_ids[t]] * scale as 32-bit, for the step's tokens; with `accumulate`, out[t] = (out[t] + delta[t])
-        + that row (`delta`, a pending contribution, may be None)."""
+        + that row (`delta`, a pending contribution, may be None).  With `positions` [P, D] (a table of the type of `table`) row p
+        of it is added to a token at position p; with `streams` S the row is written S times side by side (out [T, S D])."""
+        if accumulate and (positions is not None or streams != 1):
+            raise ValueError("embedding: rows with positions or several streams are not added to a stream that exists")
         if delta is not None and not accumulate:
             raise ValueError("embedding: a contribution is only added to a stream that exists")
-        self._add("embedding", table=table, out=out, scale=float(scale), accumulate=bool(accumulate), delta=delta)
+        self._add("embedding", table=table, out=out, scale=float(scale), accumulate=bool(accumulate), delta=delta,
+                  positions=positions, streams=int(streams))
         if accumulate:
             self.note_copy(out, None)
 
@@ -142,7 +159,7 @@ class Plan:
 
     def latent_attention(self, *, q_rot, kv_in, c_gain, eps: float, inv_freq, rot_dims: int, q, out, cache, group: int,
                          num_heads: int, kv_rank: int, rot_dim: int, scale: float, sink=None, scratch=None, window: int = 0,
-                         interleaved: bool = False) -> None:
+                         interleaved: bool = False, amplitude: float = 1.0) -> None:
         """Attention over a cache of latents, one row [c | rotated key part] per token, shared by all heads.
         `kv_in` [T, kv_rank + rot_dim] is the raw down-projection: its first kv_rank values are RMS-normed with
         `c_gain`, the rest rotated by the token's position (`inv_freq`: rot_dims / 2 frequencies; none: no positions),
@@ -150,10 +167,11 @@ class Plan:
         its last rot_dim values are filled here from `q_rot` [T, H, rot_dim] (a strided view), rotated.  Then
         score = (q . row) * scale, causal (with `window` W > 0 query i sees key j only if i - j < W), softmax (with `sink`
         [H]: the denominator also holds exp(sink_h)), and out[t, h, :] = sum_j w_j c_j  [T, H, kv_rank].  `interleaved`:
-        the rotation pairs coordinate 2i with 2i + 1 instead of i with i + rot_dims / 2."""
+        the rotation pairs coordinate 2i with 2i + 1 instead of i with i + rot_dims / 2.  `amplitude` multiplies cosine and sine."""
         self._add("latent_attention", q_rot=q_rot, kv_in=kv_in, c_gain=c_gain, eps=float(eps), inv_freq=inv_freq,
                   rot_dims=int(rot_dims), q=q, out=out, cache=cache, group=group, num_heads=num_heads, kv_rank=kv_rank,
-                  rot_dim=rot_dim, scale=float(scale), sink=sink, scratch=scratch, window=int(window), interleaved=bool(interleaved))
+                  rot_dim=rot_dim, scale=float(scale), sink=sink, scratch=scratch, window=int(window), interleaved=bool(interleaved),
+                  amplitude=float(amplitude))
 
     def token_side(self, *, x, a, b, table, offset: int, dim: int, w_gate, w_proj, gain, eps: float, xb, g, y) -> None:
         """x += a (+ b); e = table[token][offset : offset + dim]; g = gelu_tanh(w_gate x) * e; y = w_proj g;
@@ -175,7 +193,7 @@ class Plan:
                          q, out, cache, group: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int,
                          window: int, keep_first: int, scale: float, sink=None, scratch=None, q_bias=None, k_bias=None,
                          v_bias=None, head_norm: bool = False, softcap: float = 0.0, interleaved: bool = False,
-                         unit_norm: bool = False, decode_scratch=None) -> None:
+                         unit_norm: bool = False, decode_scratch=None, value_share: int = 1) -> None:
         """Grouped-query attention over a cache whose keys are `qk_dim` and whose values are `v_dim` wide, from the raw
         projections: q_in [T, H qk_dim] and, for a layer that stores, k_in [T, G qk_dim] and v_in [T, G v_dim] (column
         ranges of one product).  With gains, queries and keys are RMS-normed over the WHOLE projection (all heads at
@@ -192,12 +210,14 @@ class Plan:
         be 32-bit where everything else has the type of the products (they then come from a convolution, not a product).
         `unit_norm`: behind the rotation every query and key head is divided by its own sqrt(mean(x^2) + eps) (no gains).
         `decode_scratch`: scratch memory of the kernels of ordinary grouped-query attention, which serve the record where its
-        mask and softmax are theirs (one width for keys and values, no kept first positions, no sink, no cap)."""
+        mask and softmax are theirs (one width for keys and values, no kept first positions, no sink, no cap).
+        `value_share` n: n neighbouring key heads attend to the same value head (v_in [T, G / n v_dim], a page holds G / n value
+        heads): the maps of a differential attention."""
         self._add("window_attention", q_bias=q_bias, k_bias=k_bias, v_bias=v_bias, head_norm=bool(head_norm), q_in=q_in, k_in=k_in, v_in=v_in, q_gain=q_gain, k_gain=k_gain, eps=float(eps),
                   inv_freq=inv_freq, rot_dims=int(rot_dims), amplitude=float(amplitude), q=q, out=out, cache=cache, group=group,
                   num_heads=num_heads, num_kv_heads=num_kv_heads, qk_dim=qk_dim, v_dim=v_dim, window=int(window),
                   keep_first=int(keep_first), scale=float(scale), sink=sink, scratch=scratch, softcap=float(softcap),
-                  interleaved=bool(interleaved), unit_norm=bool(unit_norm), decode_scratch=decode_scratch)
+                  interleaved=bool(interleaved), unit_norm=bool(unit_norm), decode_scratch=decode_scratch, value_share=int(value_share))
 
     def moe_route(self, *, logits, top_k: int, scale: float, experts, weights, offsets, order, counts,
                   mode: str = "sigmoid", correction=None, groups: tuple = (1, 1)) -> None:
@@ -206,13 +226,16 @@ class Plan:
         s_e / (sum over C of s + 1e-20).  `mode` "softmax_chosen": C = the experts of largest logits and w_e = scale *
         exp(z_e) / sum over C of exp(z).  `mode` "softmax": s = softmax(z) over all E; the choice goes by s (+ `correction` [E],
         32-bit), C = the `top_k` largest among the members of the groups[1] groups with the largest best member (the E choices
-        form groups[0] equal groups of neighbours); w_e = scale * s_e.  The (token, choice) pairs are then listed expert by expert:
+        form groups[0] equal groups of neighbours); w_e = scale * s_e.  With groups in the mode "sigmoid" a group is as good as the
+        sum of its two largest s.  The (token, choice) pairs are then listed expert by expert:
         `offsets` [E + 1] int32 with the pairs of expert e at order[offsets[e] : offsets[e + 1]], a pair being
         token * top_k + choice.  `counts` [E] int32 is scratch that is zero between launches."""
         if mode not in ("sigmoid", "softmax_chosen", "softmax"):
             raise ValueError(f"moe_route: unknown mode {mode!r}")
-        if mode != "softmax" and (correction is not None or tuple(groups) != (1, 1)):
-            raise ValueError("moe_route: corrections and groups belong to the mode 'softmax'")
+        if mode != "softmax" and correction is not None:
+            raise ValueError("moe_route: corrections belong to the mode 'softmax'")
+        if mode == "softmax_chosen" and groups[1] < groups[0]:
+            raise ValueError("moe_route: groups belong to the modes 'softmax' and 'sigmoid'")
         self._add("moe_route", logits=logits, top_k=int(top_k), scale=float(scale), experts=experts, weights=weights,
                   offsets=offsets, order=order, counts=counts, mode=mode, correction=correction, groups=(int(groups[0]), int(groups[1])))
 
@@ -222,7 +245,7 @@ class Plan:
         out_row = w[e] x_row, with x_row = x[order[r] // top_k] if `gather` (the token's row) else x[r], and written
         to out[order[r]] if `scatter` (the pair's row) else out[r].  w is [E, n, k].  With `act` "silu", w[e] is
         [gate | up] by rows and the row written is silu(gate) * up, half as wide; with `act` "relu2" the row written is
-        max(product, 0)^2 (`mid` [pairs, n]: workspace of the form that runs product and activation apart).  `rows` [pairs, k]: where a kernel that wants its rows side by side puts gathered
+        max(product, 0)^2, with "gelu" it is z Phi(z), the erf form (`mid` [pairs, n]: workspace of the form that runs product and activation apart).  `rows` [pairs, k]: where a kernel that wants its rows side by side puts gathered
         ones."""
         self._add("grouped_linear", x=x, w=w, out=out, offsets=offsets, order=order, top_k=int(top_k), gather=bool(gather),
                   scatter=bool(scatter), mid=mid, act=act, rows=rows)
@@ -248,7 +271,7 @@ class Plan:
                   inv_freq=inv_freq)
 
     def recurrence(self, *, q, k, v, state, out, heads: int, n: int, p: int, qk_groups: int, decay=None, dt=None, dt_bias=None,
-                   a_log=None, skip=None, scratch=None, keep=None, take=None, unit_column: bool = False) -> None:
+                   a_log=None, skip=None, scratch=None, keep=None, take=None, unit_column: bool = False, forget: bool = False) -> None:
         """Per request and head, over the request's tokens in order: S_t = a_t S_(t-1) + s_t k_t v_t^T (S is n x p),
         y_t = S_t^T q_t + skip_h v_t.  With `decay` [H]: a_t = decay_h, s_t = 1.  With `dt` [T, H], `dt_bias` and `a_log`
         [H]: d = softplus(dt + dt_bias), a_t = exp(-exp(a_log_h) d), s_t = d.  q, k [T, qk_groups * n] and out [T, H p] are
@@ -256,10 +279,13 @@ class Plan:
         (32-bit, a few states large) a long portion is cut into pieces that run side by side.  With `keep` and `take` [T, H]
         (32-bit): a_t = keep[t, h], s_t = take[t, h], both made by an earlier record.  `unit_column`: the last of the p columns
         has no v behind it, its v_t is one (that column of S sums s_t k_t alone, and that column of y is its product with q);
-        v is then [T, H (p - 1)]."""
+        v is then [T, H (p - 1)].  `forget`: `k` holds a forget gate f per row of S, and row c decays by f_c and takes the rest:
+        S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T."""
+        if forget and (decay is not None or dt is not None or keep is not None or skip is not None or unit_column):
+            raise ValueError("recurrence: a forget gate per row excludes other decays, steps, skips and unit columns")
         self._add("recurrence", q=q, k=k, v=v, state=state, out=out, heads=int(heads), n=int(n), p=int(p), qk_groups=int(qk_groups),
                   decay=decay, dt=dt, dt_bias=dt_bias, a_log=a_log, skip=skip, scratch=scratch, keep=keep, take=take,
-                  unit_column=bool(unit_column))
+                  unit_column=bool(unit_column), forget=bool(forget))
 
     def delta_rule(self, *, q, k, v, write, forget, dt_bias, a_log, q_scale: float, unit_eps: float, state, out, heads: int, n: int,
                    p: int, qk_groups: int, unit, coef) -> None:
@@ -275,7 +301,7 @@ class Plan:
 
     def gated_norm(self, *, y, gate, weight, out, group: int, gate_first: bool, eps: float, scale: float = 1.0,
                    gate_act: str = "silu", floor=None, den_eps: float = 0.0) -> None:
-        """RMS norm of y [T, C] (32-bit) in groups of `group` columns, with g = silu(gate) (`gate_act` "sigmoid": sigmoid(gate)):
+        """RMS norm of y [T, C] (32-bit) in groups of `group` columns, with g = silu(gate) (`gate_act` "sigmoid": sigmoid(gate); `gate` None: g = 1):
         `gate_first`: u = y g, out = u / rms(u) * weight; else out = y / rms(y) * weight * g; then times `scale`.  `weight` [C]
         32-bit or None.  With `floor` [T, C / group] (32-bit) every group of y is one column wider than its group of the gate
         and of out: the extra value d stands behind the group's own, and the group is divided by max(|d|, floor) + den_eps
@@ -284,6 +310,31 @@ class Plan:
             raise ValueError(f"gated_norm: unknown gate {gate_act!r}")
         self._add("gated_norm", y=y, gate=gate, weight=weight, out=out, group=int(group), gate_first=bool(gate_first),
                   eps=float(eps), scale=float(scale), gate_act=gate_act, floor=floor, den_eps=float(den_eps))
+
+    def stream_norm(self, x: torch.Tensor, *, streams: int, read: Optional[torch.Tensor], gain: Optional[torch.Tensor], eps: float,
+                    out: Optional[torch.Tensor], update: Optional[StreamUpdate] = None, rows: str = ROWS_TOKENS) -> None:
+        """x [T, S D]: S residual streams side by side, 32-bit.  With `update` they take a sublayer's result (StreamUpdate); then
+        u = sum_s read[s] x_s (`read` [S] 32-bit) and out = u / sqrt(mean(u^2) + eps) * gain (`gain` [D] 32-bit).  `out` None: only
+        the update.  `rows` = "logits": only the step's wanted rows, gathered into the first rows of `out`, and x stays as it is
+        (the last norm of a model)."""
+        if update is None and out is None:
+            raise ValueError("stream_norm: nothing to update and nothing to write")
+        u = update
+        self._add("stream_norm", x=x, streams=int(streams), read=read, gain=gain, eps=float(eps), out=out, rows=rows,
+                  y=u.y if u else None, gate=u.gate if u else None, gate_bias=u.bias if u else None, mix=u.mix if u else None,
+                  put=u.put if u else None)
+        self.note_copy(x, None)
+
+    def forget_gates(self, *, q_in, f_in, f_bias, lower, q, f) -> None:
+        """What enters a memory with a forget gate per channel, all 32-bit: q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in +
+        f_bias), elementwise; q_in, f_in, q and f are [T, C] (any row stride), f_bias and lower [C]."""
+        self._add("forget_gates", q_in=q_in, f_in=f_in, f_bias=f_bias, lower=lower, q=q, f=f)
+
+    def difference_norm(self, *, a, weight: float, scale: float, eps: float, heads: int, rep: int, out) -> None:
+        """The two maps of a differential attention become its heads.  `a` [T, 2 heads P] holds the maps' outputs group by group of
+        `rep` heads: the group's heads of map 1, then those of map 2.  Per head u = a1 - weight * a2, out = u / sqrt(mean(u^2) +
+        eps) * scale, [T, heads P] head by head; 32-bit arithmetic."""
+        self._add("difference_norm", a=a, weight=float(weight), scale=float(scale), eps=float(eps), heads=int(heads), rep=int(rep), out=out)
 
     def row_norm(self, *, x, gain, eps: float, out) -> None:
         """out = x / sqrt(mean(x^2) + eps) * gain over the rows of x [T, C]: a norm on (a column range of) a product, in

@@ -70,7 +70,8 @@ enum LlmeOpKind {
     LLME_OP_ATTENTION, LLME_OP_CALL, LLME_OP_LINEAR_ACT, LLME_OP_POINTWISE, LLME_OP_BATCHED_LINEAR, LLME_OP_RESIDUAL_ADD,
     LLME_OP_LATENT_ATTENTION, LLME_OP_TOKEN_SIDE, LLME_OP_POSTNORM, LLME_OP_WINDOW_ATTENTION, LLME_OP_MOE_ROUTE,
     LLME_OP_GROUPED_LINEAR, LLME_OP_MOE_COMBINE, LLME_OP_SHORT_CONV, LLME_OP_ROTATE, LLME_OP_RECURRENCE, LLME_OP_GATED_NORM,
-    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES, LLME_OP_LAYERNORM, LLME_OP_DELTA_RULE
+    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES, LLME_OP_LAYERNORM, LLME_OP_DELTA_RULE, LLME_OP_STREAM_NORM, LLME_OP_FORGET_GATES,
+    LLME_OP_DIFFERENCE_NORM
 };
 
 enum { LLME_ACT_XIELU = 1, LLME_ACT_RELU2 = 2 };   /* 2: max(z, 0)^2 */
@@ -87,6 +88,8 @@ typedef struct LlmeEmbeddingOp {
     float scale;               /* every row times this constant, in 32-bit (1: none) */
     int accumulate;            /* 1: out = (out + delta) + row: the embedding output added to a stream that exists */
     const float* delta;        /* with accumulate: a contribution still to be added, or NULL */
+    const void* pos_table; int max_positions;   /* [max_positions, hidden] of the type of the table: row p added at position p; or NULL */
+    int streams;               /* copies of the row side by side: out [T, streams * hidden] (0 counts as 1) */
 } LlmeEmbeddingOp;
 
 typedef struct LlmeRmsNormOp {
@@ -108,6 +111,36 @@ typedef struct LlmeLayerNormOp {
     int size; float eps;
     int rows;                  /* LLME_ROWS_TOKENS or LLME_ROWS_LOGITS */
 } LlmeLayerNormOp;
+
+/* Residual streams x [T, streams * size], 32-bit, side by side (csrc/streams.cu).  With y: x_t <- sum_s mix[s, t] x_s + put[t] y
+ * sigmoid(gate + gate_bias) (gate NULL: no gate), all streams from the old ones.  Then, with out: u = sum_s read[s] x_s, out = u /
+ * sqrt(mean(u^2) + eps) * gain.  LLME_ROWS_LOGITS: the step's wanted rows only, and x stays as it is. */
+typedef struct LlmeStreamNormOp {
+    float* x; int streams, size;
+    const float* y;
+    const void* gate; long long ldg; int gate_dtype; const float* gate_bias;
+    const float* mix; const float* put;
+    const float* read; const float* gain; float eps;
+    void* out; int out_dtype;
+    int rows;
+} LlmeStreamNormOp;
+
+/* q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in + f_bias) over [T, cols], 32-bit. */
+typedef struct LlmeForgetGatesOp {
+    const float* q_in; const float* f_in; long long ld_in;
+    const float* f_bias; const float* lower;
+    float* q; float* f; long long ldq, ldf;
+    int cols;
+} LlmeForgetGatesOp;
+
+/* The maps of a differential attention become its heads: a [T, 2 heads dim] holds, per group of `rep` heads, the heads of map 1 and
+ * then those of map 2; u = a1 - weight a2, out = u / sqrt(mean(u^2) + eps) * scale, [T, heads dim] head by head. */
+typedef struct LlmeDifferenceNormOp {
+    const void* a; long long lda;
+    void* out; long long ldo;
+    int dtype, heads, rep, dim;
+    float weight, scale, eps;
+} LlmeDifferenceNormOp;
 
 typedef struct LlmeLinearOp {
     const void* x; long long ldx; int x_dtype;
@@ -203,6 +236,7 @@ typedef struct LlmeLatentAttentionOp {
     float* scratch; long long scratch_floats;
     int window;                                               /* W > 0: query i sees key j only if i - j < W */
     int interleaved;                                          /* 1: the rotation pairs coordinate 2i with 2i + 1 */
+    float amplitude;                                          /* cosine and sine times this constant */
 } LlmeLatentAttentionOp;
 
 /* x += a (+ b); e = table[token][offset .. offset + dim); g = gelu_tanh(w_gate x) * e; y = w_proj g;
@@ -247,6 +281,7 @@ typedef struct LlmeWindowAttentionOp {
     /* scratch of the kernels of ordinary grouped-query attention, which serve the record where its mask and softmax are theirs
      * (dk = dv, keep_first 0, no sink, no cap); NULL: they do not */
     float* decode_scratch; long long decode_scratch_floats; long long cache_pages;
+    int value_share;                                         /* n > 1: n neighbouring key heads share one value head (v_in and a page hold nkv / n) */
 } LlmeWindowAttentionOp;
 
 /* Routing of a mixture of experts: s = sigmoid(logits), the top_k largest, w_e = scale * s_e / (sum of the chosen s + 1e-20);
@@ -256,7 +291,8 @@ typedef struct LlmeMoeRouteOp {
     int* experts; float* weights; int* offsets; int* order; int* counts;
     int mode;                  /* 0: as above; 1: the largest logits chosen, w_e = scale * softmax over the chosen logits alone; 2: s = softmax over all */
     const float* correction;   /* mode 2: added to s for the choice alone ([E], or NULL); the choices form `groups` equal groups of */
-    int groups, keep;          /* neighbours, and the members of the `keep` groups with the largest best member can be chosen; w_e = scale s_e */
+    int groups, keep;          /* neighbours, and the members of the `keep` groups with the largest best member can be chosen; w_e = scale s_e.
+                                  mode 0: the groups with the largest sum of their two largest s */
 } LlmeMoeRouteOp;
 
 /* One product per expert over the pairs routed to it. */
@@ -266,7 +302,7 @@ typedef struct LlmeGroupedLinearOp {
     void* out; long long ldo; int out_dtype;
     void* mid; long long ld_mid;                              /* [pairs, n]: workspace of the unfused activation, or NULL */
     const int* offsets; const int* order;
-    int num_experts, top_k, n, k, gather, scatter, act;       /* act 1: w[e] = [gate | up], out = silu(gate) * up; 2: out = max(product, 0)^2 */
+    int num_experts, top_k, n, k, gather, scatter, act;       /* act 1: w[e] = [gate | up], out = silu(gate) * up; 2: out = max(product, 0)^2; 3: gelu (erf) */
     void* rows;                                               /* [pairs, k] in the type of x: where gathered rows come to stand side by side, or NULL */
 } LlmeGroupedLinearOp;
 
@@ -313,6 +349,7 @@ typedef struct LlmeRecurrenceOp {
     /* gate 2: a_t = keep[t, h], s_t = take[t, h] (32-bit, row stride ld_gates), made by an earlier record */
     const float* keep; const float* take; long long ld_gates;
     int unit_column;                                         /* 1: column p - 1 has no v behind it, its v_t is one; v is [T, heads (p - 1)] */
+    /* gate 3: k holds a forget gate f per row of S: S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T */
 } LlmeRecurrenceOp;
 
 /* RMS norm in groups of `group` columns with a silu gate: gate_first 1: u = y silu(g), out = u / rms(u) * weight; 0:
@@ -324,7 +361,7 @@ typedef struct LlmeGatedNormOp {
     void* out; long long ldo;
     int dtype, cols, group, gate_first;
     float eps, scale;
-    int gate_act;                                            /* 0: silu(g); 1: sigmoid(g) */
+    int gate_act;                                            /* 0: silu(g); 1: sigmoid(g); 2: no gate */
     /* with `floor` [T, cols / group] every group of y is one value wider: the extra value d stands behind the group's own, and
      * the group is divided by max(|d|, floor) + den_eps before anything else */
     const float* floor; long long ld_floor; float den_eps;
@@ -379,7 +416,7 @@ void llme_executor_destroy(LlmeExecutor*);
  * key and value sizes "window_attention_tc/<dk>x<dv>", "moe_route", "grouped_linear", "grouped_linear_tc", "moe_combine";
  * "short_conv", "rotate", "recurrence", "gated_norm", "row_norm", "exp_gates", "sigmoid_mul_grouped", "residual_add_scaled",
  * "layernorm", "embedding_add", "relu2", "delta_step", "delta_portions", "grouped_tcgen05",
- * "grouped_tcgen05_supports". */
+ * "grouped_tcgen05_supports"; "embedding_streams", "stream_norm", "forget_gates", "difference_norm". */
 int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
 /* Which implementation an operation takes.  Operations and their variants:
  *   "linear":            "auto" | "tcgen05" | "cublas" | "plain"   (bfloat16 products of 128 tokens or more / all)
@@ -474,6 +511,9 @@ public:
     int add(const LlmeExpGatesOp& r) { return add(LLME_OP_EXP_GATES, &r, sizeof r); }
     int add(const LlmeLayerNormOp& r) { return add(LLME_OP_LAYERNORM, &r, sizeof r); }
     int add(const LlmeDeltaRuleOp& r) { return add(LLME_OP_DELTA_RULE, &r, sizeof r); }
+    int add(const LlmeStreamNormOp& r) { return add(LLME_OP_STREAM_NORM, &r, sizeof r); }
+    int add(const LlmeForgetGatesOp& r) { return add(LLME_OP_FORGET_GATES, &r, sizeof r); }
+    int add(const LlmeDifferenceNormOp& r) { return add(LLME_OP_DIFFERENCE_NORM, &r, sizeof r); }
     /* One step through the whole plan; throws with the failing record's message. */
     void run(const LlmeStep& step, cudaStream_t stream) {
         if (llme_plan_run(h_, &step, 0, -1, stream)) throw std::runtime_error(ex_.error());

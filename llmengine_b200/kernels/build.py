@@ -39,6 +39,8 @@ SOURCES: Dict[str, str] = {
     # mixture of experts: routing, the grouped product (plain form), the weighted sum; and the grouped product on tensor cores
     # layers with a state of fixed size per request: short convolution, linear recurrence, gated group norm
     "recurrent": "recurrent.cu",
+    # residual streams: a sublayer's result into all of them, the next sublayer's input out of them, normed
+    "streams": "streams.cu",
     # the gated delta rule: single tokens, and portions eight tokens at a time
     "delta_rule": "delta_rule.cu",
     "moe": "moe.cu",

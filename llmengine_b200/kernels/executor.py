@@ -14,11 +14,11 @@ ROWS = {"tokens": 0, "logits": 1}
 (OP_EMBEDDING, OP_RMSNORM, OP_LINEAR, OP_LINEAR_SWIGLU, OP_QKV_POST, OP_ATTEND, OP_ATTENTION, OP_CALL, OP_LINEAR_ACT,
  OP_POINTWISE, OP_BATCHED_LINEAR, OP_RESIDUAL_ADD, OP_LATENT_ATTENTION, OP_TOKEN_SIDE, OP_POSTNORM, OP_WINDOW_ATTENTION,
  OP_MOE_ROUTE, OP_GROUPED_LINEAR, OP_MOE_COMBINE, OP_SHORT_CONV, OP_ROTATE, OP_RECURRENCE, OP_GATED_NORM, OP_ROW_NORM,
- OP_EXP_GATES, OP_LAYERNORM, OP_DELTA_RULE) = range(1, 28)
+ OP_EXP_GATES, OP_LAYERNORM, OP_DELTA_RULE, OP_STREAM_NORM, OP_FORGET_GATES, OP_DIFFERENCE_NORM) = range(1, 31)
 GATES = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}
 ROUTING = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
 ACTIVATIONS = {"xielu": 1, "relu2": 2}
-EXPERT_ACTIVATIONS = {None: 0, "silu": 1, "relu2": 2}
+EXPERT_ACTIVATIONS = {None: 0, "silu": 1, "relu2": 2, "gelu": 3}
 POINTWISE = {"sigmoid_mul": 1}
 
 
@@ -55,7 +55,24 @@ CallFn = CFUNCTYPE(c_int, c_void_p, POINTER(Step), c_void_p)
 
 class EmbeddingOp(Structure):
     _fields_ = [("table", c_void_p), ("table_dtype", c_int), ("vocab", c_int), ("hidden", c_int), ("out", c_void_p),
-                ("scale", c_float), ("accumulate", c_int), ("delta", c_void_p)]
+                ("scale", c_float), ("accumulate", c_int), ("delta", c_void_p), ("pos_table", c_void_p), ("max_positions", c_int),
+                ("streams", c_int)]
+
+
+class StreamNormOp(Structure):
+    _fields_ = [("x", c_void_p), ("streams", c_int), ("size", c_int), ("y", c_void_p), ("gate", c_void_p), ("ldg", c_longlong),
+                ("gate_dtype", c_int), ("gate_bias", c_void_p), ("mix", c_void_p), ("put", c_void_p), ("read", c_void_p), ("gain", c_void_p),
+                ("eps", c_float), ("out", c_void_p), ("out_dtype", c_int), ("rows", c_int)]
+
+
+class ForgetGatesOp(Structure):
+    _fields_ = [("q_in", c_void_p), ("f_in", c_void_p), ("ld_in", c_longlong), ("f_bias", c_void_p), ("lower", c_void_p), ("q", c_void_p),
+                ("f", c_void_p), ("ldq", c_longlong), ("ldf", c_longlong), ("cols", c_int)]
+
+
+class DifferenceNormOp(Structure):
+    _fields_ = [("a", c_void_p), ("lda", c_longlong), ("out", c_void_p), ("ldo", c_longlong), ("dtype", c_int), ("heads", c_int),
+                ("rep", c_int), ("dim", c_int), ("weight", c_float), ("scale", c_float), ("eps", c_float)]
 
 
 class LayerNormOp(Structure):
@@ -129,7 +146,7 @@ class LatentAttentionOp(Structure):
                 ("inv_freq", c_void_p), ("rot_dims", c_int), ("q", c_void_p), ("out", c_void_p), ("dtype", c_int),
                 ("cache", c_void_p), ("cache_rows", c_longlong), ("group", c_int), ("nh", c_int), ("rank", c_int), ("rot", c_int),
                 ("scale", c_float), ("sink", c_void_p), ("scratch", c_void_p), ("scratch_floats", c_longlong), ("window", c_int),
-                ("interleaved", c_int)]
+                ("interleaved", c_int), ("amplitude", c_float)]
 
 
 class TokenSideOp(Structure):
@@ -152,7 +169,8 @@ class WindowAttentionOp(Structure):
                 ("window", c_int), ("keep_first", c_int), ("scale", c_float), ("sink", c_void_p), ("scratch", c_void_p),
                 ("scratch_floats", c_longlong), ("q_bias", c_void_p), ("k_bias", c_void_p), ("v_bias", c_void_p),
                 ("head_norm", c_int), ("softcap", c_float), ("interleaved", c_int), ("in_f32", c_int), ("unit_norm", c_int),
-                ("decode_scratch", c_void_p), ("decode_scratch_floats", c_longlong), ("cache_pages", c_longlong)]
+                ("decode_scratch", c_void_p), ("decode_scratch_floats", c_longlong), ("cache_pages", c_longlong),
+                ("value_share", c_int)]
 
 
 class MoeRouteOp(Structure):
@@ -294,10 +312,12 @@ def records(op, keep: List[Any]):
     if k == "embedding":
         t, out = a["table"], a["out"]
         assert out.dtype == torch.float32 and t.is_contiguous() and out.is_contiguous()
-        d = a.get("delta")
+        d, p, streams = a.get("delta"), a.get("positions"), int(a.get("streams", 1))
         assert d is None or (d.dtype == torch.float32 and d.is_contiguous() and d.shape == out.shape)
+        assert p is None or (p.dtype == t.dtype and p.is_contiguous() and p.shape[1] == t.shape[1])
+        assert out.shape[1] == streams * t.shape[1]
         return OP_EMBEDDING, EmbeddingOp(t.data_ptr(), code(t.dtype), t.shape[0], t.shape[1], out.data_ptr(), float(a.get("scale", 1.0)),
-                                         1 if a.get("accumulate") else 0, ptr(d))
+                                         1 if a.get("accumulate") else 0, ptr(d), ptr(p), p.shape[0] if p is not None else 0, streams)
     if k == "layernorm":
         x, d, g, b, out = a["x"], a["delta"], a["gain"], a["bias"], a["out"]
         assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and out.shape[1] == x.shape[1]
@@ -389,7 +409,8 @@ def records(op, keep: List[Any]):
             kv.data_ptr(), kv.stride(0), ptr(qr), qr.stride(0) if qr is not None else 0, qr.stride(1) if qr is not None else 0,
             gain.data_ptr(), code(gain.dtype), a["eps"], ptr(freq), a["rot_dims"], q.data_ptr(), out.data_ptr(), code(q.dtype),
             cache.data_ptr(), cache.shape[0] * cache.shape[1], a["group"], H, r, dr, a["scale"], ptr(sink), ptr(scratch),
-            scratch.numel() if scratch is not None else 0, int(a.get("window", 0)), 1 if a.get("interleaved") else 0)
+            scratch.numel() if scratch is not None else 0, int(a.get("window", 0)), 1 if a.get("interleaved") else 0,
+            float(a.get("amplitude", 1.0)))
     if k == "token_side":
         x, u, v, table, wg, wp, gain, xb, g, y = (a[n] for n in ("x", "a", "b", "table", "w_gate", "w_proj", "gain", "xb", "g", "y"))
         D, dim = x.shape[1], a["dim"]
@@ -413,12 +434,15 @@ def records(op, keep: List[Any]):
         H, G, dk, dv = a["num_heads"], a["num_kv_heads"], a["qk_dim"], a["v_dim"]
         wide = qi.dtype == torch.float32 and q.dtype != torch.float32       # 32-bit projections (from a convolution)
         assert q.dtype == out.dtype == cache.dtype and (wide or qi.dtype == q.dtype) and qi.stride(1) == 1 and q.is_contiguous() and out.is_contiguous()
-        assert cache.is_contiguous() and qi.shape[1] == q.shape[1] == H * dk and out.shape[1] == H * dv and cache.shape[1] % (G * (dk + dv)) == 0
+        assert cache.is_contiguous() and qi.shape[1] == q.shape[1] == H * dk and out.shape[1] == H * dv
+        share = int(a.get("value_share", 1))
+        Gv = G // share                                                     # value heads
+        assert G % share == 0 and cache.shape[1] % (G * dk + Gv * dv) == 0
         assert (ki is None) == (vi is None) and (ki is None or (ki.dtype == vi.dtype == qi.dtype and ki.stride(1) == vi.stride(1) == 1
-                                                              and ki.shape[1] == G * dk and vi.shape[1] == G * dv))
+                                                              and ki.shape[1] == G * dk and vi.shape[1] == Gv * dv))
         per_head = bool(a.get("head_norm"))
         for t, n in ((a["q_gain"], dk if per_head else H * dk), (a["k_gain"], dk if per_head else G * dk), (a["sink"], H),
-                     (a["inv_freq"], a["rot_dims"] // 2), (a.get("q_bias"), H * dk), (a.get("k_bias"), G * dk), (a.get("v_bias"), G * dv)):
+                     (a["inv_freq"], a["rot_dims"] // 2), (a.get("q_bias"), H * dk), (a.get("k_bias"), G * dk), (a.get("v_bias"), Gv * dv)):
             assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n)
         return OP_WINDOW_ATTENTION, WindowAttentionOp(
             qi.data_ptr(), ptr(ki), ptr(vi), qi.stride(0), ki.stride(0) if ki is not None else 0, vi.stride(0) if vi is not None else 0,
@@ -427,7 +451,8 @@ def records(op, keep: List[Any]):
             ptr(a["sink"]), ptr(a.get("scratch")), a["scratch"].numel() if a.get("scratch") is not None else 0,
             ptr(a.get("q_bias")), ptr(a.get("k_bias")), ptr(a.get("v_bias")), 1 if a.get("head_norm") else 0,
             float(a.get("softcap", 0.0)), 1 if a.get("interleaved") else 0, 1 if wide else 0, 1 if a.get("unit_norm") else 0,
-            ptr(a.get("decode_scratch")), a["decode_scratch"].numel() if a.get("decode_scratch") is not None else 0, cache.shape[0])
+            ptr(a.get("decode_scratch")), a["decode_scratch"].numel() if a.get("decode_scratch") is not None else 0, cache.shape[0],
+            share)
     if k == "moe_route":
         z, ex_, wt, off, order, counts = a["logits"], a["experts"], a["weights"], a["offsets"], a["order"], a["counts"]
         assert z.dtype == wt.dtype == torch.float32 and z.stride(1) == 1 and ex_.is_contiguous() and wt.is_contiguous()
@@ -496,7 +521,7 @@ def records(op, keep: List[Any]):
         for t in ("decay", "dt_bias", "a_log", "skip"):
             assert _f32(a.get(t), H)
         return OP_RECURRENCE, RecurrenceOp(q.data_ptr(), kk.data_ptr(), q.stride(0), kk.stride(0), G, v.data_ptr(), v.stride(0), code(v.dtype),
-                                           2 if keep is not None else (0 if dt is None else 1), ptr(a.get("decay")), ptr(dt), dt.stride(0) if dt is not None else 0,
+                                           3 if a.get("forget") else 2 if keep is not None else (0 if dt is None else 1), ptr(a.get("decay")), ptr(dt), dt.stride(0) if dt is not None else 0,
                                            code(dt.dtype) if dt is not None else 0, ptr(a.get("dt_bias")), ptr(a.get("a_log")),
                                            ptr(a.get("skip")), st.data_ptr(), st.stride(0), out.data_ptr(), out.stride(0), H, n, p,
                                            ptr(scratch), scratch.numel() if scratch is not None else 0, ptr(keep), ptr(take),
@@ -504,16 +529,38 @@ def records(op, keep: List[Any]):
     if k == "gated_norm":
         y, g, w, out = a["y"], a["gate"], a["weight"], a["out"]
         cols, floor = out.shape[1], a.get("floor")
-        assert y.dtype == torch.float32 and y.stride(1) == g.stride(1) == out.stride(1) == 1 and g.dtype in (out.dtype, torch.float32)
-        assert g.shape[1] == cols and cols % a["group"] == 0 and _f32(w, cols)
+        assert y.dtype == torch.float32 and y.stride(1) == out.stride(1) == 1 and cols % a["group"] == 0 and _f32(w, cols)
+        assert (g is None and not a["gate_first"]) or (g.stride(1) == 1 and g.dtype in (out.dtype, torch.float32) and g.shape[1] == cols)
         groups = cols // a["group"]
         assert y.shape[1] == (cols + groups if floor is not None else cols)
         assert floor is None or (floor.dtype == torch.float32 and floor.stride(1) == 1 and floor.shape[1] == groups)
-        return OP_GATED_NORM, GatedNormOp(y.data_ptr(), y.stride(0), g.data_ptr(), g.stride(0), ptr(w), out.data_ptr(), out.stride(0),
+        return OP_GATED_NORM, GatedNormOp(y.data_ptr(), y.stride(0), ptr(g), g.stride(0) if g is not None else 0, ptr(w), out.data_ptr(), out.stride(0),
                                           code(out.dtype), cols, a["group"], 1 if a["gate_first"] else 0, a["eps"], a["scale"],
-                                          1 if a.get("gate_act", "silu") == "sigmoid" else 0, ptr(floor),
+                                          2 if g is None else 1 if a.get("gate_act", "silu") == "sigmoid" else 0, ptr(floor),
                                           floor.stride(0) if floor is not None else 0, float(a.get("den_eps", 0.0)),
-                                          1 if g.dtype == torch.float32 else 0)
+                                          1 if g is not None and g.dtype == torch.float32 else 0)
+    if k == "stream_norm":
+        x, S, y, g, out, gain = a["x"], a["streams"], a["y"], a["gate"], a["out"], a["gain"]
+        D = x.shape[1] // S
+        assert x.dtype == torch.float32 and x.is_contiguous() and x.shape[1] == S * D
+        assert y is None or (y.dtype == torch.float32 and y.is_contiguous() and y.shape[1] == D and _f32(a["mix"], S * S) and _f32(a["put"], S))
+        assert (g is None) == (a["gate_bias"] is None) and (g is None or (y is not None and g.stride(1) == 1 and g.shape[1] == D and _f32(a["gate_bias"], D)))
+        assert (out is None) == (gain is None) and (out is None or (out.is_contiguous() and out.shape[1] == D and _f32(gain, D) and _f32(a["read"], S)))
+        return OP_STREAM_NORM, StreamNormOp(x.data_ptr(), S, D, ptr(y), ptr(g), g.stride(0) if g is not None else 0, code(g.dtype) if g is not None else 0,
+                                            ptr(a["gate_bias"]), ptr(a["mix"]), ptr(a["put"]), ptr(a["read"]), ptr(gain), a["eps"], ptr(out),
+                                            code(out.dtype) if out is not None else 0, ROWS[a["rows"]])
+    if k == "forget_gates":
+        qi, fi, q, f = a["q_in"], a["f_in"], a["q"], a["f"]
+        for t in (qi, fi, q, f):
+            assert t.dtype == torch.float32 and t.stride(1) == 1 and t.shape[1] == q.shape[1]
+        assert qi.stride(0) == fi.stride(0) and _f32(a["f_bias"], q.shape[1]) and _f32(a["lower"], q.shape[1])
+        return OP_FORGET_GATES, ForgetGatesOp(qi.data_ptr(), fi.data_ptr(), qi.stride(0), a["f_bias"].data_ptr(), a["lower"].data_ptr(),
+                                              q.data_ptr(), f.data_ptr(), q.stride(0), f.stride(0), q.shape[1])
+    if k == "difference_norm":
+        m, out, H, rep = a["a"], a["out"], a["heads"], a["rep"]
+        assert m.dtype == out.dtype and m.stride(1) == out.stride(1) == 1 and m.shape[1] == 2 * out.shape[1] and out.shape[1] % H == 0 and H % rep == 0
+        return OP_DIFFERENCE_NORM, DifferenceNormOp(m.data_ptr(), m.stride(0), out.data_ptr(), out.stride(0), code(out.dtype), H, rep,
+                                                    out.shape[1] // H, a["weight"], a["scale"], a["eps"])
     if k == "delta_rule":
         q, kk, v, wr, fg, st, out, unit, coef = (a[n] for n in ("q", "k", "v", "write", "forget", "state", "out", "unit", "coef"))
         H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]

@@ -193,16 +193,18 @@ class CudaOps:
     _ENTRY_POINTS = {
         "elementwise": {"embedding": "llme_embedding", "rmsnorm": "llme_rmsnorm", "qkv_post": "llme_qkv_post",
                         "swiglu": "llme_swiglu", "embedding_scaled": "llme_embedding_scaled", "rmsnorm_pair": "llme_rmsnorm_pair",
-                        "embedding_add": "llme_embedding_add", "layernorm": "llme_layernorm"},
+                        "embedding_add": "llme_embedding_add", "layernorm": "llme_layernorm", "embedding_streams": "llme_embedding_streams"},
+        "streams": {"stream_norm": "llme_stream_norm"},
         "gemm_f32": {"gemm_f32": "llme_gemm_nt_f32", "gemm_f32_batched": "llme_gemm_nt_f32_batched"},
         "pointwise": {"xielu": "llme_xielu", "sigmoid_mul": "llme_sigmoid_mul", "residual_add": "llme_residual_add",
                       "gelu_gather_mul": "llme_gelu_gather_mul", "rmsnorm_add": "llme_rmsnorm_add",
                       "latent_post": "llme_latent_post", "postnorm": "llme_postnorm", "gated_act": "llme_gated_act",
                       "sigmoid_mul_scaled": "llme_sigmoid_mul_scaled", "gated_act_bias": "llme_gated_act_bias",
                       "bias_add": "llme_bias_add", "sigmoid_mul_grouped": "llme_sigmoid_mul_grouped",
-                      "residual_add_scaled": "llme_residual_add_scaled", "row_norm": "llme_row_norm", "relu2": "llme_relu2"},
+                      "residual_add_scaled": "llme_residual_add_scaled", "row_norm": "llme_row_norm", "relu2": "llme_relu2",
+                      "difference_norm": "llme_difference_norm"},
         "recurrent": {"short_conv": "llme_short_conv", "rotate": "llme_rotate", "recurrence": "llme_recurrence",
-                      "gated_norm": "llme_gated_norm", "exp_gates": "llme_exp_gates"},
+                      "gated_norm": "llme_gated_norm", "exp_gates": "llme_exp_gates", "forget_gates": "llme_forget_gates"},
         "delta_rule": {"delta_step": "llme_delta_step", "delta_portions": "llme_delta_portions"},
         "attention_window": {"window_post": "llme_window_post", "window_attention_plain": "llme_window_attention_plain"},
         "attention_window_tc": {"window_attention_tc/{hd}": "llme_window_attention_tc"},
@@ -247,13 +249,15 @@ class CudaOps:
             a = op.a
             if op.kind in ("embedding", "rmsnorm", "layernorm", "qkv_post", "attention"):
                 want("elementwise")
-            if op.kind in ("linear_act", "pointwise", "residual_add", "latent_attention", "token_side", "postnorm", "row_norm"):
+            if op.kind in ("linear_act", "pointwise", "residual_add", "latent_attention", "token_side", "postnorm", "row_norm", "difference_norm"):
                 want("pointwise")
+            if op.kind == "stream_norm":
+                want("streams")
             if op.kind == "linear_swiglu" and (a.get("act", "silu") != "silu" or a.get("bias") is not None):
                 want("pointwise")
             if op.kind == "linear" and a.get("bias") is not None:
                 want("pointwise")
-            if op.kind in ("short_conv", "rotate", "recurrence", "gated_norm", "exp_gates"):
+            if op.kind in ("short_conv", "rotate", "recurrence", "gated_norm", "exp_gates", "forget_gates"):
                 want("recurrent")
             if op.kind == "delta_rule":
                 want("delta_rule")

@@ -123,20 +123,26 @@ class SplitKVView:
 class SplitKVSpec:
     """Keys and values of different widths in pages: a page holds the keys of its tokens, [kv_heads, page_size, k_dim],
     and behind them the values, [kv_heads, page_size, v_dim].  `window` W > 0: only the last W positions are needed,
-    and beside them the first `keep_first` positions of the request, whose pages are never given back."""
+    and beside them the first `keep_first` positions of the request, whose pages are never given back.  `value_share` n: n
+    neighbouring key heads share one value head, a page then has kv_heads / n value heads."""
 
     num_kv_heads: int
     k_dim: int
     v_dim: int
     window: int = 0
     keep_first: int = 0
+    value_share: int = 1
     paged = True
 
+    @property
+    def token_values(self) -> int:
+        return self.num_kv_heads * self.k_dim + self.num_kv_heads // self.value_share * self.v_dim
+
     def allocate(self, count: int, page_size: int, dtype: torch.dtype, device: torch.device) -> torch.Tensor:
-        return torch.zeros(count, self.num_kv_heads * page_size * (self.k_dim + self.v_dim), dtype=dtype, device=device)
+        return torch.zeros(count, page_size * self.token_values, dtype=dtype, device=device)
 
     def bytes_per_token(self, dtype: torch.dtype) -> int:
-        return self.num_kv_heads * (self.k_dim + self.v_dim) * torch.empty((), dtype=dtype).element_size()
+        return self.token_values * torch.empty((), dtype=dtype).element_size()
 
     def view(self, tensor: torch.Tensor, group: Optional[int], writes: bool) -> SplitKVView:
         return SplitKVView(tensor, group, writes)
@@ -344,6 +350,88 @@ class WindowSinkAttention(Part):
         self.emit_heads(plan, proj, cache, out)
         delta = rt.workspace("mixer_out", self.hidden, torch.float32)
         plan.linear(out, self.w_o, delta)
+        return delta
+
+    def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:
+        plan = Plan()
+        delta = self.emit(plan, h, cache)
+        run_alone(self.rt, plan, batch)
+        return delta[: h.shape[0]]
+
+
+@register_part("mixer", "difference_attention")
+class DifferenceAttention(Part):
+    """Differential attention: every head has two maps, causal softmaxes with queries and keys of their own over the SAME values;
+    what is attended to is their difference.
+        q, k: RMS norm per head and map with weights q.norm, k.norm [qk_dim] (shared by heads and maps), then rotation;
+        a1, a2 = the maps' outputs; lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff, one number a layer;
+        head = (a1 - lambda a2) / sqrt(mean(.^2) + eps) * (1 - diff); the heads, side by side, are projected by o.
+    Query head a reads key/value head a // (num_heads / num_kv_heads).
+
+    Tensors: q [2 H qk_dim, hidden] and k [2 G qk_dim, hidden], head by head as [map 1 | map 2]; v [G v_dim, hidden]; q.norm, k.norm;
+    lq1, lk1, lq2, lk2 [qk_dim]; o [hidden, H v_dim].
+
+    Towards the attention kernels this is grouped-query attention of 2 H query heads on 2 G key heads of which neighbouring pairs
+    share a value head (`value_share`).  A map of a group's query heads reads one key head, so the rows of W_q are put into the
+    order [group, map, head of the group] when the weights are loaded; lambda is formed once in 32-bit and travels as a constant."""
+
+    MAPS = 2
+
+    def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int, scale: float,
+                 diff: float, norm_eps: float, position_encoding: Optional[PartSpec] = None):
+        super().__init__(rt, prefix)
+        if num_heads % num_kv_heads:
+            raise ValueError(f"{prefix}: {num_heads} query heads are not a multiple of {num_kv_heads} key/value heads")
+        self.hidden, self.nh, self.nkv, self.dk, self.dv = int(hidden_size), int(num_heads), int(num_kv_heads), int(qk_dim), int(v_dim)
+        self.rep = self.nh // self.nkv
+        self.scale, self.diff, self.eps = float(scale), float(diff), float(norm_eps)
+        self.position = build_part("position", position_encoding, rt, prefix) if position_encoding is not None else None
+        if self.position is not None and self.position.dims > self.dk:
+            raise ValueError(f"{prefix}: {self.position.dims} rotated coordinates do not fit a head of {self.dk}")
+        self.q_size, self.k_size, self.v_size = self.MAPS * self.nh * self.dk, self.MAPS * self.nkv * self.dk, self.nkv * self.dv
+        self.o_size = self.nh * self.dv
+        self.w_in = self.w_o = self.q_gain = self.k_gain = None
+        self.weight = 0.0                                     # lambda
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        v = lambda init: WeightSpec((self.dk,), role="vector", init=init)
+        return {self.name("q"): WeightSpec((self.q_size, self.hidden)), self.name("k"): WeightSpec((self.k_size, self.hidden)),
+                self.name("v"): WeightSpec((self.v_size, self.hidden)), self.name("o"): WeightSpec((self.hidden, self.o_size)),
+                self.name("q.norm"): v("gain"), self.name("k.norm"): v("gain"),
+                **{self.name(n): v("normal") for n in ("lq1", "lk1", "lq2", "lk2")}}
+
+    def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        q = t[self.name("q")].view(self.nkv, self.rep, self.MAPS, self.dk, self.hidden).transpose(1, 2).reshape(self.q_size, self.hidden)
+        self.w_in = torch.cat([q, t[self.name("k")], t[self.name("v")]], 0).contiguous()
+        self.w_o = t[self.name("o")].contiguous()
+        self.q_gain, self.k_gain = t[self.name("q.norm")].float().contiguous(), t[self.name("k.norm")].float().contiguous()
+        l = {n: t[self.name(n)].detach().to("cpu", torch.float32) for n in ("lq1", "lk1", "lq2", "lk2")}
+        self.weight = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum()) + torch.tensor(self.diff, dtype=torch.float32))
+
+    def cache_spec(self) -> SplitKVSpec:
+        return SplitKVSpec(self.MAPS * self.nkv, self.dk, self.dv, value_share=self.MAPS)
+
+    def emit(self, plan: Plan, h: torch.Tensor, cache) -> torch.Tensor:
+        rt, qs, ks = self.rt, self.q_size, self.k_size
+        if not cache.writes:
+            raise ValueError(f"{self.prefix}: this mixer keeps a cache of its own")
+        proj = rt.workspace("qkv", self.w_in.shape[0], rt.dtype)
+        plan.linear(h, self.w_in, proj)
+        q = rt.workspace("q", qs, rt.dtype)
+        maps = rt.workspace("attn_maps", self.MAPS * self.o_size, rt.dtype)
+        pos, H, G = self.position, self.MAPS * self.nh, self.MAPS * self.nkv
+        plan.window_attention(
+            q_in=proj[:, :qs], k_in=proj[:, qs:qs + ks], v_in=proj[:, qs + ks:], q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps,
+            inv_freq=pos.frequencies() if pos is not None else None, rot_dims=pos.dims if pos is not None else 0,
+            amplitude=pos.amplitude if pos is not None else 1.0, q=q, out=maps, cache=cache.kv, group=cache.group, num_heads=H, num_kv_heads=G,
+            qk_dim=self.dk, v_dim=self.dv, window=0, keep_first=0, scale=self.scale, head_norm=True, value_share=self.MAPS,
+            interleaved=bool(pos is not None and pos.interleaved),
+            scratch=(rt.buffer("window_attention_scratch", 1, rt.max_requests * H * 8 * (self.dv + 2), torch.float32, exact=True).view(-1)
+                     if rt.dtype == torch.bfloat16 else None))
+        heads = rt.workspace("attn_out", self.o_size, rt.dtype)
+        plan.difference_norm(a=maps, weight=self.weight, scale=1.0 - self.diff, eps=self.eps, heads=self.nh, rep=self.rep, out=heads)
+        delta = rt.workspace("mixer_out", self.hidden, torch.float32)
+        plan.linear(heads, self.w_o, delta)
         return delta
 
     def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:

@@ -267,14 +267,14 @@ class Runtime:
             return None
         return self.buffer("attention_scratch", 1, n, torch.float32, exact=True, zero=True).view(-1)
 
-    def recurrence_scratch(self, heads: int, p: int, n: int) -> Optional[torch.Tensor]:
+    def recurrence_scratch(self, heads: int, p: int, n: int, decays: int = 1) -> Optional[torch.Tensor]:
         """Room for the states that the pieces of long portions start from (one buffer for all layers, as large as the
         largest state among them needs): a step of T tokens cut every c tokens has fewer than 2 T / c pieces in requests
-        of several, each with a [heads, p, n] state and a product of decays per head.  Up to 64 pieces of 64 tokens or more."""
+        of several, each with a [heads, p, n] state and `decays` products of decays per head.  Up to 64 pieces of 64 tokens or more."""
         if self.max_tokens <= 64 or self.device.type != "cuda":
             return None
         pieces = min(64, max(4, 2 * ((self.max_tokens + 63) // 64)))
-        self._recurrence_scratch_floats = max(getattr(self, "_recurrence_scratch_floats", 0), pieces * heads * (p * n + 1))
+        self._recurrence_scratch_floats = max(getattr(self, "_recurrence_scratch_floats", 0), pieces * heads * (p * n + decays))
         return self.buffer("recurrence_scratch", 1, self._recurrence_scratch_floats, torch.float32, exact=True).view(-1)
 
     def delta_workspace(self, heads: int, qk_heads: int, n: int) -> Tuple[torch.Tensor, torch.Tensor]:

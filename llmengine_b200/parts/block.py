@@ -6,7 +6,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from ..config.spec import LayerSpec
-from ..engine.plan import Plan
+from ..engine.plan import Plan, StreamUpdate
 from .base import (Part, Runtime, WeightSpec, build_part, emit_feed_forward, emit_mixer, emit_norm, register_part,
                    run_alone)
 
@@ -309,5 +309,88 @@ class SandwichResidualBlock(Part):
     def forward(self, x: torch.Tensor, delta: Optional[torch.Tensor], batch, cache):
         plan = Plan()
         x, _ = self.emit(plan, x, delta, cache)
+        run_alone(self.rt, plan, batch)
+        return x, None
+
+
+@register_part("block", "stream_residual")
+class StreamResidualBlock(Part):
+    """Hyper-connections: the residual stream is S streams x_1 .. x_S side by side ([T, S D], 32-bit).  Each sublayer q (the mixer,
+    then the feed-forward, where the layer has one) reads h = norm_q(sum_s in_q[s] x_s); its result, gated, goes into all of them:
+        y = sublayer(h) * sigmoid(W_q h + b_q);   x_t <- sum_s mix_q[s, t] x_s + multiplier * out_q[t] * y  (all from the old ones).
+
+    Tensors below the layer's prefix: <connection>.in [S], .out [S], .mix [S, S] ([from, to]); the gate's <gate> [D, D] and
+    <gate>.b [D]; the norms' under their names.  A sublayer's result is not written where it is produced: it travels as a
+    `StreamUpdate` to the next norm, whose kernel updates the streams, sums what its own sublayer reads and norms it in one
+    pass.  The block reads the parts "mixer", "mixer_norm" and, where the layer has them, "feed_forward" and
+    "feed_forward_norm", the norms of a kind that takes a stream's read weights (`stream_rmsnorm`)."""
+
+    def __init__(self, rt: Runtime, prefix: str, layer: LayerSpec, hidden_size: int, streams: int, multiplier: float = 1.0,
+                 mixer_name: str = "mixer", feed_forward_name: str = "feed_forward",
+                 norm_names: Tuple[str, str] = ("mixer_norm", "feed_forward_norm"),
+                 connection_names: Tuple[str, str] = ("mixer_connection", "feed_forward_connection"),
+                 gate_names: Tuple[str, str] = ("mixer_gate", "feed_forward_gate")):
+        super().__init__(rt, prefix)
+        missing = [n for n in ("mixer", "mixer_norm") if n not in layer.parts]
+        has_ffn = "feed_forward" in layer.parts
+        if has_ffn and "feed_forward_norm" not in layer.parts:
+            missing.append("feed_forward_norm")
+        if missing:
+            raise ValueError(f"layer {prefix!r}: a stream_residual block needs the parts {', '.join(missing)}")
+        self.hidden, self.streams, self.multiplier = int(hidden_size), int(streams), float(multiplier)
+        self.norms = [build_part("norm", layer.parts["mixer_norm"], rt, self.name(norm_names[0]))]
+        self.mixer = build_part("mixer", layer.parts["mixer"], rt, self.name(mixer_name))
+        self.ffn = None
+        if has_ffn:
+            self.norms.append(build_part("norm", layer.parts["feed_forward_norm"], rt, self.name(norm_names[1])))
+            self.ffn = build_part("feed_forward", layer.parts["feed_forward"], rt, self.name(feed_forward_name))
+        self.parts = tuple(p for p in (*self.norms, self.mixer, self.ffn) if p is not None)
+        n = len(self.norms)
+        self.connections, self.gates = tuple(connection_names[:n]), tuple(gate_names[:n])
+        self.capture_safe = all(p.capture_safe and hasattr(p, "emit") for p in self.parts)
+        self.read, self.mix, self.put, self.w_gate, self.b_gate = [], [], [], [], []
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        out: Dict[str, WeightSpec] = {}
+        for p in self.parts:
+            out.update(p.weight_specs())
+        S, D = self.streams, self.hidden
+        for c, g in zip(self.connections, self.gates):
+            out[self.name(c + ".in")] = WeightSpec((S,), role="vector", init="gain")
+            out[self.name(c + ".out")] = WeightSpec((S,), role="vector", init="gain")
+            out[self.name(c + ".mix")] = WeightSpec((S, S), role="vector")
+            out[self.name(g)] = WeightSpec((D, D))
+            out[self.name(g + ".b")] = WeightSpec((D,), role="vector")
+        return out
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        for p in self.parts:
+            p.load_weights({n: tensors[n] for n in p.weight_specs()})
+        f = lambda n: tensors[self.name(n)].float().contiguous()
+        self.read, self.mix = [f(c + ".in") for c in self.connections], [f(c + ".mix") for c in self.connections]
+        self.put = [f(c + ".out") * self.multiplier for c in self.connections]
+        self.w_gate, self.b_gate = [tensors[self.name(g)].contiguous() for g in self.gates], [f(g + ".b") for g in self.gates]
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def _result(self, plan: Plan, q: int, h: torch.Tensor, y: torch.Tensor) -> StreamUpdate:
+        """Sublayer q's result `y` on its way into the streams, with the product its gate is made from."""
+        gate = self.rt.workspace("sublayer_gate", self.hidden, self.rt.dtype)
+        plan.linear(h, self.w_gate[q], gate)
+        return StreamUpdate(y=y, gate=gate, bias=self.b_gate[q], mix=self.mix[q], put=self.put[q])
+
+    def emit(self, plan: Plan, x: torch.Tensor, delta: Optional[StreamUpdate], cache):
+        h = self.norms[0].emit(plan, x, delta=delta, read=self.read[0])
+        delta = self._result(plan, 0, h, emit_mixer(plan, self.mixer, h, cache, self.hidden))
+        if self.ffn is not None:
+            h = self.norms[1].emit(plan, x, delta=delta, read=self.read[1])
+            delta = self._result(plan, 1, h, emit_feed_forward(plan, self.ffn, h, self.hidden))
+        return x, delta
+
+    def forward(self, x: torch.Tensor, delta: Optional[StreamUpdate], batch, cache):
+        plan = Plan()
+        x, delta = self.emit(plan, x, delta, cache)
+        plan.stream_norm(x, streams=self.streams, read=None, gain=None, eps=0.0, out=None, update=delta)
         run_alone(self.rt, plan, batch)
         return x, None

@@ -16,12 +16,22 @@ class TokenEmbedding(Part):
 
     `leaf` is the table's name below the prefix ("" = the prefix itself).  `extra_tables` (full tensor name ->
     width) are further per-token tables [vocab, width] that the part only stores: other parts of the model take
-    them as shared tensors and gather from them by the step's token ids."""
+    them as shared tensors and gather from them by the step's token ids.
+
+    `position_table` (full tensor name) with `max_positions` rows: row p, unscaled, is added to a token at position p.
+    `streams` S: the stream holds S copies of every row side by side, [T, S hidden] (hyper-connections)."""
 
     def __init__(self, rt: Runtime, prefix: str, vocab_size: int, hidden_size: int, leaf: str = "weight",
                  extra_tables: Optional[Dict[str, int]] = None, norm_leaf: Optional[str] = None,
-                 norm_eps: Optional[float] = None, scale: float = 1.0):
+                 norm_eps: Optional[float] = None, scale: float = 1.0, position_table: Optional[str] = None, max_positions: int = 0,
+                 streams: int = 1):
         super().__init__(rt, prefix)
+        self.streams, self.position_name, self.max_positions = int(streams), position_table, int(max_positions)
+        if self.position_name is not None and self.max_positions <= 0:
+            raise ValueError(f"{prefix}: a position table needs its number of rows")
+        if norm_leaf is not None and (self.streams > 1 or position_table is not None):
+            raise ValueError(f"{prefix}: a norm on the embedding excludes streams and a position table")
+        self.position: Optional[torch.Tensor] = None
         self.vocab, self.hidden = int(vocab_size), int(hidden_size)
         self.leaf = leaf
         self.scale = float(scale)
@@ -40,6 +50,8 @@ class TokenEmbedding(Part):
             s[n] = WeightSpec((self.vocab, w), init="unit")
         if self.norm_leaf is not None:
             s[self.name(self.norm_leaf)] = WeightSpec((self.hidden,), role="vector", init="gain")
+        if self.position_name is not None:
+            s[self.position_name] = WeightSpec((self.max_positions, self.hidden))
         return s
 
     def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
@@ -47,6 +59,8 @@ class TokenEmbedding(Part):
         self.extra = {n: t[n].contiguous() for n in self.extra_widths}
         if self.norm_leaf is not None:
             self.norm_gain = t[self.name(self.norm_leaf)].contiguous()
+        if self.position_name is not None:
+            self.position = t[self.position_name].contiguous()
 
     def shared_tensor(self, name: str) -> Optional[torch.Tensor]:
         if name in self.extra:
@@ -54,8 +68,8 @@ class TokenEmbedding(Part):
         return self.table if name == self.name(self.leaf) else None
 
     def emit(self, plan: Plan) -> torch.Tensor:
-        x = self.rt.workspace("residual", self.hidden, torch.float32)
-        plan.embedding(self.table, x, scale=self.scale)
+        x = self.rt.workspace("residual", self.streams * self.hidden, torch.float32)
+        plan.embedding(self.table, x, scale=self.scale, positions=self.position, streams=self.streams)
         if self.norm_leaf is not None:
             # the stream in the type of the products too: a block whose sublayers read the stream itself finds it there
             copy = None if self.rt.dtype == torch.float32 else self.rt.workspace("stream_copy", self.hidden, self.rt.dtype)
@@ -64,14 +78,16 @@ class TokenEmbedding(Part):
 
     def emit_again(self, plan: Plan, x: torch.Tensor, delta: Optional[torch.Tensor]) -> None:
         """x += delta (where a contribution is pending) + the embedding output, the rows gathered anew."""
-        if self.norm_leaf is not None:
-            raise ValueError(f"{self.prefix}: an embedding with a norm of its own is not added to the stream a second time")
+        if self.norm_leaf is not None or self.position is not None or self.streams > 1:
+            raise ValueError(f"{self.prefix}: an embedding with a norm, positions or streams is not added to the stream a second time")
         plan.embedding(self.table, x, scale=self.scale, accumulate=True, delta=delta)
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
         from ..engine.batch import StepBatch
         plan = Plan()
         x = self.emit(plan)
+        if self.position is not None:
+            raise ValueError(f"{self.prefix}: an embedding with positions needs a batch that has them (emit)")
         run_alone(self.rt, plan, StepBatch.bare(token_ids.numel(), token_ids.device, token_ids=token_ids))
         return x[: token_ids.numel()]
 

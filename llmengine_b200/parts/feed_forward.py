@@ -134,6 +134,7 @@ class Dense(Part):
 
 GATED_ACTIVATIONS = ("silu", "clamped_swish", "gelu_tanh")
 PLAIN_ACTIVATIONS = ("relu2",)
+EXPERT_ACTIVATIONS = ("silu", "relu2", "gelu")      # of an expert: gated, the square of relu, gelu in its erf form
 
 
 @register_part("feed_forward", "gated_dense")
@@ -202,10 +203,11 @@ class RoutedExperts(Part):
     sigmoid(W_sg h), one number a token.  Tensors: router (router.b, correction); e<i>.gate / up / down; shared.gate / up / down
     (shared.sg [1, hidden]).
 
-    Options of the "softmax" routing: `groups` (count, keep): the choices form `count` equal groups of neighbours, and only the
-    members of the `keep` groups whose largest choice score is largest can be chosen; `identity` I: the router has I outputs
-    more than there are experts, and these stand for the input itself (output h, times the weight; no tensors).
-    `activation` "relu2": an expert is down(max(up h, 0)^2), without a gate.
+    `groups` (count, keep), for the routings by scores over all: the choices form `count` equal groups of neighbours, and only
+    the members of the best `keep` groups can be chosen; "softmax": a group is as good as its largest choice score, "sigmoid": as
+    the sum of its two largest scores.  `identity` I ("softmax"): the router has I outputs more than there are experts, and these
+    stand for the input itself (output h, times the weight; no tensors).  `activation` "relu2" or "gelu": an expert is
+    down(act(up h)) with max(z, 0)^2 or z Phi(z), without a gate.
 
     The experts' matrices are stacked ([E, 2 ff, D] and [E, D, ff]) and run as two grouped products over the
     (token, choice) pairs listed expert by expert; the pairs' outputs are combined per token in the order of the
@@ -220,15 +222,17 @@ class RoutedExperts(Part):
         self.hidden, self.E, self.top, self.ff = int(hidden_size), int(num_experts), int(top_k), int(expert_size)
         self.identity, self.choices = int(identity), int(num_experts) + int(identity)
         self.groups, self.has_correction, self.correction = (int(groups[0]), int(groups[1])), bool(correction), None
-        if activation not in ("silu",) + PLAIN_ACTIVATIONS:
+        if activation not in EXPERT_ACTIVATIONS:
             raise ValueError(f"{prefix}: unknown activation {activation!r} of an expert")
         self.act = activation
         if not 0 < self.top <= self.choices:
             raise ValueError(f"{prefix}: {self.top} of {self.choices} experts cannot be chosen")
         if routing not in ("sigmoid", "softmax_chosen", "softmax"):
             raise ValueError(f"{prefix}: unknown routing {routing!r}; known: sigmoid, softmax_chosen, softmax")
-        if routing != "softmax" and (correction or identity or self.groups[1] < self.groups[0]):
-            raise ValueError(f"{prefix}: corrections, identity experts and groups belong to the routing by a softmax over all")
+        if routing != "softmax" and (correction or identity):
+            raise ValueError(f"{prefix}: corrections and identity experts belong to the routing by a softmax over all")
+        if routing == "softmax_chosen" and self.groups[1] < self.groups[0]:
+            raise ValueError(f"{prefix}: groups belong to the routings by scores over all experts")
         if self.choices % self.groups[0] or not 0 < self.groups[1] <= self.groups[0] or self.top > self.choices // self.groups[0] * self.groups[1]:
             raise ValueError(f"{prefix}: {self.groups[1]} of {self.groups[0]} groups of {self.choices} experts do not offer {self.top}")
         self.route_scale, self.routing, self.router_bias = float(route_scale), routing, bool(router_bias)

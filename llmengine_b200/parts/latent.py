@@ -196,7 +196,8 @@ class LatentAttention(Part):
                               rot_dims=self.position.dims if self.position is not None else 0, q=q, out=out,
                               cache=cache.kv, group=cache.group, num_heads=H, kv_rank=r, rot_dim=dr, scale=self.scale,
                               sink=self.sink, scratch=rt.latent_scratch(H, r), window=self.window,
-                              interleaved=bool(self.position is not None and self.position.interleaved))
+                              interleaved=bool(self.position is not None and self.position.interleaved),
+                              amplitude=self.position.amplitude if self.position is not None else 1.0)
         heads = rt.workspace("latent_heads", self.o_size, rt.dtype)
         plan.batched_linear(out.view(T, H, r), self.w_uv, heads.view(T, H, dv))
         if self.has_gate:

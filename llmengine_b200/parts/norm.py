@@ -5,7 +5,7 @@ from typing import Dict, Optional
 
 import torch
 
-from ..engine.plan import ROWS_LOGITS, ROWS_TOKENS, Plan
+from ..engine.plan import ROWS_LOGITS, ROWS_TOKENS, Plan, StreamUpdate
 from .base import Part, Runtime, WeightSpec, register_part, run_alone
 
 
@@ -113,6 +113,41 @@ class LayerNorm(Part):
 
     def forward(self, x: torch.Tensor, delta: Optional[torch.Tensor] = None,
                 out_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+        from ..engine.batch import StepBatch
+        plan = Plan()
+        out = self.emit(plan, x, delta=delta, rows=ROWS_TOKENS if out_rows is None else ROWS_LOGITS)
+        run_alone(self.rt, plan, StepBatch.bare(x.shape[0], x.device, logit_rows=out_rows))
+        return out[: x.shape[0] if out_rows is None else out_rows.numel()]
+
+
+@register_part("norm", "stream_rmsnorm")
+class StreamRMSNorm(Part):
+    """The RMS norm of a weighted sum of streams: with x [T, S size] = S streams side by side, u = sum_s read[s] x_s and
+    y = u / sqrt(mean(u^2) + eps) * gain, times the constant `scale` where a design multiplies what follows (the logits) by one.
+    `read` comes with the sublayer that asks (hyper-connections); without it the streams are summed.  `delta` is a
+    `StreamUpdate`, a sublayer's result that is not yet part of the streams: the kernel updates them in the same pass."""
+
+    def __init__(self, rt: Runtime, prefix: str, size: int, streams: int, eps: float, leaf: str = "weight", scale: float = 1.0):
+        super().__init__(rt, prefix)
+        self.size, self.streams, self.eps, self.scale, self.leaf = int(size), int(streams), float(eps), float(scale), leaf
+        self.gain: Optional[torch.Tensor] = None
+        self.sum_of_all: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        return {self.name(self.leaf): WeightSpec((self.size,), role="vector", init="gain")}
+
+    def load_weights(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.gain = (tensors[self.name(self.leaf)].float() * self.scale).contiguous()
+        self.sum_of_all = torch.ones(self.streams, dtype=torch.float32, device=self.gain.device)
+
+    def emit(self, plan: Plan, x: torch.Tensor, delta: Optional[StreamUpdate] = None, rows: str = ROWS_TOKENS,
+             read: Optional[torch.Tensor] = None, out_name: Optional[str] = None) -> torch.Tensor:
+        out = self.rt.workspace(out_name or ("normed" if rows == ROWS_TOKENS else "normed_rows"), self.size, self.rt.dtype)
+        plan.stream_norm(x, streams=self.streams, read=self.sum_of_all if read is None else read, gain=self.gain, eps=self.eps, out=out,
+                         update=delta, rows=rows)
+        return out
+
+    def forward(self, x: torch.Tensor, delta: Optional[StreamUpdate] = None, out_rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         from ..engine.batch import StepBatch
         plan = Plan()
         out = self.emit(plan, x, delta=delta, rows=ROWS_TOKENS if out_rows is None else ROWS_LOGITS)

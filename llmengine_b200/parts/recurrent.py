@@ -21,6 +21,10 @@
   a_t = exp(-exp(A_log) softplus(W_a h + dt_bias)); S <- a_t S, u = b_t (v_t - S^T k_t), S <- S + k_t u^T, o_t = S^T q_t; every
   head's o is divided by its root mean square, times a weight shared by the heads, times silu(W_g h), and projected.  State per
   request: the matrices S (32-bit) and the convolution's last taps - 1 inputs.
+* `ForgetMemory` (kind `forget_memory`): a linear memory whose forget gate, one per head and channel, also says how much is written.
+  q = silu(W_q h), v = W_v h, f = lower + (1 - lower) sigmoid(W_f h + b_f); S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T, o_t = S_t^T q_t;
+  every head's o is divided by its root mean square, times a weight shared by the heads, and projected.  State per request: the
+  matrices S (32-bit).
 * `ParallelMixer` (kind `parallel`): branches that read the same input; the result is sum_b scale_b branch_b(h).  The
   branches' input projections are ONE product, and so are their output projections: every branch writes its gated heads,
   times its scale, into its columns of one row, and the output matrices stand side by side.
@@ -300,6 +304,60 @@ class GatedDelta(Part):
                         state=cache.states["state"], out=o, heads=H, n=self.dk, p=self.dv, qk_groups=self.nqk, unit=unit, coef=coef)
         heads = rt.workspace("delta_heads", hs, rt.dtype)
         plan.gated_norm(y=o, gate=proj[:, C:C + hs], weight=self.norm_w, out=heads, group=self.dv, gate_first=False, eps=self.eps)
+        delta = rt.workspace("mixer_out", self.hidden, torch.float32)
+        plan.linear(heads, self.w_o, delta)
+        return delta
+
+    def forward(self, h: torch.Tensor, batch, cache) -> torch.Tensor:
+        plan = Plan()
+        buf = self.rt.workspace("normed", self.hidden, self.rt.dtype)
+        buf[: h.shape[0]].copy_(h)
+        delta = self.emit(plan, buf, cache)
+        run_alone(self.rt, plan, batch)
+        return delta[: h.shape[0]]
+
+
+@register_part("mixer", "forget_memory")
+class ForgetMemory(Part):
+    """Tensors: q, f [heads qk_dim, hidden]; f.b, lower [heads qk_dim]; v [heads v_dim, hidden]; norm [v_dim]; o [hidden, heads v_dim].
+    The three projections are ONE product with 32-bit results: gates and queries enter the recurrence unrounded."""
+
+    def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, qk_dim: int, v_dim: int, norm_eps: float):
+        super().__init__(rt, prefix)
+        self.hidden, self.nh, self.dk, self.dv, self.eps = int(hidden_size), int(num_heads), int(qk_dim), int(v_dim), float(norm_eps)
+        self.qk_size, self.heads_size = self.nh * self.dk, self.nh * self.dv
+        used = 2 * self.qk_size + self.heads_size
+        self.in_size = used + -used % 8          # rows of zeros up to a multiple of 8: the product's rows start on 32 bytes
+        self.w_in = self.w_o = self.f_bias = self.lower = self.norm_w = None
+
+    def weight_specs(self) -> Dict[str, WeightSpec]:
+        m = lambda n: WeightSpec((n, self.hidden))
+        v = lambda n, init: WeightSpec((n,), role="vector", init=init)
+        return {self.name("q"): m(self.qk_size), self.name("f"): m(self.qk_size), self.name("f.b"): v(self.qk_size, "unit"),
+                self.name("lower"): v(self.qk_size, "normal"), self.name("v"): m(self.heads_size), self.name("norm"): v(self.dv, "gain"),
+                self.name("o"): WeightSpec((self.hidden, self.heads_size))}
+
+    def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
+        rows = [t[self.name(n)] for n in ("q", "f", "v")]
+        rows.append(rows[0].new_zeros(self.in_size - sum(r.shape[0] for r in rows), self.hidden))
+        self.w_in, self.w_o = torch.cat(rows, 0).contiguous(), t[self.name("o")].contiguous()
+        self.f_bias, self.lower = t[self.name("f.b")].float().contiguous(), t[self.name("lower")].float().contiguous()
+        self.norm_w = t[self.name("norm")].float().repeat(self.nh).contiguous()
+
+    def cache_spec(self) -> StatesSpec:
+        return StatesSpec((("state", (self.nh, self.dv, self.dk)),))
+
+    def emit(self, plan: Plan, h: torch.Tensor, cache: StatesView) -> torch.Tensor:
+        rt, H, qs, hs = self.rt, self.nh, self.qk_size, self.heads_size
+        proj = rt.workspace("forget_in", self.in_size, torch.float32)
+        plan.linear(h, self.w_in, proj)
+        q, f = rt.workspace("forget_q", qs, torch.float32), rt.workspace("forget_f", qs, torch.float32)
+        plan.forget_gates(q_in=proj[:, :qs], f_in=proj[:, qs:2 * qs], f_bias=self.f_bias, lower=self.lower, q=q, f=f)
+        o = rt.workspace("forget_o", hs, torch.float32)
+        plan.recurrence(q=q, k=f, v=proj[:, 2 * qs:2 * qs + hs], state=cache.states["state"], out=o, heads=H, n=self.dk, p=self.dv, qk_groups=H,
+                        forget=True, scratch=rt.recurrence_scratch(H, self.dv, self.dk, decays=self.dk))
+        heads = rt.workspace("forget_heads", hs, rt.dtype)
+        plan.gated_norm(y=o, gate=None, weight=self.norm_w, out=heads, group=self.dv, gate_first=False, eps=self.eps)
         delta = rt.workspace("mixer_out", self.hidden, torch.float32)
         plan.linear(heads, self.w_o, delta)
         return delta

@@ -23,8 +23,11 @@ class HostOps:
     def compile(self, plan):
         return HostPlan(self, plan)
 
-    def embedding(self, ids, table, out, scale=1.0, accumulate=False, delta=None):
+    def embedding(self, ids, table, out, scale=1.0, accumulate=False, delta=None, positions=None, pos_table=None, streams=1):
         rows = table[ids.long()].float() * scale
+        if pos_table is not None:
+            rows = rows + pos_table[positions.long()].float()
+        rows = rows.repeat(1, streams)
         if delta is not None:
             out += delta.float()
         out.copy_(out + rows if accumulate else rows)
@@ -187,6 +190,10 @@ class HostOps:
                     v = torch.cat([a["v"][t].float().view(H, p - 1), torch.ones(H, 1)], 1)
                 else:
                     v = a["v"][t].float().view(H, p)
+                if a.get("forget"):
+                    S.mul_(k[:, None, :]).add_(v[:, :, None] * (1.0 - k)[:, None, :])
+                    a["out"][t] = torch.einsum("hpn,hn->hp", S, q).reshape(-1)
+                    continue
                 if a.get("keep") is not None:
                     decay, step = a["keep"][t], a["take"][t]
                 elif a["dt"] is None:
@@ -218,8 +225,8 @@ class HostOps:
                 a["out"][t] = torch.einsum("hpn,hn->hp", S, q).reshape(-1)
 
     def gated_norm(self, a, T):
-        y, g = a["y"][:T], a["gate"][:T].float()
-        gate = torch.sigmoid(g) if a.get("gate_act", "silu") == "sigmoid" else g * torch.sigmoid(g)
+        y, g = a["y"][:T], a["gate"][:T].float() if a["gate"] is not None else None
+        gate = 1.0 if g is None else torch.sigmoid(g) if a.get("gate_act", "silu") == "sigmoid" else g * torch.sigmoid(g)
         if a.get("floor") is not None:
             wide = y.reshape(T, -1, a["group"] + 1)
             den = torch.maximum(wide[..., -1].abs(), a["floor"][:T]) + a["den_eps"]
@@ -232,6 +239,35 @@ class HostOps:
         if not a["gate_first"]:
             u = u * gate
         a["out"][:T] = (u * a["scale"]).to(a["out"].dtype)
+
+    def stream_norm(self, a, T, rows):
+        S = a["streams"]
+        x = a["x"][:T].view(T, S, -1)
+        if a["y"] is not None:
+            y = a["y"][:T]
+            if a["gate"] is not None:
+                y = y * torch.sigmoid(a["gate"][:T].float() + a["gate_bias"])
+            new = torch.einsum("tsd,sb->tbd", x, a["mix"]) + a["put"][None, :, None] * y[:, None, :]
+            if rows is None:
+                x.copy_(new)
+            x = new
+        if a["out"] is None:
+            return
+        u = torch.einsum("tsd,s->td", x, a["read"])
+        u = u if rows is None else u[rows.long()]
+        a["out"][: u.shape[0]] = (u * (1.0 / torch.sqrt((u * u).mean(-1, keepdim=True) + a["eps"])) * a["gain"]).to(a["out"].dtype)
+
+    def forget_gates(self, a, T):
+        z = a["q_in"][:T]
+        a["q"][:T] = z * torch.sigmoid(z)
+        a["f"][:T] = a["lower"] + (1.0 - a["lower"]) * torch.sigmoid(a["f_in"][:T] + a["f_bias"])
+
+    def difference_norm(self, a, T):
+        H, rep = a["heads"], a["rep"]
+        m = a["a"][:T].float().view(T, H // rep, 2, rep, -1)
+        u = (m[:, :, 0] - a["weight"] * m[:, :, 1]).reshape(T, H, -1)
+        u = u / torch.sqrt((u * u).mean(-1, keepdim=True) + a["eps"]) * a["scale"]
+        a["out"][:T] = u.reshape(T, -1).to(a["out"].dtype)
 
     def row_norm(self, a, T):
         x = a["x"][:T].float()
@@ -275,9 +311,9 @@ class HostOps:
         c = c * (1.0 / torch.sqrt((c * c).mean(-1, keepdim=True) + a["eps"])) * a["c_gain"].float()
         row = c
         if dr:
-            il = bool(a.get("interleaved"))
-            row = torch.cat([c, self._rotate(kv[:, r:], positions, a["inv_freq"], a["rot_dims"], il)], -1)
-            q[:, :, r:] = self._rotate(a["q_rot"][:T].float(), positions, a["inv_freq"], a["rot_dims"], il).to(q.dtype)
+            il, amp = bool(a.get("interleaved")), a.get("amplitude", 1.0)
+            row = torch.cat([c, self._rotate(kv[:, r:], positions, a["inv_freq"], a["rot_dims"], il, amp)], -1)
+            q[:, :, r:] = self._rotate(a["q_rot"][:T].float(), positions, a["inv_freq"], a["rot_dims"], il, amp).to(q.dtype)
         flat = cache.view(-1, r + dr)
         for t in range(T):
             if int(slot_mapping[t]) >= 0:
@@ -324,7 +360,8 @@ class HostOps:
         cache, ps = a["cache"], page_size
         pages = cache.view(cache.shape[0], -1)
         keys = pages[:, :G * ps * dk].view(-1, G, ps, dk)
-        vals = pages[:, G * ps * dk:].view(-1, G, ps, dv)
+        share = a.get("value_share", 1)
+        vals = pages[:, G * ps * dk:].view(-1, G // share, ps, dv)
 
         def biased(x, bias):
             return x[:T] if bias is None else (x[:T].float() + bias).to(x.dtype)
@@ -346,7 +383,7 @@ class HostOps:
         a["q"][:T] = q.reshape(T, -1)
         if a["k_in"] is not None:
             k = finish(a["k_in"], G, a["k_gain"], a.get("k_bias")).to(cache.dtype)
-            v = biased(a["v_in"], a.get("v_bias")).reshape(T, G, dv).to(cache.dtype)
+            v = biased(a["v_in"], a.get("v_bias")).reshape(T, G // share, dv).to(cache.dtype)
             for t in range(T):
                 slot = int(slot_mapping[t])
                 if slot >= 0:
@@ -370,7 +407,7 @@ class HostOps:
                 if a["sink"] is not None:
                     s = torch.cat([s, a["sink"][h:h + 1]])
                 w = torch.softmax(s, 0)[: js.numel()]
-                a["out"][t, h * dv:(h + 1) * dv] = (w @ vv[:, h // rep]).to(a["out"].dtype)
+                a["out"][t, h * dv:(h + 1) * dv] = (w @ vv[:, h // rep // share]).to(a["out"].dtype)
 
     def moe_route(self, a, T):
         top, E = a["top_k"], a["logits"].shape[1]
@@ -387,6 +424,12 @@ class HostOps:
             wt = s.gather(1, idx) * a["scale"]
         else:
             s = torch.sigmoid(a["logits"][:T].float())
+            count, keep = a.get("groups", (1, 1))
+            if keep < count:
+                best = torch.topk(s.view(T, count, -1), min(2, E // count), dim=-1).values.sum(-1)
+                kept = torch.topk(best, keep, dim=-1).indices
+                allowed = torch.zeros(T, count, dtype=torch.bool).scatter_(1, kept, True).repeat_interleave(E // count, 1)
+                s = s.masked_fill(~allowed, -1.0)
             val, idx = torch.topk(s, top, dim=-1)
             wt = val / (val.sum(-1, keepdim=True) + 1e-20) * a["scale"]
         a["experts"][:T] = idx.to(torch.int32)
@@ -408,6 +451,8 @@ class HostOps:
                 y = w[e].float() @ row
                 if a["act"] == "relu2":
                     y = torch.clamp(y, min=0) ** 2
+                elif a["act"] == "gelu":
+                    y = 0.5 * y * (1.0 + torch.erf(y / math.sqrt(2.0)))
                 elif a["act"]:
                     n = y.numel() // 2
                     g, u = y[:n].to(a["x"].dtype).float(), y[n:].to(a["x"].dtype).float()
@@ -457,7 +502,8 @@ class HostPlan:
         for op in self.plan.ops[first:last]:
             a, k = op.a, op.kind
             if k == "embedding":
-                o.embedding(batch.token_ids, a["table"], a["out"][:T], a.get("scale", 1.0), bool(a.get("accumulate")), cut(a.get("delta")))
+                o.embedding(batch.token_ids, a["table"], a["out"][:T], a.get("scale", 1.0), bool(a.get("accumulate")), cut(a.get("delta")),
+                            positions=batch.positions, pos_table=a.get("positions"), streams=a.get("streams", 1))
             elif k == "layernorm":
                 o.layernorm(a["x"][:T], a["gain"], a["bias"], a["eps"], a["out"][:n_rows(a["rows"])], delta=cut(a["delta"]),
                             rows=batch.logit_rows if a["rows"] == "logits" else None)
@@ -482,6 +528,12 @@ class HostPlan:
                 o.gated_norm(a, T)
             elif k == "row_norm":
                 o.row_norm(a, T)
+            elif k == "stream_norm":
+                o.stream_norm(a, T, batch.logit_rows if a["rows"] == "logits" else None)
+            elif k == "forget_gates":
+                o.forget_gates(a, T)
+            elif k == "difference_norm":
+                o.difference_norm(a, T)
             elif k == "exp_gates":
                 o.exp_gates(a, batch)
             elif k == "linear_swiglu":
