@@ -17,8 +17,8 @@ TOL_F32 = 3e-4          # for logits of order one to ten (only the order of sums
 
 def keep_away_from_close_calls(model: PlainLopilix, reqs: Dict[str, List[int]], margin: float) -> None:
     """Changes the requests IN PLACE until the model makes no close call on them: where two experts' (or two groups') choice
-    scores lie closer together than rounding moves them (`margin`, in units of the scores at the boundary), and where a memory's
-    query is nearly orthogonal to what the memory holds (its first token; a token behind a decay that emptied it), rounding
+    scores lie closer together than rounding moves them (`margin`, how far a logit would have to move), and where a memory's
+    query is nearly orthogonal to what the memory holds (above all its first token), rounding
     decides, and no comparison can rest on that.  The token at the first such position is exchanged for the next one of the
     vocabulary (positions before it are not affected: the model is causal)."""
     vocab = model.cfg["vocab"]
@@ -61,7 +61,7 @@ def _settle(model_dir: str, reqs: Dict[str, List[int]], dtype: str):
     reqs = {r: list(ids) for r, ids in reqs.items()}
     plain = PlainLopilix(model_dir)
     rounded = PlainLopilix(model_dir, round_to=torch.bfloat16)
-    keep_away_from_close_calls(rounded if dtype == "bfloat16" else plain, reqs, 0.12 if dtype == "bfloat16" else 2e-4)
+    keep_away_from_close_calls(rounded if dtype == "bfloat16" else plain, reqs, 0.06 if dtype == "bfloat16" else 1e-4)
     ref = {r: plain.logits(ids) for r, ids in reqs.items()}
     if dtype != "bfloat16":
         return reqs, ref, TOL_F32 * max(1.0, max(float(v.abs().max()) for v in ref.values()) / 10.0)

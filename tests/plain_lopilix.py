@@ -110,9 +110,9 @@ def difference_attention(h, w, pre, m, eps, positions, round_to):
     return (unit_rms(o, eps) * (1.0 - m["diff"])).reshape(T, H * P)
 
 
-def gated_memory(q, f, v, S=None):
+def gated_memory(q, f, v, S=None, sizes=None):
     """q, f [T, H, d], v [T, H, P]: S <- f S + (1 - f) v^T row by row (row c of S decays by f_c and takes (1 - f_c) v), then
-    o = S^T q.  Returns o [T, H, P] and S [H, d, P]."""
+    o = S^T q.  Returns o [T, H, P] and S [H, d, P]; `sizes` (a list) receives the norm of every head's S per token."""
     T, H, d = q.shape
     if S is None:
         S = torch.zeros(H, d, v.shape[-1], dtype=q.dtype)
@@ -120,17 +120,27 @@ def gated_memory(q, f, v, S=None):
     for t in range(T):
         S = f[t][:, :, None] * S + (1.0 - f[t])[:, :, None] * v[t][:, None, :]
         out.append(torch.einsum("adp,ad->ap", S, q[t]))
+        if sizes is not None:
+            sizes.append(S.flatten(1).norm(dim=-1))
     return torch.stack(out), S
 
 
-def memory_mixer(h, w, pre, m, eps):
+def memory_mixer(h, w, pre, m, eps, calls=None):
     """q = silu(W_q h), v = W_v h, f = lower + (1 - lower) sigmoid(W_f h + b_f) per head and channel; the memory; every head's o
-    normed over its P values with a weight shared by the heads.  Returns [T, H P]."""
+    normed over its P values with a weight shared by the heads.  Returns [T, H P].
+
+    `calls` (a list) receives per token how far the model is from a close call: the norm leaves only the direction of S^T q, and
+    where q is nearly orthogonal to what the memory holds (a memory of one token: the SIGN of a sum) rounding decides it.
+    2.5 sqrt(d) |S^T q| / (|S| |q|), the least over the heads."""
     H, d, P = m["heads"], m["dim"], m["vdim"]
     T, lower = h.shape[0], w[pre + "lower"]
     q = silu(h @ w[pre + "q"].t()).view(T, H, d)
     f = (lower + (1.0 - lower) * torch.sigmoid(h @ w[pre + "f"].t() + w[pre + "f.b"])).view(T, H, d)
-    o, _ = gated_memory(q, f, (h @ w[pre + "v"].t()).view(T, H, P))
+    sizes = None if calls is None else []
+    o, _ = gated_memory(q, f, (h @ w[pre + "v"].t()).view(T, H, P), sizes=sizes)
+    if calls is not None:
+        hold = torch.stack(sizes) * q.norm(dim=-1)
+        calls.append((2.5 * math.sqrt(d) * (o.norm(dim=-1) / hold.clamp_min(1e-30)).amin(-1)).to(torch.float32))
     return (unit_rms(o, eps) * w[pre + "norm"]).reshape(T, H * P)
 
 
@@ -244,7 +254,7 @@ class PlainLopilix:
         if L["type"] == "attention":
             heads = difference_attention(h, w, pre, m, eps, pos, rt)
         elif L["type"] == "hgrn2":
-            heads = memory_mixer(h, w, pre, m, eps)
+            heads = memory_mixer(h, w, pre, m, eps, calls=self._gaps)
         elif L["type"] == "latent_attention":
             heads = latent_attention(h, w, pre, m, eps, pos, rt)
         else:
@@ -281,7 +291,7 @@ class PlainLopilix:
                 x = self.sublayer(i, 2, x, lambda h: self.feed_forward(i, L["mlp"], h))
             if layers_out is not None:
                 layers_out.append(x.sum(1))
-        # per position, the closest call any router of the model made on it
+        # per position, the closest call any router or memory of the model made on it
         self.gaps = torch.stack(self._gaps).amin(0) if self._gaps else torch.full((len(ids),), float("inf"))
         return (self.norm(x.sum(1), "final.norm") @ self.w["embed"].t()) * cfg["logit_scale"]
 
