@@ -56,6 +56,12 @@
 // which the pipe drains; a tile's softmax took 0.85 us of exponentials plus 0.4 us to hand the probabilities over.
 // Two Q tiles that share every key tile, as here, pay those once for 256 rows.
 //
+// Two maps over the same values (-DHEAD_DIM=64 -DVALUE_DIM=128 -DMAPS=2: differential attention).  The block's two Q tiles are then the
+// SAME 128 rows under the two maps: the key tile is the two maps' keys side by side, Q tile t meets half t of it, and both use
+// the one value tile.  At the end both maps' outputs of a row are in the block, and what is written is the finished head:
+// u = a1 - weight a2, u / sqrt(mean(u^2) + eps) * scale; the maps' outputs never reach memory.  A page of the cache holds the keys
+// [nkv][page_size][64] (neighbouring key heads are a value head's two maps) and then the values [nkv / 2][page_size][128].
+//
 // Reference counterpart: flash_sdpa_tiled_kernel (src/runtime/kernels/cuda_kernels.cu:558-645): one block per
 // query row, scalar FMA, keys of the same launch only.
 #include <cuda.h>
@@ -66,6 +72,13 @@
 #error "compile with -DHEAD_DIM=64 or -DHEAD_DIM=128"
 #endif
 static_assert(HEAD_DIM == 64 || HEAD_DIM == 128, "HEAD_DIM must be 64 or 128");
+#ifndef VALUE_DIM
+#define VALUE_DIM HEAD_DIM
+#endif
+#ifndef MAPS
+#define MAPS 1
+#endif
+static_assert(MAPS == 1 ? VALUE_DIM == HEAD_DIM : (MAPS == 2 && HEAD_DIM == 64 && VALUE_DIM == 128), "two maps come with keys of 64 and values of 128");
 
 LLME_API const char* llme_last_error() { return llme_error_buffer(); }
 
@@ -73,14 +86,19 @@ namespace {
 
 typedef __nv_bfloat16 bf16;
 constexpr int HD = HEAD_DIM;
-constexpr int HALVES = HD / 64;        // 64-column (128-byte) halves of a row
+constexpr int VD = VALUE_DIM;
+constexpr int HALVES = HD / 64;        // 64-column (128-byte) halves of a query row
+constexpr int PARTS = VD / 64;         // 64-column parts of a value row, and of a key tile (halves of a row, or the two maps' keys)
+static_assert(PARTS == HALVES * MAPS, "key and value tiles have the same shape");
 constexpr int BM = 128;                // rows per Q tile
 constexpr int QT = 2;                  // Q tiles per block: they share every key/value tile the block loads
 constexpr int BN = 128;                // keys per tile
 constexpr int BOX_ROWS = 32;           // most keys one TMA load brings; a tile's loads are started by as many lanes
 constexpr int THREADS = 32 * (2 + 8 * QT);   // producer, matrix warp, eight softmax warps per Q tile
 constexpr int HALF_BYTES = 128 * 128;  // a [128 rows x 64 columns] bfloat16 tile with 128-byte rows
-constexpr int TILE_BYTES = HALVES * HALF_BYTES;
+constexpr int TILE_BYTES = HALVES * HALF_BYTES;     // a Q tile
+constexpr int KV_BYTES = PARTS * HALF_BYTES;        // a key tile, a value tile
+constexpr int BLOCK_ROWS = MAPS == 2 ? BM : QT * BM;   // (token, head) rows a block serves
 constexpr unsigned WAIT_LIMIT = 1u << 20;
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -96,6 +114,7 @@ struct TcAttnArgs {
     const int* block_tables;     // [*, max_blocks]
     int max_blocks, n_rows, nh, nkv, page_size, window;
     float scale;
+    float diff_weight, diff_scale, diff_eps;     // two maps: what a row's two outputs become (out is then [T, nh / 2, VD])
 };
 #include "kernel_args.h"
 static_assert(sizeof(TcAttnArgs) == sizeof(LlmeTcAttnArgs), "the argument block must match kernel_args.h");
@@ -265,30 +284,33 @@ struct Barriers {
 };
 
 __global__ void __launch_bounds__(THREADS, 1)
-attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, TcAttnArgs a) {
+attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
+                    TcAttnArgs a) {
     extern __shared__ unsigned char smem_raw[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
     unsigned char* q_tiles = smem;                             // QT x HALVES x [128 rows x 128 B]
     unsigned char* k_tiles = q_tiles + QT * TILE_BYTES;        // 2 stages
-    unsigned char* v_tiles = k_tiles + 2 * TILE_BYTES;         // 2 stages
-    Barriers* bar = reinterpret_cast<Barriers*>(v_tiles + 2 * TILE_BYTES);
+    unsigned char* v_tiles = k_tiles + 2 * KV_BYTES;           // 2 stages
+    Barriers* bar = reinterpret_cast<Barriers*>(v_tiles + 2 * KV_BYTES);
     volatile int* abort_flag = &bar->abort_flag;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = a.rows[blockIdx.z];
     // blockIdx.x = pair * nkv + head: the blocks with the most keys, of all heads, start first
-    const int kvh = (int)(blockIdx.x % (unsigned)a.nkv), pair_index = (int)(blockIdx.x / (unsigned)a.nkv);
+    const int n_heads = a.nkv / MAPS;                          // value heads
+    const int kvh = (int)(blockIdx.x % (unsigned)n_heads), pair_index = (int)(blockIdx.x / (unsigned)n_heads);
     const int G = a.nh / a.nkv;
     const int q0 = a.cu_q_lens[r];
     const int q_len = a.cu_q_lens[r + 1] - q0;
     const int M = q_len * G;
-    const int m0 = ((M + QT * BM - 1) / (QT * BM) - 1 - pair_index) * (QT * BM);    // first row of the block's first Q tile
+    const int m0 = ((M + BLOCK_ROWS - 1) / BLOCK_ROWS - 1 - pair_index) * BLOCK_ROWS;    // first row of the block's first Q tile
     if (m0 < 0) return;
-    const int n_q = m0 + BM < M ? QT : 1;                             // Q tiles of this block that hold rows
+    const int n_q = MAPS == 2 || m0 + BM < M ? QT : 1;                // Q tiles of this block that hold rows
+    const int row_tiles = MAPS == 2 ? 1 : n_q;                        // tiles of different rows among them
     const int start = a.ctx_lens[r] - q_len;
     const int* bt = a.block_tables + (size_t)a.table_rows[r] * a.max_blocks;
     const int ps = a.page_size;
-    const int t_lo = m0 / G, t_hi = min(q_len - 1, (m0 + n_q * BM - 1) / G);
+    const int t_lo = m0 / G, t_hi = min(q_len - 1, (m0 + row_tiles * BM - 1) / G);
     const int hi_max = start + t_hi;                                  // last key any row of the block sees
     const int lo_min = a.window > 0 ? max(0, start + t_lo - a.window + 1) : 0;
     const int tile_first = lo_min / BN, tile_last = hi_max / BN;
@@ -311,7 +333,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     // the value tiles start as zeros: rows that are never loaded (before a window, past the last key) must not be NaN
-    for (int i = threadIdx.x; i < 2 * TILE_BYTES / 16; i += THREADS) reinterpret_cast<uint4*>(v_tiles)[i] = make_uint4(0, 0, 0, 0);
+    for (int i = threadIdx.x; i < 2 * KV_BYTES / 16; i += THREADS) reinterpret_cast<uint4*>(v_tiles)[i] = make_uint4(0, 0, 0, 0);
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     if (warp == 1) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&bar->tmem_base)), "r"(512u));
@@ -331,10 +353,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             mbar_expect_tx(&bar->q_full, (unsigned)(n_q * TILE_BYTES));
             for (int t = 0; t < n_q; ++t)
                 for (int h = 0; h < HALVES; ++h)
-                    tma_load_3d(q_tiles + t * TILE_BYTES + h * HALF_BYTES, &map_q, h * 64, kvh * G, q0 + (m0 + t * BM) / G, &bar->q_full);
+                    tma_load_3d(q_tiles + t * TILE_BYTES + h * HALF_BYTES, &map_q, h * 64, (MAPS == 2 ? 2 * kvh + t : kvh) * G,
+                                q0 + (MAPS == 2 ? m0 : m0 + t * BM) / G, &bar->q_full);
         }
         // Rows one TMA load of the cache brings: a power of two (pages of 8..32 tokens, or 32 rows of a larger
-        // page).  A lane looks after one TMA load of a tile (box lane / HALVES, 64-column half lane % HALVES): it
+        // page).  A lane looks after one TMA load of a tile (box lane / PARTS, 64-column part lane % PARTS): it
         // looks up the box's page (two tiles ahead of its use, so that the look-up's latency is not in front of
         // the copies), and decides whether the box is needed whole (a TMA load), in part (copied by hand), or
         // not at all.  No division in the loop: the producer's instructions are a dependent chain, and nothing
@@ -343,17 +366,21 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int box_shift = __ffs(rows_per_box) - 1;
         const int n_boxes = BN >> box_shift;
         const int ps_shift = (ps & (ps - 1)) == 0 ? __ffs(ps) - 1 : -1;
-        constexpr int H_SHIFT = HALVES == 2 ? 1 : 0;
+        constexpr int H_SHIFT = PARTS == 2 ? 1 : 0;
         const unsigned load_bytes = (unsigned)(rows_per_box * 128);     // one TMA load: a box of one 64-column half
-        const int my_box = lane >> H_SHIFT, my_half = lane & (HALVES - 1);
-        const long long head_rows = (long long)kvh * ps;                 // row of this head within a page's K (or V) block
-        const long long page_rows = (long long)2 * a.nkv * ps, v_rows = (long long)a.nkv * ps;
+        const int my_box = lane >> H_SHIFT, my_half = lane & (PARTS - 1);
+        // A page in rows of HD values (keys) and of VD values (values): 2 nkv ps rows of either width where the two are the same;
+        // with two maps the keys are nkv ps rows of half the width of the nkv / 2 ps rows of values behind them.
+        const long long key_page = (long long)2 * a.nkv * ps, key_head = (long long)(MAPS == 2 ? 2 * kvh + my_half : kvh) * ps;
+        const long long value_page = key_page / MAPS, value_head = (MAPS == 2 ? (long long)a.nkv / 2 * ps : (long long)a.nkv * ps) + (long long)kvh * ps;
+        struct BoxRows { long long k, v; };                               // rows of this lane's box in the key and in the value map, or -1
         bool ok = true;
-        auto first_row = [&](int i) -> long long {                       // cache row of this lane's box in tile i (its K rows), or -1
+        auto first_row = [&](int i) -> BoxRows {
             const int ja = (tile_first + i) * BN + (my_box << box_shift);
-            if (i >= n_tiles || my_box >= n_boxes || ja + rows_per_box - 1 < lo_min || ja > hi_max) return -1;
+            if (i >= n_tiles || my_box >= n_boxes || ja + rows_per_box - 1 < lo_min || ja > hi_max) return {-1, -1};
             const int blk = ps_shift >= 0 ? ja >> ps_shift : ja / ps;
-            return (long long)bt[blk] * page_rows + head_rows + (ja - blk * ps);
+            const long long page = bt[blk], off = ja - blk * ps;
+            return {page * key_page + key_head + off, page * value_page + value_head + off};
         };
         // One load of a tile: its keys (which = 0) or its values (1), into the stage i % 2; `full` counts its bytes,
         // `empty` (if any) with `empty_parity` says when the stage may be overwritten.
@@ -364,7 +391,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             const unsigned whole_mask = __ballot_sync(0xffffffffu, whole);                 // one bit per TMA load
             const unsigned part_mask = __ballot_sync(0xffffffffu, my_row >= 0 && !whole && my_half == 0);
             const unsigned tx = (unsigned)__popc(whole_mask) * load_bytes;
-            unsigned char* tile = (which ? v_tiles : k_tiles) + (i & 1) * TILE_BYTES;
+            unsigned char* tile = (which ? v_tiles : k_tiles) + (i & 1) * KV_BYTES;
             if (empty) ok = mbar_wait(empty, empty_parity, abort_flag, 10 + which);
             ok = ok && !*abort_flag;
             if (!ok) return;
@@ -374,13 +401,15 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             if (part_mask) {
                 for (unsigned rest = part_mask; rest; rest &= rest - 1) {
                     const int src_lane = __ffs(rest) - 1, b = (src_lane >> H_SHIFT) << box_shift;
-                    const long long row0 = __shfl_sync(0xffffffffu, my_row, src_lane) + (which ? v_rows : 0);
-                    for (int c = lane; c < rows_per_box * (HD / 8); c += 32) {
-                        const int rr = c / (HD / 8), ch = c % (HD / 8);
+                    const long long row0 = __shfl_sync(0xffffffffu, my_row, src_lane);
+                    for (int c = lane; c < rows_per_box * (VD / 8); c += 32) {
+                        const int rr = c / (VD / 8), ch = c % (VD / 8);
                         const int j = j0 + b + rr;
-                        uint4 v = make_uint4(0, 0, 0, 0);
-                        if (j >= lo_min && j <= hi_max) v = *reinterpret_cast<const uint4*>(a.cache + (row0 + rr) * HD + ch * 8);
                         const int h = ch >> 3, q = ch & 7, row = b + rr;
+                        uint4 v = make_uint4(0, 0, 0, 0);
+                        if (j >= lo_min && j <= hi_max)
+                            v = *reinterpret_cast<const uint4*>(MAPS == 2 && !which ? a.cache + (row0 + (long long)h * ps + rr) * HD + q * 8
+                                                                                    : a.cache + (row0 + rr) * VD + ch * 8);
                         *reinterpret_cast<uint4*>(tile + h * HALF_BYTES + row * 128 + ((q ^ (row & 7)) << 4)) = v;
                     }
                 }
@@ -392,27 +421,27 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // every lane starts the load of its own box: issued from one thread, the many small boxes of
             // small pages went out one after the other and took longer than the arithmetic on them
             if (whole)
-                tma_load_2d(tile + my_half * HALF_BYTES + (my_box << box_shift) * 128, &map_kv, my_half * 64,
-                            (int)(my_row + (which ? v_rows : 0)), full);
+                tma_load_2d(tile + my_half * HALF_BYTES + (my_box << box_shift) * 128, which ? &map_v : &map_k,
+                            MAPS == 2 && !which ? 0 : my_half * 64, (int)my_row, full);
             __syncwarp();
         };
         // The keys run one tile ahead of the values: the matrix warp takes V(i) and K(i+1) together (O += P V(i),
         // then S = Q K(i+1)^T), and gives both stages back together when tile i is done.
-        long long row_cur = first_row(0), row_next = first_row(1);
-        load_tile(0, 0, row_cur, &bar->k0_full, nullptr, 0u);
+        BoxRows row_cur = first_row(0), row_next = first_row(1);
+        load_tile(0, 0, row_cur.k, &bar->k0_full, nullptr, 0u);
         for (int i = 0; i < n_tiles && ok; ++i) {
-            const long long row_after = first_row(i + 2);
+            const BoxRows row_after = first_row(i + 2);
             unsigned long long* full = &bar->kv_full[i & 1];
             unsigned long long* empty = &bar->kv_empty[i & 1];
             const unsigned parity = ((unsigned)(i >> 1) & 1u) ^ 1u;          // passes at once while the stages are fresh
             // K(2) goes where K(0) lay, which no kv_empty speaks for
             if (i == 1) ok = mbar_wait(&bar->k0_empty, 0, abort_flag, 12);
             if (i + 1 < n_tiles) {
-                if (ok) load_tile(i + 1, 0, row_next, full, empty, parity);
+                if (ok) load_tile(i + 1, 0, row_next.k, full, empty, parity);
             } else if (lane == 0) {
                 mbar_arrive(full);                                           // no keys behind the last tile
             }
-            if (ok) load_tile(i, 1, row_cur, full, empty, parity);
+            if (ok) load_tile(i, 1, row_cur.v, full, empty, parity);
             row_cur = row_next;
             row_next = row_after;
         }
@@ -427,30 +456,34 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // softmax of the other runs: S_0(0) S_1(0) | O_0(0) S_0(1) O_1(0) S_1(1) | O_0(1) S_0(2) ...
         if (lane == 0) {
             constexpr unsigned id_s = idesc(BM, BN, 0);
-            constexpr unsigned id_o = idesc(BM, HD, 1);
+            constexpr unsigned id_o = idesc(BM, VD, 1);
             bool ok = mbar_wait(&bar->q_full, 0, abort_flag, 20);
             // The one thread that issues the matrix instructions runs a dependent chain of its own: every
             // instruction it spends between two products delays both Q tiles (measured: 0.7 us per group of
             // eight products when the descriptors were built inside the loop, against 0.27 us that the tensor
             // pipe needs for them).  So the descriptors are built once, and a group is waits, eight
             // instructions and commits.
-            unsigned long long dq[QT][HALVES], dk[2][HALVES], dv[2];
+            unsigned long long dq[QT][HALVES], dk[2][PARTS], dv[2];
 #pragma unroll
-            for (int h = 0; h < HALVES; ++h) {
+            for (int h = 0; h < PARTS; ++h) {
+                if (h < HALVES) {
 #pragma unroll
-                for (int t = 0; t < QT; ++t) dq[t][h] = desc_k_major(q_tiles + t * TILE_BYTES + h * HALF_BYTES);
+                    for (int t = 0; t < QT; ++t) dq[t][h < HALVES ? h : 0] = desc_k_major(q_tiles + t * TILE_BYTES + h * HALF_BYTES);
+                }
 #pragma unroll
-                for (int s = 0; s < 2; ++s) dk[s][h] = desc_k_major(k_tiles + s * TILE_BYTES + h * HALF_BYTES);
+                for (int s = 0; s < 2; ++s) dk[s][h] = desc_k_major(k_tiles + s * KV_BYTES + h * HALF_BYTES);
             }
 #pragma unroll
-            for (int s = 0; s < 2; ++s) dv[s] = desc_mn_major(v_tiles + s * TILE_BYTES);
+            for (int s = 0; s < 2; ++s) dv[s] = desc_mn_major(v_tiles + s * KV_BYTES);
+            // the keys of stage s that Q tile t meets first: the first 64 columns of the rows, or map t's keys
+            auto dk_first = [&](int s, int t) { return MAPS == 2 && t == 1 ? (s == 0 ? dk[0][PARTS - 1] : dk[1][PARTS - 1]) : (s == 0 ? dk[0][0] : dk[1][0]); };
             auto issue_first = [&](int t) {                           // S_t(0) = Q_t K(0)^T
                 ok = ok && mbar_wait(&bar->k0_full, 0, abort_flag, 21);
                 if (!ok) return;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const unsigned d = t == 0 ? tmem_s[0] : tmem_s[1];
-                umma_qk_half<true>(d, t == 0 ? dq[0][0] : dq[QT - 1][0], dk[0][0], id_s);
-                if (HALVES == 2) umma_qk_half<false>(d, t == 0 ? dq[0][HALVES - 1] : dq[QT - 1][HALVES - 1], dk[0][HALVES - 1], id_s);
+                umma_qk_half<true>(d, t == 0 ? dq[0][0] : dq[QT - 1][0], dk_first(0, t), id_s);
+                if (HALVES == 2) umma_qk_half<false>(d, t == 0 ? dq[0][HALVES - 1] : dq[QT - 1][HALVES - 1], dk[0][PARTS - 1], id_s);
                 if (t == n_q - 1) umma_commit(&bar->k0_empty);        // both Q tiles have read K(0)
                 umma_commit(&bar->s_full[t]);
             };
@@ -475,9 +508,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 umma_pv_half(d, pa + 64u, b0 + 4ull * (2048 >> 4), id_o, 1u);
                 if (more) {
                     // S_t is free again once the products above have read P_t(i); the pipe runs them in order
-                    umma_qk_half<true>(pa, t == 0 ? dq[0][0] : dq[QT - 1][0], s1 == 0 ? dk[0][0] : dk[1][0], id_s);
+                    umma_qk_half<true>(pa, t == 0 ? dq[0][0] : dq[QT - 1][0], dk_first(s1, t), id_s);
                     if (HALVES == 2)
-                        umma_qk_half<false>(pa, t == 0 ? dq[0][HALVES - 1] : dq[QT - 1][HALVES - 1], s1 == 0 ? dk[0][HALVES - 1] : dk[1][HALVES - 1], id_s);
+                        umma_qk_half<false>(pa, t == 0 ? dq[0][HALVES - 1] : dq[QT - 1][HALVES - 1], s1 == 0 ? dk[0][PARTS - 1] : dk[1][PARTS - 1], id_s);
                     umma_commit(&bar->s_full[t]);
                 }
                 if (t == n_q - 1) {
@@ -500,13 +533,13 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         // through registers and a second reading of the scores, which then happens only in the first few tiles.
         constexpr float RESCALE = 8.0f;
         constexpr int BH = BN / 2;                           // keys of a tile per thread
-        constexpr int OC = HD / 2;                           // columns of the output accumulator per thread
+        constexpr int OC = VD / 2;                           // columns of the output accumulator per thread
         const int quarter = warp & 3;
         const int role = (warp - 2) >> 2;                    // 0..3
         const int t = role >> 1, ch = role & 1;              // Q tile, half of the columns
         if (t < n_q) {
             const int row = quarter * 32 + lane;             // this thread's row of its Q tile
-            const int mt0 = m0 + t * BM;
+            const int mt0 = MAPS == 2 ? m0 : m0 + t * BM;
             const int m = mt0 + row;
             const bool row_ok = m < M;
             const int p = start + min(m, M - 1) / G;         // its position
@@ -629,10 +662,67 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // of a row are swizzled with the row, so that neither the writes (eight rows, the same piece) nor the
             // reads (one row, pieces in turn) meet in a bank; the two warps of a (Q tile, quarter) then write their
             // 32 rows out whole, two rows to a store.
-            constexpr int ROW_PIECES = HD / 8;
-            unsigned char* stage = q_tiles + t * TILE_BYTES;     // [BM rows][2 x HEAD_DIM bytes]
+            constexpr int ROW_PIECES = VD / 8;
+            unsigned char* stage = MAPS == 2 ? k_tiles : q_tiles + t * TILE_BYTES;     // [BM rows][2 x HEAD_DIM bytes]
             const bool good = ok && !*abort_flag;
-            if (good) {
+            if (MAPS == 2) {
+                // The maps' outputs meet in shared memory, in the place of the key tiles, which nothing reads any more: the second
+                // map's warps leave weight * a2 there (32-bit, the 16-byte pieces of a row swizzled with the row), the first map's
+                // take the difference, sum its squares over the row's two halves and put it back; then the four warps of a
+                // quarter write their 32 finished rows out.  Every warp comes to every barrier, also after a wait has given up.
+                auto quarter_sync = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(9 + quarter) : "memory"); };
+                const float inv = (t == 0 ? 1.0f : a.diff_weight) / l_run;
+                auto slot = [&](int r, int piece) { return reinterpret_cast<float4*>(stage + r * (VD * 4) + ((piece ^ (r & 7)) << 4)); };
+                if (good) asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                if (t == 1 && good) {
+#pragma unroll 1
+                    for (int c = 0; c < OC; c += 32) {
+                        float v[32];
+                        tmem_ld32(tmem_o[1] + lane_off + (unsigned)(ch * OC + c), v);
+#pragma unroll
+                        for (int q4 = 0; q4 < 8; ++q4)
+                            *slot(row, (ch * OC + c) / 4 + q4) = make_float4(v[4 * q4] * inv, v[4 * q4 + 1] * inv, v[4 * q4 + 2] * inv, v[4 * q4 + 3] * inv);
+                    }
+                }
+                quarter_sync();
+                float ss = 0.0f;
+                if (t == 0 && good) {
+#pragma unroll 1
+                    for (int c = 0; c < OC; c += 32) {
+                        float v[32];
+                        tmem_ld32(tmem_o[0] + lane_off + (unsigned)(ch * OC + c), v);
+#pragma unroll
+                        for (int q4 = 0; q4 < 8; ++q4) {
+                            float4* at = slot(row, (ch * OC + c) / 4 + q4);
+                            float4 u = *at;
+                            u = make_float4(fmaf(v[4 * q4], inv, -u.x), fmaf(v[4 * q4 + 1], inv, -u.y), fmaf(v[4 * q4 + 2], inv, -u.z), fmaf(v[4 * q4 + 3], inv, -u.w));
+                            ss = fmaf(u.x, u.x, fmaf(u.y, u.y, fmaf(u.z, u.z, fmaf(u.w, u.w, ss))));
+                            *at = u;
+                        }
+                    }
+                }
+                if (t == 0) bar->row_max[0][0][ch][row] = ss;
+                quarter_sync();
+                if (good) {
+                    const int tid = (t * 2 + ch) * 32 + lane;        // 0..127 among the quarter's four warps
+#pragma unroll 2
+                    for (int k = 0; k < 32 * ROW_PIECES / 128; ++k) {
+                        const int idx = k * 128 + tid;
+                        const int r = quarter * 32 + idx / ROW_PIECES, piece = idx % ROW_PIECES;
+                        const int mm = mt0 + r;
+                        if (mm >= M) continue;
+                        const float f = a.diff_scale / sqrtf((bar->row_max[0][0][0][r] + bar->row_max[0][0][1][r]) / (float)VD + a.diff_eps);
+                        const float4 lo = *slot(r, 2 * piece), hi = *slot(r, 2 * piece + 1);
+                        uint4 pk;
+                        *reinterpret_cast<__nv_bfloat162*>(&pk.x) = __floats2bfloat162_rn(lo.x * f, lo.y * f);
+                        *reinterpret_cast<__nv_bfloat162*>(&pk.y) = __floats2bfloat162_rn(lo.z * f, lo.w * f);
+                        *reinterpret_cast<__nv_bfloat162*>(&pk.z) = __floats2bfloat162_rn(hi.x * f, hi.y * f);
+                        *reinterpret_cast<__nv_bfloat162*>(&pk.w) = __floats2bfloat162_rn(hi.z * f, hi.w * f);
+                        *reinterpret_cast<uint4*>(a.out + ((size_t)(q0 + mm / G) * (a.nh / 2) + kvh * G + mm % G) * VD + piece * 8) = pk;
+                    }
+                }
+            }
+            if (MAPS == 1 && good) {
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const float inv = 1.0f / l_run;
 #pragma unroll 1
@@ -653,8 +743,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     }
                 }
             }
-            pair_sync();
-            if (good) {
+            if (MAPS == 1) pair_sync();
+            if (MAPS == 1 && good) {
                 const int tid = ch * 32 + lane;                  // 0..63 among the two warps
 #pragma unroll 4
                 for (int k = 0; k < 32 * ROW_PIECES / 64; ++k) {
@@ -690,7 +780,8 @@ EncodeTiledFn encode_fn() {
     return fn;
 }
 
-constexpr size_t SMEM_BYTES = 1024 + (size_t)(QT + 4) * TILE_BYTES + sizeof(Barriers) + 64;
+constexpr size_t SMEM_BYTES = 1024 + (size_t)QT * TILE_BYTES + 4 * (size_t)KV_BYTES + sizeof(Barriers) + 64;
+static_assert(MAPS == 1 || (size_t)BM * VD * 4 <= 2 * (size_t)KV_BYTES, "the rows' differences take the place of the key tiles");
 static_assert(SMEM_BYTES <= 232448, "the block's shared memory must fit an SM");
 
 }  // namespace
@@ -706,7 +797,7 @@ LLME_API int llme_attention_tc_supports(int nh, int nkv, int page_size) {
 }
 
 // q, out [T, nh, HD] bfloat16 (q_tokens = T rows in all); the other arguments as for the portion kernel of
-// attention_fast.cu.  total_cache_rows = pages * 2 * nkv * page_size.
+// attention_fast.cu.  total_cache_rows = pages * 2 * nkv * page_size (rows of HD values).  Two maps: out [T, nh / 2, VD].
 LLME_API int llme_attention_tc(const void* q, long long q_tokens, long long total_cache_rows, const TcAttnArgs* args,
                                int max_q_len, cudaStream_t stream) {
     const TcAttnArgs& a = *args;
@@ -714,11 +805,12 @@ LLME_API int llme_attention_tc(const void* q, long long q_tokens, long long tota
     if (!q || !a.out || !a.cache || !a.rows || !a.cu_q_lens || !a.ctx_lens || !a.table_rows || !a.block_tables)
         LLME_REFUSE("attention_tc: null pointer");
     if (!llme_attention_tc_supports(a.nh, a.nkv, a.page_size)) LLME_REFUSE("attention_tc: %d/%d heads with pages of %d are not supported", a.nh, a.nkv, a.page_size);
+    if (a.nkv % MAPS || (MAPS == 2 && !(a.diff_eps > 0.0f))) LLME_REFUSE("attention_tc: two maps come in pairs of key heads, with a positive eps");
     if (a.n_rows > 65535) LLME_REFUSE("attention_tc: grid too large");
     EncodeTiledFn enc = encode_fn();
     if (!enc) LLME_REFUSE("attention_tc: cuTensorMapEncodeTiled is not available in this driver");
     const int G = a.nh / a.nkv;
-    alignas(64) CUtensorMap mq, mkv;
+    alignas(64) CUtensorMap mq, mk, mv;
     {   // q as [token][head][column]; a box is 128/G tokens x G heads x 64 columns = 128 rows of 128 bytes
         cuuint64_t dims[3] = {(cuuint64_t)HD, (cuuint64_t)a.nh, (cuuint64_t)q_tokens};
         cuuint64_t strides[2] = {(cuuint64_t)HD * 2, (cuuint64_t)a.nh * HD * 2};
@@ -729,26 +821,29 @@ LLME_API int llme_attention_tc(const void* q, long long q_tokens, long long tota
                          CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
         if (r != CUDA_SUCCESS) LLME_REFUSE("attention_tc: cuTensorMapEncodeTiled (q) failed with code %d", (int)r);
     }
-    {   // the cache as rows of HD columns; a box is one page (or 128 rows of a larger page) x 64 columns
-        cuuint64_t dims[2] = {(cuuint64_t)HD, (cuuint64_t)total_cache_rows};
-        cuuint64_t strides[1] = {(cuuint64_t)HD * 2};
+    // the cache as rows of HD columns (and, where the values are wider, as rows of VD columns); a box is one page (or 32 rows of a
+    // larger page) x 64 columns
+    auto cache_map = [&](CUtensorMap* map, int cols, long long rows) -> CUresult {
+        cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+        cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
         cuuint32_t box[2] = {64, (cuuint32_t)(a.page_size < BOX_ROWS ? a.page_size : BOX_ROWS)};
         cuuint32_t es[2] = {1, 1};
-        CUresult r = enc(&mkv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(a.cache), dims, strides, box, es,
-                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                         CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-        if (r != CUDA_SUCCESS) LLME_REFUSE("attention_tc: cuTensorMapEncodeTiled (cache) failed with code %d", (int)r);
-    }
+        return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(a.cache), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    };
+    CUresult r = cache_map(&mk, HD, total_cache_rows);
+    if (r == CUDA_SUCCESS) r = cache_map(&mv, VD, total_cache_rows / MAPS);
+    if (r != CUDA_SUCCESS) LLME_REFUSE("attention_tc: cuTensorMapEncodeTiled (cache) failed with code %d", (int)r);
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);
         if (e != cudaSuccess) LLME_REFUSE("attention_tc: cannot reserve %zu bytes of shared memory: %s", SMEM_BYTES, cudaGetErrorString(e));
         configured = true;
     }
-    const long long tiles = ((long long)max_q_len * G + QT * BM - 1) / (QT * BM);
-    if (tiles * a.nkv > 2147483647LL) LLME_REFUSE("attention_tc: grid too large");
-    dim3 grid((unsigned)(tiles * a.nkv), 1, a.n_rows);
-    attention_tc_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(mq, mkv, a);
+    const long long tiles = ((long long)max_q_len * G + BLOCK_ROWS - 1) / BLOCK_ROWS;
+    if (tiles * (a.nkv / MAPS) > 2147483647LL) LLME_REFUSE("attention_tc: grid too large");
+    dim3 grid((unsigned)(tiles * (a.nkv / MAPS)), 1, a.n_rows);
+    attention_tc_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(mq, mk, mv, a);
     LLME_LAUNCH_STATUS();
 }
 

@@ -81,6 +81,8 @@ typedef int (*EmbeddingStreamsFn)(const int*, const void*, int, const int*, cons
 typedef int (*StreamNormFn)(const LlmeStreamNormArgs*, cudaStream_t);
 typedef int (*ForgetGatesFn)(const LlmeForgetGatesArgs*, cudaStream_t);
 typedef int (*DifferenceNormFn)(const LlmeDifferenceNormArgs*, cudaStream_t);
+typedef int (*MapsDecodeFn)(const LlmeMapsDecodeArgs*, cudaStream_t);
+typedef long long (*MapsScratchFn)(int, int, int, int);
 typedef int (*RowNormFn)(const void*, long long, int, const void*, int, void*, long long, int, int, int, float, cudaStream_t);
 typedef int (*ExpGatesFn)(const LlmeExpGatesArgs*, int, cudaStream_t);
 typedef int (*GemmF32BatchedFn)(const float*, const void*, int, float*, int, int, int, long long, long long, long long, int, long long,
@@ -204,7 +206,6 @@ size_t record_size(int kind) {
         case LLME_OP_DELTA_RULE: return sizeof(LlmeDeltaRuleOp);
         case LLME_OP_STREAM_NORM: return sizeof(LlmeStreamNormOp);
         case LLME_OP_FORGET_GATES: return sizeof(LlmeForgetGatesOp);
-        case LLME_OP_DIFFERENCE_NORM: return sizeof(LlmeDifferenceNormOp);
     }
     return 0;
 }
@@ -213,8 +214,8 @@ const char* kind_name(int kind) {
                                   "linear_act", "pointwise", "batched_linear", "residual_add", "latent_attention", "token_side",
                                   "postnorm", "window_attention", "moe_route", "grouped_linear", "moe_combine", "short_conv", "rotate",
                                   "recurrence", "gated_norm", "row_norm", "exp_gates", "layernorm", "delta_rule",
-                                  "stream_norm", "forget_gates", "difference_norm"};
-    return kind >= 1 && kind <= 30 ? names[kind] : names[0];
+                                  "stream_norm", "forget_gates"};
+    return kind >= 1 && kind <= 29 ? names[kind] : names[0];
 }
 
 constexpr int SKINNY_ROWS = 16;      // most rows the weight-streaming product takes (gemm_skinny.cu)
@@ -718,9 +719,56 @@ int op_postnorm(LlmeExecutor& ex, const LlmePostNormOp& o, const LlmeStep& s, cu
     return ex.launched(f(o.x, o.y, o.y_dtype, o.gain, o.gain_dtype, o.copy, o.copy_dtype, s.num_tokens, o.size, o.eps, o.accumulate, st), "postnorm");
 }
 
-int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st) {
-    if (s.num_tokens <= 0) return 0;
-    if (o.group < 0 || o.group >= s.num_groups) return ex.fail("window attention: the step has no cache group %d", o.group);
+// Differential attention behind its post step where kernels finish the heads themselves: prompt portions on tcgen05 (two maps a block),
+// single tokens in shares.  `done` stays false where these kernels do not serve the step.
+int difference_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st, bool* done) {
+    const LlmeStepGroup& g = s.groups[o.group];
+    if (o.dtype != LLME_DT_BF16 || ex.choice("attention") != "fast") return 0;
+    const std::string sizes = std::to_string(o.dk) + "x" + std::to_string(o.dv);
+    const int rep = o.nh / o.nkv, ps = g.page_size, groups = o.nkv / 2;
+    auto* tc = (AttnTcFn)ex.find("attention_tc/" + sizes + "x2");
+    auto* decode = (MapsDecodeFn)ex.find("maps_decode/" + sizes);
+    auto* need = (MapsScratchFn)ex.find("maps_decode_scratch/" + sizes);
+    if (s.num_portion > 0 && !(tc && ex.choice("attention.portion") == "tcgen05" && ps >= 8 && (ps <= 128 ? 128 % ps == 0 : ps % 128 == 0) && 128 % rep == 0)) return 0;
+    long long splits = 1;
+    if (s.num_decode > 0) {
+        if (!decode || !need || !o.maps_scratch) return 0;
+        // shares: three blocks an SM, no share shorter than two sub-tiles of 16 keys a warp, at most 32
+        const long long units = need(s.num_decode, o.nh / 2, groups, 1) / (16 * (o.dv + 2)), subs = (s.max_decode_ctx + 15) / 16;
+        splits = 3LL * ex.sms / (units > 0 ? units : 1);
+        if (splits > subs / 8) splits = subs / 8;
+        if (splits > 32) splits = 32;
+        if (splits < 1) splits = 1;
+        while (splits > 1 && need(s.num_decode, o.nh / 2, groups, (int)splits) > o.maps_scratch_floats) --splits;
+        if (need(s.num_decode, o.nh / 2, groups, (int)splits) > o.maps_scratch_floats) return 0;
+    }
+    if (s.num_portion > 0) {
+        LlmeTcAttnArgs a = {o.heads, o.cache, s.portion_rows, s.cu_q_lens, s.ctx_lens, s.state_slots, g.block_tables, g.max_blocks, s.num_portion, o.nh,
+                            o.nkv, ps, 0, o.scale, o.diff_weight, o.diff_scale, o.diff_eps};
+        const long long key_rows = o.cache_pages * ps * (o.nkv + (long long)groups * o.dv / o.dk);        // the cache in rows of dk values
+        if (int rc = ex.launched(tc(o.q, s.num_tokens, key_rows, &a, s.max_portion_len, st), "attention_tc")) return rc;
+    }
+    if (s.num_decode > 0) {
+        LlmeMapsDecodeArgs a = {o.q, o.cache, o.heads, s.decode_rows, s.cu_q_lens, s.ctx_lens, s.state_slots, g.block_tables, o.maps_scratch, g.max_blocks,
+                                s.num_decode, o.nh / 2, groups, ps, (int)splits, o.scale, o.diff_weight, o.diff_scale, o.diff_eps};
+        if (int rc = ex.launched(decode(&a, st), "maps_decode")) return rc;
+        ++ex.launches;                                          // the shares and their sum are two kernels
+    }
+    *done = true;
+    return 0;
+}
+
+// The difference of the maps as a step of its own, behind the attention.
+int difference_norm(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st) {
+    auto* f = (DifferenceNormFn)ex.find("difference_norm");
+    if (!f) return ex.fail("no difference_norm kernel is registered");
+    LlmeDifferenceNormArgs a = {o.out, (long long)o.nh * o.dv, o.heads, (long long)o.nh / 2 * o.dv, o.dtype, s.num_tokens, o.nh / 2, o.nh / o.nkv, o.dv,
+                                o.diff_weight, o.diff_scale, o.diff_eps};
+    return ex.launched(f(&a, st), "difference_norm");
+}
+
+// Norm, rotation and cache write of a window attention.
+int window_post(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st) {
     const LlmeStepGroup& g = s.groups[o.group];
     auto* post = (WindowPostFn)ex.find("window_post");
     if (!post) return ex.fail("no window_post kernel is registered");
@@ -732,7 +780,12 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
     p.q_bias = o.q_bias; p.k_bias = o.k_bias; p.v_bias = o.v_bias; p.head_norm = o.head_norm;
     p.interleaved = o.interleaved; p.in_f32 = o.in_f32; p.unit_norm = o.unit_norm;
     p.value_share = o.value_share;
-    if (int rc = ex.launched(post(&p, o.dtype, st), "window_post")) return rc;
+    return ex.launched(post(&p, o.dtype, st), "window_post");
+}
+
+// Its attention, queries finished and keys stored.
+int window_attend(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st) {
+    const LlmeStepGroup& g = s.groups[o.group];
     // ordinary causal attention with keys and values of one width: a page holds its keys and then its values in both layouts, so the
     // kernels of plain grouped-query attention (tcgen05 portions, split-context decode) read the cache as it is
     if (o.decode_scratch && o.dk == o.dv && o.value_share <= 1 && !o.keep_first && !o.sink && !(o.softcap > 0.0f) && fast_attention(ex, o.dtype, o.dk)) {
@@ -773,6 +826,18 @@ int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const 
     LlmeWindowAttnArgs a = {o.q, o.cache, o.out, o.sink, s.positions, s.token_request, g.block_tables, g.max_blocks, s.num_tokens,
                             o.nh, o.nkv, o.dk, o.dv, g.page_size, o.window, o.keep_first, o.scale, o.softcap, o.value_share};
     return ex.launched(plain(&a, o.dtype, st), "window_attention_plain");
+}
+
+int op_window_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const LlmeStep& s, cudaStream_t st) {
+    if (s.num_tokens <= 0) return 0;
+    if (o.group < 0 || o.group >= s.num_groups) return ex.fail("window attention: the step has no cache group %d", o.group);
+    if (int rc = window_post(ex, o, s, st)) return rc;
+    if (!o.heads) return window_attend(ex, o, s, st);
+    bool done = false;
+    if (int rc = difference_attention(ex, o, s, st, &done)) return rc;
+    if (done) return 0;
+    if (int rc = window_attend(ex, o, s, st)) return rc;
+    return difference_norm(ex, o, s, st);
 }
 
 int op_short_conv(LlmeExecutor& ex, const LlmeShortConvOp& o, const LlmeStep& s, cudaStream_t st) {
@@ -865,14 +930,6 @@ int op_forget_gates(LlmeExecutor& ex, const LlmeForgetGatesOp& o, const LlmeStep
     if (!f) return ex.fail("no forget_gates kernel is registered");
     LlmeForgetGatesArgs a = {o.q_in, o.f_in, o.ld_in, o.f_bias, o.lower, o.q, o.f, o.ldq, o.ldf, s.num_tokens, o.cols};
     return ex.launched(f(&a, st), "forget_gates");
-}
-
-int op_difference_norm(LlmeExecutor& ex, const LlmeDifferenceNormOp& o, const LlmeStep& s, cudaStream_t st) {
-    if (s.num_tokens <= 0) return 0;
-    auto* f = (DifferenceNormFn)ex.find("difference_norm");
-    if (!f) return ex.fail("no difference_norm kernel is registered");
-    LlmeDifferenceNormArgs a = {o.a, o.lda, o.out, o.ldo, o.dtype, s.num_tokens, o.heads, o.rep, o.dim, o.weight, o.scale, o.eps};
-    return ex.launched(f(&a, st), "difference_norm");
 }
 
 int op_exp_gates(LlmeExecutor& ex, const LlmeExpGatesOp& o, const LlmeStep& s, cudaStream_t st) {
@@ -1088,7 +1145,6 @@ LLME_EXPORT int llme_plan_run(LlmePlan* p, const LlmeStep* step, int first, int 
             case LLME_OP_DELTA_RULE: rc = op_delta_rule(ex, *(const LlmeDeltaRuleOp*)b, s, stream); break;
             case LLME_OP_STREAM_NORM: rc = op_stream_norm(ex, *(const LlmeStreamNormOp*)b, s, stream); break;
             case LLME_OP_FORGET_GATES: rc = op_forget_gates(ex, *(const LlmeForgetGatesOp*)b, s, stream); break;
-            case LLME_OP_DIFFERENCE_NORM: rc = op_difference_norm(ex, *(const LlmeDifferenceNormOp*)b, s, stream); break;
             case LLME_OP_EXP_GATES: rc = op_exp_gates(ex, *(const LlmeExpGatesOp*)b, s, stream); break;
             case LLME_OP_CALL: {
                 const LlmeCallOp& c = *(const LlmeCallOp*)b;

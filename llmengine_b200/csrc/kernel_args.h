@@ -45,6 +45,7 @@ typedef struct LlmeTcAttnArgs {
     const int* rows; const int* cu_q_lens; const int* ctx_lens; const int* table_rows; const int* block_tables;
     int max_blocks, n_rows, nh, nkv, page_size, window;
     float scale;
+    float diff_weight, diff_scale, diff_eps;     /* the form for two maps: out = (a1 - weight a2) / rms * scale, [T, nh / 2, dv] */
 } LlmeTcAttnArgs;
 
 /* Norm of the latent, rotation of the shared key part and of the heads' rotated query parts, cache write. */
@@ -259,3 +260,13 @@ typedef struct LlmeDifferenceNormArgs {
     int dtype, tokens, heads, rep, dim;
     float weight, scale, eps;
 } LlmeDifferenceNormArgs;
+
+/* Differential attention of the single tokens `rows` (csrc/attention_maps.cu): q [T, 2 heads dk] finished queries, per value head its
+ * heads under map 1 and then under map 2; out [T, heads dv] the finished heads.  A page: [2 groups][page][dk] keys, [groups][page][dv] values. */
+typedef struct LlmeMapsDecodeArgs {
+    const void* q; const void* cache; void* out;
+    const int* rows; const int* cu_q_lens; const int* ctx_lens; const int* table_rows; const int* block_tables;
+    float* scratch;
+    int max_blocks, n_rows, heads, groups, page_size, splits;
+    float scale, diff_weight, diff_scale, diff_eps;
+} LlmeMapsDecodeArgs;

@@ -1,4 +1,4 @@
-"""A design beside its closest existing model at equal size (`python bench.py --design bepuzen | torisun | vifelix | funevik | vaderax`).
+"""A design beside its closest existing model at equal size (`python bench.py --design bepuzen | torisun | vifelix | funevik | vaderax | lopilix`).
 
 For each size: prefill of one 2,048-token prompt and decode at batch 1 / 8 / 64 over 2,048 cached tokens, tokens/s,
 for the design and for the grouped-query model of the same width, depth and (active) weight count per layer;
@@ -112,6 +112,25 @@ def vaderax_shape(width: int, heads: int, kv_heads: int, ff: int, experts: int, 
             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in kinds], "loop": {"start": 1, "stop": 3, "times": 2}}
 
 
+def lopilix_shape(width: int, heads: int, kv_heads: int, ff: int, experts: int, top: int, expert_ff: int, streams: int = 4, dim: int = 128,
+                  vocab: int = 32768) -> Dict[str, Any]:
+    """Four stored layers that run as six, on four residual streams: a differential attention (two maps of 64 on values of 128, so its
+    projections have the grouped-query model's sizes) with a dense gated feed-forward, a loop of two passes over a memory with forget
+    gates and a latent attention (a latent of 512, a shared rotated part of 64, stretched) with routed experts, and a memory with a
+    dense feed-forward.  An active routed feed-forward has about the weights of the dense one."""
+    at = {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5, "diff": 0.5,
+          "rot": {"base": 250000.0, "dims": dim // 4}}
+    me = {"heads": heads, "dim": dim, "vdim": dim}
+    la = {"heads": heads, "dim": dim, "rot_dim": 64, "vdim": dim, "kv_rank": 512, "scale": (dim + 64) ** -0.5,
+          "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "scale": 2.5, "groups": {"count": 4, "keep": 2}}}
+    kinds = [("attention", at, dense), ("hgrn2", me, routed), ("latent_attention", la, routed), ("hgrn2", me, dense)]
+    return {"architecture": "Lopilix", "vocab": vocab, "width": width, "streams": streams, "max_positions": 4096, "norm": {"eps": 1e-6},
+            "residual_mult": 0.7, "logit_scale": 0.5, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in kinds],
+            "loop": {"start": 1, "stop": 3, "times": 2}}
+
+
 # 32-bit multiply-adds outside the tensor cores: 148 SMs x 128 lanes x 2 x 1.965 GHz (nominal), the compute ceiling of a
 # recurrence whose state and inputs are 32-bit
 FP32_TFLOPS = 74.4
@@ -136,6 +155,10 @@ FUNEVIK_SIZES = {
 VADERAX_SIZES = {
     "2048": (6, vaderax_shape(2048, 16, 4, 8192, 32, 4, 2048, 16), gqa_shape(6, 2048, 16, 5504)),
     "4096": (6, vaderax_shape(4096, 32, 8, 16384, 64, 4, 4096, 32), gqa_shape(6, 4096, 32, 10944)),
+}
+LOPILIX_SIZES = {
+    "2048": (6, lopilix_shape(2048, 16, 4, 5504, 32, 4, 2048), gqa_shape(6, 2048, 16, 5504)),
+    "4096": (6, lopilix_shape(4096, 32, 8, 10944, 64, 4, 4096), gqa_shape(6, 4096, 32, 10944)),
 }
 CACHED, PROMPT = 2048, 2048
 
@@ -189,9 +212,11 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
             else:
                 keys = min(keys_per_row, W + first)
                 rows_read = cache_rows * keys / keys_per_row
+        Gv = G // a.get("value_share", 1)
         proj = a["q_in"].shape[1] + (a["k_in"].shape[1] + a["v_in"].shape[1] if a["k_in"] is not None else 0)
-        return (f"window attention {H}/{G} heads of {dk}/{dv}, window {W}+{first}" + ("" if a["k_in"] is not None else ", reads another layer's keys"),
-                2.0 * T * H * keys * (dk + dv), rows_read * G * (dk + dv) * el + T * (proj + 2 * H * dk + H * dv) * el)
+        return (f"window attention {H}/{G} heads of {dk}/{dv}, window {W}+{first}" + ("" if a["k_in"] is not None else ", reads another layer's keys")
+                + (f", {Gv} value heads" if Gv != G else "") + (", difference" if a.get("heads") is not None else ""),
+                2.0 * T * H * keys * (dk + dv), rows_read * (G * dk + Gv * dv) * el + T * (proj + 2 * H * dk + (H // 2 if a.get("heads") is not None else H) * dv) * el)
     if k == "postnorm":
         D = a["x"].shape[1]
         return "norm of a sublayer's output + residual add", 0.0, T * D * (4 + 4 + 4 + el)
@@ -203,7 +228,7 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
         E, n, kk = w.shape
         used = E * (1.0 - (1.0 - top / E) ** T)                       # experts that some token of the step uses, in the mean
         n_out = n // 2 if a["act"] == "silu" else n
-        what = {"silu": "gate|up + silu", "relu2": "up + relu^2", None: "down"}[a["act"]]
+        what = {"silu": "gate|up + silu", "relu2": "up + relu^2", "gelu": "up + gelu", None: "down"}[a["act"]]
         if (E, top) in ROUTED_SHARE:                                  # identity experts take their share of the pairs
             top = top * ROUTED_SHARE[E, top]
             used = E * (1.0 - (1.0 - top / E) ** T)
@@ -214,6 +239,13 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
         return "weighted sum of the chosen experts", 0.0, T * D * (top * 4 + (4 if a["base"] is not None else 0) + 4)
     if k == "layernorm":
         return "layer norm" + (" + residual add" if a["delta"] is not None else ""), 0.0, T * a["x"].shape[1] * ((12 if a["delta"] is not None else 4) + el)
+    if k == "stream_norm":
+        S, D = a["streams"], a["x"].shape[1] // a["streams"]
+        update = a["y"] is not None
+        return (f"{S} streams" + (": update, read, norm" if update else ": read, norm"), 0.0,
+                T * D * (S * (8 if update else 4) + (4 + a["gate"].element_size() if update else 0) + el))
+    if k == "forget_gates":
+        return f"forget gates and queries, {a['q'].shape[1]} channels", 0.0, T * a["q"].shape[1] * 16
     if k == "embedding":
         return "embedding added again", 0.0, T * a["out"].shape[1] * (12 + el)
     if k == "rmsnorm":
@@ -240,7 +272,8 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
     if k == "recurrence":
         H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]
         return (f"recurrence {H} heads, state {n}x{p}" + (", decay per token" if a.get("dt") is not None else
-                                                          ", given gates" if a.get("keep") is not None else ", fixed decay"),
+                                                          ", given gates" if a.get("keep") is not None else
+                                                          ", a gate per row" if a.get("forget") else ", fixed decay"),
                 4.0 * T * H * n * p * FP32_SHARE, requests * 2 * H * n * p * 4 + T * (2 * G * n * 4 + H * p * (a["v"].element_size() + 4)))
     if k == "delta_rule":
         H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]
@@ -248,6 +281,8 @@ def record_cost(op, T: int, keys_per_row: float, cache_rows: float):
                 requests * 2 * H * n * p * 4 + T * (2 * G * n * 4 + 2 * H * p * 4 + 2 * H * 4))
     if k == "gated_norm":
         cols = a["y"].shape[1]
+        if a["gate"] is None:
+            return f"norm in groups of {a['group']}", 0.0, T * cols * (4 + el)
         return f"gate + norm in groups of {a['group']}" + (", normalised" if a.get("floor") is not None else ""), 0.0, T * cols * (4 + a["gate"].element_size() + el)
     return k, 0.0, 0.0
 
@@ -396,7 +431,7 @@ def run(args, pk) -> int:
     import torch
     design_name = getattr(args, "design", None) or "bepuzen"
     table_of_sizes = {"bepuzen": SIZES, "torisun": TORISUN_SIZES, "vifelix": VIFELIX_SIZES, "funevik": FUNEVIK_SIZES,
-                      "vaderax": VADERAX_SIZES}[design_name]
+                      "vaderax": VADERAX_SIZES, "lopilix": LOPILIX_SIZES}[design_name]
     global FP32_SHARE
     FP32_SHARE = pk["bf16_tflops"] / FP32_TFLOPS
     sizes = [args.size] if getattr(args, "size", None) else list(table_of_sizes)

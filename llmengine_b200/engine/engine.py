@@ -432,6 +432,6 @@ class Engine:
         status = status or (self.ops.grouped_tcgen05_status() if "moe_tcgen05" in libs else 0)
         for key in libs:
             if key.startswith("attention_tc@HEAD_DIM="):
-                status = status or self.ops.attention_tc_status(int(key.split("=")[1]))
+                status = status or int(libs[key].llme_attention_tc_status())
         if status:
             raise RuntimeError(f"a tcgen05 kernel gave up waiting (code {status}): its results are not valid")

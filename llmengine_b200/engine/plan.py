@@ -193,7 +193,8 @@ class Plan:
                          q, out, cache, group: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int,
                          window: int, keep_first: int, scale: float, sink=None, scratch=None, q_bias=None, k_bias=None,
                          v_bias=None, head_norm: bool = False, softcap: float = 0.0, interleaved: bool = False,
-                         unit_norm: bool = False, decode_scratch=None, value_share: int = 1) -> None:
+                         unit_norm: bool = False, decode_scratch=None, value_share: int = 1,
+                         difference: Optional[tuple] = None, heads=None, maps_scratch=None) -> None:
         """Grouped-query attention over a cache whose keys are `qk_dim` and whose values are `v_dim` wide, from the raw
         projections: q_in [T, H qk_dim] and, for a layer that stores, k_in [T, G qk_dim] and v_in [T, G v_dim] (column
         ranges of one product).  With gains, queries and keys are RMS-normed over the WHOLE projection (all heads at
@@ -212,12 +213,18 @@ class Plan:
         `decode_scratch`: scratch memory of the kernels of ordinary grouped-query attention, which serve the record where its
         mask and softmax are theirs (one width for keys and values, no kept first positions, no sink, no cap).
         `value_share` n: n neighbouring key heads attend to the same value head (v_in [T, G / n v_dim], a page holds G / n value
-        heads): the maps of a differential attention."""
+        heads): the maps of a differential attention.  `difference` (weight, scale, eps), with a value_share of two: the maps become
+        heads, u = a1 - weight a2, u / sqrt(mean(u^2) + eps) * scale per head, written to `heads` [T, H / 2 v_dim] head by head; `out`
+        [T, H v_dim] (per value head its query heads under map 1, then under map 2) is then the workspace of the form that runs
+        attention and difference apart, `maps_scratch` (32-bit) that of the form for single tokens."""
+        if (difference is None) != (heads is None) or (difference is not None and (value_share != 2 or window or keep_first or sink is not None or softcap)):
+            raise ValueError("window_attention: a difference is one of two plain causal maps, with a place for its heads")
         self._add("window_attention", q_bias=q_bias, k_bias=k_bias, v_bias=v_bias, head_norm=bool(head_norm), q_in=q_in, k_in=k_in, v_in=v_in, q_gain=q_gain, k_gain=k_gain, eps=float(eps),
                   inv_freq=inv_freq, rot_dims=int(rot_dims), amplitude=float(amplitude), q=q, out=out, cache=cache, group=group,
                   num_heads=num_heads, num_kv_heads=num_kv_heads, qk_dim=qk_dim, v_dim=v_dim, window=int(window),
                   keep_first=int(keep_first), scale=float(scale), sink=sink, scratch=scratch, softcap=float(softcap),
-                  interleaved=bool(interleaved), unit_norm=bool(unit_norm), decode_scratch=decode_scratch, value_share=int(value_share))
+                  interleaved=bool(interleaved), unit_norm=bool(unit_norm), decode_scratch=decode_scratch, value_share=int(value_share),
+                  difference=None if difference is None else tuple(float(v) for v in difference), heads=heads, maps_scratch=maps_scratch)
 
     def moe_route(self, *, logits, top_k: int, scale: float, experts, weights, offsets, order, counts,
                   mode: str = "sigmoid", correction=None, groups: tuple = (1, 1)) -> None:
@@ -329,12 +336,6 @@ class Plan:
         """What enters a memory with a forget gate per channel, all 32-bit: q = silu(q_in), f = lower + (1 - lower) sigmoid(f_in +
         f_bias), elementwise; q_in, f_in, q and f are [T, C] (any row stride), f_bias and lower [C]."""
         self._add("forget_gates", q_in=q_in, f_in=f_in, f_bias=f_bias, lower=lower, q=q, f=f)
-
-    def difference_norm(self, *, a, weight: float, scale: float, eps: float, heads: int, rep: int, out) -> None:
-        """The two maps of a differential attention become its heads.  `a` [T, 2 heads P] holds the maps' outputs group by group of
-        `rep` heads: the group's heads of map 1, then those of map 2.  Per head u = a1 - weight * a2, out = u / sqrt(mean(u^2) +
-        eps) * scale, [T, heads P] head by head; 32-bit arithmetic."""
-        self._add("difference_norm", a=a, weight=float(weight), scale=float(scale), eps=float(eps), heads=int(heads), rep=int(rep), out=out)
 
     def row_norm(self, *, x, gain, eps: float, out) -> None:
         """out = x / sqrt(mean(x^2) + eps) * gain over the rows of x [T, C]: a norm on (a column range of) a product, in

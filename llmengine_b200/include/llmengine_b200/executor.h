@@ -70,8 +70,7 @@ enum LlmeOpKind {
     LLME_OP_ATTENTION, LLME_OP_CALL, LLME_OP_LINEAR_ACT, LLME_OP_POINTWISE, LLME_OP_BATCHED_LINEAR, LLME_OP_RESIDUAL_ADD,
     LLME_OP_LATENT_ATTENTION, LLME_OP_TOKEN_SIDE, LLME_OP_POSTNORM, LLME_OP_WINDOW_ATTENTION, LLME_OP_MOE_ROUTE,
     LLME_OP_GROUPED_LINEAR, LLME_OP_MOE_COMBINE, LLME_OP_SHORT_CONV, LLME_OP_ROTATE, LLME_OP_RECURRENCE, LLME_OP_GATED_NORM,
-    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES, LLME_OP_LAYERNORM, LLME_OP_DELTA_RULE, LLME_OP_STREAM_NORM, LLME_OP_FORGET_GATES,
-    LLME_OP_DIFFERENCE_NORM
+    LLME_OP_ROW_NORM, LLME_OP_EXP_GATES, LLME_OP_LAYERNORM, LLME_OP_DELTA_RULE, LLME_OP_STREAM_NORM, LLME_OP_FORGET_GATES
 };
 
 enum { LLME_ACT_XIELU = 1, LLME_ACT_RELU2 = 2 };   /* 2: max(z, 0)^2 */
@@ -132,15 +131,6 @@ typedef struct LlmeForgetGatesOp {
     float* q; float* f; long long ldq, ldf;
     int cols;
 } LlmeForgetGatesOp;
-
-/* The maps of a differential attention become its heads: a [T, 2 heads dim] holds, per group of `rep` heads, the heads of map 1 and
- * then those of map 2; u = a1 - weight a2, out = u / sqrt(mean(u^2) + eps) * scale, [T, heads dim] head by head. */
-typedef struct LlmeDifferenceNormOp {
-    const void* a; long long lda;
-    void* out; long long ldo;
-    int dtype, heads, rep, dim;
-    float weight, scale, eps;
-} LlmeDifferenceNormOp;
 
 typedef struct LlmeLinearOp {
     const void* x; long long ldx; int x_dtype;
@@ -282,6 +272,10 @@ typedef struct LlmeWindowAttentionOp {
      * (dk = dv, keep_first 0, no sink, no cap); NULL: they do not */
     float* decode_scratch; long long decode_scratch_floats; long long cache_pages;
     int value_share;                                         /* n > 1: n neighbouring key heads share one value head (v_in and a page hold nkv / n) */
+    /* differential attention (heads given, value_share 2, plain causal masks): the two maps' outputs of a head become u = a1 - diff_weight a2,
+     * u / sqrt(mean(u^2) + diff_eps) * diff_scale, [T, nh / 2, dv]; `out` is then the workspace of the form that runs the two apart */
+    void* heads; float diff_weight, diff_scale, diff_eps;
+    float* maps_scratch; long long maps_scratch_floats;
 } LlmeWindowAttentionOp;
 
 /* Routing of a mixture of experts: s = sigmoid(logits), the top_k largest, w_e = scale * s_e / (sum of the chosen s + 1e-20);
@@ -416,7 +410,8 @@ void llme_executor_destroy(LlmeExecutor*);
  * key and value sizes "window_attention_tc/<dk>x<dv>", "moe_route", "grouped_linear", "grouped_linear_tc", "moe_combine";
  * "short_conv", "rotate", "recurrence", "gated_norm", "row_norm", "exp_gates", "sigmoid_mul_grouped", "residual_add_scaled",
  * "layernorm", "embedding_add", "relu2", "delta_step", "delta_portions", "grouped_tcgen05",
- * "grouped_tcgen05_supports"; "embedding_streams", "stream_norm", "forget_gates", "difference_norm". */
+ * "grouped_tcgen05_supports"; "embedding_streams", "stream_norm", "forget_gates", "difference_norm"; per pair
+ * of sizes "maps_decode/<dk>x<dv>", "maps_decode_scratch/<dk>x<dv>" and, for keys of 64 and values of 128, "attention_tc/64x128x2". */
 int llme_executor_register(LlmeExecutor*, const char* name, void* entry_point);
 /* Which implementation an operation takes.  Operations and their variants:
  *   "linear":            "auto" | "tcgen05" | "cublas" | "plain"   (bfloat16 products of 128 tokens or more / all)
@@ -513,7 +508,6 @@ public:
     int add(const LlmeDeltaRuleOp& r) { return add(LLME_OP_DELTA_RULE, &r, sizeof r); }
     int add(const LlmeStreamNormOp& r) { return add(LLME_OP_STREAM_NORM, &r, sizeof r); }
     int add(const LlmeForgetGatesOp& r) { return add(LLME_OP_FORGET_GATES, &r, sizeof r); }
-    int add(const LlmeDifferenceNormOp& r) { return add(LLME_OP_DIFFERENCE_NORM, &r, sizeof r); }
     /* One step through the whole plan; throws with the failing record's message. */
     void run(const LlmeStep& step, cudaStream_t stream) {
         if (llme_plan_run(h_, &step, 0, -1, stream)) throw std::runtime_error(ex_.error());

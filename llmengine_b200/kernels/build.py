@@ -36,6 +36,8 @@ SOURCES: Dict[str, str] = {
     "attention_window": "attention_window.cu",
     # the same on the tensor cores, per pair of sizes: "attention_window_tc@DK=64,DV=64"
     "attention_window_tc": "attention_window_tc.cu",
+    # differential attention of single tokens: two maps over the same values, per pair of sizes: "attention_maps@DK=64,DV=128"
+    "attention_maps": "attention_maps.cu",
     # mixture of experts: routing, the grouped product (plain form), the weighted sum; and the grouped product on tensor cores
     # layers with a state of fixed size per request: short convolution, linear recurrence, gated group norm
     "recurrent": "recurrent.cu",
@@ -58,7 +60,8 @@ SOURCES: Dict[str, str] = {
     "engine": "native/engine.cu",
     # compiled per head size: ask for "attention_fast@HEAD_DIM=128"
     "attention_fast": "attention_fast.cu",
-    # the tcgen05 portion kernel, per head size (64 or 128): "attention_tc@HEAD_DIM=128"
+    # the tcgen05 portion kernel, per head size (64 or 128): "attention_tc@HEAD_DIM=128"; its form for two maps over the same values:
+    # "attention_tc@HEAD_DIM=64,VALUE_DIM=128,MAPS=2"
     "attention_tc": "attention_tc.cu",
     # the same kernels with built-in scratch memory: "attention_decode_static@HEAD_DIM=128"
     "attention_decode_static": "attention_decode_static.cu",
@@ -71,7 +74,8 @@ INCLUDES: Dict[str, List[str]] = {"attention_decode_static": ["attention_fast.cu
 VARIANTS: Dict[str, List[str]] = {
     "attention_fast": ["attention_fast@HEAD_DIM=64", "attention_fast@HEAD_DIM=128"],
     "attention_decode_static": ["attention_decode_static@HEAD_DIM=128"],
-    "attention_tc": ["attention_tc@HEAD_DIM=64", "attention_tc@HEAD_DIM=128"],
+    "attention_tc": ["attention_tc@HEAD_DIM=64", "attention_tc@HEAD_DIM=128", "attention_tc@HEAD_DIM=64,VALUE_DIM=128,MAPS=2"],
+    "attention_maps": ["attention_maps@DK=64,DV=128"],
     "attention_latent_tc": ["attention_latent_tc@RANK=128", "attention_latent_tc@RANK=512"],
     "attention_window_tc": ["attention_window_tc@DK=64,DV=64", "attention_window_tc@DK=128,DV=128"],
 }

@@ -14,7 +14,7 @@ ROWS = {"tokens": 0, "logits": 1}
 (OP_EMBEDDING, OP_RMSNORM, OP_LINEAR, OP_LINEAR_SWIGLU, OP_QKV_POST, OP_ATTEND, OP_ATTENTION, OP_CALL, OP_LINEAR_ACT,
  OP_POINTWISE, OP_BATCHED_LINEAR, OP_RESIDUAL_ADD, OP_LATENT_ATTENTION, OP_TOKEN_SIDE, OP_POSTNORM, OP_WINDOW_ATTENTION,
  OP_MOE_ROUTE, OP_GROUPED_LINEAR, OP_MOE_COMBINE, OP_SHORT_CONV, OP_ROTATE, OP_RECURRENCE, OP_GATED_NORM, OP_ROW_NORM,
- OP_EXP_GATES, OP_LAYERNORM, OP_DELTA_RULE, OP_STREAM_NORM, OP_FORGET_GATES, OP_DIFFERENCE_NORM) = range(1, 31)
+ OP_EXP_GATES, OP_LAYERNORM, OP_DELTA_RULE, OP_STREAM_NORM, OP_FORGET_GATES) = range(1, 30)
 GATES = {"silu": 0, "clamped_swish": 1, "gelu_tanh": 2}
 ROUTING = {"sigmoid": 0, "softmax_chosen": 1, "softmax": 2}
 ACTIVATIONS = {"xielu": 1, "relu2": 2}
@@ -68,11 +68,6 @@ class StreamNormOp(Structure):
 class ForgetGatesOp(Structure):
     _fields_ = [("q_in", c_void_p), ("f_in", c_void_p), ("ld_in", c_longlong), ("f_bias", c_void_p), ("lower", c_void_p), ("q", c_void_p),
                 ("f", c_void_p), ("ldq", c_longlong), ("ldf", c_longlong), ("cols", c_int)]
-
-
-class DifferenceNormOp(Structure):
-    _fields_ = [("a", c_void_p), ("lda", c_longlong), ("out", c_void_p), ("ldo", c_longlong), ("dtype", c_int), ("heads", c_int),
-                ("rep", c_int), ("dim", c_int), ("weight", c_float), ("scale", c_float), ("eps", c_float)]
 
 
 class LayerNormOp(Structure):
@@ -170,7 +165,8 @@ class WindowAttentionOp(Structure):
                 ("scratch_floats", c_longlong), ("q_bias", c_void_p), ("k_bias", c_void_p), ("v_bias", c_void_p),
                 ("head_norm", c_int), ("softcap", c_float), ("interleaved", c_int), ("in_f32", c_int), ("unit_norm", c_int),
                 ("decode_scratch", c_void_p), ("decode_scratch_floats", c_longlong), ("cache_pages", c_longlong),
-                ("value_share", c_int)]
+                ("value_share", c_int), ("heads", c_void_p), ("diff_weight", c_float), ("diff_scale", c_float), ("diff_eps", c_float),
+                ("maps_scratch", c_void_p), ("maps_scratch_floats", c_longlong)]
 
 
 class MoeRouteOp(Structure):
@@ -437,6 +433,8 @@ def records(op, keep: List[Any]):
         assert cache.is_contiguous() and qi.shape[1] == q.shape[1] == H * dk and out.shape[1] == H * dv
         share = int(a.get("value_share", 1))
         Gv = G // share                                                     # value heads
+        heads = a.get("heads")
+        assert heads is None or (share == 2 and heads.dtype == out.dtype and heads.is_contiguous() and heads.shape[1] * 2 == out.shape[1])
         assert G % share == 0 and cache.shape[1] % (G * dk + Gv * dv) == 0
         assert (ki is None) == (vi is None) and (ki is None or (ki.dtype == vi.dtype == qi.dtype and ki.stride(1) == vi.stride(1) == 1
                                                               and ki.shape[1] == G * dk and vi.shape[1] == Gv * dv))
@@ -452,7 +450,8 @@ def records(op, keep: List[Any]):
             ptr(a.get("q_bias")), ptr(a.get("k_bias")), ptr(a.get("v_bias")), 1 if a.get("head_norm") else 0,
             float(a.get("softcap", 0.0)), 1 if a.get("interleaved") else 0, 1 if wide else 0, 1 if a.get("unit_norm") else 0,
             ptr(a.get("decode_scratch")), a["decode_scratch"].numel() if a.get("decode_scratch") is not None else 0, cache.shape[0],
-            share)
+            share, ptr(heads), *(a.get("difference") or (0.0, 0.0, 0.0)), ptr(a.get("maps_scratch")),
+            a["maps_scratch"].numel() if a.get("maps_scratch") is not None else 0)
     if k == "moe_route":
         z, ex_, wt, off, order, counts = a["logits"], a["experts"], a["weights"], a["offsets"], a["order"], a["counts"]
         assert z.dtype == wt.dtype == torch.float32 and z.stride(1) == 1 and ex_.is_contiguous() and wt.is_contiguous()
@@ -556,11 +555,6 @@ def records(op, keep: List[Any]):
         assert qi.stride(0) == fi.stride(0) and _f32(a["f_bias"], q.shape[1]) and _f32(a["lower"], q.shape[1])
         return OP_FORGET_GATES, ForgetGatesOp(qi.data_ptr(), fi.data_ptr(), qi.stride(0), a["f_bias"].data_ptr(), a["lower"].data_ptr(),
                                               q.data_ptr(), f.data_ptr(), q.stride(0), f.stride(0), q.shape[1])
-    if k == "difference_norm":
-        m, out, H, rep = a["a"], a["out"], a["heads"], a["rep"]
-        assert m.dtype == out.dtype and m.stride(1) == out.stride(1) == 1 and m.shape[1] == 2 * out.shape[1] and out.shape[1] % H == 0 and H % rep == 0
-        return OP_DIFFERENCE_NORM, DifferenceNormOp(m.data_ptr(), m.stride(0), out.data_ptr(), out.stride(0), code(out.dtype), H, rep,
-                                                    out.shape[1] // H, a["weight"], a["scale"], a["eps"])
     if k == "delta_rule":
         q, kk, v, wr, fg, st, out, unit, coef = (a[n] for n in ("q", "k", "v", "write", "forget", "state", "out", "unit", "coef"))
         H, n, p, G = a["heads"], a["n"], a["p"], a["qk_groups"]

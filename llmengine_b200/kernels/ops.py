@@ -91,7 +91,7 @@ class _TcAttnArgs(Structure):
         ("out", c_void_p), ("cache", c_void_p), ("rows", c_void_p), ("cu_q_lens", c_void_p), ("ctx_lens", c_void_p),
         ("table_rows", c_void_p), ("block_tables", c_void_p),
         ("max_blocks", c_int), ("n_rows", c_int), ("nh", c_int), ("nkv", c_int), ("page_size", c_int),
-        ("window", c_int), ("scale", c_float),
+        ("window", c_int), ("scale", c_float), ("diff_weight", c_float), ("diff_scale", c_float), ("diff_eps", c_float),
     ]
 
 
@@ -207,6 +207,7 @@ class CudaOps:
                       "gated_norm": "llme_gated_norm", "exp_gates": "llme_exp_gates", "forget_gates": "llme_forget_gates"},
         "delta_rule": {"delta_step": "llme_delta_step", "delta_portions": "llme_delta_portions"},
         "attention_window": {"window_post": "llme_window_post", "window_attention_plain": "llme_window_attention_plain"},
+        "attention_maps": {"maps_decode/{hd}": "llme_maps_decode", "maps_decode_scratch/{hd}": "llme_maps_decode_scratch_floats"},
         "attention_window_tc": {"window_attention_tc/{hd}": "llme_window_attention_tc"},
         "moe": {"moe_route": "llme_moe_route", "grouped_linear": "llme_grouped_linear", "moe_combine": "llme_moe_combine"},
         "moe_tcgen05": {"grouped_tcgen05": "llme_grouped_tcgen05", "grouped_tcgen05_supports": "llme_grouped_tcgen05_supports"},
@@ -249,7 +250,7 @@ class CudaOps:
             a = op.a
             if op.kind in ("embedding", "rmsnorm", "layernorm", "qkv_post", "attention"):
                 want("elementwise")
-            if op.kind in ("linear_act", "pointwise", "residual_add", "latent_attention", "token_side", "postnorm", "row_norm", "difference_norm"):
+            if op.kind in ("linear_act", "pointwise", "residual_add", "latent_attention", "token_side", "postnorm", "row_norm"):
                 want("pointwise")
             if op.kind == "stream_norm":
                 want("streams")
@@ -263,6 +264,12 @@ class CudaOps:
                 want("delta_rule")
             if op.kind == "window_attention":
                 want("attention_window")
+                if a.get("heads") is not None:
+                    want("pointwise")                                                   # (the difference as a step of its own)
+                    if fast_attention and self.window_tc_supports(a["qk_dim"], a["v_dim"], a["q"].dtype):
+                        want(f"attention_maps@DK={a['qk_dim']},DV={a['v_dim']}")
+                        if (a["qk_dim"], a["v_dim"]) == (64, 128) and self.chosen("attention.portion") == "tcgen05":
+                            want("attention_tc@HEAD_DIM=64,VALUE_DIM=128,MAPS=2")
                 if fast_attention and a.get("decode_scratch") is not None and self.fast_attention_supports(a["qk_dim"], a["q"].dtype):
                     want(f"attention_fast@HEAD_DIM={a['qk_dim']}")       # ordinary attention: the grouped-query kernels
                     if a["qk_dim"] in (64, 128) and self.chosen("attention.portion") == "tcgen05":

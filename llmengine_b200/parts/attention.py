@@ -419,6 +419,7 @@ class DifferenceAttention(Part):
         plan.linear(h, self.w_in, proj)
         q = rt.workspace("q", qs, rt.dtype)
         maps = rt.workspace("attn_maps", self.MAPS * self.o_size, rt.dtype)
+        heads = rt.workspace("attn_out", self.o_size, rt.dtype)
         pos, H, G = self.position, self.MAPS * self.nh, self.MAPS * self.nkv
         plan.window_attention(
             q_in=proj[:, :qs], k_in=proj[:, qs:qs + ks], v_in=proj[:, qs + ks:], q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps,
@@ -427,9 +428,8 @@ class DifferenceAttention(Part):
             qk_dim=self.dk, v_dim=self.dv, window=0, keep_first=0, scale=self.scale, head_norm=True, value_share=self.MAPS,
             interleaved=bool(pos is not None and pos.interleaved),
             scratch=(rt.buffer("window_attention_scratch", 1, rt.max_requests * H * 8 * (self.dv + 2), torch.float32, exact=True).view(-1)
-                     if rt.dtype == torch.bfloat16 else None))
-        heads = rt.workspace("attn_out", self.o_size, rt.dtype)
-        plan.difference_norm(a=maps, weight=self.weight, scale=1.0 - self.diff, eps=self.eps, heads=self.nh, rep=self.rep, out=heads)
+                     if rt.dtype == torch.bfloat16 else None),
+            difference=(self.weight, 1.0 - self.diff, self.eps), heads=heads, maps_scratch=rt.maps_scratch(self.nh, self.nkv, self.dv))
         delta = rt.workspace("mixer_out", self.hidden, torch.float32)
         plan.linear(heads, self.w_o, delta)
         return delta

@@ -298,6 +298,16 @@ class Runtime:
         self._latent_scratch_floats = max(getattr(self, "_latent_scratch_floats", 0), n)
         return self.buffer("latent_scratch", 1, self._latent_scratch_floats, torch.float32, exact=True).view(-1)
 
+    def maps_scratch(self, heads: int, groups: int, v_dim: int) -> Optional[torch.Tensor]:
+        """Scratch memory of the differential attention of single tokens whose keys are cut into shares (one buffer for all layers): a
+        maximum, a sum and an output row for each of 16 rows per (request, value head, eight query heads, share); as many shares as
+        three blocks an SM take, or one where the requests alone are more."""
+        if self.dtype != torch.bfloat16 or self.device.type != "cuda":
+            return None
+        units = self.max_requests * groups * ((heads // groups + 7) // 8)
+        self._maps_scratch_floats = max(getattr(self, "_maps_scratch_floats", 0), max(512, units) * 16 * (v_dim + 2))
+        return self.buffer("maps_scratch", 1, self._maps_scratch_floats, torch.float32, exact=True).view(-1)
+
     def rows(self, t: Optional[torch.Tensor], n: Optional[int] = None) -> Optional[torch.Tensor]:
         """The first rows of a workspace buffer: those of the running step's tokens (or `n` of them)."""
         if t is None:

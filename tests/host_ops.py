@@ -262,13 +262,6 @@ class HostOps:
         a["q"][:T] = z * torch.sigmoid(z)
         a["f"][:T] = a["lower"] + (1.0 - a["lower"]) * torch.sigmoid(a["f_in"][:T] + a["f_bias"])
 
-    def difference_norm(self, a, T):
-        H, rep = a["heads"], a["rep"]
-        m = a["a"][:T].float().view(T, H // rep, 2, rep, -1)
-        u = (m[:, :, 0] - a["weight"] * m[:, :, 1]).reshape(T, H, -1)
-        u = u / torch.sqrt((u * u).mean(-1, keepdim=True) + a["eps"]) * a["scale"]
-        a["out"][:T] = u.reshape(T, -1).to(a["out"].dtype)
-
     def row_norm(self, a, T):
         x = a["x"][:T].float()
         a["out"][:T] = (x * (1.0 / torch.sqrt((x * x).mean(-1, keepdim=True) + a["eps"])) * a["gain"].float()).to(a["out"].dtype)
@@ -408,6 +401,11 @@ class HostOps:
                     s = torch.cat([s, a["sink"][h:h + 1]])
                 w = torch.softmax(s, 0)[: js.numel()]
                 a["out"][t, h * dv:(h + 1) * dv] = (w @ vv[:, h // rep // share]).to(a["out"].dtype)
+        if a.get("heads") is not None:
+            weight, scale, eps = a["difference"]
+            m = a["out"][:T].float().view(T, G // 2, 2, rep, dv)
+            u = m[:, :, 0] - weight * m[:, :, 1]
+            a["heads"][:T] = (u / torch.sqrt((u * u).mean(-1, keepdim=True) + eps) * scale).reshape(T, -1).to(a["heads"].dtype)
 
     def moe_route(self, a, T):
         top, E = a["top_k"], a["logits"].shape[1]
@@ -532,8 +530,6 @@ class HostPlan:
                 o.stream_norm(a, T, batch.logit_rows if a["rows"] == "logits" else None)
             elif k == "forget_gates":
                 o.forget_gates(a, T)
-            elif k == "difference_norm":
-                o.difference_norm(a, T)
             elif k == "exp_gates":
                 o.exp_gates(a, batch)
             elif k == "linear_swiglu":
