@@ -24,7 +24,7 @@ LLME_API const char* llme_last_error() { return llme_error_buffer(); }
 namespace {
 
 typedef __nv_bfloat16 bf16;
-constexpr int THREADS = 128, WARPS = THREADS / 32, SUB = 16, HEADS = 8, STAGES = 2;
+constexpr int THREADS = 128, WARPS = THREADS / 32, SUB = 16, HEADS = 8, STAGES = 3;
 constexpr int LDK = DK + 8, LDV = DV + 8;                      // rows apart from one another's banks
 constexpr int STAGE_ELEMS = SUB * (2 * LDK + LDV);
 constexpr int PART = DV + 2;                                   // a row's part: maximum (base 2), sum, outputs
@@ -56,6 +56,24 @@ __device__ __forceinline__ unsigned pack_bf16(float a, float b) {
     return *reinterpret_cast<const unsigned*>(&v);
 }
 
+// Sixteen rows of N values, one behind the other in a page: every lane's addresses are a constant apart.
+template <int N, int LD>
+__device__ __forceinline__ void load_rows(bf16* dst, const bf16* src, int lane) {
+    constexpr int C = N / 8, PASSES = (SUB * C + 31) / 32;
+    if (32 % C == 0) {
+        dst += (lane / C) * LD + (lane % C) * 8;
+        src += (lane / C) * N + (lane % C) * 8;
+#pragma unroll
+        for (int i = 0; i < PASSES; ++i) cp_async16(dst + i * (32 / C) * LD, src + i * (32 / C) * N, true);
+    } else {
+#pragma unroll
+        for (int i = 0; i < PASSES; ++i) {
+            const int idx = lane + 32 * i;
+            if (SUB * C % 32 == 0 || idx < SUB * C) cp_async16(dst + (idx / C) * LD + (idx % C) * 8, src + idx * 8, true);
+        }
+    }
+}
+
 // grid (splits, value heads * chunks of eight query heads, requests)
 __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs a) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -72,61 +90,36 @@ __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs
     const bool one_page = ps % SUB == 0;                       // a sub-tile then lies in one page
     const int ps_shift = (ps & (ps - 1)) == 0 ? __ffs(ps) - 1 : -1;
 
-    auto load = [&](int sub, int stage) {
+    auto block_of = [&](int j) { return ps_shift >= 0 ? j >> ps_shift : j / ps; };
+    // The page of a warp's sub-tile, looked up one sub-tile before its keys are asked for: the look-up's latency is then not in
+    // front of theirs.
+    auto page_of = [&](int sub) -> int { return one_page && sub < last ? bt[block_of(sub * SUB)] : 0; };
+    const size_t k1_at = (size_t)2 * g * ps * DK, k2_at = k1_at + (size_t)ps * DK, v_at = (size_t)2 * a.groups * ps * DK + (size_t)g * ps * DV;
+    auto load = [&](int sub, int stage, int page) {
         bf16* dst = stages + (size_t)stage * STAGE_ELEMS;
         const int j0 = sub * SUB;
-        constexpr int KC = DK / 8, VC = DV / 8, CH = 2 * KC + VC;
-        size_t page_at = 0;
-        int off0 = 0;
-        if (one_page) {
-            const int blk = ps_shift >= 0 ? j0 >> ps_shift : j0 / ps;
-            page_at = (size_t)bt[blk] * page_elems;
-            off0 = j0 - blk * ps;
+        if (one_page && j0 + SUB <= ctx) {                     // the usual case: sixteen rows of one page, addresses a constant apart
+            const bf16* at = cache + (size_t)page * page_elems;
+            const int off = j0 - block_of(j0) * ps;
+            load_rows<DK, LDK>(dst, at + k1_at + (size_t)off * DK, lane);
+            load_rows<DK, LDK>(dst + SUB * LDK, at + k2_at + (size_t)off * DK, lane);
+            load_rows<DV, LDV>(dst + 2 * SUB * LDK, at + v_at + (size_t)off * DV, lane);
+            return;
         }
-#pragma unroll
-        for (int i = lane; i < SUB * CH; i += 32) {
-            const int r = i / CH, c = i - r * CH, j = j0 + r;
+#pragma unroll 1
+        for (int r = 0; r < SUB; ++r) {                        // row by row; rows behind the last key become zeros
+            const int j = j0 + r;
             const bool ok = j < ctx;
-            size_t at = page_at;
-            int off = off0 + r;
-            if (!one_page && ok) {
-                const int blk = ps_shift >= 0 ? j >> ps_shift : j / ps;
-                at = (size_t)bt[blk] * page_elems;
-                off = j - blk * ps;
-            }
-            const bf16* src;
-            bf16* to;
-            if (c < 2 * KC) {
-                const int m = c / KC, cc = c - m * KC;
-                src = cache + at + ((size_t)(2 * g + m) * ps + off) * DK + cc * 8;
-                to = dst + (size_t)m * SUB * LDK + r * LDK + cc * 8;
-            } else {
-                const int cc = c - 2 * KC;
-                src = cache + at + (size_t)2 * a.groups * ps * DK + ((size_t)g * ps + off) * DV + cc * 8;
-                to = dst + (size_t)2 * SUB * LDK + r * LDV + cc * 8;
-            }
-            cp_async16(to, ok ? src : cache, ok);
+            const int blk = ok ? block_of(j) : 0;
+            const bf16* at = cache + (ok ? (size_t)bt[blk] * page_elems : 0);
+            const size_t off = ok ? j - blk * ps : 0;
+            if (lane < DK / 8) cp_async16(dst + r * LDK + lane * 8, at + (ok ? k1_at + off * DK : 0) + lane * 8, ok);
+            if (lane < DK / 8) cp_async16(dst + (SUB + r) * LDK + lane * 8, at + (ok ? k2_at + off * DK : 0) + lane * 8, ok);
+            if (lane < DV / 8) cp_async16(dst + 2 * SUB * LDK + r * LDV + lane * 8, at + (ok ? v_at + off * DV : 0) + lane * 8, ok);
         }
     };
-    // Keys that earlier steps stored may be on their way before the kernel before this one (it stores the newest key and finishes
-    // the queries) is done.
-    const bool early = first < last && (first + 1) * SUB < ctx;
-    if (early) load(first, 0);
-    pdl_wait();
-    if (first < last && !early) load(first, 0);
-    cp_async_commit();
 
     unsigned qf[DK / 16][4];                                   // rows: map 1's heads, then map 2's
-    {
-        const bf16* q = (const bf16*)a.q + ((size_t)a.cu_q_lens[req] * a.heads * 2 + (size_t)2 * g * rep) * DK;
-        const int h = h0 + (lane >> 2);
-        const bool ok = h < rep;
-#pragma unroll
-        for (int k = 0; k < DK / 16; ++k)
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                qf[k][e] = ok ? *reinterpret_cast<const unsigned*>(q + ((size_t)(e & 1) * rep + h) * DK + k * 16 + (e >> 1) * 8 + (lane & 3) * 2) : 0u;
-    }
     const float sc = a.scale * LOG2E;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f}, o[DV / 8][4];
 #pragma unroll
@@ -134,11 +127,34 @@ __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[n][e] = 0.0f;
 
-    int stage = 0;
-    for (int sub = first; sub < last; sub += WARPS, stage ^= 1) {
-        if (sub + WARPS < last) load(sub + WARPS, stage ^ 1);
+    // Two sub-tiles are on their way while one is worked on.  Keys that earlier steps stored are asked for before the kernel before
+    // this one (it stores the newest key and finishes the queries) is done.
+    int stage = 0, fill = 0, page = page_of(first);
+    bool waited = false;
+#pragma unroll 1
+    for (int it = 0;; ++it) {
+        const int ahead = first + it * WARPS, sub = ahead - 2 * WARPS;
+        if (!waited && (it == 2 || (ahead + 1) * SUB >= ctx)) {
+            pdl_wait();
+            waited = true;
+        }
+        if (ahead < last) load(ahead, fill, page);
         cp_async_commit();
-        cp_async_wait<1>();
+        fill = fill == STAGES - 1 ? 0 : fill + 1;
+        page = page_of(ahead + WARPS);
+        if (it < 2) continue;
+        if (it == 2) {
+            const bf16* q = (const bf16*)a.q + ((size_t)a.cu_q_lens[req] * a.heads * 2 + (size_t)2 * g * rep) * DK;
+            const int h = h0 + (lane >> 2);
+            const bool ok = h < rep;
+#pragma unroll
+            for (int k = 0; k < DK / 16; ++k)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    qf[k][e] = ok ? *reinterpret_cast<const unsigned*>(q + ((size_t)(e & 1) * rep + h) * DK + k * 16 + (e >> 1) * 8 + (lane & 3) * 2) : 0u;
+        }
+        if (sub >= last) break;
+        cp_async_wait<2>();
         __syncwarp();
         const bf16* K = stages + (size_t)stage * STAGE_ELEMS;
         const bf16* V = K + 2 * SUB * LDK;
@@ -179,10 +195,12 @@ __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs
             }
 #pragma unroll
         for (int h = 0; h < 2; ++h) l[h] = l[h] * corr[h] + sum[h];      // (this lane's share; the lanes are added up at the end)
+        if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f)) {      // (a maximum moves in the first few sub-tiles, hardly ever later)
 #pragma unroll
-        for (int n = 0; n < DV / 8; ++n) {
-            o[n][0] *= corr[0]; o[n][1] *= corr[0];
-            o[n][2] *= corr[1]; o[n][3] *= corr[1];
+            for (int n = 0; n < DV / 8; ++n) {
+                o[n][0] *= corr[0]; o[n][1] *= corr[0];
+                o[n][2] *= corr[1]; o[n][3] *= corr[1];
+            }
         }
         const unsigned pf[4] = {pack_bf16(p[0][0], p[0][1]), pack_bf16(p[0][2], p[0][3]), pack_bf16(p[1][0], p[1][1]), pack_bf16(p[1][2], p[1][3])};
 #pragma unroll
@@ -193,6 +211,7 @@ __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs
             mma_bf16(o[n + 1], pf, b2, b3);
         }
         __syncwarp();                                          // every lane is done with the stage before it is filled again
+        stage = stage == STAGES - 1 ? 0 : stage + 1;
     }
     cp_async_wait<0>();
     __syncthreads();
@@ -243,47 +262,49 @@ __global__ void __launch_bounds__(THREADS) maps_decode_kernel(LlmeMapsDecodeArgs
     }
 }
 
-// One warp per (request, head): the shares of both maps are added up, then the difference and its norm.
+// One block per (request, head): its warps deal the shares of both maps among themselves; then the difference and its norm.
 __global__ void __launch_bounds__(THREADS) maps_finish_kernel(LlmeMapsDecodeArgs a) {
+    __shared__ float sums[WARPS][DV], red[32];
     pdl_launch_dependents();
     pdl_wait();
-    const int lane = threadIdx.x & 31, h = blockIdx.x * WARPS + (threadIdx.x >> 5);
-    if (h >= a.heads) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, h = blockIdx.x;
     const int req = a.rows[blockIdx.y], rep = a.heads / a.groups, chunks = (rep + HEADS - 1) / HEADS;
     const int g = h / rep, hh = h - g * rep, unit = g * chunks + hh / HEADS;
     const float* parts = a.scratch + ((size_t)blockIdx.y * a.groups * chunks + unit) * a.splits * 16 * PART + (size_t)(hh % HEADS) * PART;
     constexpr int R = (DV + 31) / 32;
-    float u[R];
+    float f[2], u[R];
+#pragma unroll
+    for (int mp = 0; mp < 2; ++mp) {                           // lane s looks after share s
+        const float* mine = parts + (size_t)lane * 16 * PART + (size_t)mp * 8 * PART;
+        const bool in = lane < a.splits;
+        const float ms = in ? mine[0] : -INFINITY, ls = in ? mine[1] : 0.0f;
+        const float top = warp_max(ms), w = in ? exp2f(ms - top) : 0.0f;
+        f[mp] = (mp == 0 ? 1.0f : -a.diff_weight) / warp_sum(ls * w) * w;
+    }
 #pragma unroll
     for (int i = 0; i < R; ++i) u[i] = 0.0f;
-#pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-        const float* mine = parts + (size_t)mp * 8 * PART;
-        const bool in = lane < a.splits;                       // lane s looks after share s
-        const float ms = in ? mine[(size_t)lane * 16 * PART] : -INFINITY;
-        const float top = warp_max(ms), w = in ? exp2f(ms - top) : 0.0f;
-        const float sum = warp_sum(in ? mine[(size_t)lane * 16 * PART + 1] * w : 0.0f);
-        const float f = (mp == 0 ? 1.0f : -a.diff_weight) / sum * w;
 #pragma unroll 4
-        for (int s = 0; s < a.splits; ++s) {
-            const float fs = __shfl_sync(0xffffffffu, f, s);
+    for (int s = warp; s < a.splits; s += WARPS) {
+        const float f1 = __shfl_sync(0xffffffffu, f[0], s), f2 = __shfl_sync(0xffffffffu, f[1], s);
+        const float* mine = parts + (size_t)s * 16 * PART + 2;
 #pragma unroll
-            for (int i = 0; i < R; ++i) {
-                const int d = lane + 32 * i;
-                if (d < DV) u[i] = fmaf(fs, mine[(size_t)s * 16 * PART + 2 + d], u[i]);
-            }
+        for (int i = 0; i < R; ++i) {
+            const int d = lane + 32 * i;
+            if (d < DV) u[i] = fmaf(f2, mine[8 * PART + d], fmaf(f1, mine[d], u[i]));
         }
     }
-    float ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < R; ++i) ss = fmaf(u[i], u[i], ss);
-    const float r = a.diff_scale / sqrtf(warp_sum(ss) / (float)DV + a.diff_eps);
-    bf16* out = (bf16*)a.out + ((size_t)a.cu_q_lens[req] * a.heads + h) * DV;
+    for (int i = 0; i < R; ++i)
+        if (lane + 32 * i < DV) sums[warp][lane + 32 * i] = u[i];
+    __syncthreads();
+    const int d = threadIdx.x;                                 // (DV is at most the block's width)
+    float v = 0.0f;
+    if (d < DV) {
 #pragma unroll
-    for (int i = 0; i < R; ++i) {
-        const int d = lane + 32 * i;
-        if (d < DV) out[d] = __float2bfloat16_rn(u[i] * r);
+        for (int w = 0; w < WARPS; ++w) v += sums[w][d];
     }
+    const float r = a.diff_scale / sqrtf(block_sum(v * v, red) / (float)DV + a.diff_eps);
+    if (d < DV) ((bf16*)a.out)[((size_t)a.cu_q_lens[req] * a.heads + h) * DV + d] = __float2bfloat16_rn(v * r);
 }
 
 }  // namespace
@@ -316,6 +337,6 @@ LLME_API int llme_maps_decode(const LlmeMapsDecodeArgs* args, cudaStream_t strea
         snprintf(llme_error_buffer(), 512, "%s", cudaGetErrorString(e));
         return (int)e;
     }
-    llme_launch(maps_finish_kernel, dim3((a.heads + WARPS - 1) / WARPS, a.n_rows), dim3(THREADS), 0, stream, a);
+    llme_launch(maps_finish_kernel, dim3(a.heads, a.n_rows), dim3(THREADS), 0, stream, a);
     LLME_LAUNCH_STATUS();
 }

@@ -733,14 +733,18 @@ int difference_attention(LlmeExecutor& ex, const LlmeWindowAttentionOp& o, const
     long long splits = 1;
     if (s.num_decode > 0) {
         if (!decode || !need || !o.maps_scratch) return 0;
-        // shares: three blocks an SM, no share shorter than two sub-tiles of 16 keys a warp, at most 32
+        // Shares, by what the time is made of: rounds of two blocks an SM, each as long as the sub-tiles of 16 keys a warp walks and
+        // the time of about five beside them, and a little for every share that is added up afterwards (8 requests of 4 / 8 value
+        // heads at 2,048 keys: 9 / 4 shares; 64 requests: one).
         const long long units = need(s.num_decode, o.nh / 2, groups, 1) / (16 * (o.dv + 2)), subs = (s.max_decode_ctx + 15) / 16;
-        splits = 3LL * ex.sms / (units > 0 ? units : 1);
-        if (splits > subs / 8) splits = subs / 8;
-        if (splits > 32) splits = 32;
-        if (splits < 1) splits = 1;
-        while (splits > 1 && need(s.num_decode, o.nh / 2, groups, (int)splits) > o.maps_scratch_floats) --splits;
-        if (need(s.num_decode, o.nh / 2, groups, (int)splits) > o.maps_scratch_floats) return 0;
+        long long best = -1;
+        for (long long n = 1; n <= 32 && n <= subs; ++n) {
+            if (need(s.num_decode, o.nh / 2, groups, (int)n) > o.maps_scratch_floats) break;
+            const long long rounds = (units * n + 2LL * ex.sms - 1) / (2LL * ex.sms), walk = ((subs + n - 1) / n + 3) / 4;
+            const long long cost = 8 * rounds * (walk + 5) + n;
+            if (best < 0 || cost < best) { best = cost; splits = n; }
+        }
+        if (best < 0) return 0;                                 // no room for the parts
     }
     if (s.num_portion > 0) {
         LlmeTcAttnArgs a = {o.heads, o.cache, s.portion_rows, s.cu_q_lens, s.ctx_lens, s.state_slots, g.block_tables, g.max_blocks, s.num_portion, o.nh,

@@ -301,7 +301,7 @@ class Runtime:
     def maps_scratch(self, heads: int, groups: int, v_dim: int) -> Optional[torch.Tensor]:
         """Scratch memory of the differential attention of single tokens whose keys are cut into shares (one buffer for all layers): a
         maximum, a sum and an output row for each of 16 rows per (request, value head, eight query heads, share); as many shares as
-        three blocks an SM take, or one where the requests alone are more."""
+        the GPU's SMs take blocks, or one where the requests alone are more."""
         if self.dtype != torch.bfloat16 or self.device.type != "cuda":
             return None
         units = self.max_requests * groups * ((heads // groups + 7) // 8)
