@@ -376,6 +376,7 @@ class DifferenceAttention(Part):
     order [group, map, head of the group] when the weights are loaded; lambda is formed once in 32-bit and travels as a constant."""
 
     MAPS = 2
+    carries_rows = True
 
     def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, num_kv_heads: int, qk_dim: int, v_dim: int, scale: float,
                  diff: float, norm_eps: float, position_encoding: Optional[PartSpec] = None):
@@ -392,6 +393,7 @@ class DifferenceAttention(Part):
         self.o_size = self.nh * self.dv
         self.w_in = self.w_o = self.q_gain = self.k_gain = None
         self.weight = 0.0                                     # lambda
+        self.carried_at: Optional[int] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         v = lambda init: WeightSpec((self.dk,), role="vector", init=init)
@@ -406,7 +408,11 @@ class DifferenceAttention(Part):
         self.w_o = t[self.name("o")].contiguous()
         self.q_gain, self.k_gain = t[self.name("q.norm")].float().contiguous(), t[self.name("k.norm")].float().contiguous()
         l = {n: t[self.name(n)].detach().to("cpu", torch.float32) for n in ("lq1", "lk1", "lq2", "lk2")}
+        self.carried_at = None
         self.weight = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum()) + torch.tensor(self.diff, dtype=torch.float32))
+
+    def carry_rows(self, rows: torch.Tensor) -> None:
+        self.w_in, self.carried_at = self.with_carried_rows(self.w_in, rows)
 
     def cache_spec(self) -> SplitKVSpec:
         return SplitKVSpec(self.MAPS * self.nkv, self.dk, self.dv, value_share=self.MAPS)
@@ -417,12 +423,13 @@ class DifferenceAttention(Part):
             raise ValueError(f"{self.prefix}: this mixer keeps a cache of its own")
         proj = rt.workspace("qkv", self.w_in.shape[0], rt.dtype)
         plan.linear(h, self.w_in, proj)
+        self.carried = proj[:, self.carried_at:] if self.carried_at is not None else None
         q = rt.workspace("q", qs, rt.dtype)
         maps = rt.workspace("attn_maps", self.MAPS * self.o_size, rt.dtype)
         heads = rt.workspace("attn_out", self.o_size, rt.dtype)
         pos, H, G = self.position, self.MAPS * self.nh, self.MAPS * self.nkv
         plan.window_attention(
-            q_in=proj[:, :qs], k_in=proj[:, qs:qs + ks], v_in=proj[:, qs + ks:], q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps,
+            q_in=proj[:, :qs], k_in=proj[:, qs:qs + ks], v_in=proj[:, qs + ks:qs + ks + self.v_size], q_gain=self.q_gain, k_gain=self.k_gain, eps=self.eps,
             inv_freq=pos.frequencies() if pos is not None else None, rot_dims=pos.dims if pos is not None else 0,
             amplitude=pos.amplitude if pos is not None else 1.0, q=q, out=maps, cache=cache.kv, group=cache.group, num_heads=H, num_kv_heads=G,
             qk_dim=self.dk, v_dim=self.dv, window=0, keep_first=0, scale=self.scale, head_norm=True, value_share=self.MAPS,

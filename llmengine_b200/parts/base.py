@@ -204,10 +204,26 @@ class Part:
     # False for a part whose forward reads device data on the host (it then cannot be captured in a
     # CUDA graph, and steps of a model that holds such a part always run eagerly)
     capture_safe = True
+    # True for a part whose first product of its input can carry further rows for someone else who multiplies the same input
+    # (`carry_rows`)
+    carries_rows = False
 
     def __init__(self, rt: "Runtime", prefix: str):
         self.rt = rt
         self.prefix = prefix
+        self.carried: Optional[torch.Tensor] = None        # after `emit`: the carried rows' columns of the product
+
+    @staticmethod
+    def with_carried_rows(w: torch.Tensor, rows: torch.Tensor) -> Tuple[torch.Tensor, int]:
+        """(`w` with `rows` below it, the column of the product where theirs begin): rows of zeros between them up to a multiple of 8,
+        so that the columns begin on whole 16-byte pieces."""
+        at = w.shape[0] + -w.shape[0] % 8
+        return torch.cat([w, w.new_zeros(at - w.shape[0], w.shape[1]), rows], 0).contiguous(), at
+
+    def carry_rows(self, rows: torch.Tensor) -> None:
+        """Takes over `rows` [n, hidden] as further rows of the first product; called after `load_weights`.  `emit` then leaves the
+        columns of the product that belong to them in `carried`."""
+        raise NotImplementedError(f"{self.prefix}: this part carries no rows")
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         """Full tensor name -> spec, for every tensor this part (and its sub-parts) reads."""

@@ -345,6 +345,7 @@ class StreamResidualBlock(Part):
             self.norms.append(build_part("norm", layer.parts["feed_forward_norm"], rt, self.name(norm_names[1])))
             self.ffn = build_part("feed_forward", layer.parts["feed_forward"], rt, self.name(feed_forward_name))
         self.parts = tuple(p for p in (*self.norms, self.mixer, self.ffn) if p is not None)
+        self.sublayers = tuple(p for p in (self.mixer, self.ffn) if p is not None)
         n = len(self.norms)
         self.connections, self.gates = tuple(connection_names[:n]), tuple(gate_names[:n])
         self.capture_safe = all(p.capture_safe and hasattr(p, "emit") for p in self.parts)
@@ -370,14 +371,21 @@ class StreamResidualBlock(Part):
         self.read, self.mix = [f(c + ".in") for c in self.connections], [f(c + ".mix") for c in self.connections]
         self.put = [f(c + ".out") * self.multiplier for c in self.connections]
         self.w_gate, self.b_gate = [tensors[self.name(g)].contiguous() for g in self.gates], [f(g + ".b") for g in self.gates]
+        for q, part in enumerate(self.sublayers):
+            if part.carries_rows:                     # the gate reads the sublayer's own input: it rides in its first product
+                part.carry_rows(self.w_gate[q])
+                self.w_gate[q] = None
 
     def cache_spec(self):
         return self.mixer.cache_spec()
 
     def _result(self, plan: Plan, q: int, h: torch.Tensor, y: torch.Tensor) -> StreamUpdate:
-        """Sublayer q's result `y` on its way into the streams, with the product its gate is made from."""
-        gate = self.rt.workspace("sublayer_gate", self.hidden, self.rt.dtype)
-        plan.linear(h, self.w_gate[q], gate)
+        """Sublayer q's result `y` on its way into the streams, with what its gate is made from: columns of the sublayer's first
+        product, or a product of its own where the sublayer carries no rows."""
+        gate = self.sublayers[q].carried
+        if self.w_gate[q] is not None:
+            gate = self.rt.workspace("sublayer_gate", self.hidden, self.rt.dtype)
+            plan.linear(h, self.w_gate[q], gate)
         return StreamUpdate(y=y, gate=gate, bias=self.b_gate[q], mix=self.mix[q], put=self.put[q])
 
     def emit(self, plan: Plan, x: torch.Tensor, delta: Optional[StreamUpdate], cache):

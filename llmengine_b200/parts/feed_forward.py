@@ -214,6 +214,8 @@ class RoutedExperts(Part):
     choices, so a token's result does not depend on what else is in the step.  The shared expert's gate is one more row
     of the router's matrix, so one product gives both."""
 
+    carries_rows = True
+
     def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_experts: int, top_k: int, expert_size: int,
                  route_scale: float = 1.0, shared_size: int = 0, routing: str = "sigmoid", router_bias: bool = False,
                  shared_gate: bool = False, activation: str = "silu", correction: bool = False, identity: int = 0,
@@ -241,6 +243,12 @@ class RoutedExperts(Part):
         if self.shared_gate and self.shared is None:
             raise ValueError(f"{prefix}: a gate on the shared expert needs a shared expert")
         self.w_router = self.w_gate_up = self.w_down = self.b_router = None
+        self.carried_at: Optional[int] = None
+
+    def carry_rows(self, rows: torch.Tensor) -> None:
+        if self.b_router is not None:
+            raise ValueError(f"{self.prefix}: a router with a bias carries no rows")
+        self.w_router, self.carried_at = self.with_carried_rows(self.w_router, rows)
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         s = {self.name("router"): WeightSpec((self.choices, self.hidden))}
@@ -265,7 +273,7 @@ class RoutedExperts(Part):
         pad = -used % 8                 # rows of zeros up to a multiple of 8: the product's 32-bit output rows then start on 32 bytes
         if pad:
             rows.append(rows[0].new_zeros(pad, self.hidden))
-        self.w_router = torch.cat(rows, 0).contiguous()
+        self.w_router, self.carried_at = torch.cat(rows, 0).contiguous(), None
         if self.router_bias:
             b = t[self.name("router.b")].float()
             self.b_router = torch.cat([b, b.new_zeros(self.w_router.shape[0] - self.choices)]).contiguous()
@@ -283,6 +291,7 @@ class RoutedExperts(Part):
         wide = rt.workspace("router_logits", self.w_router.shape[0], torch.float32)    # [logits | gate of the shared expert]
         plan.linear(h, self.w_router, wide, bias=self.b_router)
         logits = wide[:, :E]
+        self.carried = wide[:, self.carried_at:] if self.carried_at is not None else None
         experts = rt.workspace("route_experts", top, torch.int32)
         weights = rt.workspace("route_weights", top, torch.float32)
         offsets = rt.buffer("route_offsets", 1, E + 1, torch.int32, exact=True, zero=True).view(-1)

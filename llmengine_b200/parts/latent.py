@@ -113,6 +113,8 @@ class LatentAttention(Part):
     [H, kv_rank, nope_dim] (it carries queries into the latent space), W_uv per head [H, v_dim, kv_rank].
     """
 
+    carries_rows = True
+
     def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, nope_dim: int, rot_dim: int,
                  v_dim: int, kv_rank: int, scale: float, norm_eps: float, position_encoding: Optional[PartSpec] = None,
                  sink: bool = False, output_gate: bool = False, q_rank: int = 0, window: int = 0):
@@ -130,6 +132,7 @@ class LatentAttention(Part):
         self.kv_size = self.rank + self.dr
         self.o_size = self.nh * self.dv
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.c_gain = self.sink = self.w_uq = self.q_gain = None
+        self.carried_at: Optional[int] = None
 
     # ------------------------------------------------------------------ weights
     def weight_specs(self) -> Dict[str, WeightSpec]:
@@ -154,7 +157,7 @@ class LatentAttention(Part):
 
     def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
         parts = [t[self.name("dq" if self.q_rank else "q")], t[self.name("dkv")]] + ([t[self.name("g")]] if self.has_gate else [])
-        self.w_in = torch.cat(parts, dim=0).contiguous()
+        self.w_in, self.carried_at = torch.cat(parts, dim=0).contiguous(), None
         if self.q_rank:
             self.w_uq = t[self.name("uq")].contiguous()
             self.q_gain = t[self.name("dq.norm")].contiguous()
@@ -163,6 +166,9 @@ class LatentAttention(Part):
         self.w_o = t[self.name("o")].contiguous()
         self.c_gain = t[self.name("dkv.norm")].contiguous()
         self.sink = t[self.name("sink")].float().contiguous() if self.has_sink else None
+
+    def carry_rows(self, rows: torch.Tensor) -> None:
+        self.w_in, self.carried_at = self.with_carried_rows(self.w_in, rows)
 
     def cache_spec(self) -> LatentKVSpec:
         return LatentKVSpec(self.kv_size, self.window)
@@ -177,6 +183,7 @@ class LatentAttention(Part):
         width = self.w_in.shape[0]
         proj = rt.workspace("latent_in", width, rt.dtype)
         plan.linear(h, self.w_in, proj)
+        self.carried = proj[:, self.carried_at:] if self.carried_at is not None else None
         first = self.q_rank or self.q_size                       # columns of the product that belong to the queries
         if self.q_rank:
             cq = rt.workspace("latent_cq", self.q_rank, rt.dtype)
@@ -201,7 +208,8 @@ class LatentAttention(Part):
         heads = rt.workspace("latent_heads", self.o_size, rt.dtype)
         plan.batched_linear(out.view(T, H, r), self.w_uv, heads.view(T, H, dv))
         if self.has_gate:
-            plan.pointwise("sigmoid_mul", heads, proj[:, first + self.kv_size:], heads)
+            gate = first + self.kv_size
+            plan.pointwise("sigmoid_mul", heads, proj[:, gate:gate + self.o_size], heads)
         delta = rt.workspace("mixer_out", self.hidden, torch.float32)
         plan.linear(heads, self.w_o, delta)
         return delta

@@ -322,6 +322,8 @@ class ForgetMemory(Part):
     """Tensors: q, f [heads qk_dim, hidden]; f.b, lower [heads qk_dim]; v [heads v_dim, hidden]; norm [v_dim]; o [hidden, heads v_dim].
     The three projections are ONE product with 32-bit results: gates and queries enter the recurrence unrounded."""
 
+    carries_rows = True
+
     def __init__(self, rt: Runtime, prefix: str, hidden_size: int, num_heads: int, qk_dim: int, v_dim: int, norm_eps: float):
         super().__init__(rt, prefix)
         self.hidden, self.nh, self.dk, self.dv, self.eps = int(hidden_size), int(num_heads), int(qk_dim), int(v_dim), float(norm_eps)
@@ -329,6 +331,7 @@ class ForgetMemory(Part):
         used = 2 * self.qk_size + self.heads_size
         self.in_size = used + -used % 8          # rows of zeros up to a multiple of 8: the product's rows start on 32 bytes
         self.w_in = self.w_o = self.f_bias = self.lower = self.norm_w = None
+        self.carried_at: Optional[int] = None
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         m = lambda n: WeightSpec((n, self.hidden))
@@ -340,17 +343,21 @@ class ForgetMemory(Part):
     def load_weights(self, t: Dict[str, torch.Tensor]) -> None:
         rows = [t[self.name(n)] for n in ("q", "f", "v")]
         rows.append(rows[0].new_zeros(self.in_size - sum(r.shape[0] for r in rows), self.hidden))
-        self.w_in, self.w_o = torch.cat(rows, 0).contiguous(), t[self.name("o")].contiguous()
+        self.w_in, self.w_o, self.carried_at = torch.cat(rows, 0).contiguous(), t[self.name("o")].contiguous(), None
         self.f_bias, self.lower = t[self.name("f.b")].float().contiguous(), t[self.name("lower")].float().contiguous()
         self.norm_w = t[self.name("norm")].float().repeat(self.nh).contiguous()
+
+    def carry_rows(self, rows: torch.Tensor) -> None:
+        self.w_in, self.carried_at = self.with_carried_rows(self.w_in, rows)
 
     def cache_spec(self) -> StatesSpec:
         return StatesSpec((("state", (self.nh, self.dv, self.dk)),))
 
     def emit(self, plan: Plan, h: torch.Tensor, cache: StatesView) -> torch.Tensor:
         rt, H, qs, hs = self.rt, self.nh, self.qk_size, self.heads_size
-        proj = rt.workspace("forget_in", self.in_size, torch.float32)
+        proj = rt.workspace("forget_in", self.w_in.shape[0], torch.float32)
         plan.linear(h, self.w_in, proj)
+        self.carried = proj[:, self.carried_at:] if self.carried_at is not None else None
         q, f = rt.workspace("forget_q", qs, torch.float32), rt.workspace("forget_f", qs, torch.float32)
         plan.forget_gates(q_in=proj[:, :qs], f_in=proj[:, qs:2 * qs], f_bias=self.f_bias, lower=self.lower, q=q, f=f)
         o = rt.workspace("forget_o", hs, torch.float32)
