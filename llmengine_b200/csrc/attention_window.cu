@@ -236,12 +236,14 @@ template <> struct Four<__nv_bfloat16> {
     }
 };
 
-template <typename T>
-__global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowPostArgs a) {
+// LANES lanes hold a head (its size in fours, rounded up to 8, 16 or 32), so a warp finishes 32 / LANES heads at a time.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(256) window_post_fours_kernel(LlmeWindowPostArgs a) {
     extern __shared__ __align__(16) float cs4[];                     // [rot_dims / 2] cosines, then sines
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, warps = blockDim.x >> 5, lane = threadIdx.x & 31, d = 4 * lane;
+    constexpr int EACH = 32 / LANES;                                 // heads a warp has in hand
+    const int t = blockIdx.x, warps = blockDim.x >> 5, lane = threadIdx.x & (LANES - 1), d = 4 * lane;
     const int dk = a.dk, dv = a.dv, ps = a.page_size, half = a.inv_freq ? a.rot_dims >> 1 : 0;
     for (int i = threadIdx.x; i < half; i += blockDim.x) {
         float s, c;
@@ -253,19 +255,29 @@ __global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowP
     const int page = slot >= 0 ? slot / ps : 0, off = slot - page * ps;
     const int nv = value_heads(a.nkv, a.value_share);
     T* kpage = (T*)a.cache + (size_t)page * page_values(a.nkv, nv, ps, dk, dv);
-    const int heads = a.nh + (slot >= 0 ? a.nkv + nv : 0), stride = gridDim.y * warps;
+    const int heads = a.nh + (slot >= 0 ? a.nkv : 0), stride = gridDim.y * warps * EACH;
     const T* qrow = (const T*)a.q_in + (size_t)t * a.q_stride;
     const T* krow = (const T*)a.k_in + (size_t)t * a.k_stride;
-    const T* vrow = (const T*)a.v_in + (size_t)t * a.v_stride;
     const bool turned = d < 2 * half, first = d < half, inside = d < dk;
     const int partner = !turned ? lane : first ? lane + half / 4 : lane - half / 4;
-    auto source = [&](int hh) -> const T* {
-        return hh < a.nh ? qrow + hh * dk : hh < a.nh + a.nkv ? krow + (hh - a.nh) * dk : vrow + (hh - a.nh - a.nkv) * dv;
+    auto source = [&](int hh) -> const T* { return hh < a.nh ? qrow + hh * dk : krow + (hh - a.nh) * dk; };
+    auto head_sum = [&](float v) {                                   // over the lanes of a head
+#pragma unroll
+        for (int o = LANES / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        return v;
     };
     const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    int hh = blockIdx.y * warps + (threadIdx.x >> 5);
-    float4 x = zero, ahead = zero;
-    if (hh < heads && d < (hh < a.nh + a.nkv ? dk : dv)) x = Four<T>::load(source(hh) + d);
+    int hh = (blockIdx.y * warps + (threadIdx.x >> 5)) * EACH + (threadIdx.x & 31) / LANES;
+    float4 x = hh < heads && inside ? Four<T>::load(source(hh) + d) : zero, ahead = zero;
+    if (slot >= 0) {                                                 // the values, as they are
+        const T* vrow = (const T*)a.v_in + (size_t)t * a.v_stride;
+        T* vpage = kpage + (size_t)a.nkv * ps * dk + (size_t)off * dv;
+        const int pieces = dv / 4;
+        for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < nv * pieces; i += gridDim.y * blockDim.x) {
+            const int g = i / pieces, e = 4 * (i - g * pieces);
+            Four<T>::store(vpage + (size_t)g * ps * dv + e, Four<T>::load(vrow + g * dv + e));
+        }
+    }
     __syncthreads();
     float4 c = make_float4(1.0f, 1.0f, 1.0f, 1.0f), s = zero, gq = c, gk = c;
     if (a.head_norm && inside && a.q_gain) {
@@ -281,36 +293,33 @@ __global__ void __launch_bounds__(256) window_post_unit_fours_kernel(LlmeWindowP
         s = *(const float4*)&cs4[half + (first ? d : d - half)];
         if (first) s = make_float4(-s.x, -s.y, -s.z, -s.w);          // u cos - v sin, v cos + u sin
     }
-    for (; hh < heads; hh += stride, x = ahead) {
+    // (every lane of a warp takes the same number of turns: exchanges are between all of them)
+    for (int h0 = hh - (threadIdx.x & 31) / LANES; h0 < heads; h0 += stride, hh += stride, x = ahead) {
         const int nx = hh + stride;
-        ahead = nx < heads && d < (nx < a.nh + a.nkv ? dk : dv) ? Four<T>::load(source(nx) + d) : zero;
-        if (hh >= a.nh + a.nkv) {
-            if (d < dv) Four<T>::store(kpage + (size_t)a.nkv * ps * dk + ((size_t)(hh - a.nh - a.nkv) * ps + off) * dv + d, x);
-            continue;
-        }
+        ahead = nx < heads && inside ? Four<T>::load(source(nx) + d) : zero;
         if (a.head_norm) {
-            const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+            const float ss = head_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
             const float rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
             const float4 g = hh < a.nh ? gq : gk;
             x = make_float4(x.x * rinv * g.x, x.y * rinv * g.y, x.z * rinv * g.z, x.w * rinv * g.w);
         }
         const float4 o = a.interleaved ? make_float4(x.y, x.x, x.w, x.z)
-                                       : make_float4(__shfl_sync(0xffffffffu, x.x, partner), __shfl_sync(0xffffffffu, x.y, partner),
-                                                     __shfl_sync(0xffffffffu, x.z, partner), __shfl_sync(0xffffffffu, x.w, partner));
+                                       : make_float4(__shfl_sync(0xffffffffu, x.x, partner, LANES), __shfl_sync(0xffffffffu, x.y, partner, LANES),
+                                                     __shfl_sync(0xffffffffu, x.z, partner, LANES), __shfl_sync(0xffffffffu, x.w, partner, LANES));
         if (turned) x = make_float4(x.x * c.x + o.x * s.x, x.y * c.y + o.y * s.y, x.z * c.z + o.z * s.z, x.w * c.w + o.w * s.w);
         float rinv = 1.0f;
         if (a.unit_norm) {
-            const float ss = warp_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
+            const float ss = head_sum(fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))));
             rinv = 1.0f / sqrtf(ss / (float)dk + a.eps);
         }
         T* out = hh < a.nh ? (T*)a.q_out + ((size_t)t * a.nh + hh) * dk : kpage + ((size_t)(hh - a.nh) * ps + off) * dk;
-        if (inside) Four<T>::store(out + d, make_float4(x.x * rinv, x.y * rinv, x.z * rinv, x.w * rinv));
+        if (inside && hh < heads) Four<T>::store(out + d, make_float4(x.x * rinv, x.y * rinv, x.z * rinv, x.w * rinv));
     }
 }
 
-// A block per token, or several where the step has few.
-static dim3 post_grid(const LlmeWindowPostArgs& a) {
-    const int heads = a.nh + (a.k_in ? a.nkv + (a.value_share > 1 ? a.nkv / a.value_share : a.nkv) : 0), most = (heads + 7) / 8;
+// A block per token, or several where the step has few; a block has eight warps of `each` heads.
+static dim3 post_grid(const LlmeWindowPostArgs& a, int each = 1) {
+    const int heads = a.nh + (a.k_in ? a.nkv + (a.value_share > 1 ? a.nkv / a.value_share : a.nkv) : 0), most = (heads + 8 * each - 1) / (8 * each);
     const int fill = (592 + a.tokens - 1) / a.tokens;
     return dim3(a.tokens, most < fill ? most : fill);
 }
@@ -318,11 +327,14 @@ static dim3 post_grid(const LlmeWindowPostArgs& a) {
 template <typename T>
 static bool launch_post_fours(const LlmeWindowPostArgs& a, cudaStream_t s) {
     const size_t smem = (size_t)(a.inv_freq ? a.rot_dims : 0) * sizeof(float), piece = 4 * sizeof(T);
-    const bool fours = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && a.dv <= 128 && (!a.inv_freq || a.rot_dims % (a.interleaved ? 4 : 8) == 0) &&
+    const bool fours = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && (!a.inv_freq || a.rot_dims % (a.interleaved ? 4 : 8) == 0) &&
                        a.q_stride % 4 == 0 && a.k_stride % 4 == 0 && a.v_stride % 4 == 0 && ((uintptr_t)a.q_gain | (uintptr_t)a.k_gain) % 16 == 0 &&
                        ((uintptr_t)a.q_in | (uintptr_t)a.k_in | (uintptr_t)a.v_in | (uintptr_t)a.q_out | (uintptr_t)a.cache) % piece == 0;
-    if (fours) llme_launch(window_post_unit_fours_kernel<T>, post_grid(a), dim3(256), smem, s, a);
-    return fours;
+    if (!fours) return false;
+    if (a.dk <= 32) llme_launch(window_post_fours_kernel<T, 8>, post_grid(a, 4), dim3(256), smem, s, a);
+    else if (a.dk <= 64) llme_launch(window_post_fours_kernel<T, 16>, post_grid(a, 2), dim3(256), smem, s, a);
+    else llme_launch(window_post_fours_kernel<T, 32>, post_grid(a), dim3(256), smem, s, a);
+    return true;
 }
 
 template <typename T>

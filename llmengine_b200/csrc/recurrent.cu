@@ -922,48 +922,63 @@ template <> __device__ __forceinline__ void store_four<__nv_bfloat16>(__nv_bfloa
     *(uint2*)p = raw;
 }
 
-template <typename T, typename GT, int V>
+// A warp takes N neighbouring items one behind the other, the loads of all of them on their way before the first sum.
+template <typename T, typename GT, int V, int N>
 __global__ void __launch_bounds__(128) gated_norm_fours_kernel(LlmeGatedNormArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, groups = a.cols / a.group;
-    const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);          // (token, group)
-    if (item >= (long long)a.tokens * groups) return;
-    const int t = (int)(item / groups), c0 = (int)(item - (long long)t * groups) * a.group;
-    const float* y = a.y + (size_t)t * a.ldy + c0;
-    const GT* g = (const GT*)a.gate + (size_t)t * a.ldg + c0;
-    T* o = (T*)a.out + (size_t)t * a.ldo + c0;
-    float u[V][4], gate[V][4], ss = 0.0f;
+    const long long item0 = ((long long)blockIdx.x * 4 + (threadIdx.x >> 5)) * N, items = (long long)a.tokens * groups;     // (token, group)
+    if (item0 >= items) return;
+    const int t0 = (int)(item0 / groups), g0 = (int)(item0 - (long long)t0 * groups);
+    float u[N][V][4], gate[N][V][4];
 #pragma unroll
-    for (int i = 0; i < V; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        if (c < a.group) {
-            load_four<float>(y + c, u[i]);
-            if (a.gate) load_four<GT>(g + c, gate[i]);
-        } else {
+    for (int k = 0; k < N; ++k) {
+        const int t = t0 + (g0 + k) / groups, c0 = (g0 + k) % groups * a.group;
+        const bool on = item0 + k < items;
+        const float* y = a.y + (size_t)t * a.ldy + c0;
+        const GT* g = (const GT*)a.gate + (size_t)t * a.ldg + c0;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) u[i][e] = gate[i][e] = 0.0f;
+        for (int i = 0; i < V; ++i) {
+            const int c = 4 * (lane + 32 * i);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) u[k][i][e] = gate[k][i][e] = 0.0f;
+            if (on && c < a.group) {
+                load_four<float>(y + c, u[k][i]);
+                if (a.gate) load_four<GT>(g + c, gate[k][i]);
+            }
         }
     }
 #pragma unroll
-    for (int i = 0; i < V; ++i)
+    for (int k = 0; k < N; ++k) {
+        const int t = t0 + (g0 + k) / groups, c0 = (g0 + k) % groups * a.group;
+        float ss = 0.0f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) ss = fmaf(u[i][e], u[i][e], ss);
-    const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.group + a.eps);
+        for (int i = 0; i < V; ++i)
 #pragma unroll
-    for (int i = 0; i < V; ++i) {
-        const int c = 4 * (lane + 32 * i);
-        if (c >= a.group) continue;
-        float w[4] = {1.0f, 1.0f, 1.0f, 1.0f};
-        if (a.weight) load_four<float>(a.weight + c0 + c, w);
+            for (int e = 0; e < 4; ++e) ss = fmaf(u[k][i][e], u[k][i][e], ss);
+        const float rinv = 1.0f / sqrtf(warp_sum(ss) / (float)a.group + a.eps);
+        if (item0 + k >= items) break;
+        T* o = (T*)a.out + (size_t)t * a.ldo + c0;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            // (a result that goes to bfloat16 takes the hardware's exponential and reciprocal)
-            const float z = a.gate ? gate[i][e] : 0.0f;
-            const float s = sizeof(T) == 2 ? __frcp_rn(1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
-            u[i][e] = u[i][e] * rinv * w[e] * (!a.gate ? 1.0f : a.gate_act == 1 ? s : z * s) * a.scale;
+        for (int i = 0; i < V; ++i) {
+            const int c = 4 * (lane + 32 * i);
+            if (c >= a.group) continue;
+            float w[4] = {1.0f, 1.0f, 1.0f, 1.0f};
+            if (a.weight) load_four<float>(a.weight + c0 + c, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float f = 1.0f;
+                if (a.gate) {
+                    // (a result that goes to bfloat16 takes the hardware's exponential and reciprocal)
+                    const float z = gate[k][i][e];
+                    const float s = sizeof(T) == 2 ? __frcp_rn(1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
+                    f = a.gate_act == 1 ? s : z * s;
+                }
+                u[k][i][e] = u[k][i][e] * rinv * w[e] * f * a.scale;
+            }
+            store_four<T>(o + c, u[k][i]);
         }
-        store_four<T>(o + c, u[i]);
     }
 }
 
@@ -973,9 +988,10 @@ static bool launch_fours(const LlmeGatedNormArgs& a, long long items, cudaStream
     if (a.gate_first || a.floor || a.group % 4 || a.group > 512 || items > (1LL << 32)) return false;
     if (a.ldy % 4 || a.ldg % 4 || a.ldo % 4 || (uintptr_t)a.y % 16 || (uintptr_t)a.weight % 16 || (uintptr_t)a.gate % gate_bytes || (uintptr_t)a.out % bytes) return false;
     const dim3 grid((unsigned)((items + 3) / 4)), block(128);
-    if (a.group <= 128) llme_launch(gated_norm_fours_kernel<T, GT, 1>, grid, block, 0, s, a);
-    else if (a.group <= 256) llme_launch(gated_norm_fours_kernel<T, GT, 2>, grid, block, 0, s, a);
-    else llme_launch(gated_norm_fours_kernel<T, GT, 4>, grid, block, 0, s, a);
+    if (a.group <= 128 && items >= 148 * 64) llme_launch(gated_norm_fours_kernel<T, GT, 1, 4>, dim3((unsigned)((items + 15) / 16)), block, 0, s, a);
+    else if (a.group <= 128) llme_launch(gated_norm_fours_kernel<T, GT, 1, 1>, grid, block, 0, s, a);
+    else if (a.group <= 256) llme_launch(gated_norm_fours_kernel<T, GT, 2, 1>, grid, block, 0, s, a);
+    else llme_launch(gated_norm_fours_kernel<T, GT, 4, 1>, grid, block, 0, s, a);
     return true;
 }
 

@@ -123,8 +123,8 @@ def test_small_records_of_the_design(dtype, tol):
         assert float((q.cpu() - silu(wide[:, :C])).abs().max()) < 1e-5
         assert float((f.cpu() - (low + (1 - low) * torch.sigmoid(wide[:, C:2 * C] + bias))).abs().max()) < 1e-6
         assert float(f.max()) <= 1.0 and float((f[1, 0].cpu() - low[0]).abs()) < 1e-6
-    for groups, group in ((3, 5), (4, 32), (2, 300), (1, 1500)):
-        T, cols = 7, groups * group
+    for T, groups, group in ((7, 3, 5), (7, 4, 32), (7, 2, 300), (7, 1, 1500), (999, 10, 128), (1201, 9, 20)):
+        cols = groups * group
         y, w = 3 * rnd(T, cols), 1 + 0.2 * rnd(cols)
         out = torch.zeros(T + 1, cols, dtype=dtype, device=DEV)
         _run(ops, lambda p: p.gated_norm(y=y.to(DEV), gate=None, weight=w.to(DEV), out=out, group=group, gate_first=False, eps=1e-5), _batch([T], [0]))
